@@ -5,7 +5,7 @@ What the reference does in one PagedAllocator + KVCache for one uniform tensor
 (engine/core/kv_cache.py:124-301, 305-437) is done here per GROUP: execution steps whose
 mixers need the same thing (kv heads, head size, window) share a pool of pages and one block
 table per request.  A group with a window gives a page back as soon as every key in it lies
-before the window of the next position.  Storage of a group is
+before the window of the next position (the pages of the first keep_first keys stay).  Storage of a group is
 [steps, planes (k, v; or one), pages + 1, kv_heads, page_size, head_dim]: one (page, kv head) is a
 contiguous page_size x head_dim tile that a kernel can fetch in one bulk copy.
 
@@ -147,7 +147,16 @@ class CacheManager:
         W = g.need.window
         if W is None or max_span is None:
             return full
-        return min(full, self.pages_for(W + max_span) + 1)
+        return min(full, self.pages_for(g.need.keep_first) + self.pages_for(W + max_span) + 1)
+
+    def _kept_pages(self, g: "_Group") -> int:
+        """Pages at the start of every request that no window passes: those of the first keep_first keys."""
+        return 0 if g.need.window is None else self.pages_for(g.need.keep_first)
+
+    def _live_pages(self, gi: int, seq: "SeqCache"):
+        """Page indices of group gi that the request holds: the kept start, and from first_live on."""
+        start, first = self._kept_pages(self.kv_groups[gi]), seq.first_live[gi]
+        return [*range(min(start, first)), *range(first, seq.num_pages[gi])]
 
     def _first_needed_page(self, g: _Group, num_cached: int) -> int:
         """First page index that holds a key some position >= num_cached may still read."""
@@ -206,7 +215,7 @@ class CacheManager:
             keep_from = min(self._first_needed_page(g, num_tokens), seq.num_pages[gi])
             row = g.tables[seq.slot]
             base = seq.slot * self.max_pages_per_seq
-            for idx in range(seq.first_live[gi], keep_from):
+            for idx in range(max(seq.first_live[gi], self._kept_pages(g)), keep_from):
                 g.pool.give(int(row[idx]))
                 row[idx] = PagePool.NULL_PAGE
                 g.dirty[base + idx] = None
@@ -221,7 +230,7 @@ class CacheManager:
         for gi, g in enumerate(self.kv_groups):
             row = g.tables[seq.slot]
             base = seq.slot * self.max_pages_per_seq
-            for idx in range(seq.first_live[gi], seq.num_pages[gi]):
+            for idx in self._live_pages(gi, seq):
                 g.pool.give(int(row[idx]))
                 row[idx] = PagePool.NULL_PAGE
                 g.dirty[base + idx] = None
@@ -265,10 +274,10 @@ class CacheManager:
             held = []
             for seq in self.seqs.values():
                 row = g.tables[seq.slot]
-                live = [int(p) for p in row[seq.first_live[gi]:seq.num_pages[gi]]]
+                at = self._live_pages(gi, seq)
+                live = [int(p) for p in row[at]]
                 assert all(p != 0 for p in live), f"group {gi}: a live table entry is the null page"
-                assert not row[:seq.first_live[gi]].any() and not row[seq.num_pages[gi]:].any(), \
-                    f"group {gi}: table entries outside the live range are not null"
+                assert not np.delete(row, at).any(), f"group {gi}: table entries outside the live range are not null"
                 held += live
             for slot in range(g.tables.shape[0]):
                 if slot not in {s.slot for s in self.seqs.values()}:

@@ -78,7 +78,11 @@ constexpr int DEC_WARPS_ALONE = 8; // warps of a block that has its SM to itself
 //               in flight per SM at no register cost.
 // SPLIT: every softmax weight enters the P V product as two bfloat16 numbers, its rounding and what the rounding left behind
 // (16 mantissa bits in all, summed in float32), for designs that want their attention weights in more than 16-bit precision.
-template <int D, bool BULK, int WARPS, bool SPLIT = false, bool BIAS = false>
+// EXT: the scaled score s becomes cap * tanh(s / cap) (cap > 0), the first `keep` keys of a request stay visible whatever the window,
+// and the output is multiplied by sigmoid(gate), gate bfloat16 [T, H D] with rows gate_stride apart (null: no gate).
+struct DecodeExt { float cap; int keep; const __nv_bfloat16* gate; int gate_stride; };
+
+template <int D, bool BULK, int WARPS, bool SPLIT = false, bool BIAS = false, bool EXT = false>
 __global__ void __launch_bounds__(WARPS * 32, WARPS > DEC_WARPS ? 1 : BULK ? 2 : 3)
 attn_decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap vmap,
                        const __nv_bfloat16* __restrict__ q, int q_stride, const __nv_bfloat16* __restrict__ k_cache,
@@ -89,7 +93,7 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
                        int H, int KV, int ps, float scale_log2, int window, int* __restrict__ merge_counters,
                        int* __restrict__ error_word, int cluster_merge, int block, int sink,
                        const float* __restrict__ sink_values, const float* __restrict__ bias_t, int bias_last,
-                       const float* __restrict__ slopes) {
+                       const float* __restrict__ slopes, const DecodeExt ext) {
     // BIAS: bias_t float32 [H, bias_last + 1] is added to the scaled score by the distance len - 1 - key (beyond bias_last: the last
     // entry), one row per head; sink_values float32 [H] (or null: 0) is the score of the sink; slopes float32 [H] (or null):
     // slopes[h] * distance is taken off the scaled score as well.
@@ -111,7 +115,11 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
     const int S = gridDim.z, s = blockIdx.z;
     const int tok = seg_q_start[seg], len = seg_kv_len[seg];
     const int lo = max(window > 0 ? max(0, len - window) : 0, block > 0 ? (len - 1) / block * block : 0);
-    const int blk_lo = lo / 16, blk_hi = (len + 15) / 16;
+    // EXT: the blocks of the kept keys come first (those that the window's own blocks do not hold), so block number blk is blk_of(blk)
+    const int blk_first = lo / 16, blk_hi = (len + 15) / 16;
+    const int kept_blocks = EXT && window > 0 ? min((ext.keep + 15) / 16, blk_first) : 0;
+    const int blk_lo = blk_first - kept_blocks;
+    auto blk_of = [&](int b) { return EXT && b < blk_first ? b - blk_lo : b; };
     const int per = (blk_hi - blk_lo + S - 1) / S;
     const int b0 = blk_lo + s * per, b1 = min(b0 + per, blk_hi);
     // an entry's pages: row `seg` of the table, or row table_rows[seg] of a table that holds a row per live request
@@ -139,8 +147,9 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
         sm100::mbar_init_fence();
     }
     // BULK: lane 0 asks for the K and V tiles of block `blk` into ring stage st
-    auto issue = [&](int blk, int st) {
+    auto issue = [&](int nth_blk, int st) {
         if (lane == 0) {
+            const int blk = blk_of(nth_blk);
             asm volatile("fence.proxy.async.shared::cta;\n" ::: "memory");      // the stage was just read with ordinary loads
             const uint32_t dst = sm100::smem_u32(ring + st * 2 * TILE), bar = bar0 + 8 * st;
             const int page = table_row[(blk * 16) / ps];
@@ -182,6 +191,16 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
     for (int t = 0; t < NT; ++t) { o[t][0] = o[t][1] = o[t][2] = o[t][3] = 0.f; }
     const bool has_sink = sink && s == 0 && warp == 0;
     constexpr float LOG2E = 1.4426950408889634f;
+    // cap * tanh(s / cap) = cap - 2 cap / (1 + e^(2 s / cap)), everything in base 2
+    const float cap_log2 = EXT ? ext.cap * LOG2E : 0.f, cap_rate = EXT && ext.cap > 0.f ? 2.f * scale_log2 / ext.cap : 0.f;
+    auto score = [&](float dot) {
+        if (!EXT || ext.cap <= 0.f) return dot * scale_log2;
+        return cap_log2 - __fdividef(2.f * cap_log2, 1.f + exp2f(dot * cap_rate));
+    };
+    auto gated = [&](float v, int h, int d) {             // what the kernel's three ways of finishing a row write
+        if (!EXT || ext.gate == nullptr) return v;
+        return v / (1.f + expf(-__bfloat162float(ext.gate[(size_t)tok * ext.gate_stride + (size_t)h * D + d])));
+    };
     const int head0 = kvh * G + min(g, G - 1), head1 = kvh * G + min(g + 8, G - 1);        // rows beyond G are padding
     const float* __restrict__ bias_row0 = BIAS && bias_t ? bias_t + (size_t)head0 * (bias_last + 1) : nullptr;     // no table: slopes alone
     const float* __restrict__ bias_row1 = BIAS && bias_t ? bias_t + (size_t)head1 * (bias_last + 1) : nullptr;
@@ -228,7 +247,8 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
                 vreg[i][hb] = *reinterpret_cast<const uint4*>(tile + hb * 2048 + key * 128 + ((g ^ (key & 7)) << 4));
         }
     };
-    auto tile_of = [&](const __nv_bfloat16* cache, int blk) {
+    auto tile_of = [&](const __nv_bfloat16* cache, int nth_blk) {
+        const int blk = blk_of(nth_blk);
         const int page = table_row[(blk * 16) / ps];
         return cache + ((size_t)(page * KV + kvh) * ps + (blk * 16) % ps) * D;
     };
@@ -271,16 +291,16 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
         for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
             for (int e = 0; e < 2; ++e) {
-                const int key = blk * 16 + nt * 8 + 2 * c + e;
-                const bool ok = key >= lo && key < len;
+                const int key = blk_of(blk) * 16 + nt * 8 + 2 * c + e;
+                const bool ok = (key >= lo || (EXT && key < ext.keep)) && key < len;
                 if (BIAS) {
                     const int far = max(len - 1 - key, 0), dist = min(far, bias_last);
                     const float t0 = bias_row0 ? bias_row0[dist] * LOG2E : 0.f, t1 = bias_row1 ? bias_row1[dist] * LOG2E : 0.f;
                     sc[nt][e] = ok ? fmaf(sc[nt][e], scale_log2, fmaf(-slope0, (float)far, t0)) : -INFINITY;
                     sc[nt][2 + e] = ok ? fmaf(sc[nt][2 + e], scale_log2, fmaf(-slope1, (float)far, t1)) : -INFINITY;
                 } else {
-                    sc[nt][e] = ok ? sc[nt][e] * scale_log2 : -INFINITY;
-                    sc[nt][2 + e] = ok ? sc[nt][2 + e] * scale_log2 : -INFINITY;
+                    sc[nt][e] = ok ? score(sc[nt][e]) : -INFINITY;
+                    sc[nt][2 + e] = ok ? score(sc[nt][2 + e]) : -INFINITY;
                 }
                 mx0 = fmaxf(mx0, sc[nt][e]);
                 mx1 = fmaxf(mx1, sc[nt][2 + e]);
@@ -366,7 +386,7 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
         const float val = den > 0.f ? num / den : 0.f;
         const int h = kvh * G + row;
         if (S == 1) {
-            out[((size_t)tok * H + h) * D + d] = __float2bfloat16_rn(val);
+            out[((size_t)tok * H + h) * D + d] = __float2bfloat16_rn(gated(val, h, d));
         } else if (BULK && cluster_merge) {
             float* cpart = smem + CLUSTER_OFF;             // [16][D] this split's rows, then [16] their log-sum-exp
             cpart[idx] = val;
@@ -400,7 +420,7 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
                     den += w;
                     num += w * v[r];
                 }
-                out[((size_t)tok * H + h) * D + d] = __float2bfloat16_rn(num / den);
+                out[((size_t)tok * H + h) * D + d] = __float2bfloat16_rn(gated(num / den, h, d));
             }
         }
         cluster_sync();                                    // the others' shared memory stays until split 0 has read it
@@ -443,7 +463,7 @@ attn_decode_mma_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_co
                 num += w * v[j];
             }
         }
-        out[((size_t)tok * H + h) * D + d] = __float2bfloat16_rn(num / den);
+        out[((size_t)tok * H + h) * D + d] = __float2bfloat16_rn(gated(num / den, h, d));
     }
     if (threadIdx.x == 0) merge_counters[blockIdx.x * KV + kvh] = 0;       // ready for the next call
 }
@@ -546,7 +566,7 @@ MI_EXPORT int mi_attn_decode_cluster_fit(int D, int splits) {
 // the device) and entry i reads row table_rows[i]; null: entry i reads row i.  cluster_merge != 0: with 2..8 splits the
 // splits of a (request, kv head) are launched as one thread-block cluster and merged through distributed shared memory
 // (o_part, lse_part, merge_counters unused).
-template <bool SPLIT, bool BIAS = false>
+template <bool SPLIT, bool BIAS = false, bool EXT = false>
 static int decode_mma_rows_launch(const void* q, int q_stride, const void* k_cache, const void* v_cache, void* out,
                                   float* o_part, float* lse_part, const int* decode_segs, int num_decode,
                                   const int* seg_q_start, const int* seg_kv_len, const int* block_table,
@@ -554,7 +574,7 @@ static int decode_mma_rows_launch(const void* q, int q_stride, const void* k_cac
                                   float scale, int window, int* merge_counters, int* error_word, int cache_pages,
                                   int cluster_merge, cudaStream_t stream, int block = 0, int sink = 0,
                                   const float* sink_values = nullptr, const float* bias_t = nullptr, int bias_last = 0,
-                                  const float* slopes = nullptr) {
+                                  const float* slopes = nullptr, const DecodeExt& ext = DecodeExt{0.f, 0, nullptr, 0}) {
     if (num_decode == 0) return 0;
     if ((D != 64 && D != 128) || H % KV || H / KV > 16 || ps % 16 || q_stride % 8) return -2;
     dim3 grid(num_decode, KV, splits);
@@ -583,7 +603,7 @@ static int decode_mma_rows_launch(const void* q, int q_stride, const void* k_cac
 #define LAUNCH(DD, BB, WW) do { \
         static bool configured = false; \
         if (!configured && smem > 48 * 1024) { \
-            cudaError_t e = cudaFuncSetAttribute(attn_decode_mma_kernel<DD, BB, WW, SPLIT, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            cudaError_t e = cudaFuncSetAttribute(attn_decode_mma_kernel<DD, BB, WW, SPLIT, BIAS, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (e != cudaSuccess) return (int)e; \
             configured = true; \
         } \
@@ -601,17 +621,17 @@ static int decode_mma_rows_launch(const void* q, int q_stride, const void* k_cac
             if (fit[splits] == 0) { \
                 cfg.attrs = attr; cfg.numAttrs = 1; \
                 int n = 0; \
-                if (cudaOccupancyMaxActiveClusters(&n, attn_decode_mma_kernel<DD, BB, WW, SPLIT, BIAS>, &cfg) != cudaSuccess || n < 1) n = -1; \
+                if (cudaOccupancyMaxActiveClusters(&n, attn_decode_mma_kernel<DD, BB, WW, SPLIT, BIAS, EXT>, &cfg) != cudaSuccess || n < 1) n = -1; \
                 fit[splits] = n; \
             } \
             /* (with a margin: blocks of the kernels before and after share the SMs for a moment) */ \
             if (fit[splits] < 0 || (long long)num_decode * KV * 100 > (long long)fit[splits] * 92) use_cluster = 0; \
         } \
         cfg.attrs = use_cluster ? attr : attr + 1; cfg.numAttrs = use_cluster ? 2 : 1; \
-        return (int)cudaLaunchKernelEx(&cfg, attn_decode_mma_kernel<DD, BB, WW, SPLIT, BIAS>, kmap, vmap, \
+        return (int)cudaLaunchKernelEx(&cfg, attn_decode_mma_kernel<DD, BB, WW, SPLIT, BIAS, EXT>, kmap, vmap, \
             (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, \
             (__nv_bfloat16*)out, o_part, lse_part, decode_segs, seg_q_start, seg_kv_len, block_table, table_rows, \
-            table_stride, H, KV, ps, scale_log2, window, merge_counters, error_word, use_cluster, block, sink, sink_values, bias_t, bias_last, slopes); } while (0)
+            table_stride, H, KV, ps, scale_log2, window, merge_counters, error_word, use_cluster, block, sink, sink_values, bias_t, bias_last, slopes, ext); } while (0)
     if (D == 128) { if (alone) LAUNCH(128, true, DEC_WARPS_ALONE); else if (bulk) LAUNCH(128, true, DEC_WARPS); else LAUNCH(128, false, DEC_WARPS); }
     else { if (alone) LAUNCH(64, true, DEC_WARPS_ALONE); else if (bulk) LAUNCH(64, true, DEC_WARPS); else LAUNCH(64, false, DEC_WARPS); }
 #undef LAUNCH
@@ -673,5 +693,19 @@ MI_EXPORT int mi_attn_decode_mma_rows_sloped(const void* q, int q_stride, const 
                                              int bias_last, const float* slopes, cudaStream_t stream) {
     if (!slopes) return -2;                                // bias_t may be null: slopes alone
     return decode_mma_rows_launch<true, true>(DECODE_ROWS_ARGS, block, sink, sink_values, bias_t, bias_last, slopes);
+}
+
+// The masked form (no sink, no blocks) with a cap on the scores (cap <= 0: none), the first `keep` keys kept whatever the window, and a
+// gate on the output (gate bfloat16 [T, H D], rows gate_stride apart; null: none).  With splits > 1 the kernel must merge them itself
+// (merge_counters, or splits that fit a cluster): a separate merge launch knows no gate.
+MI_EXPORT int mi_attn_decode_mma_rows_capped(const void* q, int q_stride, const void* k_cache, const void* v_cache, void* out,
+                                             float* o_part, float* lse_part, const int* decode_segs, int num_decode,
+                                             const int* seg_q_start, const int* seg_kv_len, const int* block_table,
+                                             const int* table_rows, int table_stride, int H, int KV, int D, int ps, int splits,
+                                             float scale, int window, int* merge_counters, int* error_word, int cache_pages,
+                                             int cluster_merge, float cap, int keep, const void* gate, int gate_stride, cudaStream_t stream) {
+    if (gate && splits > 1 && !merge_counters) return -2;
+    const DecodeExt ext{cap, keep, (const __nv_bfloat16*)gate, gate_stride};
+    return decode_mma_rows_launch<true, false, true>(DECODE_ROWS_ARGS, 0, 0, nullptr, nullptr, 0, nullptr, ext);
 }
 #undef DECODE_ROWS_ARGS

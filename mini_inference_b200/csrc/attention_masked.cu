@@ -8,6 +8,9 @@
 //   bias      a float32 table [bias_last + 1, H] added to the scaled score by the distance i - j (distances beyond bias_last
 //             read the last row)
 //   slopes    float32 [H]: slopes[h] * (i - j) is taken off the scaled score of head h (a straight line in the distance, no table)
+//   cap       (> 0) the score becomes cap * tanh(score / cap), last of all
+//   keep      with window > 0: the first `keep` keys of a sequence stay visible to every later position
+//   gate      [T, H Dv] in the rows' type (rows gate_stride apart) or null: the output is multiplied by sigmoid(gate), element by element
 //   sizes     key rows of D and value rows of Dv entries (up to 256; any size, 16-byte loads where rows allow), each in a pool of its own:
 //             k_cache [pages, KV, page_size, D], v_cache [pages, KV, page_size, Dv]
 //
@@ -35,7 +38,7 @@ __device__ __forceinline__ void attend_keys(const float* q_s, const T* __restric
                                             const int* __restrict__ table_row, int kvh, int KV, int D, int Dv, int ps,
                                             int lo, int hi, float& m, float& l, float (&acc)[MAX_D / 32],
                                             const float* __restrict__ bias = nullptr, int bias_last = 0, int H = 0, int h = 0, int qpos = 0,
-                                            float slope = 0.f) {
+                                            float slope = 0.f, float cap = 0.f) {
     const int lane = threadIdx.x & 31;
     constexpr int VN = Vec16<T>::N;
     for (int j0 = lo; j0 < hi; j0 += 32) {
@@ -58,6 +61,7 @@ __device__ __forceinline__ void attend_keys(const float* q_s, const T* __restric
             }
             s = bias ? dot + bias[(size_t)min(qpos - j, bias_last) * H + h] : dot;
             if (slope != 0.f) s -= slope * (float)(qpos - j);
+            if (cap > 0.f) s = cap * tanhf(s / cap);
         }
         const float m_new = fmaxf(m, warp_max(s));
         const float alpha = expf(m - m_new);              // nothing seen yet and no sink: exp(-inf) = 0
@@ -86,6 +90,11 @@ __device__ __forceinline__ int first_key(int p, int block, int window) {
     return lo;
 }
 
+template <typename T>
+__device__ __forceinline__ float gated(float v, const T* __restrict__ gate_row, int i) {
+    return gate_row ? v / (1.f + expf(-to_f32(gate_row[i]))) : v;
+}
+
 // grid (tiles, H): tile = (entry, first row); each warp takes rows of the tile in turn.
 template <typename T>
 __global__ void masked_prefill_kernel(const T* __restrict__ q, int q_stride, const T* __restrict__ k_cache, const T* __restrict__ v_cache,
@@ -94,7 +103,7 @@ __global__ void masked_prefill_kernel(const T* __restrict__ q, int q_stride, con
                                       const int* __restrict__ table_rows, int table_stride, int H, int KV, int D, int Dv, int ps,
                                       int tile_rows, float scale, int block, int window, int sink,
                                       const float* __restrict__ sink_values, const float* __restrict__ bias, int bias_last,
-                                      const float* __restrict__ slopes) {
+                                      const float* __restrict__ slopes, float cap, int keep, const T* __restrict__ gate, int gate_stride) {
     __shared__ float q_s[WARPS][MAX_D];
     const int seg = tiles[2 * blockIdx.x], r0 = tiles[2 * blockIdx.x + 1];
     const int h = blockIdx.y, kvh = h / (H / KV);
@@ -110,13 +119,18 @@ __global__ void masked_prefill_kernel(const T* __restrict__ q, int q_stride, con
         float m = sink ? (sink_values ? sink_values[h] : 0.f) : -INFINITY, l = sink ? 1.f : 0.f, acc[MAX_D / 32];
 #pragma unroll
         for (int k = 0; k < MAX_D / 32; ++k) acc[k] = 0.f;
-        attend_keys<T>(q_s[warp], k_cache, v_cache, table_row, kvh, KV, D, Dv, ps, first_key(p, block, window), p + 1, m, l, acc,
-                       bias, bias_last, H, h, p, slopes ? slopes[h] : 0.f);
+        const int lo = first_key(p, block, window), kept = min(keep, lo);
+        if (kept > 0)
+            attend_keys<T>(q_s[warp], k_cache, v_cache, table_row, kvh, KV, D, Dv, ps, 0, kept, m, l, acc, bias, bias_last, H, h, p,
+                           slopes ? slopes[h] : 0.f, cap);
+        attend_keys<T>(q_s[warp], k_cache, v_cache, table_row, kvh, KV, D, Dv, ps, lo, p + 1, m, l, acc,
+                       bias, bias_last, H, h, p, slopes ? slopes[h] : 0.f, cap);
         T* orow = out + ((size_t)tok * H + h) * Dv;
+        const T* grow = gate ? gate + (size_t)tok * gate_stride + (size_t)h * Dv : nullptr;
 #pragma unroll
         for (int k = 0; k < MAX_D / 32; ++k) {
             const int d = lane + 32 * k;
-            if (d < Dv) orow[d] = from_f32<T>(acc[k] / l);
+            if (d < Dv) orow[d] = from_f32<T>(gated(acc[k] / l, grow, d));
         }
         __syncwarp();
     }
@@ -132,7 +146,7 @@ __global__ void masked_decode_kernel(const T* __restrict__ q, int q_stride, cons
                                      const int* __restrict__ table_rows, int table_stride, int H, int KV, int D, int Dv, int ps,
                                      float scale, int block, int window, int sink,
                                      const float* __restrict__ sink_values, const float* __restrict__ bias, int bias_last,
-                                     const float* __restrict__ slopes) {
+                                     const float* __restrict__ slopes, float cap, int keep, const T* __restrict__ gate, int gate_stride) {
     __shared__ float q_s[WARPS][MAX_D];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int h = blockIdx.y * WARPS + warp;
@@ -141,9 +155,10 @@ __global__ void masked_decode_kernel(const T* __restrict__ q, int q_stride, cons
     const int tok = seg_q_start[seg], len = seg_kv_len[seg];
     const int S = gridDim.z, s = blockIdx.z;
     const int lo0 = first_key(len - 1, block, window);           // the query's position is len - 1
-    // every request cuts ITS OWN key range into S pieces of whole 32-key chunks
-    const int piece = (((len - lo0) + S - 1) / S + 31) / 32 * 32;
-    const int lo = lo0 + s * piece, hi = min(lo + piece, len);
+    // every request cuts ITS OWN visible keys (the kept ones first, then the range from lo0) into S pieces of whole 32-key chunks
+    const int kept = min(keep, lo0), seen = kept + len - lo0;
+    const int piece = ((seen + S - 1) / S + 31) / 32 * 32;
+    const int a = s * piece, b = min(a + piece, seen), shift = lo0 - kept;
     const T* qr = q + (size_t)tok * q_stride + (size_t)h * D;
     for (int d = lane; d < D; d += 32) q_s[warp][d] = to_f32(qr[d]) * scale;
     __syncwarp();
@@ -151,14 +166,19 @@ __global__ void masked_decode_kernel(const T* __restrict__ q, int q_stride, cons
     float m = own_sink ? (sink_values ? sink_values[h] : 0.f) : -INFINITY, l = own_sink ? 1.f : 0.f, acc[MAX_D / 32];
 #pragma unroll
     for (int k = 0; k < MAX_D / 32; ++k) acc[k] = 0.f;
-    if (lo < hi)
-        attend_keys<T>(q_s[warp], k_cache, v_cache, block_table + (size_t)(table_rows ? table_rows[seg] : seg) * table_stride, kvh, KV,
-                       D, Dv, ps, lo, hi, m, l, acc, bias, bias_last, H, h, len - 1, slopes ? slopes[h] : 0.f);
+    const int* table_row = block_table + (size_t)(table_rows ? table_rows[seg] : seg) * table_stride;
+    const T* grow = gate ? gate + (size_t)tok * gate_stride + (size_t)h * Dv : nullptr;
+    if (a < min(b, kept))
+        attend_keys<T>(q_s[warp], k_cache, v_cache, table_row, kvh, KV, D, Dv, ps, a, min(b, kept), m, l, acc, bias, bias_last, H, h,
+                       len - 1, slopes ? slopes[h] : 0.f, cap);
+    if (max(a, kept) < b)
+        attend_keys<T>(q_s[warp], k_cache, v_cache, table_row, kvh, KV, D, Dv, ps, max(a, kept) + shift, b + shift, m, l, acc, bias,
+                       bias_last, H, h, len - 1, slopes ? slopes[h] : 0.f, cap);
     const float inv = l > 0.f ? 1.f / l : 0.f;                  // empty piece: output 0, lse -inf
     if (S == 1) {
         T* orow = out + ((size_t)tok * H + h) * Dv;
 #pragma unroll
-        for (int k = 0; k < MAX_D / 32; ++k) { const int d = lane + 32 * k; if (d < Dv) orow[d] = from_f32<T>(acc[k] * inv); }
+        for (int k = 0; k < MAX_D / 32; ++k) { const int d = lane + 32 * k; if (d < Dv) orow[d] = from_f32<T>(gated(acc[k] * inv, grow, d)); }
     } else {
         const size_t idx = ((size_t)blockIdx.x * H + h) * S + s;
         float* orow = o_part + idx * Dv;
@@ -172,7 +192,7 @@ __global__ void masked_decode_kernel(const T* __restrict__ q, int q_stride, cons
 template <typename T>
 __global__ void masked_merge_kernel(const float* __restrict__ o_part, const float* __restrict__ lse_part, T* __restrict__ out,
                                     const int* __restrict__ decode_segs, const int* __restrict__ seg_q_start, int H, int Dv, int S, int sink,
-                                    const float* __restrict__ sink_values) {
+                                    const float* __restrict__ sink_values, const T* __restrict__ gate, int gate_stride) {
     const int i = blockIdx.x, h = blockIdx.y;
     const float sv = sink_values ? sink_values[h] : 0.f;
     const int tok = seg_q_start[decode_segs[i]];
@@ -184,7 +204,7 @@ __global__ void masked_merge_kernel(const float* __restrict__ o_part, const floa
     for (int d = threadIdx.x; d < Dv; d += blockDim.x) {
         float num = 0.f;
         for (int s = 0; s < S; ++s) num += expf(lse_part[base + s] - mx) * o_part[(base + s) * Dv + d];
-        out[((size_t)tok * H + h) * Dv + d] = from_f32<T>(num / den);
+        out[((size_t)tok * H + h) * Dv + d] = from_f32<T>(gated(num / den, gate ? gate + (size_t)tok * gate_stride + (size_t)h * Dv : (const T*)nullptr, d));
     }
 }
 
@@ -265,12 +285,12 @@ MI_EXPORT int mi_masked_prefill(const void* q, int q_stride, const void* k_cache
                                 int num_tiles, const int* seg_q_start, const int* seg_pos0, const int* block_table,
                                 const int* table_rows, int table_stride, int H, int KV, int D, int Dv, int ps, int tile_rows, float scale,
                                 int block, int window, int sink, const float* sink_values, const float* bias, int bias_last,
-                                const float* slopes, int dtype, cudaStream_t stream) {
+                                const float* slopes, float cap, int keep, const void* gate, int gate_stride, int dtype, cudaStream_t stream) {
     if (num_tiles == 0) return 0;
     if (D > MAX_D || Dv > MAX_D || H > 65535) return -2;
     dim3 grid(num_tiles, H);
 #define ARGS(T) (const T*)q, q_stride, (const T*)k_cache, (const T*)v_cache, (T*)out, tiles, seg_q_start, seg_pos0, block_table, table_rows, \
-        table_stride, H, KV, D, Dv, ps, tile_rows, scale, block, window, sink, sink_values, bias, bias_last, slopes
+        table_stride, H, KV, D, Dv, ps, tile_rows, scale, block, window, sink, sink_values, bias, bias_last, slopes, cap, keep, (const T*)gate, gate_stride
     if (dtype == MI_BF16) masked_prefill_kernel<__nv_bfloat16><<<grid, WARPS * 32, 0, stream>>>(ARGS(__nv_bfloat16));
     else masked_prefill_kernel<float><<<grid, WARPS * 32, 0, stream>>>(ARGS(float));
 #undef ARGS
@@ -281,12 +301,13 @@ MI_EXPORT int mi_masked_decode(const void* q, int q_stride, const void* k_cache,
                                float* lse_part, const int* decode_segs, int num_decode, const int* seg_q_start, const int* seg_kv_len,
                                const int* block_table, const int* table_rows, int table_stride, int H, int KV, int D, int Dv, int ps,
                                int splits, float scale, int block, int window, int sink, const float* sink_values, const float* bias,
-                               int bias_last, const float* slopes, int dtype, cudaStream_t stream) {
+                               int bias_last, const float* slopes, float cap, int keep, const void* gate, int gate_stride, int dtype,
+                               cudaStream_t stream) {
     if (num_decode == 0) return 0;
     if (D > MAX_D || Dv > MAX_D || H > 65535 * WARPS) return -2;
     dim3 grid(num_decode, (H + WARPS - 1) / WARPS, splits);
 #define ARGS(T) (const T*)q, q_stride, (const T*)k_cache, (const T*)v_cache, (T*)out, o_part, lse_part, decode_segs, seg_q_start, seg_kv_len, \
-        block_table, table_rows, table_stride, H, KV, D, Dv, ps, scale, block, window, sink, sink_values, bias, bias_last, slopes
+        block_table, table_rows, table_stride, H, KV, D, Dv, ps, scale, block, window, sink, sink_values, bias, bias_last, slopes, cap, keep, (const T*)gate, gate_stride
     if (dtype == MI_BF16) masked_decode_kernel<__nv_bfloat16><<<grid, WARPS * 32, 0, stream>>>(ARGS(__nv_bfloat16));
     else masked_decode_kernel<float><<<grid, WARPS * 32, 0, stream>>>(ARGS(float));
 #undef ARGS
@@ -294,8 +315,8 @@ MI_EXPORT int mi_masked_decode(const void* q, int q_stride, const void* k_cache,
     if (err || splits == 1) return err;
     dim3 mgrid(num_decode, H);
     if (dtype == MI_BF16)
-        masked_merge_kernel<__nv_bfloat16><<<mgrid, 128, 0, stream>>>(o_part, lse_part, (__nv_bfloat16*)out, decode_segs, seg_q_start, H, Dv, splits, sink, sink_values);
+        masked_merge_kernel<__nv_bfloat16><<<mgrid, 128, 0, stream>>>(o_part, lse_part, (__nv_bfloat16*)out, decode_segs, seg_q_start, H, Dv, splits, sink, sink_values, (const __nv_bfloat16*)gate, gate_stride);
     else
-        masked_merge_kernel<float><<<mgrid, 128, 0, stream>>>(o_part, lse_part, (float*)out, decode_segs, seg_q_start, H, Dv, splits, sink, sink_values);
+        masked_merge_kernel<float><<<mgrid, 128, 0, stream>>>(o_part, lse_part, (float*)out, decode_segs, seg_q_start, H, Dv, splits, sink, sink_values, (const float*)gate, gate_stride);
     return (int)cudaGetLastError();
 }

@@ -58,7 +58,11 @@ __device__ __forceinline__ float bf16_rest(float x) { return x - __bfloat162floa
 // BIAS: a learned number per head and distance, bias_t float32 [H, bias_last + 1] (distances beyond bias_last read the last entry),
 // is added to the scaled score; sink_values float32 [H] (with sink != 0) is the sink's score instead of 0; slopes float32 [H]
 // (or null): slopes[h] * distance is taken off the scaled score as well (a straight line beside, or instead of, the table).
-template <int D, bool SPLIT, bool BIAS>
+// EXT: the scaled score s becomes cap * tanh(s / cap) (cap > 0), the first `keep` keys of a sequence stay visible whatever the window,
+// and the output is multiplied by sigmoid(gate), gate bfloat16 [T, H D] with rows gate_stride apart (null: no gate).
+struct MmaExt { float cap; int keep; const __nv_bfloat16* gate; int gate_stride; };
+
+template <int D, bool SPLIT, bool BIAS, bool EXT>
 __global__ void __launch_bounds__(PF_WARPS * 32, 3)
 attn_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const __nv_bfloat16* __restrict__ k_cache,
                         const __nv_bfloat16* __restrict__ v_cache, __nv_bfloat16* __restrict__ out,
@@ -66,7 +70,7 @@ attn_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
                         const int* __restrict__ seg_pos0, const int* __restrict__ block_table,
                         const int* __restrict__ table_rows, int table_stride, int H, int KV, int ps, float scale_log2, int window,
                         int block, int sink, const float* __restrict__ sink_values, const float* __restrict__ bias_t, int bias_last,
-                        const float* __restrict__ slopes) {
+                        const float* __restrict__ slopes, const MmaExt ext) {
     // block > 0: a query at p sees only keys of its own block of positions, j >= floor(p / block) * block.  sink: the softmax has
     // one more term of score 0 without a value: the running maximum starts at 0 and the running sum at 1.
     auto first_key = [&](int p) { return max(block > 0 ? p / block * block : 0, window > 0 ? p - window + 1 : 0); };
@@ -89,8 +93,12 @@ attn_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
     const int rows = min(BQ, n - r0);
     const int* table_row = block_table + (size_t)(table_rows ? table_rows[seg] : seg) * table_stride;
     const int p_first = pos0 + r0, p_last = pos0 + r0 + rows - 1;
-    const int kt_lo = first_key(p_first) / BK;
+    const int kt_first = first_key(p_first) / BK;
     const int kt_hi = p_last / BK;                                          // inclusive
+    // EXT: the tiles of the kept keys come first (what the window's tiles do not hold anyway), so tile number it is kt_of(it)
+    const int kept_tiles = EXT && window > 0 ? min((ext.keep + BK - 1) / BK, kt_first) : 0;
+    const int kt_lo = kt_first - kept_tiles;
+    auto kt_of = [&](int it) { return EXT && it < kt_first ? it - kt_lo : it; };
 
     // ---- loads
     {
@@ -112,7 +120,7 @@ attn_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
             cp_async16(sV + buf * TILE_BYTES + swz<D>(row, ch), v_cache + off, ok);
         }
     };
-    load_kv(kt_lo, 0);
+    load_kv(kt_of(kt_lo), 0);
     cp_async_commit();
 
     uint32_t qa[KS][4];
@@ -124,6 +132,12 @@ attn_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
     const float* __restrict__ bias_row = BIAS && bias_t ? bias_t + (size_t)h * (bias_last + 1) : nullptr;      // no table: slopes alone
     const float slope_log2 = BIAS && slopes ? slopes[h] * LOG2E : 0.f;        // slopes: slopes[h] * distance is taken off the scaled score
     auto bias_at = [&](int dist) { return fmaf(-slope_log2, (float)dist, bias_row ? bias_row[min(dist, bias_last)] * LOG2E : 0.f); };
+    // cap * tanh(s / cap) = cap - 2 cap / (1 + e^(2 s / cap)), everything in base 2
+    const float cap_log2 = EXT ? ext.cap * LOG2E : 0.f, cap_rate = EXT && ext.cap > 0.f ? 2.f * scale_log2 / ext.cap : 0.f;
+    auto score = [&](float dot) {
+        if (!EXT || ext.cap <= 0.f) return dot * scale_log2;
+        return cap_log2 - __fdividef(2.f * cap_log2, 1.f + exp2f(dot * cap_rate));
+    };
     float m0 = sink ? sink_score : -INFINITY, m1 = m0, l0 = sink && c == 0 ? 1.f : 0.f, l1 = l0;      // a row's sum is spread over four lanes
     const int p_row0 = pos0 + r0 + warp * 16 + g, p_row1 = p_row0 + 8;     // positions of this thread's two rows
 
@@ -136,9 +150,9 @@ attn_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
     }
     __syncthreads();                               // the borrowed buffer is free again
 
-    for (int kt = kt_lo; kt <= kt_hi; ++kt) {
-        const int buf = (kt - kt_lo) & 1;
-        if (kt < kt_hi) { load_kv(kt + 1, buf ^ 1); cp_async_commit(); }      // lands while this tile is computed
+    for (int it = kt_lo; it <= kt_hi; ++it) {
+        const int buf = (it - kt_lo) & 1, kt = kt_of(it);
+        if (it < kt_hi) { load_kv(kt_of(it + 1), buf ^ 1); cp_async_commit(); }      // lands while this tile is computed
         const uint32_t kbuf = sK + buf * TILE_BYTES, vbuf = sV + buf * TILE_BYTES;
         // ---- S = Q K^T : 16 rows x 64 keys per warp
         float s[BK / 8][4];
@@ -170,7 +184,7 @@ attn_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
                     }
                 } else {
 #pragma unroll
-                    for (int e = 0; e < 4; ++e) s[nt][e] *= scale_log2;
+                    for (int e = 0; e < 4; ++e) s[nt][e] = score(s[nt][e]);
                 }
                 mx0 = fmaxf(mx0, fmaxf(s[nt][0], s[nt][1]));
                 mx1 = fmaxf(mx1, fmaxf(s[nt][2], s[nt][3]));
@@ -181,14 +195,14 @@ attn_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
                     const int j = kt * BK + nt * 8 + 2 * c + e;
-                    const bool ok0 = j <= p_row0 && j >= lo_row0;
-                    const bool ok1 = j <= p_row1 && j >= lo_row1;
+                    const bool ok0 = j <= p_row0 && (j >= lo_row0 || (EXT && j < ext.keep));
+                    const bool ok1 = j <= p_row1 && (j >= lo_row1 || (EXT && j < ext.keep));
                     if (BIAS) {
                         s[nt][e] = ok0 ? fmaf(s[nt][e], scale_log2, bias_at(p_row0 - j)) : -INFINITY;
                         s[nt][2 + e] = ok1 ? fmaf(s[nt][2 + e], scale_log2, bias_at(p_row1 - j)) : -INFINITY;
                     } else {
-                        s[nt][e] = ok0 ? s[nt][e] * scale_log2 : -INFINITY;
-                        s[nt][2 + e] = ok1 ? s[nt][2 + e] * scale_log2 : -INFINITY;
+                        s[nt][e] = ok0 ? score(s[nt][e]) : -INFINITY;
+                        s[nt][2 + e] = ok1 ? score(s[nt][2 + e]) : -INFINITY;
                     }
                     mx0 = fmaxf(mx0, s[nt][e]);
                     mx1 = fmaxf(mx1, s[nt][2 + e]);
@@ -247,6 +261,16 @@ attn_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
 #pragma unroll
     for (int t = 0; t < DT; ++t) {
         const int d = t * 8 + 2 * c;
+        if (EXT && ext.gate) {
+            const __nv_bfloat16* gr = ext.gate + (size_t)(qs + row0) * ext.gate_stride + (size_t)h * D + d;
+#pragma unroll
+            for (int half = 0; half < 2; ++half) {
+                if (row0 + 8 * half >= n) continue;
+                const float2 gv = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gr + (size_t)(8 * half) * ext.gate_stride));
+                o[t][2 * half] = __fdividef(o[t][2 * half], 1.f + exp2f(-LOG2E * gv.x));
+                o[t][2 * half + 1] = __fdividef(o[t][2 * half + 1], 1.f + exp2f(-LOG2E * gv.y));
+            }
+        }
         if (row0 < n) *reinterpret_cast<uint32_t*>(obase + (size_t)row0 * H * D + d) = pack2(o[t][0] * i0, o[t][1] * i0);
         if (row1 < n) *reinterpret_cast<uint32_t*>(obase + (size_t)row1 * H * D + d) = pack2(o[t][2] * i1, o[t][3] * i1);
     }
@@ -254,13 +278,13 @@ attn_prefill_mma_kernel(const __nv_bfloat16* __restrict__ q, int q_stride, const
 
 }  // namespace
 
-template <bool SPLIT, bool BIAS = false>
+template <bool SPLIT, bool BIAS = false, bool EXT = false>
 static int prefill_mma_launch(const void* q, int q_stride, const void* k_cache, const void* v_cache, void* out,
                               const int* tiles, int num_tiles, const int* seg_q_start, const int* seg_pos0,
                               const int* block_table, const int* table_rows, int table_stride, int H, int KV, int D, int ps,
                               int tile_rows, float scale, int window, int block, int sink, cudaStream_t stream,
                               const float* sink_values = nullptr, const float* bias_t = nullptr, int bias_last = 0,
-                              const float* slopes = nullptr) {
+                              const float* slopes = nullptr, const MmaExt& ext = MmaExt{0.f, 0, nullptr, 0}) {
     if (num_tiles == 0) return 0;
     if ((D != 64 && D != 128) || H % KV || tile_rows != BQ || q_stride % 8) return -2;
     static bool configured[2] = {false, false};
@@ -269,13 +293,13 @@ static int prefill_mma_launch(const void* q, int q_stride, const void* k_cache, 
     const float scale_log2 = scale * 1.4426950408889634f;
 #define LAUNCH(DD, IDX) do { \
         if (!configured[IDX]) { \
-            cudaError_t e = cudaFuncSetAttribute(attn_prefill_mma_kernel<DD, SPLIT, BIAS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
+            cudaError_t e = cudaFuncSetAttribute(attn_prefill_mma_kernel<DD, SPLIT, BIAS, EXT>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem); \
             if (e != cudaSuccess) return (int)e; \
             configured[IDX] = true; \
         } \
-        attn_prefill_mma_kernel<DD, SPLIT, BIAS><<<grid, PF_WARPS * 32, smem, stream>>>( \
+        attn_prefill_mma_kernel<DD, SPLIT, BIAS, EXT><<<grid, PF_WARPS * 32, smem, stream>>>( \
             (const __nv_bfloat16*)q, q_stride, (const __nv_bfloat16*)k_cache, (const __nv_bfloat16*)v_cache, \
-            (__nv_bfloat16*)out, tiles, seg_q_start, seg_pos0, block_table, table_rows, table_stride, H, KV, ps, scale_log2, window, block, sink, sink_values, bias_t, bias_last, slopes); \
+            (__nv_bfloat16*)out, tiles, seg_q_start, seg_pos0, block_table, table_rows, table_stride, H, KV, ps, scale_log2, window, block, sink, sink_values, bias_t, bias_last, slopes, ext); \
     } while (0)
     if (D == 128) LAUNCH(128, 0); else LAUNCH(64, 1);
 #undef LAUNCH
@@ -331,4 +355,18 @@ MI_EXPORT int mi_attn_prefill_mma_sloped(const void* q, int q_stride, const void
     return prefill_mma_launch<true, true>(q, q_stride, k_cache, v_cache, out, tiles, num_tiles, seg_q_start, seg_pos0, block_table, table_rows,
                                           table_stride, H, KV, D, ps, tile_rows, scale, window, block, sink, stream, sink_values, bias_t, bias_last,
                                           slopes);
+}
+
+// The masked form (no sink, no blocks) with a cap on the scores (cap <= 0: none), the first `keep` keys kept whatever the window, and a
+// gate on the output (gate bfloat16 [T, H D], rows gate_stride apart, 4-byte aligned; null: none).
+MI_EXPORT int mi_attn_prefill_mma_capped(const void* q, int q_stride, const void* k_cache, const void* v_cache, void* out,
+                                         const int* tiles, int num_tiles, const int* seg_q_start, const int* seg_pos0,
+                                         const int* block_table, const int* table_rows, int table_stride, int H, int KV, int D, int ps,
+                                         int tile_rows, float scale, int window, float cap, int keep, const void* gate, int gate_stride,
+                                         cudaStream_t stream) {
+    if (gate && ((uintptr_t)gate % 4 || gate_stride % 2)) return -2;
+    const MmaExt ext{cap, keep, (const __nv_bfloat16*)gate, gate_stride};
+    return prefill_mma_launch<true, false, true>(q, q_stride, k_cache, v_cache, out, tiles, num_tiles, seg_q_start, seg_pos0, block_table,
+                                                 table_rows, table_stride, H, KV, D, ps, tile_rows, scale, window, 0, 0, stream, nullptr, nullptr, 0,
+                                                 nullptr, ext);
 }

@@ -713,6 +713,30 @@ __global__ void memory_output_kernel(const float* __restrict__ full, const float
     }
 }
 
+// ------------------------------------------------------------------ state space with one decay per head (scan form), prologue
+// xbc [T, ldx] = x | B | C behind their convolution; dt_in: the dt columns as projected.  out [T, ldo] float32 = C [G N] | B [G N] | dt x [H V] |
+// e^(A dt) [H] with dt = softplus(. + dt_bias): what mode 3 of the scan stages.
+template <typename T>
+__global__ void state_space_prepare_kernel(const T* __restrict__ xbc, int ldx, const T* __restrict__ dt_in, int ld_dt, const float* __restrict__ dt_bias,
+                                           const float* __restrict__ A, float* __restrict__ out, int ldo, int H, int V, int GN) {
+    extern __shared__ float dsm[];                                // [H] dt
+    const size_t t = blockIdx.x;
+    const T* row = xbc + t * ldx;
+    float* o = out + t * ldo;
+    const int I = H * V;
+    for (int h = threadIdx.x; h < H; h += blockDim.x) {
+        const float v = to_f32(dt_in[t * ld_dt + h]) + dt_bias[h], dt = v > 20.f ? v : log1pf(expf(v));
+        dsm[h] = dt;
+        o[2 * GN + I + h] = expf(A[h] * dt);
+    }
+    for (int i = threadIdx.x; i < GN; i += blockDim.x) {
+        o[i] = to_f32(row[I + GN + i]);
+        o[GN + i] = to_f32(row[I + i]);
+    }
+    __syncthreads();
+    for (int i = threadIdx.x; i < I; i += blockDim.x) o[2 * GN + i] = dsm[i / V] * to_f32(row[i]);
+}
+
 // ------------------------------------------------------------------ selective state-space scan
 // grid (entries, ceil(I / 32)), 256 threads: 8 lanes share a channel, lane l holding the states n = l + 8 g in registers.
 // Per chunk of SS_TC tokens the block stages B and C [N] of each token, and for its 32 channels the step softplus(dt + dt_b),
@@ -1007,4 +1031,23 @@ MI_EXPORT int mi_selective_scan(const void* x, const float* dt, const float* dt_
 #undef PICK
 #undef GO
     return (int)cudaGetLastError();
+}
+
+// xbc [T, ldx] = x | B | C behind their convolution (H V, G N, G N columns), dt_in the dt columns as projected; prep: float32 scratch
+// [T, ldprep], ldprep >= 2 G N + H V + H; out float32 [T, H V] = S^T C.
+MI_EXPORT int mi_state_space_scan(const void* xbc, int ldx, const void* dt_in, int ld_dt, const float* dt_bias, const float* A, float* prep, int ldprep,
+                                  float* state, long long state_stride, float* out, const int* seg_q_start, const int* seg_slot, int T_, int num_segs,
+                                  int H, int V, int N, int G, int dtype, cudaStream_t stream) {
+    if (T_ == 0 || num_segs == 0) return 0;
+    if (H % G || (size_t)H * sizeof(float) > 48 * 1024) return -2;
+    const int GN = G * N;
+    if (dtype == MI_BF16)
+        state_space_prepare_kernel<__nv_bfloat16><<<T_, 256, H * sizeof(float), stream>>>((const __nv_bfloat16*)xbc, ldx, (const __nv_bfloat16*)dt_in, ld_dt, dt_bias, A, prep,
+                                                                                         ldprep, H, V, GN);
+    else
+        state_space_prepare_kernel<float><<<T_, 256, H * sizeof(float), stream>>>((const float*)xbc, ldx, (const float*)dt_in, ld_dt, dt_bias, A, prep, ldprep, H, V, GN);
+    const int err = (int)cudaGetLastError();
+    if (err) return err;
+    const ScanLayout L{ldprep, 0, GN, 2 * GN, 0, 2 * GN + H * V, 0, 0};
+    return launch_scan<3>(prep, L, nullptr, state, state_stride, out, seg_q_start, seg_slot, T_, num_segs, H, G, N, V, stream);
 }

@@ -129,6 +129,7 @@ class CudaOps:
         self.fast_attention = True           # tests clear this to run the generic attention kernels in bfloat16
         self.biased_attention_tc = True      # prompts of attention with a distance table or a learned sink on the tensor cores (bfloat16)
         self._zero_bias = {}
+        self.chunked_scan = True             # prompts of a state space with one decay per head in chunks on the tensor cores (tests clear this)
         # Latent attention whose cached rows have 64 or 128 entries can run on the tensor-core paged attention kernels.  Those
         # round the softmax weights to bfloat16 before the weighted sum; a design that asks for float32 weights gets the
         # float32 kernels of csrc/attention_latent.cu unless MI_LATENT_TC=1 (or this flag) says otherwise.
@@ -863,12 +864,14 @@ class CudaOps:
         return p[:, :H * D]
 
     def masked_attention(self, q, k_cache, v_cache, meta, H, KV, D, V, scale, block_size, window, sink, sink_values=None, distance_bias=None,
-                         distance_bias_by_head=None, distance_slopes=None):
+                         distance_bias_by_head=None, distance_slopes=None, softcap=None, keep_first=0, gate=None):
         """q [T, H D] (a strided view is allowed) over the pages; keys of D and values of V entries; block_size / window / sink as
         csrc/attention_masked.cu states them.  sink_values float32 [H]: the sink's score per head (None: 0); distance_bias float32
         [far + 1, H]: added to the scaled score by the distance i - j (beyond far: the last row); distance_bias_by_head: the same
         table as float32 [H, far + 1], for the kernels that read it along the distance.  distance_slopes float32 [H]: slope_h * (i - j)
-        is taken off the scaled score of head h.  Scores, weights and sums are float32.  Returns [T, H V]."""
+        is taken off the scaled score of head h.  softcap: the score becomes softcap * tanh(score / softcap), last of all; keep_first: with
+        a window, the first keep_first keys of a sequence stay visible; gate [T, H V] (a strided view is allowed): the output is multiplied by
+        sigmoid(gate).  Scores, weights and sums are float32.  Returns [T, H V]."""
         T = q.shape[0]
         assert q.stride(1) == 1
         out = torch.empty((T, H * V), dtype=q.dtype, device=q.device)
@@ -877,12 +880,25 @@ class CudaOps:
         num_decode, num_tiles = meta.decode_segs.shape[0], meta.prefill_tiles.shape[0]
         slopes = distance_slopes
         plain = sink_values is None and distance_bias is None and slopes is None
+        # a cap, kept keys or a gate: forms of their own of the tensor-core kernels (not beside a sink, blocks or distance terms)
+        extended = softcap is not None or keep_first > 0 or gate is not None
+        cap, keep, gate_stride = float(softcap or 0.0), int(keep_first if win else 0), 0 if gate is None else gate.stride(0)
+        assert gate is None or (gate.stride(1) == 1 and gate.dtype == q.dtype and gate.shape == (T, H * V))
+        tc_ext = extended and plain and not sink and not blk and (gate is None or (gate.data_ptr() % 4 == 0 and gate_stride % 2 == 0))
+        tc_form = tc_ext if extended else True
         if not plain:
             assert slopes is None or (slopes.dtype == torch.float32 and slopes.is_contiguous() and slopes.numel() == H)
             assert sink_values is None or (sink and sink_values.dtype == torch.float32 and sink_values.numel() == H)
             assert distance_bias is None or (distance_bias.dtype == torch.float32 and distance_bias.is_contiguous() and distance_bias.shape[1] == H)
         bias_last = 0 if distance_bias is None else distance_bias.shape[0] - 1
-        if (num_tiles and plain and self.fast_attention and q.dtype == torch.bfloat16 and D == V and D in (64, 128) and meta.tile == 64
+        if (num_tiles and tc_ext and self.fast_attention and q.dtype == torch.bfloat16 and D == V and D in (64, 128) and meta.tile == 64
+                and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0):
+            _check(self.lib.mi_attn_prefill_mma_capped(
+                _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(meta.prefill_tiles), num_tiles, _p(meta.seg_q_start),
+                _p(meta.seg_pos0), _p(meta.block_table), _p(rows), meta.max_pages, H, KV, D, meta.page_size, meta.tile,
+                _c.c_float(scale), win, _c.c_float(cap), keep, _p(gate), gate_stride, self._stream()), "attn_prefill_mma_capped")
+            self.launches += 1
+        elif (num_tiles and plain and not extended and self.fast_attention and q.dtype == torch.bfloat16 and D == V and D in (64, 128) and meta.tile == 64
                 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0):
             # key and value rows of 64 or 128 entries: the mma.sync prompt kernel, every softmax weight entering P V as two
             # bfloat16 numbers (float32 scores and softmax, 16 mantissa bits of each weight, float32 sums)
@@ -891,7 +907,7 @@ class CudaOps:
                 _p(meta.seg_pos0), _p(meta.block_table), _p(rows), meta.max_pages, H, KV, D, meta.page_size, meta.tile,
                 _c.c_float(scale), win, blk, int(bool(sink)), self._stream()), "attn_prefill_mma_masked")
             self.launches += 1
-        elif (num_tiles and self.fast_attention and self.biased_attention_tc and q.dtype == torch.bfloat16 and D == V and D in (64, 128)
+        elif (num_tiles and not extended and self.fast_attention and self.biased_attention_tc and q.dtype == torch.bfloat16 and D == V and D in (64, 128)
                 and meta.tile == 64 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0):
             # the same kernel with the learned sink's score and the distance table (one row per head) in its softmax
             no_table = slopes is not None and distance_bias is None and distance_bias_by_head is None        # slopes alone: the kernel reads no table
@@ -908,13 +924,14 @@ class CudaOps:
             _check(self.lib.mi_masked_prefill(
                 _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(meta.prefill_tiles), num_tiles, _p(meta.seg_q_start),
                 _p(meta.seg_pos0), _p(meta.block_table), _p(rows), meta.max_pages, H, KV, D, V, meta.page_size, meta.tile,
-                _c.c_float(scale), blk, win, int(bool(sink)), _p(sink_values), _p(distance_bias), bias_last, _p(slopes), code, self._stream()), "masked_prefill")
+                _c.c_float(scale), blk, win, int(bool(sink)), _p(sink_values), _p(distance_bias), bias_last, _p(slopes), _c.c_float(cap), keep,
+                _p(gate), gate_stride, code, self._stream()), "masked_prefill")
             self.launches += 1
         if not num_decode:
             return out
         reach = meta.max_kv_len if not blk else min(meta.max_kv_len, blk)              # the most keys a decoded token can see
-        reach = reach if not win else min(reach, win)
-        if ((plain or self.biased_attention_tc) and self.fast_attention and q.dtype == torch.bfloat16 and D == V and D in (64, 128) and H // KV <= 16
+        reach = reach if not win else min(reach, win + keep)
+        if ((plain or self.biased_attention_tc) and tc_form and self.fast_attention and q.dtype == torch.bfloat16 and D == V and D in (64, 128) and H // KV <= 16
                 and meta.page_size % 16 == 0 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0):
             # the tensor-core decode kernel (the G query heads of a kv head are the rows of one tile), split weights
             S = self.choose_splits(num_decode * KV, reach, 2 if self.bulk_decode else 3, cluster=self.bulk_decode and self.cluster_merge, head_dim=D)
@@ -922,7 +939,7 @@ class CudaOps:
             if S > 1:
                 o_part = torch.empty((num_decode, H, S, D), dtype=torch.float32, device=q.device)
                 lse = torch.empty((num_decode, H, S), dtype=torch.float32, device=q.device)
-                if self.fused_merge:
+                if self.fused_merge or gate is not None:       # the gate is applied where the splits are merged
                     if num_decode * KV > self._merge_counters.numel():
                         raise ValueError(f"attn_decode: {num_decode} rows x {KV} kv heads exceed the {self._merge_counters.numel()} "
                                          "merge counters allocated at start-up")
@@ -931,7 +948,10 @@ class CudaOps:
                     _p(meta.seg_q_start), _p(meta.seg_kv_len), _p(meta.block_table), _p(rows), meta.max_pages, H, KV, D, meta.page_size, S,
                     _c.c_float(scale), win, _p(counters), _p(self._stream_error if self.bulk_decode else None), k_cache.shape[0],
                     int(self.cluster_merge and counters is not None), blk, int(bool(sink)))
-            if plain:
+            if extended:                                   # args without its last two (blocks, sink)
+                _check(self.lib.mi_attn_decode_mma_rows_capped(*args[:-2], _c.c_float(cap), keep, _p(gate), gate_stride, self._stream()),
+                       "attn_decode_mma_capped")
+            elif plain:
                 _check(self.lib.mi_attn_decode_mma_rows_masked(*args, self._stream()), "attn_decode_mma_masked")
             else:                                          # the learned sink's score and the distance table (one row per head) in the softmax
                 if slopes is None:
@@ -959,8 +979,8 @@ class CudaOps:
             _check(self.lib.mi_masked_decode(
                 _p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(o_part), _p(lse), _p(meta.decode_segs), num_decode,
                 _p(meta.seg_q_start), _p(meta.seg_kv_len), _p(meta.block_table), _p(rows), meta.max_pages, H, KV, D, V,
-                meta.page_size, S, _c.c_float(scale), blk, win, int(bool(sink)), _p(sink_values), _p(distance_bias), bias_last, _p(slopes), code,
-                self._stream()), "masked_decode")
+                meta.page_size, S, _c.c_float(scale), blk, win, int(bool(sink)), _p(sink_values), _p(distance_bias), bias_last, _p(slopes),
+                _c.c_float(cap), keep, _p(gate), gate_stride, code, self._stream()), "masked_decode")
             self.launches += 2 if S > 1 else 1
         return out
 
@@ -1266,6 +1286,73 @@ class CudaOps:
                                           batch.num_segs, I, N, _code(x.dtype), self._stream()), "selective_scan")
         self.launches += 1
         return out
+
+    # ---------------------------------------------------------------- norms behind the sums, filtered attention, Mamba-2
+    def sum_rmsnorm(self, x, y, weight, alpha, eps, rows_dtype):
+        """x (float32 stream, in place) <- weight * N(alpha * x + y), N(z) = z / rms(z).  Returns x's rows in rows_dtype (x itself when that is float32)."""
+        assert x.dtype == torch.float32 and x.is_contiguous() and y.is_contiguous() and y.shape == x.shape and weight.dtype == torch.float32
+        rows = None if rows_dtype == torch.float32 else torch.empty(x.shape, dtype=rows_dtype, device=x.device)
+        _check(self.lib.mi_sum_rmsnorm(_p(x), _p(y), _p(weight), _p(rows), x.shape[0], x.shape[1], _c.c_float(alpha), _c.c_float(eps), _code(y.dtype),
+                                       self._stream()), "sum_rmsnorm")
+        self.launches += 1
+        return x if rows is None else rows
+
+    def conv_qkv_cache(self, p, H, KV, D, V, bias, conv, taps, q_norm, k_norm, eps, inv_freq, state, batch, meta, k_cache, v_cache):
+        """p [T, >= C] = q | k | v | .., C = H D + KV (D + V).  u = p + bias passes a causal convolution per channel (conv [C, taps] in p's
+        dtype; earlier inputs from, and the newest to, state float32 [slots, (taps - 1) C]); q and k are divided by the root mean square over
+        the whole projection, weighted (q_norm [H D], k_norm [KV D]) and rotated pairwise in the first 2 len(inv_freq) coordinates of each head;
+        k and v go to the rows' slots of the caches.  Returns q [T, H D].  KV = 0: p has no k and v, nothing is cached."""
+        T, C = p.shape[0], H * D + KV * (D + V)
+        assert p.stride(1) == 1 and p.shape[1] >= C and conv.dtype == p.dtype and conv.is_contiguous() and conv.shape == (C, taps)
+        assert bias.dtype == q_norm.dtype == torch.float32 and bias.numel() == C and q_norm.numel() == H * D
+        assert KV == 0 or (k_norm.dtype == torch.float32 and k_norm.numel() == KV * D and k_cache is not None and v_cache is not None)
+        assert taps == 1 or (state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] == (taps - 1) * C)
+        q = torch.empty((T, H * D), dtype=p.dtype, device=p.device)
+        single = T == batch.num_segs
+        _check(self.lib.mi_conv_qkv_cache(_p(p), p.stride(0), _p(bias), _p(conv), taps, _p(q_norm), _p(k_norm if KV else None), _c.c_float(eps), _p(inv_freq),
+                                          0 if inv_freq is None else inv_freq.numel(), _p(state if taps > 1 else None),
+                                          _c.c_longlong(state.stride(0) if taps > 1 else 0), _p(q), _p(k_cache if KV else None), _p(v_cache if KV else None),
+                                          _p(batch.positions), _p(meta.slots), _p(batch.token_seg), _p(batch.seg_q_start), _p(batch.seg_slot), T, batch.num_segs,
+                                          H, KV, D, V, meta.page_size, _code(p.dtype), self._stream()), "conv_qkv_cache")
+        self.launches += 1 if taps == 1 or single else 2
+        return q
+
+    def mamba2_mix(self, p, conv, conv_b, taps, dt_bias, A, Dv, H, V, N, G, norm, parts, eps, state, batch):
+        """p [T, >= I + C + H] = z | x | B | C | dt as projected (I = H V, C = I + 2 G N).  x, B and C pass the convolution and silu,
+        dt <- softplus(dt + dt_bias); S <- e^(A dt) S + dt B x^T, y = S^T C + Dv x per head from the slot's state (float32 H N V, the
+        convolution's last inputs behind it); returns rows [T, I] = N(y * silu(z)) in `parts` equal parts, * norm, in p's dtype."""
+        T, I = p.shape[0], H * V
+        C, off, dev = I + 2 * G * N, H * N * V, p.device
+        assert p.stride(1) == 1 and p.shape[1] >= I + C + H and state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] >= off + (taps - 1) * C
+        y = torch.empty((T, I), dtype=torch.float32, device=dev)
+        rows = torch.empty((T, I), dtype=p.dtype, device=dev)
+        code, stride = _code(p.dtype), _c.c_longlong(state.stride(0))
+        if T == batch.num_segs:                             # every entry brings one token
+            _check(self.lib.mi_ssd_step(_p(p), p.stride(0), _p(conv), _p(conv_b), taps, _p(dt_bias), _p(A), _p(Dv), _p(state), stride, _p(y),
+                                        _p(batch.seg_q_start), _p(batch.seg_slot), batch.num_segs, H, V, N, G, code, self._stream()), "ssd_step")
+            _check(self.lib.mi_gated_part_norm(_p(y), _p(None), 0, _p(None), V, _p(p), p.stride(0), _p(norm), _p(rows), T, I, parts, _c.c_float(eps),
+                                               _p(state), stride, _c.c_longlong(off), _p(batch.seg_slot), C, taps, code, self._stream()), "gated_part_norm")
+            self.launches += 2
+            return rows
+        xbc = self.short_conv(p[:, I:I + C], conv, conv_b, taps, state, off, batch, act="silu")
+        dt = p[:, I + C:I + C + H]
+        rc = -2
+        if p.dtype == torch.bfloat16 and self.chunked_scan:
+            rc = self.lib.mi_ssd_chunk(_p(xbc), xbc.stride(0), _p(dt), dt.stride(0), _p(dt_bias), _p(A), _p(state), stride, _p(y), _p(batch.seg_q_start),
+                                       _p(batch.seg_slot), T, batch.num_segs, H, V, N, G, self._stream())
+            if rc != -2:
+                _check(rc, "ssd_chunk")
+                self.launches += 1
+        if rc == -2:                                        # float32, or a size without a chunked form: the token-by-token scan
+            prep = torch.empty((T, (2 * G * N + I + H + 3) // 4 * 4), dtype=torch.float32, device=dev)
+            _check(self.lib.mi_state_space_scan(_p(xbc), xbc.stride(0), _p(dt), dt.stride(0), _p(dt_bias), _p(A), _p(prep), prep.stride(0), _p(state), stride,
+                                                _p(y), _p(batch.seg_q_start), _p(batch.seg_slot), T, batch.num_segs, H, V, N, G, code, self._stream()),
+                   "state_space_scan")
+            self.launches += 2
+        _check(self.lib.mi_gated_part_norm(_p(y), _p(xbc), xbc.stride(0), _p(Dv), V, _p(p), p.stride(0), _p(norm), _p(rows), T, I, parts, _c.c_float(eps),
+                                           _p(None), _c.c_longlong(0), _c.c_longlong(0), _p(None), 0, 1, code, self._stream()), "gated_part_norm")
+        self.launches += 1
+        return rows
 
     # ---------------------------------------------------------------- sampling
     def argmax(self, logits):

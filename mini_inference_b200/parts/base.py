@@ -71,8 +71,10 @@ a block reads the attributes, it never probes with hasattr:
 """
 from __future__ import annotations
 
-from dataclasses import dataclass
+from dataclasses import dataclass, replace
 from typing import Callable, Dict, Optional, Tuple
+
+import torch
 
 from ..config.spec import PartSpec
 
@@ -88,7 +90,7 @@ class WeightSpec:
 
 @dataclass(frozen=True)
 class KVCacheNeed:
-    """Keys and values in pages; window=None keeps every key, W keeps the last W.  planes: 2 = a key and a value
+    """Keys and values in pages; window=None keeps every key, W keeps the last W (and the first keep_first, whatever the window).  planes: 2 = a key and a value
     pool; 1 = one pool of rows per token (a mixer that caches one compressed vector per token and derives both
     keys and values from it); the LayerCache then has no v.  value_dim: the size of a value row when it differs from a
     key row's (head_dim); the value pool is then a tensor of its own."""
@@ -97,6 +99,16 @@ class KVCacheNeed:
     window: Optional[int] = None
     planes: int = 2
     value_dim: Optional[int] = None
+    keep_first: int = 0
+
+    def covering(self, other: "KVCacheNeed") -> "KVCacheNeed":
+        """The need of pages that serve both this one and another reader of the same rows: the wider window, the longer kept start."""
+        mine, theirs = (replace(n, window=None, keep_first=0) for n in (self, other))
+        if mine != theirs:
+            raise ValueError(f"a step reads another step's pages, but their rows differ: {mine} and {theirs}")
+        if self.window is None or other.window is None:
+            return mine
+        return replace(mine, window=max(self.window, other.window), keep_first=max(self.keep_first, other.keep_first))
 
 
 @dataclass(frozen=True)
@@ -117,6 +129,12 @@ def flatten_needs(need):
             raise ValueError("an execution step can own the pages of one cache group only")
         return out
     return (need,)
+
+
+def pad_rows(w, multiple: int):
+    """w [N, K] with zero rows behind it up to the next multiple: the rows of a product with it then start on aligned addresses."""
+    extra = -w.shape[0] % multiple
+    return (torch.cat([w, w.new_zeros(extra, w.shape[1])], dim=0) if extra else w).contiguous()
 
 
 class GatedDelta:
@@ -153,6 +171,10 @@ class LayerCache:
         """The view a sub-part gets: the pages (or none) and the given slice of the state tensors."""
         return LayerCache(self.group if pages else -1, self.k if pages else None, self.v if pages else None, states=self.states[states])
 
+    def with_states(self, own: "Optional[LayerCache]"):
+        """These pages with the states of another step's cache (a step that reads an earlier step's pages and keeps states of its own)."""
+        return LayerCache(self.group, self.k, self.v, states=() if own is None else own.states)
+
 
 class StepContext:
     """What a part sees of the step being run."""
@@ -188,6 +210,9 @@ class Part:
     takes_pair_delta = False         # Norm: `delta` may be a PairDelta; pre_add may be a [T, hidden] float32 tensor added row by row
     adds_to_embedding = False        # Position: owns an absolute_table (known before the weights are loaded)
     absolute_table = None            # Position: a [rows, hidden] table whose row p the embedding kernel adds to the token at position p
+    # Mixer: a step that reads an earlier step's pages (ExecStep.cache_from) still keeps the states its cache_need() declares for itself;
+    # the pages are kept long enough for the windows of all who read them
+    keeps_states_when_borrowing = False
     owns_state = False               # Block: cache_need() gives the step's whole need (its own parts' state beside the mixer's)
     offers_unbiased = False          # FeedForward: forward_unbiased(h, ctx) -> (y, bias): forward == y + bias, the addition left to the caller
     step_arrays_key: Optional[str] = None

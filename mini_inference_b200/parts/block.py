@@ -90,6 +90,35 @@ class OutputNormMixerOnly(OutputNormBlock):
     roles = {"mixer": "mixer", "norm1": "norm", "position": "position"}
 
 
+@register_block("postnorm")
+class PostNormBlock(Part):
+    """Sublayers read the stream itself and the norms stand behind the sums:
+    x <- norm1(alpha x + mixer(x)); x <- norm2(alpha x + feed_forward(x)), the norms being of the kind that offers norm_sum (they own
+    alpha).  The stream is float32; the sublayers get its rows in the run's dtype, which the norm kernel that last wrote the stream
+    has left in the step context."""
+    roles = {"mixer": "mixer", "feed_forward": "feed_forward", "norm1": "norm", "norm2": "norm", "position": "position"}
+
+    def __init__(self, spec, parts):
+        super().__init__(spec)
+        self.parts = dict(parts)
+        self.mixer, self.feed_forward = parts["mixer"], parts.get("feed_forward")
+        self.norm1, self.norm2, self.position = parts["norm1"], parts.get("norm2"), parts["position"]
+
+    def forward(self, x, delta, ctx, cache, owns_cache=True, pre_add=None):
+        if delta is not None or pre_add is not None:
+            raise ValueError("the arrangement with norms behind the sums carries no pending addition and takes no pass vector")
+        h = self.norm1.norm_sum(x, self.mixer.forward(ctx.rows_of(x), ctx, cache, self.position, owns_cache), ctx)
+        if self.feed_forward is not None:
+            self.norm2.norm_sum(x, self.feed_forward.forward(h, ctx), ctx)
+        return x, None
+
+
+@register_block("postnorm_mixer")
+class PostNormMixerOnly(PostNormBlock):
+    """A layer without feed-forward: x <- norm1(alpha x + mixer(x))."""
+    roles = {"mixer": "mixer", "norm1": "norm", "position": "position"}
+
+
 @register_block("gated_prenorm")
 class GatedPreNormBlock(Part):
     """Pre-norm arrangement whose sublayers read a FILTERED copy of the normed rows and whose outputs are GATED by the

@@ -254,3 +254,31 @@ class GatedMLP(Part):
     def forward(self, h, ctx):
         y, b = self.forward_unbiased(h, ctx)
         return y if b is None else ctx.ops.bias_act(y, b, "none")
+
+
+@register_feed_forward("clamped_mlp")
+class ClampedMLP(Part):
+    """W_down y,  g = min(W_gate h, limit), u = clamp(W_up h, -limit, limit), y = g * sigmoid(gate_slope * g) * (u + 1).
+    gate and up are one [2 I, hidden] product; clamps, gate and product of the halves are one kernel."""
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.hidden, self.inter = int(spec.get("hidden_size")), int(spec.get("intermediate_size"))
+        self.limit, self.slope = float(spec.get("limit")), float(spec.get("gate_slope"))
+        self.gate_up = self.down = None
+
+    def weight_specs(self):
+        return [WeightSpec("gate", (self.inter, self.hidden)), WeightSpec("up", (self.inter, self.hidden)),
+                WeightSpec("down", (self.hidden, self.inter))]
+
+    def load(self, tensors, dtype, device):
+        self.gate_up = torch.cat([tensors.pop("gate"), tensors.pop("up")], dim=0).contiguous()
+        self.down = tensors.pop("down")
+
+    @property
+    def first_weight(self):
+        return self.gate_up
+
+    def forward(self, h, ctx):
+        ops = ctx.ops
+        return ops.linear(ops.clamped_glu(ops.linear(h, self.gate_up), self.limit, self.slope), self.down)

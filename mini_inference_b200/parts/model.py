@@ -8,7 +8,7 @@ from typing import Dict, List, Tuple
 import torch
 
 from ..config.spec import ModelSpec, PartSpec
-from .base import Part, WeightSpec, build_part, lookup
+from .base import KVCacheNeed, Part, StateNeed, WeightSpec, build_part, flatten_needs, lookup
 
 
 class DecoderModel:
@@ -184,14 +184,23 @@ class DecoderModel:
     # ---------------------------------------------------------------- cache needs
     def cache_needs(self):
         """Per execution step: the mixer's need (the block's, when its own parts keep state too), or None when the step
-        reads another's cache.  An embedding part that keeps state adds one more entry behind the steps'."""
+        reads another's cache (its states alone, when its mixer keeps them all the same).  Pages that several steps read are kept
+        for the widest of their windows.  An embedding part that keeps state adds one more entry behind the steps'."""
         needs = []
         for step in self.spec.order:
             block = self.blocks[step.layer]
-            if step.cache_from is not None:
-                needs.append(None)
-            else:
-                needs.append(block.cache_need() if block.owns_state else block.mixer.cache_need())
+            need = block.cache_need() if block.owns_state else block.mixer.cache_need()
+            if step.cache_from is None:
+                needs.append(need)
+                continue
+            flat = flatten_needs(need)
+            reads = [n for n in flat if isinstance(n, KVCacheNeed)]
+            if reads:
+                src = flatten_needs(needs[step.cache_from])
+                wide = tuple(n.covering(reads[0]) if isinstance(n, KVCacheNeed) else n for n in src)
+                needs[step.cache_from] = wide if len(wide) != 1 else wide[0]
+            own = tuple(n for n in flat if isinstance(n, StateNeed)) if block.mixer.keeps_states_when_borrowing else ()
+            needs.append(own or None)
         if self.embedder is not None and self.embedder.cache_need() is not None:
             needs.append(self.embedder.cache_need())
         return needs
@@ -220,14 +229,16 @@ class DecoderModel:
         delta = None
         entered = x.clone() if self._adds_embedding else None  # the stream is rewritten in place; the passes add what entered it
         for i, step in enumerate(self.spec.order):
-            src = i if step.cache_from is None else step.cache_from
             block = self.blocks[step.layer]
+            cache = caches[i if step.cache_from is None else step.cache_from]
+            if step.cache_from is not None and block.mixer.keeps_states_when_borrowing:
+                cache = cache.with_states(caches[i])
             if step.add_embedding:
-                x, delta = block.forward(x, delta, ctx, caches[src], step.cache_from is None, pre_add=entered)
+                x, delta = block.forward(x, delta, ctx, cache, step.cache_from is None, pre_add=entered)
             elif step.add_row is None:
-                x, delta = block.forward(x, delta, ctx, caches[src], step.cache_from is None)
+                x, delta = block.forward(x, delta, ctx, cache, step.cache_from is None)
             else:
-                x, delta = block.forward(x, delta, ctx, caches[src], step.cache_from is None,
+                x, delta = block.forward(x, delta, ctx, cache, step.cache_from is None,
                                          pre_add=self.pass_vectors[step.add_row])
         if b.num_logit_rows == 0:
             return None

@@ -59,7 +59,8 @@ class ScalarRMSNorm(Part):
 @register_norm("stream_rmsnorm")
 class StreamRMSNorm(Part):
     """y = w * x / sqrt(mean(x^2) + eps) on a float32 residual stream, rows handed out in the run's dtype
-    (a pending delta, if any, is added to the stream first, in float32; a GatedDelta is gated in the same kernel)."""
+    (a pending delta, if any, is added to the stream first, in float32; a GatedDelta is gated in the same kernel).
+    one_plus=True: the checkpoint holds w - 1 (a weight stored around zero)."""
     keeps_float32_stream = True
     takes_gated_delta = True
     takes_pair_delta = True
@@ -67,13 +68,15 @@ class StreamRMSNorm(Part):
     def __init__(self, spec):
         super().__init__(spec)
         self.size, self.eps = int(spec.get("size")), float(spec.get("eps"))
+        self.one_plus = bool(spec.get("one_plus", False))
         self.weight = None
 
     def weight_specs(self):
-        return [WeightSpec("weight", (self.size,), kind="vector", init="norm")]
+        return [WeightSpec("weight", (self.size,), kind="vector", init="zeros" if self.one_plus else "norm")]
 
     def load(self, tensors, dtype, device):
-        self.weight = tensors["weight"].float().contiguous()
+        w = tensors["weight"].float()
+        self.weight = (1.0 + w if self.one_plus else w).contiguous()
 
     def forward(self, x, delta, ctx, rows=None, pre_add=None):
         """pre_add: float32 [hidden] (a vector for every row) or [T, hidden] (row by row), added to the stream with the delta."""
@@ -114,3 +117,33 @@ class OutputRMSNorm(Part):
 
     def forward(self, x, delta, ctx, rows=None, pre_add=None):
         raise TypeError("out_rmsnorm norms a sublayer's output (add_normed); it is not a norm of the stream")
+
+
+@register_norm("sum_rmsnorm")
+class SumRMSNorm(Part):
+    """The norm of an arrangement that norms the SUM of the stream and a sublayer's output: x <- w * N(alpha * x + y), N(z) = z / rms(z).
+    x is the float32 stream; one kernel adds, norms, rewrites x in float32 and hands out its rows in the run's dtype for the next
+    reader of the stream.  one_plus=True: the checkpoint holds w - 1 (a weight stored around zero)."""
+    keeps_float32_stream = True
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.size, self.eps, self.alpha = int(spec.get("size")), float(spec.get("eps")), float(spec.get("alpha", 1.0))
+        self.one_plus = bool(spec.get("one_plus", False))
+        self.weight = None
+
+    def weight_specs(self):
+        return [WeightSpec("weight", (self.size,), kind="vector", init="zeros" if self.one_plus else "norm")]
+
+    def load(self, tensors, dtype, device):
+        w = tensors["weight"].float()
+        self.weight = (1.0 + w if self.one_plus else w).contiguous()
+
+    def norm_sum(self, x, y, ctx):
+        """x <- w * N(alpha * x + y), in place; returns x's rows in the run's dtype."""
+        rows = ctx.ops.sum_rmsnorm(x, y, self.weight, self.alpha, self.eps, ctx.dtype)
+        ctx.note_rows(x, rows)
+        return rows
+
+    def forward(self, x, delta, ctx, rows=None, pre_add=None):
+        raise TypeError("sum_rmsnorm norms the sum of the stream and a sublayer's output (norm_sum); it hands out no rows of its own")

@@ -18,7 +18,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import Part, StateNeed, WeightSpec, register_mixer
+from .base import Part, StateNeed, WeightSpec, pad_rows, register_mixer
 
 
 @register_mixer("lightning")
@@ -347,3 +347,57 @@ class SelectiveScan(Part):
         dt = ops.linear(p[:, :R], self.w_dt, out_dtype=torch.float32)    # [T, I] float32, before bias and softplus
         y = ops.selective_scan(x, dt, self.dt_b, self.A, p[:, R:R + N], p[:, R + N:], self.Dv, xz[:, I:], cache.state, ctx.batch, ctx.dtype)
         return ops.linear(y, self.o)
+
+
+@register_mixer("mamba2")
+class Mamba2(Part):
+    """Mamba-2: a state-space recurrence with ONE decay per head and token over a state S [heads, N, V] (head h uses the B and C of
+    group floor(h / (heads / groups))):
+        z | x | B | C | dt = W_in h;  x, B, C <- silu(conv(.) + b) (causal, per channel, conv_taps taps);  dt <- softplus(dt + dt_bias);
+        S <- exp(-exp(A_log) dt) S + dt B x^T;   y = S^T C + D x;
+    rows: y * silu(z), divided by the root mean square in norm_groups equal parts, * weight; then W_o.
+    The state slot holds S (float32) and behind it the convolution's last conv_taps - 1 inputs.  dt, decays, state and read-out are
+    float32.  Prompts walk a request in chunks of 64 tokens on the tensor cores (the decayed sums inside a chunk are a masked product,
+    the state enters and leaves once a chunk); a decode step is one kernel over the state."""
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        g = spec.get
+        self.hidden, self.H, self.V, self.N = int(g("hidden_size")), int(g("num_heads")), int(g("value_dim")), int(g("state_dim"))
+        self.G, self.parts, self.taps, self.eps = int(g("groups")), int(g("norm_groups")), int(g("conv_taps")), float(g("out_norm_eps"))
+        self.I, self.C = self.H * self.V, self.H * self.V + 2 * self.G * self.N           # inner size; channels of the convolution
+        if self.H % self.G or self.I % self.parts or self.taps < 1:
+            raise ValueError(f"mamba2: {self.H} heads of {self.V} in {self.G} groups, {self.parts} norm parts, {self.taps} taps")
+        self.proj = self.conv = self.conv_b = self.dt_bias = self.A = self.Dv = self.norm = self.o = None
+
+    def weight_specs(self):
+        H, I, C, hid = self.H, self.I, self.C, self.hidden
+        return [WeightSpec("in", (I + C + H, hid)), WeightSpec("conv", (C, self.taps), kind="vector"),
+                WeightSpec("conv.b", (C,), kind="vector", init="zeros"), WeightSpec("dt_bias", (H,), kind="vector", init="zeros"),
+                WeightSpec("A_log", (H,), kind="vector", init="zeros"), WeightSpec("D", (H,), kind="vector", init="norm"),
+                WeightSpec("norm", (I,), kind="vector", init="norm"), WeightSpec("o", (hid, I))]
+
+    def cache_need(self):
+        floats = self.H * self.N * self.V + (self.taps - 1) * self.C
+        return StateNeed(((floats + 3) // 4 * 4,), "float32")              # whole 16-byte pieces a slot
+
+    def load(self, tensors, dtype, device):
+        self.proj, self.o = pad_rows(tensors.pop("in"), 8), tensors.pop("o")
+        self.conv, self.conv_b = tensors.pop("conv").float().contiguous(), tensors.pop("conv.b").float().contiguous()
+        self.dt_bias, self.Dv = tensors.pop("dt_bias").float().contiguous(), tensors.pop("D").float().contiguous()
+        self.A = (-torch.exp(tensors.pop("A_log").float())).contiguous()
+        self.norm = tensors.pop("norm").float().contiguous()
+
+    @property
+    def first_weight(self):
+        return self.proj
+
+    def step_flops(self, rows, pairs):
+        return 4 * self.I * self.N * rows                          # state update and read-out, a multiply and an add each
+
+    def forward(self, h, ctx, cache, position, owns_cache=True):
+        ops = ctx.ops
+        p = ops.linear(h, self.proj)                               # [T, I + C + H (+ unused)]: z | x | B | C | dt
+        rows = ops.mamba2_mix(p, self.conv, self.conv_b, self.taps, self.dt_bias, self.A, self.Dv, self.H, self.V, self.N, self.G,
+                              self.norm, self.parts, self.eps, cache.state, ctx.batch)
+        return ops.linear(rows, self.o)

@@ -772,6 +772,95 @@ _stream_rmsnorm, _masked_attention, _route_topk, _expert_ffn = _stream_rmsnorm_g
 _latent_prepare, _head_gate, _unit_qk_cache, _masked_attention, _route_topk = _latent_prepare_general, _head_gate_optional, _unit_qk_cache_general, _masked_attention_sloped, _route_topk_any
 
 
+# ---------------------------------------------------------------- norms behind the sums, filtered attention, Mamba-2
+def _sum_rmsnorm(self, x, y, weight, alpha, eps, rows_dtype):
+    x.copy_(_rms(alpha * x + y.float(), eps) * weight.float())
+    return x if rows_dtype == torch.float32 else x.to(rows_dtype)
+
+
+def _conv_qkv_cache(self, p, H, KV, D, V, bias, conv, taps, q_norm, k_norm, eps, inv_freq, state, batch, meta, k_cache, v_cache):
+    T, C = p.shape[0], H * D + KV * (D + V)
+    u = p[:, :C].float() + bias.float()
+    y = torch.empty_like(u)
+    for a, b, slot in _segments(batch):
+        hist = state[slot].view(taps - 1, C) if taps > 1 else u[:0]
+        ext = torch.cat([hist, u[a:b]], dim=0)
+        y[a:b] = sum(conv[:, j].float() * ext[j:j + b - a] for j in range(taps))
+        if taps > 1:
+            state[slot] = ext[ext.shape[0] - (taps - 1):].reshape(-1)
+    def turned(t, w, heads):
+        t = (_rms(t, eps) * w.float()).view(T, heads, D)
+        if inv_freq is None or inv_freq.numel() == 0:
+            return t
+        n = inv_freq.numel()
+        ang = batch.positions.float()[:, None] * inv_freq.float()[None, :]
+        cos, sin = ang.cos()[:, None, :], ang.sin()[:, None, :]
+        a, b = t[..., 0:2 * n:2].clone(), t[..., 1:2 * n:2].clone()
+        t[..., 0:2 * n:2], t[..., 1:2 * n:2] = a * cos - b * sin, b * cos + a * sin
+        return t
+    if KV:
+        page, off = meta.slots.long() // meta.page_size, meta.slots.long() % meta.page_size
+        k_cache[page, :, off, :] = turned(y[:, H * D:(H + KV) * D], k_norm, KV).to(p.dtype)
+        v_cache[page, :, off, :] = y[:, (H + KV) * D:].view(T, KV, V).to(p.dtype)
+    return turned(y[:, :H * D], q_norm, H).reshape(T, H * D).to(p.dtype)
+
+
+_masked_attention_before = _masked_attention
+
+
+def _masked_attention_capped(self, q, k_cache, v_cache, meta, H, KV, D, V, scale, block_size, window, sink, sink_values=None,
+                             distance_bias=None, distance_bias_by_head=None, distance_slopes=None, softcap=None, keep_first=0, gate=None):
+    if softcap is None and not keep_first and gate is None:
+        return _masked_attention_before(self, q, k_cache, v_cache, meta, H, KV, D, V, scale, block_size, window, sink, sink_values,
+                                        distance_bias, distance_bias_by_head, distance_slopes)
+    assert block_size is None and not sink and distance_bias is None and distance_slopes is None
+    T = q.shape[0]
+    out = torch.empty((T, H * V), dtype=torch.float32, device=q.device)
+    q_start, pos0, kv_len = meta.seg_q_start.tolist(), meta.seg_pos0.tolist(), meta.seg_kv_len.tolist()
+    ps, rows = meta.page_size, getattr(meta, "table_rows", None)
+    rows = list(range(len(pos0))) if rows is None else rows.tolist()
+    for s in range(len(pos0)):
+        a, b, L = q_start[s], q_start[s + 1], kv_len[s]
+        j = torch.arange(L, device=q.device)
+        pages = meta.block_table[rows[s], j // ps].long()
+        k = k_cache[pages, :, j % ps, :].float().repeat_interleave(H // KV, dim=1)
+        v = v_cache[pages, :, j % ps, :].float().repeat_interleave(H // KV, dim=1)
+        dist = (pos0[s] + torch.arange(b - a, device=q.device))[:, None] - j[None, :]
+        visible = dist >= 0
+        if window is not None:
+            visible &= (dist < window) | (j[None, :] < keep_first)
+        sc = torch.einsum("phd,jhd->hpj", q[a:b].reshape(b - a, H, D).float(), k) * scale
+        if softcap is not None:
+            sc = softcap * torch.tanh(sc / softcap)
+        w = torch.softmax(sc.masked_fill(~visible[None], float("-inf")), dim=-1)
+        out[a:b] = torch.einsum("hpj,jhd->phd", w, v).reshape(b - a, H * V)
+    if gate is not None:
+        out = out * torch.sigmoid(gate.float())
+    return out.to(q.dtype)
+
+
+def _mamba2_mix(self, p, conv, conv_b, taps, dt_bias, A, Dv, H, V, N, G, norm, parts, eps, state, batch):
+    T, I, GN = p.shape[0], H * V, G * N
+    C = I + 2 * GN
+    xbc = _short_conv(self, p[:, I:I + C], conv, conv_b, taps, state, H * N * V, batch, act="silu").float()
+    dt = torch.nn.functional.softplus(p[:, I + C:I + C + H].float() + dt_bias)
+    x = xbc[:, :I].view(T, H, V)
+    B = xbc[:, I:I + GN].view(T, G, N).repeat_interleave(H // G, dim=1)
+    Cm = xbc[:, I + GN:].view(T, G, N).repeat_interleave(H // G, dim=1)
+    y = torch.empty(T, H, V, device=p.device)
+    for a, b, slot in _segments(batch):
+        S = state[slot, :H * N * V].view(H, N, V).clone()
+        for t in range(a, b):
+            S = torch.exp(A * dt[t])[:, None, None] * S + dt[t][:, None, None] * B[t][:, :, None] * x[t][:, None, :]
+            y[t] = torch.einsum("hnv,hn->hv", S, Cm[t]) + Dv[:, None] * x[t]
+        state[slot, :H * N * V] = S.reshape(-1)
+    g = y.reshape(T, I) * torch.nn.functional.silu(p[:, :I].float())
+    return (_rms(g.view(T, parts, -1), eps).reshape(T, I) * norm).to(p.dtype)
+
+
+_masked_attention = _masked_attention_capped
+
+
 for _name, _fn in list(globals().items()):
     if _name.startswith("_") and _name[1:] in ("embed_scaled_norm", "add_scaled_rmsnorm", "polynorm", "lightning_scan", "group_rmsnorm_gate",
                                                "delta_prepare", "delta_scan", "batched_linear", "latent_prepare", "latent_attention", "head_gate",
@@ -779,5 +868,6 @@ for _name, _fn in list(globals().items()):
                                                "retention_scan", "route_topk", "clamped_glu", "expert_ffn",
                                                "embed_bigram_stream", "short_conv", "general_delta_prepare", "general_delta_scan", "matrix_memory",
                                                "selective_scan", "dual_rmsnorm_mix", "bias_act", "softcap",
-                                               "embed_scaled_stream", "stream_rmsnorm_pair", "rows_rmsnorm", "bias_glu", "scale_logits"):
+                                               "embed_scaled_stream", "stream_rmsnorm_pair", "rows_rmsnorm", "bias_glu", "scale_logits",
+                                               "sum_rmsnorm", "conv_qkv_cache", "mamba2_mix"):
         setattr(TorchRefOps, _name[1:], _fn)
