@@ -727,7 +727,8 @@ __global__ void state_space_prepare_kernel(const T* __restrict__ xbc, int ldx, c
     for (int h = threadIdx.x; h < H; h += blockDim.x) {
         const float v = to_f32(dt_in[t * ld_dt + h]) + dt_bias[h], dt = v > 20.f ? v : log1pf(expf(v));
         dsm[h] = dt;
-        o[2 * GN + I + h] = expf(A[h] * dt);
+        // a decay near one acts on a state hundreds of times in a row: its last bit is worth an exponential in double, rounded once
+        o[2 * GN + I + h] = (float)exp((double)A[h] * (double)dt);
     }
     for (int i = threadIdx.x; i < GN; i += blockDim.x) {
         o[i] = to_f32(row[I + GN + i]);

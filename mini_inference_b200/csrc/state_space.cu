@@ -312,7 +312,9 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(const T* __restrict__ p, 
     const int col = threadIdx.x % cols, r0 = threadIdx.x / cols;
     float* S = slot + (long long)h * N * V;
     const float dt = softplus(to_f32(p[t * ldp + I + C + h]) + dt_bias[h]);
-    const float decay = expf(A[h] * dt);
+    __shared__ float decay_s;
+    // a decay near one acts on a state hundreds of times in a row: its last bit is worth an exponential in double, rounded once
+    if (threadIdx.x == 255) decay_s = (float)exp((double)A[h] * (double)dt);
     for (int i = threadIdx.x; i < V + 2 * N; i += 256) {
         const int c = i < V ? h * V + i : i < V + N ? I + grp * N + (i - V) : I + G * N + grp * N + (i - V - N);
         float a = conv_b[c];
@@ -322,6 +324,7 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(const T* __restrict__ p, 
         sm[i] = i >= V && i < V + N ? a * dt : a;
     }
     __syncthreads();
+    const float decay = decay_s;
     constexpr int U = VEC == 4 ? 8 : 4;                            // state pieces in flight a thread
     for (int cc = col; cc < cols; cc += 256) {
         float acc[VEC], x[VEC];

@@ -385,7 +385,7 @@ class Mamba2(Part):
         self.proj, self.o = pad_rows(tensors.pop("in"), 8), tensors.pop("o")
         self.conv, self.conv_b = tensors.pop("conv").float().contiguous(), tensors.pop("conv.b").float().contiguous()
         self.dt_bias, self.Dv = tensors.pop("dt_bias").float().contiguous(), tensors.pop("D").float().contiguous()
-        self.A = (-torch.exp(tensors.pop("A_log").float())).contiguous()
+        self.A = (-torch.exp(tensors.pop("A_log").double())).float().contiguous()
         self.norm = tensors.pop("norm").float().contiguous()
 
     @property
