@@ -122,12 +122,14 @@ def err(got, want):
 
 
 def assert_close(got, want, tol, what=""):
-    """float32 (tol < 1e-2): every logit within tol of the largest.  bfloat16: the root mean square of every position within tol."""
+    """float32 (tol < 1e-2): every logit within tol of the largest.  bfloat16: the root mean square over the vocabulary within tol at
+    every position and within a fifth of it at the median one (the norms behind the sums pass a rounding on undamped, and the stand-in
+    kernels in bfloat16 show the same largest error at the same position)."""
     if tol < 1e-2:
         assert err(got, want) < tol, (what, err(got, want))
         return
     per = (got - want).pow(2).mean(-1).sqrt() / want.pow(2).mean(-1).sqrt()
-    assert per.max().item() < tol and per.median().item() < tol / 2, (what, per.median().item(), per.max().item())
+    assert per.max().item() < tol and per.median().item() < tol / 5, (what, per.median().item(), per.max().item())
 
 
 def engine(d, page, pages, dtype="float32", device="cpu", max_seqs=4):
@@ -482,3 +484,311 @@ def test_trace_replay_in_process(dirs, tmp_path, monkeypatch, capsys):
     g1 = torch.from_numpy(np.fromfile(os.path.join(tmp_path, "1.f32"), dtype="<f4").reshape(3, -1))
     g2 = torch.from_numpy(np.fromfile(os.path.join(tmp_path, "2.f32"), dtype="<f4").reshape(1, -1))
     assert err(g0, wa[4:5]) < 2e-5 and err(g1, torch.stack([wb[2], wb[5], wa[5]])) < 2e-5 and err(g2, wa[8:9]) < 2e-5
+
+
+# ---------------------------------------------------------------- inputs made so that a fault shows
+def _i32(v, device):
+    return torch.tensor(v, dtype=torch.int32, device=device)
+
+
+def hot_key_case(ops, device, dtype, L, hot, window, keep, page=16, rows=1, H=4, KV=2, D=24, V=24, cap=12.0):
+    """L cached keys over shuffled pages, every one orthogonal to the last query except key `hot`, whose scaled score is 30 before the cap.
+    The last query's weights are then known in closed form: e^(cap tanh(30 / cap)) for `hot` and 1 for every other key it sees.  Pages
+    that hold only keys the window has passed are given to the null page (as the cache manager leaves them), which holds large rows.
+    A key that is lost, one too many at either end, or a cap left out shows in every head."""
+    g = torch.Generator().manual_seed(L * 1000 + hot)
+    keys, vals = torch.randn(L, KV, D, generator=g) * 0.3, torch.randn(L, KV, V, generator=g)
+    target = torch.randn(D, generator=g)
+    target = target / target.norm()
+    keys -= (keys @ target)[..., None] * target
+    keys[hot] += 6.0 * target
+    pages = -(-L // page)
+    order = (torch.randperm(pages, generator=g) + 1).tolist()
+    kc, vc = torch.full((pages + 1, KV, page, D), 50.0), torch.full((pages + 1, KV, page, V), 50.0)
+    for j in range(L):
+        kc[order[j // page], :, j % page], vc[order[j // page], :, j % page] = keys[j], vals[j]
+    first = L - rows                                              # the first query's position
+    table = torch.zeros(2, pages, dtype=torch.int32)
+    for i in range(pages):
+        if i * page < keep or (i + 1) * page > first - window + 1:
+            table[1, i] = order[i]
+    tiles = [(0, r) for r in range(0, rows, 64)] if rows > 1 else []
+    meta = SimpleNamespace(seg_q_start=_i32([0, rows], device), seg_pos0=_i32([first], device), seg_kv_len=_i32([L], device),
+                           table_rows=_i32([1], device), block_table=table.to(device), max_pages=pages, page_size=page,
+                           decode_segs=_i32([0] if rows == 1 else [], device), prefill_tiles=_i32(tiles, device).view(-1, 2), tile=64, max_kv_len=L)
+    q = torch.randn(rows, H, D, generator=g)
+    q[-1] = 10.0 * target                                         # times the scale of 0.5: 5, times the key's 6: a score of 30
+    gate = torch.randn(rows, 3 + H * V + 1, generator=g).to(dtype)
+    out = ops.masked_attention(q.reshape(rows, H * D).to(device, dtype), kc.to(device, dtype), vc.to(device, dtype), meta, H, KV, D, V, 0.5, None,
+                               window, False, softcap=cap, keep_first=keep, gate=gate.to(device)[:, 2:2 + H * V]).float().cpu()[-1].view(H, V)
+    j = torch.arange(L)
+    s = torch.zeros(L, dtype=torch.float64)
+    s[hot] = 30.0 if cap is None else cap * math.tanh(30.0 / cap)
+    s[~((L - 1 - j < window) | (j < keep))] = float("-inf")
+    kvh = torch.arange(H) // (H // KV)
+    want = torch.einsum("j,jhd->hd", torch.softmax(s, -1), vals.double()[:, kvh]) * torch.sigmoid(gate[-1, 2:2 + H * V].double()).view(H, V)
+    return out, want.float()
+
+
+# (L, hot, window, keep): the oldest key inside the window and the newest outside it, the last kept key and the first that is not, a
+# window and kept keys that overlap, touch or leave a gap of one, edges on page borders, everything visible, one key
+HOT = [(90, 53, 37, 5), (90, 52, 37, 5), (90, 4, 37, 5), (90, 5, 37, 5), (90, 0, 37, 5), (90, 89, 37, 5), (90, 26, 64, 16), (90, 25, 64, 16), (90, 15, 64, 16),
+       (90, 16, 64, 17), (90, 60, 30, 60), (90, 59, 30, 60), (90, 59, 30, 59), (90, 30, 100, 4), (40, 20, 20, 19), (40, 19, 20, 19), (40, 3, 1, 0), (40, 39, 1, 0),
+       (17, 0, 17, 0), (18, 0, 17, 0), (1, 0, 4, 2), (3, 0, 1, 2), (130, 64, 66, 0), (130, 63, 66, 0), (200, 70, 20, 100)]
+
+
+@pytest.mark.parametrize("L,hot,window,keep", HOT)
+def test_window_and_kept_edges_on_cpu(L, hot, window, keep):
+    for rows in (1, min(3, L)):
+        out, want = hot_key_case(TorchRefOps(), "cpu", torch.float32, L, hot, window, keep, rows=rows)
+        assert (out - want).abs().max() < 1e-4 * want.abs().max() + 1e-6
+
+
+def remembering_case(ops, device, dtype, cuts, H=2, V=32, N=64, G=1, taps=3):
+    """A state that must remember: token 0 alone writes (its B and x are large), 300 quiet tokens follow, and the last one reads.  The
+    decay is the same at every token, so what is read is known: C . B x dt e^(A dt 300) -- a lost or restarted state, a chunk's decay that
+    is one token off, or a wrong slot shows.  Returns (rows of the last token before the gated norm's scale, the wanted ones)."""
+    g = torch.Generator().manual_seed(5)
+    T, I, C = 301, H * V, H * V + 2 * G * N
+    p = torch.zeros(T, (I + C + H + 7) // 8 * 8)
+    p[:, :I] = 3.0                                                # z: the gate, the same everywhere
+    p[0, I:I + C] = torch.randn(C, generator=g).abs() + 0.5
+    p[T - 1, 2 * I + G * N:2 * I + 2 * G * N] = torch.randn(G * N, generator=g).abs() + 0.5          # C of the last token
+    p[:, I + C:I + C + H] = -5.0                                  # dt before its bias
+    p = p.to(dtype)
+    conv = torch.zeros(C, taps)
+    conv[:, -1] = 1.0                                             # the filter passes the token itself
+    dt_bias, A, Dv = torch.tensor([0.3, 0.5][:H]), torch.tensor([-0.2, -0.6][:H]), torch.zeros(H)
+    norm = torch.ones(I)
+    state = torch.full((2, (H * N * V + (taps - 1) * C + 3) // 4 * 4), 0.0)
+    mv = lambda t: t.to(device)                                   # noqa: E731
+    args = [mv(conv), torch.zeros(C, device=device), taps, mv(dt_bias), mv(A), mv(Dv), H, V, N, G, mv(norm), 1, 1e-12, mv(state)]
+    at = 0
+    for n in cuts:
+        batch = SimpleNamespace(num_segs=1, host={"seg_q_start": [0, n], "seg_slot": [1]}, seg_q_start=_i32([0, n], device), seg_slot=_i32([1], device), token_seg=_i32([0] * n, device),
+                                positions=_i32(list(range(at, at + n)), device))
+        out = ops.mamba2_mix(p[at:at + n].to(device), *args, batch)
+        at += n
+    assert at == T
+    dt = torch.nn.functional.softplus(p[0, I + C:I + C + H].double() + dt_bias.double())
+    silu = lambda t: torch.nn.functional.silu(t.double())         # noqa: E731
+    x0, B0 = silu(p[0, I:2 * I]).view(H, V), silu(p[0, 2 * I:2 * I + N])
+    CT = silu(p[T - 1, 2 * I + N:2 * I + 2 * N])
+    y = (torch.exp(A.double() * dt * 300) * dt * (B0 @ CT))[:, None] * x0
+    y = (y * silu(p[T - 1, :1])).reshape(-1)
+    return out[-1].float().cpu(), (y / y.pow(2).mean().sqrt()).float(), args[-1][1].float().cpu()
+
+
+CUTS_301 = [[301], [300, 1], [1] * 301, [64, 64, 64, 64, 45], [2, 63, 65, 1, 1, 2, 100, 67], [299, 2]]
+
+
+@pytest.mark.parametrize("cuts", CUTS_301, ids=lambda c: f"{len(c)}cuts")
+def test_a_state_that_must_remember_on_cpu(cuts):
+    out, want, _ = remembering_case(TorchRefOps(), "cpu", torch.float32, cuts)
+    assert (out - want).abs().max() < 1e-4 * want.abs().max()
+
+
+# ================================================================ on the GPU
+TOL = {"float32": 1e-4, "bfloat16": 0.15}
+
+
+def cuda_ops():
+    from mini_inference_b200.ops import get_ops
+    return get_ops("cuda:0")
+
+
+@gpu
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", sorted(CONFIGS))
+def test_cuts_on_gpu(dirs, name, dtype):
+    d, cfg, page = dirs[name]
+    check_cuts(engine(d, page, 40, dtype, "cuda:0"), d, cfg["vocab"], TOL[dtype])
+    cuda_ops().check_errors()
+
+
+@gpu
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", ["mix", "pages"])
+def test_mixed_batches_on_gpu(dirs, name, dtype):
+    d, cfg, page = dirs[name]
+    check_mixed(lambda pages: engine(d, page, pages, dtype, "cuda:0"), d, cfg["vocab"], page, TOL[dtype])
+    cuda_ops().check_errors()
+
+
+@gpu
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+@pytest.mark.parametrize("name", sorted(SINGLE))
+def test_each_mechanism_alone_on_gpu(tmp_path, name, dtype):
+    cfg = SINGLE[name]
+    d = single_dir(tmp_path, name)
+    ids = tokens(cfg["vocab"], 150, seed=1)
+    want = plain_logits(d, ids)
+    runner = engine(d, 16, 16, dtype, "cuda:0")
+    assert_close(feed(runner, "w", ids, [150]), want, TOL[dtype], "whole")
+    assert_close(feed(runner, "d", ids, [110] + [1] * 40), want, TOL[dtype], "decode")
+    assert_close(feed(runner, "p", ids, [2, 64, 3, 17, 2, 33, 29]), want, TOL[dtype], "portions")
+    cuda_ops().check_errors()
+
+
+@gpu
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("L,hot,window,keep", HOT + [(1500, 1363, 137, 20), (1500, 1362, 137, 20), (1500, 19, 137, 20), (1500, 20, 137, 20), (1500, 475, 1025, 3)])
+def test_window_and_kept_edges_on_gpu(L, hot, window, keep, dtype):
+    ops = cuda_ops()
+    for D, V in ((24, 24), (64, 64), (40, 12), (128, 128)):
+        for rows in (1, 3, 70):
+            for splits in (None, 3):
+                ops.force_splits = splits
+                try:
+                    out, want = hot_key_case(ops, "cuda:0", dtype, L, hot, window, keep, rows=min(rows, L), D=D, V=V)
+                finally:
+                    ops.force_splits = None
+                assert (out - want).abs().max() < (1e-4 if dtype == torch.float32 else 2e-2) * want.abs().max() + 1e-6, (D, V, rows, splits)
+    ops.check_errors()
+
+
+@gpu
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+@pytest.mark.parametrize("cuts", CUTS_301, ids=lambda c: f"{len(c)}cuts")
+def test_a_state_that_must_remember_on_gpu(cuts, dtype):
+    ops = cuda_ops()
+    for V, N in ((32, 64), (64, 128), (6, 20)):
+        for chunked in (True, False):
+            ops.chunked_scan = chunked
+            try:
+                out, want, state = remembering_case(ops, "cuda:0", dtype, cuts, V=V, N=N)
+            finally:
+                ops.chunked_scan = True
+            assert (out - want).abs().max() < (1e-4 if dtype == torch.float32 else 2e-2) * want.abs().max(), (V, N, chunked)
+            ref = remembering_case(TorchRefOps(), "cpu", dtype, [301], V=V, N=N)[2]
+            assert (state - ref).abs().max() < (1e-4 if dtype == torch.float32 else 2e-3) * ref.abs().max(), (V, N, chunked)
+    ops.check_errors()
+
+
+@gpu
+@pytest.mark.parametrize("lens,starts", [([1, 23, 6, 2], [40, 0, 100, 0]), ([300, 1, 59, 2, 130], [0, 7, 300, 3, 0]), ([1, 1, 1], [5, 0, 62]), ([700], [11])])
+@pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
+def test_kernels_against_the_stand_ins(dtype, lens, starts):
+    """Every kernel the design added, alone, at sizes no model above has (odd ones too), several entries of unequal length in one launch,
+    states and histories that earlier steps left, against the plain PyTorch statement of the same op."""
+    ops, ref, dev = cuda_ops(), TorchRefOps(), "cuda:0"
+    g = torch.Generator().manual_seed(0)
+    tol = 3e-5 if dtype == torch.float32 else 2e-2
+    rnd = lambda *s: torch.randn(*s, generator=g).to(dtype)      # noqa: E731
+    f32 = lambda *s: torch.randn(*s, generator=g)                # noqa: E731
+    close = lambda a, b, t=tol: (a.float().cpu() - b.float().cpu()).abs().max() <= t * max(1.0, b.float().abs().max().item())  # noqa: E731
+    T, S = sum(lens), len(lens)
+    pos = [p0 + i for p0, ln in zip(starts, lens) for i in range(ln)]
+    starts_q = [sum(lens[:i]) for i in range(S + 1)]
+    slots_of = random.Random(1).sample(range(1, S + 3), S)
+    def batch(device):
+        return SimpleNamespace(num_segs=S, host={"seg_q_start": starts_q, "seg_slot": slots_of}, seg_q_start=_i32(starts_q, device), seg_slot=_i32(slots_of, device), positions=_i32(pos, device),
+                               token_seg=_i32([i for i, n in enumerate(lens) for _ in range(n)], device))
+    cpu, gpu_b = batch("cpu"), batch(dev)
+    for hid in (77, 192, 1030, 2052, 9000):
+        x, y, w = f32(T, hid), rnd(T, hid), f32(hid)
+        xa, xb = x.clone().to(dev), x.clone()
+        ra, rb = ops.sum_rmsnorm(xa, y.to(dev), w.to(dev), 1.75, 1e-5, dtype), ref.sum_rmsnorm(xb, y, w, 1.75, 1e-5, dtype)
+        assert close(xa, xb, 3e-5 if dtype == torch.float32 else 1e-4) and close(ra, rb) and ra.dtype == dtype
+    page = 16
+    cache_slots = (torch.randperm(2 * T, generator=g)[:T] + page).to(torch.int32)
+    n_pages = 2 * T // page + 2
+    for H, KV, D, V, taps, nf in ((6, 2, 8, 24, 4, 3), (3, 1, 7, 5, 3, 2), (4, 4, 16, 16, 2, 8), (5, 0, 24, 24, 4, 12), (4, 2, 64, 64, 1, 16), (2, 1, 10, 10, 5, 0),
+                                  (32, 4, 128, 128, 4, 32), (40, 2, 128, 64, 3, 64)):
+        C = H * D + KV * (D + V)
+        p, bias, conv = rnd(T, (C + 11 + 7) // 8 * 8), f32(C), rnd(C, taps)
+        qn, kn, inv = f32(H * D), f32(KV * D) if KV else None, torch.rand(nf, generator=g)
+        state = f32(S + 3, max((taps - 1) * C, 1))
+        ka, va = torch.zeros(n_pages, max(KV, 1), page, D, dtype=dtype), torch.zeros(n_pages, max(KV, 1), page, V, dtype=dtype)
+        kb, vb, sa, sb = ka.to(dev), va.to(dev), state.clone(), state.to(dev)
+        mv = lambda t: None if t is None else t.to(dev)          # noqa: E731
+        want = ref.conv_qkv_cache(p, H, KV, D, V, bias, conv, taps, qn, kn, 1e-5, inv, sa, cpu, SimpleNamespace(slots=cache_slots, page_size=page), ka, va)
+        got = ops.conv_qkv_cache(p.to(dev), H, KV, D, V, mv(bias), mv(conv), taps, mv(qn), mv(kn), 1e-5, mv(inv), sb, gpu_b,
+                                 SimpleNamespace(slots=cache_slots.to(dev), page_size=page), kb, vb)
+        assert close(got, want) and close(kb, ka) and close(vb, va) and close(sb, sa, 1e-6), (H, KV, D, V, taps)
+    for H, V, N, G, taps, parts in ((4, 6, 10, 2, 4, 3), (3, 5, 7, 1, 3, 1), (2, 32, 64, 2, 4, 2), (4, 64, 128, 2, 3, 4), (2, 96, 64, 1, 2, 1), (1, 33, 24, 1, 1, 1), (6, 8, 200, 3, 5, 2)):
+        I, C = H * V, H * V + 2 * G * N
+        p = rnd(T, (I + C + H + 7) // 8 * 8)
+        conv, cb, dtb, A, Dv, norm = f32(C, taps) * 0.5, f32(C) * 0.3, f32(H) - 2.0, -torch.exp(f32(H) - 1.0), f32(H), f32(I)
+        state = f32(S + 3, (H * N * V + (taps - 1) * C + 3) // 4 * 4)
+        sa = state.clone()
+        want = ref.mamba2_mix(p, conv, cb, taps, dtb, A, Dv, H, V, N, G, norm, parts, 1e-5, sa, cpu)
+        for chunked in (True, False):
+            ops.chunked_scan, sb = chunked, state.to(dev)
+            try:
+                got = ops.mamba2_mix(p.to(dev), conv.to(dev), cb.to(dev), taps, dtb.to(dev), A.to(dev), Dv.to(dev), H, V, N, G, norm.to(dev), parts, 1e-5, sb, gpu_b)
+            finally:
+                ops.chunked_scan = True
+            assert close(got, want) and close(sb, sa, 1e-4 if dtype == torch.float32 else 5e-3), (H, V, N, G, taps, parts, chunked)
+    ops.check_errors()
+
+
+def plain_judged(d, prompts, got):
+    """Generated tokens judged by the plain logits: each is within a rounding's reach of the largest."""
+    for p, out in zip(prompts, got):
+        logits = plain_logits(d, p + out)
+        for i, tok in enumerate(out):
+            row = logits[len(p) + i - 1]
+            assert row[tok] >= row.max() - 0.1 * row.abs().max()
+
+
+@gpu
+@pytest.mark.parametrize("graphs", [False, True])
+@pytest.mark.parametrize("name", ["mix", "pages"])
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_generate_through_the_entry_point_on_gpu(dirs, dtype, name, graphs):
+    d, cfg, page = dirs[name]
+    prompts = [tokens(cfg["vocab"], n, seed=40 + n) for n in (5, 13, 22, 9, 3, 30)]
+    llm = LLM(d, dtype=dtype, kv_block_size=page, kv_cache_tokens=1024, max_num_seqs=4, cuda_graphs=graphs)
+    got = llm.generate(prompts, SamplingParams(max_new_tokens=12, ignore_eos=True))
+    assert llm.cache.free_pages() == llm.cache.num_pages
+    if graphs:
+        assert llm.graphs.replays > 0
+    if dtype == "float32":
+        assert got == [plain_greedy(d, p, 12) for p in prompts]
+    else:
+        plain_judged(d, prompts, got)
+
+
+@gpu
+def test_long_decoding_on_gpu(dirs):
+    """300 tokens generated one by one after a short prompt, through the scheduler: pages fill, the windows' pages are given back and taken
+    again, the kept ones stay, and the plain implementation agrees on the whole sequence at the end."""
+    d, cfg, page = dirs["pages"]
+    prompt = tokens(cfg["vocab"], 11, seed=77)
+    llm = LLM(d, dtype="float32", kv_block_size=page, kv_cache_tokens=512, max_num_seqs=2)
+    out = llm.generate([prompt], SamplingParams(max_new_tokens=300, ignore_eos=True))[0]
+    logits = plain_logits(d, prompt + out)
+    picks = logits[len(prompt) - 1:-1].argmax(-1).tolist()
+    assert sum(a == b for a, b in zip(picks, out)) >= 297          # a near tie may fall the other way; it does not derail the rest
+
+
+@gpu
+def test_trace_run_program_on_gpu(dirs, tmp_path):
+    d, cfg, page = dirs["pages"]
+    a = tokens(cfg["vocab"], 70, seed=5)
+    steps = [{"step": 0, "entries": [{"id": "a", "tokens": a[:64], "want": list(range(64))}], "end": []},
+             {"step": 1, "entries": [{"id": "a", "tokens": a[64:], "want": list(range(6))}], "end": ["a"]}]
+    for dtype in ("float32", "bfloat16"):
+        out = tmp_path / dtype
+        r = subprocess.run([os.path.join(ROOT, "bin", "trace_run"), "--model", d, "--dtype", dtype, "--out", str(out), "--max-tokens", "128"],
+                           input="\n".join(json.dumps(s) for s in steps) + "\n", capture_output=True, text=True, timeout=600)
+        assert r.returncode == 0, r.stderr[-2000:]
+        want = plain_logits(d, a)
+        g0 = torch.from_numpy(np.fromfile(out / "0.f32", dtype="<f4").reshape(64, -1))
+        g1 = torch.from_numpy(np.fromfile(out / "1.f32", dtype="<f4").reshape(6, -1))
+        assert_close(torch.cat([g0, g1]), want, TOL[dtype])
+
+
+@gpu
+def test_run_engine_command_line_on_gpu(dirs, tmp_path):
+    """The serving command line on a model folder of this design: the scheduler, temperature sampling and CUDA graphs."""
+    d, cfg, page = dirs["mix"]
+    out = tmp_path / "m.json"
+    r = subprocess.run([os.path.join(ROOT, "bin", "run_engine"), "--model", d, "--dtype", "bfloat16", "-n", "5", "-c", "3", "--warmup", "1",
+                        "--max-new-tokens", "9", "--prompt-len", "5:30", "--kv-tokens", "512", "--page-size", str(page), "--temperature", "0.8",
+                        "--cuda-graphs", "on", "--out", str(out)], capture_output=True, text=True, timeout=600)
+    assert r.returncode == 0, r.stderr[-2000:]
+    data = json.loads(out.read_text())
+    assert data["summary"]["engine"]["architecture"] == "Fetodra"
+    assert all(run["generated_tokens"] == 9 and run["error"] is None for run in data["runs"])
