@@ -826,15 +826,164 @@ def bench_megovik(args, ops, peak, out=print):
     return rows
 
 
+FETODRA_SIZES = {
+    # the widths, heads and dense feed-forwards of NAMESUN_SIZES; Mamba-2 with an inner size of twice the width, heads of 64, states of 128
+    "2k": dict(width=2048, ff=8192, heads=16, kv_heads=8, dim=128, window=1024, keep=4, m_heads=64, m_vdim=64, state=128),
+    "4k": dict(width=4096, ff=12288, heads=32, kv_heads=8, dim=128, window=1024, keep=4, m_heads=128, m_vdim=64, state=128),
+}
+
+
+def fetodra_config(size, layers, vocab=65536):
+    z = FETODRA_SIZES[size]
+    dense = {"kind": "dense", "ff": z["ff"], "limit": 7.0}
+    att = {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["dim"], "conv": 4, "scale": z["dim"] ** -0.5, "softcap": 30.0,
+           "rot": {"dims": 64, "base": 1e6}, "mask": {"size": z["window"], "keep_first": z["keep"]}}
+    ssm = {"heads": z["m_heads"], "vdim": z["m_vdim"], "state": z["state"], "groups": 1, "norm_groups": 1, "conv": 4}
+    out = []
+    for i in range(layers):                                      # own keys, own keys, state space without feed-forward, the keys of the second
+        out.append({"type": "mamba2", "mixer": ssm, "mlp": None} if i % 4 == 2 else
+                   {"type": "attention", "mixer": dict(att, kv_from=i - 2) if i % 4 == 3 else att, "mlp": dense})
+    return {"architecture": "Fetodra", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6}, "postln_alpha": 2.0, "layers": out}
+
+
+def namesun_config_like_fetodra(size, layers, vocab=65536):
+    """Namesun (float32 stream, masked attention, a scanned state, norms behind the sublayers) of the same width, depth, vocabulary, attention
+    heads and dense feed-forwards, its retention where Fetodra has its state space: the closest design the engine already serves."""
+    cfg, z = namesun_config(size, layers, vocab), FETODRA_SIZES[size]
+    pattern = namesun_config(size, 4, vocab)["layers"]
+    dense = {"kind": "dense", "ff": z["ff"]}
+    cfg["layers"] = [dict(pattern[0], mlp=None) if i % 4 == 2 else dict(pattern[2], mlp=dense) for i in range(layers)]
+    return cfg
+
+
+def bench_fetodra(args, ops, peak, out=print):
+    """Each kernel that the Fetodra design added or widened, at the layer sizes of --design-size, beside the like kernel of Namesun, with the
+    bytes or operations it cannot avoid as a share of its bound: the measured copy bandwidth, the measured bf16 peak, or (token-by-token
+    scans) the float32 FMA rate of the CUDA cores."""
+    import numpy as np
+    z = FETODRA_SIZES[args.design_size]
+    here = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+    bf16_peak = 1590.0
+    if os.path.isfile(os.path.join(here, "MEASURED_PEAKS.json")):
+        with open(os.path.join(here, "MEASURED_PEAKS.json")) as f:
+            bf16_peak = json.load(f)["bf16_tflops"]
+    fma_peak = ops.NUM_SMS * 128 * 2 * 1.965e9 / 1e12
+    rows = []
+
+    def line(kernel, shape, us, amount, bound):
+        got, top, unit = {"hbm": (amount / us / 1e3, peak, "GB/s"), "bf16": (amount / us / 1e6, bf16_peak, "TFLOP/s"),
+                          "fma": (amount / us / 1e6, fma_peak, "TF(f32)")}[bound]
+        rows.append({"kernel": kernel, "shape": shape, "us": round(us, 2), "achieved": round(got, 2), "unit": unit, "frac": round(got / top, 3)})
+        out(f"{kernel:52s} {shape:46s} {us:9.2f} us {got:9.2f} {unit:10s} {100 * got / top:5.1f} % of bound", flush=True)
+
+    t = lambda a: torch.tensor(np.asarray(a, dtype=np.int32), device="cuda")       # noqa: E731
+    bf = torch.bfloat16
+    W, T, it = z["width"], args.tokens, args.iters
+    rb = lambda *s: torch.randn(*s, device="cuda", dtype=bf)                       # noqa: E731
+    rf = lambda *s: torch.randn(*s, device="cuda")                                 # noqa: E731
+    for n in (T, 64, 8):
+        reps = 4 if n > 64 else 2
+        x, a, wn = rf(reps, n, W), rb(reps, n, W), torch.ones(W, device="cuda")
+        us = timed(lambda i: ops.sum_rmsnorm(x[i % reps], a[i % reps], wn, 2.0, 1e-6, bf), it)
+        line("norm behind the sum (f32 stream)", f"T={n} width={W}", us, n * W * 12.0, "hbm")
+        us = timed(lambda i: ops.out_rmsnorm_add(x[i % reps], a[i % reps], wn, wn, 0.3, 1e-6, bf), it)
+        line("  Namesun: output norm + add (f32 stream)", f"T={n} width={W}", us, n * W * 12.0, "hbm")
+    F = z["ff"]
+    gu = rb(2, T, 2 * F)
+    us = timed(lambda i: ops.clamped_glu(gu[i % 2], 7.0, 1.702), it)
+    line("clamped gate (Namesun's kernel)", f"T={T} ff={F}", us, T * F * 6.0, "hbm")
+    del gu
+    # ---- attention: filter, norm, rotation and cache write; capped windowed attention with kept keys and a gate
+    H, KV, D, page, taps, win, keep = z["heads"], z["kv_heads"], z["dim"], 16, 4, z["window"], z["keep"]
+    C = (H + 2 * KV) * D
+    bias, conv, qn, kn, inv = rf(C), rb(C, taps), rf(H * D), rf(KV * D), torch.full((32,), 0.01, device="cuda")
+    for B, n, ctx in ((1, T, T), (8, 1, args.ctx), (64, 1, args.ctx)):
+        pages_per = -(-ctx // page)
+        n_pages = B * pages_per + 1
+        kc, vc = rb(n_pages, KV, page, D), rb(n_pages, KV, page, D)
+        tiles = [(s, r) for s in range(B) for r in range(0, n, 64)] if n > 1 else []
+        meta = types.SimpleNamespace(seg_q_start=t(np.arange(B + 1) * n), seg_pos0=t([ctx - n] * B), seg_kv_len=t([ctx] * B), table_rows=t(np.arange(B)),
+                                     block_table=t(np.arange(1, n_pages).reshape(B, pages_per)), max_pages=pages_per, page_size=page,
+                                     decode_segs=t(np.arange(B) if n == 1 else []), prefill_tiles=t(tiles).view(-1, 2), tile=64, max_kv_len=ctx,
+                                     slots=t((np.arange(B)[:, None] * pages_per * page + page + ctx - n + np.arange(n)[None, :]).reshape(-1)),
+                                     positions=t(np.tile(np.arange(ctx - n, ctx), B)), token_seg=t(np.repeat(np.arange(B), n)), seg_slot=t(np.arange(B) + 1),
+                                     num_segs=B)
+        Tn, reps = B * n, 3
+        state = torch.zeros(B + 1, (taps - 1) * C, device="cuda")
+        p, p3 = rb(reps, Tn, C + H * D), rb(Tn, C)
+        moved = Tn * C * 4.0 + (B * (taps - 1) * C * 8.0 if n == 1 else 0.0)          # rows in and out; a decode step's filter inputs in and out
+        us = timed(lambda i: ops.conv_qkv_cache(p[i % reps], H, KV, D, D, bias, conv, taps, qn, kn, 1e-6, inv, state, meta, meta, kc, vc), it)
+        line("filter, norm, rotation, k and v -> pools", f"rows={Tn} H={H} KV={KV} D={D} taps={taps}", us, moved, "hbm")
+        us = timed(lambda i: ops.unit_qk_cache(p3, H, KV, D, D, 1e-6, None, None, meta, kc, vc), it)
+        line("  Namesun: unit q/k, k and v -> pools", f"rows={Tn} H={H} KV={KV} D={D}", us, Tn * C * 4.0, "hbm")
+        q, gate = p3[:, :H * D], p[0][:, C:]
+        pairs = sum(min(i + 1, win) + max(0, min(keep, i + 1 - win)) for i in range(n))
+        pairs_b = sum(i % win + 1 for i in range(n))
+        kv_bytes = lambda k: B * k * KV * D * 2 * 2.0             # noqa: E731
+        amount, bound = (4.0 * H * D * pairs * B, "bf16") if n > 1 else (kv_bytes(min(ctx, win + keep)), "hbm")
+        us = timed(lambda i: ops.masked_attention(q, kc, vc, meta, H, KV, D, D, D ** -0.5, None, win, False, softcap=30.0, keep_first=keep, gate=gate), it)
+        line("attention: window, kept keys, cap, gate", f"B={B} rows={n} ctx={ctx} window={win}+{keep} H={H}/{KV}", us, amount, bound)
+        us = timed(lambda i: ops.masked_attention(q, kc, vc, meta, H, KV, D, D, D ** -0.5, None, win, False, keep_first=keep, gate=gate), it)
+        line("  the same without the cap", f"B={B} rows={n} ctx={ctx} window={win}+{keep} H={H}/{KV}", us, amount, bound)
+        amount, bound = (4.0 * H * D * pairs_b * B, "bf16") if n > 1 else (kv_bytes((ctx - 1) % win + 1), "hbm")
+        us = timed(lambda i: ops.masked_attention(q, kc, vc, meta, H, KV, D, D, D ** -0.5, win, None, True), it)
+        line("  Namesun: attention in blocks, sink", f"B={B} rows={n} ctx={ctx} block={win} H={H}/{KV}", us, amount, bound)
+        del kc, vc
+    # ---- Mamba-2 beside retention
+    MH, V, N = z["m_heads"], z["m_vdim"], z["state"]
+    I, C = MH * V, MH * V + 2 * N
+    ns = NAMESUN_SIZES[args.design_size]
+    RH, RD, RV = ns["heads"], ns["dim"], ns["vdim"]
+    decay, rinv = torch.full((RH,), 0.99, device="cuda"), torch.full((RD // 2,), 0.01, device="cuda")
+    conv, cb, dtb, A, Dv, norm = rf(C, taps) * 0.5, rf(C), rf(MH) - 3.0, -torch.rand(MH, device="cuda"), rf(MH), torch.ones(I, device="cuda")
+    for B, n in ((1, T), (8, 1), (64, 1)):
+        Tn = B * n
+        reps = 1 if n > 1 else max(2, (300 << 20) // (B * MH * N * V * 4) + 1)        # decode: states rotated through more than the L2 holds
+        batch = types.SimpleNamespace(num_segs=B, seg_q_start=t(np.arange(B + 1) * n), seg_slot=t(np.arange(B) + 1), positions=t(np.tile(np.arange(n), B)),
+                                      token_seg=t(np.repeat(np.arange(B), n)))
+        state = torch.zeros(reps, B + 1, MH * N * V + (taps - 1) * C, device="cuda")
+        p = rb(2, Tn, (I + C + MH + 7) // 8 * 8)
+        us = timed(lambda i: ops.mamba2_mix(p[i % 2], conv, cb, taps, dtb, A, Dv, MH, V, N, 1, norm, 1, 1e-6, state[i % reps], batch), it)
+        shape = f"{'prompt' if n > 1 else 'decode'} B={B} T={n} heads={MH} {N}x{V}"
+        if n > 1:
+            line("Mamba-2: filter, scan, gated norm", shape, us, 4.0 * I * N * Tn, "fma")
+            xbc = rb(Tn, C)
+            dt = p[0][:, I + C:I + C + MH]
+            us = timed(lambda i: ops.short_conv(p[i % 2][:, I:I + C], conv, cb, taps, state[0], MH * N * V, batch, act="silu"), it)
+            line("  its filter", shape, us, Tn * C * 4.0, "hbm")
+            us = timed(lambda i: ops.state_space_scan(xbc, dt, dtb, A, MH, V, N, 1, state[0], batch), it)
+            line("  its scan in chunks on the tensor cores", shape, us, 4.0 * I * N * Tn, "fma")
+            line("  (the same against the bytes it moves)", shape, us, Tn * C * 2.0 + Tn * I * 4.0 + 2.0 * B * MH * N * V * 4, "hbm")
+            ops.chunked_scan = False
+            us = timed(lambda i: ops.mamba2_mix(p[i % 2], conv, cb, taps, dtb, A, Dv, MH, V, N, 1, norm, 1, 1e-6, state[0], batch), it)
+            ops.chunked_scan = True
+            line("  (filter, token-by-token scan, gated norm)", shape, us, 4.0 * I * N * Tn, "fma")
+        else:
+            line("Mamba-2: filter, state, gated norm", shape, us, 2.0 * B * (MH * N * V + (taps - 1) * C) * 4 + Tn * (2 * I + C) * 2.0, "hbm")
+        rreps = 1 if n > 1 else max(2, (300 << 20) // (B * RH * RD * RV * 4) + 1)
+        rstate = torch.zeros(rreps, B + 1, RH * RD * RV, device="cuda")
+        rp = rb(Tn, 2 * RH * RD + 2 * RH * RV)
+        us = timed(lambda i: ops.retention_scan(rp, RH, RD, RV, rinv, 0.1, decay, rstate[i % rreps], batch), it)
+        shape = f"{'prompt' if n > 1 else 'decode'} B={B} T={n} heads={RH} {RD}x{RV}"
+        if n > 1:
+            line("  Namesun: retention (rotation + scan)", shape, us, 4.0 * RH * RD * RV * Tn, "fma")
+        else:
+            line("  Namesun: retention (rotation + scan)", shape, us, 2.0 * B * RH * RD * RV * 4, "hbm")
+        del state, rstate
+    ops.check_errors()
+    return rows
+
+
 DESIGNS = {"naditar": (naditar_config, qwen3_config_like, bench_design), "namesun": (namesun_config, qwen3_config_like_namesun, bench_namesun),
            "nununex": (nununex_config, namesun_config_like_nununex, bench_nununex),
-           "megovik": (megovik_config, namesun_config_like_megovik, bench_megovik)}
-BESIDE = {"nununex": "namesun", "megovik": "namesun"}            # the design an entry of DESIGNS is set beside (default: qwen3)
+           "megovik": (megovik_config, namesun_config_like_megovik, bench_megovik),
+           "fetodra": (fetodra_config, namesun_config_like_fetodra, bench_fetodra)}
+BESIDE = {"nununex": "namesun", "megovik": "namesun", "fetodra": "namesun"}            # the design an entry of DESIGNS is set beside (default: qwen3)
 
 
 def main(argv=None):
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
-    ap.add_argument("what", choices=["gemm", "attention", "prefill", "design", "namesun", "nununex", "megovik"])
+    ap.add_argument("what", choices=["gemm", "attention", "prefill", "design", "namesun", "nununex", "megovik", "fetodra"])
     ap.add_argument("--design-size", default="2k", choices=sorted(NADITAR_SIZES), help="design: layer sizes of the Naditar kernels")
     ap.add_argument("--size", default="4b", choices=sorted(SIZES))
     ap.add_argument("--rows", default="1,8,64", type=lambda s: [int(v) for v in s.split(",")])
@@ -853,7 +1002,7 @@ def main(argv=None):
     ops = get_ops("cuda:0")
     peak, src = peak_gbs()
     print(f"# peak {peak} GB/s ({src})")
-    {"gemm": bench_gemm, "attention": bench_attention, "prefill": bench_prefill_attention, "design": bench_design, "namesun": bench_namesun, "nununex": bench_nununex, "megovik": bench_megovik}[args.what](args, ops, peak)
+    {"gemm": bench_gemm, "attention": bench_attention, "prefill": bench_prefill_attention, "design": bench_design, "namesun": bench_namesun, "nununex": bench_nununex, "megovik": bench_megovik, "fetodra": bench_fetodra}[args.what](args, ops, peak)
     return 0
 
 

@@ -1324,10 +1324,10 @@ class CudaOps:
         T, I = p.shape[0], H * V
         C, off, dev = I + 2 * G * N, H * N * V, p.device
         assert p.stride(1) == 1 and p.shape[1] >= I + C + H and state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] >= off + (taps - 1) * C
-        y = torch.empty((T, I), dtype=torch.float32, device=dev)
         rows = torch.empty((T, I), dtype=p.dtype, device=dev)
         code, stride = _code(p.dtype), _c.c_longlong(state.stride(0))
         if T == batch.num_segs:                             # every entry brings one token
+            y = torch.empty((T, I), dtype=torch.float32, device=dev)
             _check(self.lib.mi_ssd_step(_p(p), p.stride(0), _p(conv), _p(conv_b), taps, _p(dt_bias), _p(A), _p(Dv), _p(state), stride, _p(y),
                                         _p(batch.seg_q_start), _p(batch.seg_slot), batch.num_segs, H, V, N, G, code, self._stream()), "ssd_step")
             _check(self.lib.mi_gated_part_norm(_p(y), _p(None), 0, _p(None), V, _p(p), p.stride(0), _p(norm), _p(rows), T, I, parts, _c.c_float(eps),
@@ -1336,23 +1336,34 @@ class CudaOps:
             return rows
         xbc = self.short_conv(p[:, I:I + C], conv, conv_b, taps, state, off, batch, act="silu")
         dt = p[:, I + C:I + C + H]
-        rc = -2
-        if p.dtype == torch.bfloat16 and self.chunked_scan:
-            rc = self.lib.mi_ssd_chunk(_p(xbc), xbc.stride(0), _p(dt), dt.stride(0), _p(dt_bias), _p(A), _p(state), stride, _p(y), _p(batch.seg_q_start),
-                                       _p(batch.seg_slot), T, batch.num_segs, H, V, N, G, self._stream())
-            if rc != -2:
-                _check(rc, "ssd_chunk")
-                self.launches += 1
-        if rc == -2:                                        # float32, or a size without a chunked form: the token-by-token scan
-            prep = torch.empty((T, (2 * G * N + I + H + 3) // 4 * 4), dtype=torch.float32, device=dev)
-            _check(self.lib.mi_state_space_scan(_p(xbc), xbc.stride(0), _p(dt), dt.stride(0), _p(dt_bias), _p(A), _p(prep), prep.stride(0), _p(state), stride,
-                                                _p(y), _p(batch.seg_q_start), _p(batch.seg_slot), T, batch.num_segs, H, V, N, G, code, self._stream()),
-                   "state_space_scan")
-            self.launches += 2
+        y = self.state_space_scan(xbc, dt, dt_bias, A, H, V, N, G, state, batch)
         _check(self.lib.mi_gated_part_norm(_p(y), _p(xbc), xbc.stride(0), _p(Dv), V, _p(p), p.stride(0), _p(norm), _p(rows), T, I, parts, _c.c_float(eps),
                                            _p(None), _c.c_longlong(0), _c.c_longlong(0), _p(None), 0, 1, code, self._stream()), "gated_part_norm")
         self.launches += 1
         return rows
+
+    def state_space_scan(self, xbc, dt, dt_bias, A, H, V, N, G, state, batch):
+        """S <- e^(A step) S + step B x^T, step = softplus(dt + dt_bias), y = S^T C per head; xbc [T, H V + 2 G N] = x | B | C contiguous, dt
+        [T, H] a strided view in the same dtype; the slot's first H N V floats are S.  Returns float32 [T, H V].  bfloat16: chunks of 64
+        tokens on the tensor cores where the sizes have that form; otherwise token by token in float32."""
+        T, I = xbc.shape[0], H * V
+        assert xbc.is_contiguous() and dt.stride(1) == 1 and dt.dtype == xbc.dtype and state.dtype == torch.float32 and state.is_contiguous()
+        y = torch.empty((T, I), dtype=torch.float32, device=xbc.device)
+        stride = _c.c_longlong(state.stride(0))
+        if xbc.dtype == torch.bfloat16 and self.chunked_scan:
+            rc = self.lib.mi_ssd_chunk(_p(xbc), xbc.stride(0), _p(dt), dt.stride(0), _p(dt_bias), _p(A), _p(state), stride, _p(y), _p(batch.seg_q_start),
+                                       _p(batch.seg_slot), T, batch.num_segs, H, V, N, G, self._stream())
+            if rc == 0:
+                self.launches += 1
+                return y
+            if rc != -2:
+                _check(rc, "ssd_chunk")
+        prep = torch.empty((T, (2 * G * N + I + H + 3) // 4 * 4), dtype=torch.float32, device=xbc.device)
+        _check(self.lib.mi_state_space_scan(_p(xbc), xbc.stride(0), _p(dt), dt.stride(0), _p(dt_bias), _p(A), _p(prep), prep.stride(0), _p(state), stride,
+                                            _p(y), _p(batch.seg_q_start), _p(batch.seg_slot), T, batch.num_segs, H, V, N, G, _code(xbc.dtype), self._stream()),
+               "state_space_scan")
+        self.launches += 2
+        return y
 
     # ---------------------------------------------------------------- sampling
     def argmax(self, logits):
