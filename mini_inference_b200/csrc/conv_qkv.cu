@@ -103,6 +103,15 @@ __global__ void __launch_bounds__(MAXT) conv_qkv_vec_kernel(const __nv_bfloat16*
     const int c0 = kv ? HD : 0, n = kv ? C - HD : HD, normed = kv ? KD : HD;
     const int i0 = threadIdx.x * 8, c = c0 + i0;
     const bool live = i0 < n;
+    // inside one entry, beyond its first taps: all rows that the TOK tokens read are fetched at once (no history, no look-ups between)
+    constexpr int ROWS = TOK + TAPS - 1;
+    const int seg0 = a.token_seg[t0];
+    const bool inside = TOK > 1 && t0 + TOK <= a.T && a.token_seg[min(t0 + TOK, a.T) - 1] == seg0 && t0 - a.seg_q_start[seg0] >= TAPS - 1;
+    uint4 raw[ROWS];
+    if (inside && live) {
+#pragma unroll
+        for (int i = 0; i < ROWS; ++i) raw[i] = *reinterpret_cast<const uint4*>(p + (size_t)(t0 - (TAPS - 1) + i) * ldp + c);
+    }
     for (int i = threadIdx.x; i < TOK * a.nf; i += blockDim.x) {
         const int k = i / a.nf, f = i - k * a.nf;
         sincosf((float)a.positions[min(t0 + k, a.T - 1)] * a.inv_freq[f], &csm[TOK * a.nf + i], &csm[i]);
@@ -124,6 +133,19 @@ __global__ void __launch_bounds__(MAXT) conv_qkv_vec_kernel(const __nv_bfloat16*
             const int at = e * TAPS + j;
             return __uint_as_float(at & 1 ? wr[at >> 1] & 0xffff0000u : wr[at >> 1] << 16);
         };
+        if (inside) {
+#pragma unroll
+            for (int k = 0; k < TOK; ++k)
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) {                 // the order of the general form: per token, taps ascending
+                    const uint32_t q[4] = {raw[k + j].x, raw[k + j].y, raw[k + j].z, raw[k + j].w};
+#pragma unroll
+                    for (int e = 0; e < 8; ++e) {
+                        const float u = __uint_as_float(e & 1 ? q[e >> 1] & 0xffff0000u : q[e >> 1] << 16) + bias[e];
+                        y[k][e] = fmaf(tap(e, j), u, y[k][e]);
+                    }
+                }
+        } else
 #pragma unroll
         for (int k = 0; k < TOK; ++k) {
             const int t = t0 + k;
@@ -149,10 +171,12 @@ __global__ void __launch_bounds__(MAXT) conv_qkv_vec_kernel(const __nv_bfloat16*
                     *reinterpret_cast<float4*>(hw + 4) = make_float4(u[4], u[5], u[6], u[7]);
                 }
             }
-            if (i0 < normed) {
+        }
+        if (i0 < normed) {
+#pragma unroll
+            for (int k = 0; k < TOK; ++k)
 #pragma unroll
                 for (int e = 0; e < 8; ++e) ss[k] += y[k][e] * y[k][e];
-            }
         }
     }
 #pragma unroll

@@ -490,6 +490,35 @@ __global__ void short_conv_vec_kernel(const __nv_bfloat16* __restrict__ h, int l
 #pragma unroll
         for (int e = 0; e < 8; ++e) breg[e] = 0.f;
     }
+    // inside one entry, beyond its first taps: the rows are fetched all at once, so that their latencies overlap
+    constexpr int ROWS = TOK + TAPS - 1;
+    if (t0 + TOK <= T_ && qs_[0] == qs_[TOK - 1] && t0 - qs_[0] >= TAPS - 1) {
+        uint4 raw[ROWS];
+#pragma unroll
+        for (int i = 0; i < ROWS; ++i) raw[i] = *reinterpret_cast<const uint4*>(h + (size_t)(t0 - (TAPS - 1) + i) * ldh + c);
+        auto entry = [&](int i, int e) {
+            const uint32_t w32 = e < 2 ? raw[i].x : e < 4 ? raw[i].y : e < 6 ? raw[i].z : raw[i].w;
+            return __uint_as_float(e & 1 ? w32 & 0xffff0000u : w32 << 16);
+        };
+#pragma unroll
+        for (int k = 0; k < TOK; ++k) {
+            float acc[8];
+#pragma unroll
+            for (int e = 0; e < 8; ++e) {
+                acc[e] = breg[e];
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) acc[e] = fmaf(wreg[e][j], entry(k + j, e), acc[e]);
+                if (act == 1) acc[e] = silu(acc[e]);
+                if (residual) acc[e] += entry(k + TAPS - 1, e);
+            }
+            uint4 o;
+            __nv_bfloat162* oh = reinterpret_cast<__nv_bfloat162*>(&o);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) oh[e] = __floats2bfloat162_rn(acc[2 * e], acc[2 * e + 1]);
+            *reinterpret_cast<uint4*>(out + (size_t)(t0 + k) * C + c) = o;
+        }
+        return;
+    }
 #pragma unroll
     for (int k = 0; k < TOK; ++k) {
         const int t = t0 + k;

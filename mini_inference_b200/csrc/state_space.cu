@@ -293,7 +293,8 @@ __global__ void __launch_bounds__(CH_THREADS, 2) ssd_chunk_kernel(const __nv_bfl
 
 // ------------------------------------------------------------------ decode step
 // grid (entries, heads), every entry brings ONE token.  VEC neighbouring columns a thread; the threads of a block are cols x rows of them.
-template <typename T, int VEC>
+// TAPS: the convolution's taps when known (0: any number), so that a channel's inputs are fetched together.
+template <typename T, int VEC, int TAPS>
 __global__ void __launch_bounds__(256) ssd_step_kernel(const T* __restrict__ p, int ldp, const float* __restrict__ conv, const float* __restrict__ conv_b, int taps,
                                                        const float* __restrict__ dt_bias, const float* __restrict__ A, const float* __restrict__ Dv,
                                                        float* __restrict__ state, long long state_stride, float* __restrict__ out,
@@ -311,40 +312,47 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(const T* __restrict__ p, 
     const int cols = V / VEC, rows = max(1, 256 / cols);
     const int col = threadIdx.x % cols, r0 = threadIdx.x / cols;
     float* S = slot + (long long)h * N * V;
+    constexpr int U = VEC == 4 ? 8 : 4;                            // state pieces in flight a thread
+    float s[U][VEC];
+    auto fetch = [&](int n0, int cc) {
+#pragma unroll
+        for (int u = 0; u < U; ++u) {
+            const int nn = n0 + u * rows;
+            if (nn < N) {
+                if constexpr (VEC == 4) {
+                    const float4 f = *reinterpret_cast<const float4*>(S + (size_t)nn * V + cc * 4);
+                    s[u][0] = f.x; s[u][1] = f.y; s[u][2] = f.z; s[u][3] = f.w;
+                } else {
+                    s[u][0] = S[(size_t)nn * V + cc];
+                }
+            }
+        }
+    };
+    if (r0 < rows) fetch(r0, col);                                 // the first pieces travel while the convolution is made
     const float dt = softplus(to_f32(p[t * ldp + I + C + h]) + dt_bias[h]);
     __shared__ float decay_s;
     // a decay near one acts on a state hundreds of times in a row: its last bit is worth an exponential in double, rounded once
     if (threadIdx.x == 255) decay_s = (float)exp((double)A[h] * (double)dt);
     for (int i = threadIdx.x; i < V + 2 * N; i += 256) {
         const int c = i < V ? h * V + i : i < V + N ? I + grp * N + (i - V) : I + G * N + grp * N + (i - V - N);
+        const int nt = TAPS ? TAPS : taps;
         float a = conv_b[c];
-        for (int j = 0; j + 1 < taps; ++j) a = fmaf(conv[(size_t)c * taps + j], hist[(size_t)j * C + c], a);
-        a = fmaf(conv[(size_t)c * taps + taps - 1], to_f32(row[c]), a);
+        const float own = to_f32(row[c]);
+#pragma unroll
+        for (int j = 0; j + 1 < nt; ++j) a = fmaf(conv[(size_t)c * nt + j], hist[(size_t)j * C + c], a);
+        a = fmaf(conv[(size_t)c * nt + nt - 1], own, a);
         a = round_to<T>(silu(a));
         sm[i] = i >= V && i < V + N ? a * dt : a;
     }
     __syncthreads();
     const float decay = decay_s;
-    constexpr int U = VEC == 4 ? 8 : 4;                            // state pieces in flight a thread
     for (int cc = col; cc < cols; cc += 256) {
         float acc[VEC], x[VEC];
 #pragma unroll
         for (int e = 0; e < VEC; ++e) { acc[e] = 0.f; x[e] = xs[cc * VEC + e]; }
         if (r0 < rows) {
             for (int n0 = r0; n0 < N; n0 += rows * U) {
-                float s[U][VEC];
-#pragma unroll
-                for (int u = 0; u < U; ++u) {
-                    const int nn = n0 + u * rows;
-                    if (nn < N) {
-                        if constexpr (VEC == 4) {
-                            const float4 f = *reinterpret_cast<const float4*>(S + (size_t)nn * V + cc * 4);
-                            s[u][0] = f.x; s[u][1] = f.y; s[u][2] = f.z; s[u][3] = f.w;
-                        } else {
-                            s[u][0] = S[(size_t)nn * V + cc];
-                        }
-                    }
-                }
+                if (n0 != r0 || cc != col) fetch(n0, cc);
 #pragma unroll
                 for (int u = 0; u < U; ++u) {
                     const int nn = n0 + u * rows;
@@ -373,30 +381,32 @@ __global__ void __launch_bounds__(256) ssd_step_kernel(const T* __restrict__ p, 
 }
 
 // ------------------------------------------------------------------ (y + D x) * silu(z), norm in parts, weight
-struct Tail { float* state; long long stride, off; const int* seg_slot; int C, taps; };      // state null: nothing to move
+struct Tail { float* state; long long stride, off; const int* seg_slot; int C, taps, parts; };      // state null: nothing to move
 
 template <typename T>
 __device__ __forceinline__ void shift_inputs(const T* __restrict__ zrow, int I, const Tail& k) {
-    // a step of single tokens: entry == token; the convolution's inputs x | B | C stand behind z in the token's row
+    // a step of single tokens: entry == token; the convolution's inputs x | B | C stand behind z in the token's row.  A block behind the
+    // norm's parts takes blockDim.x channels.
     float* hist = k.state + (long long)k.seg_slot[blockIdx.x] * k.stride + k.off;
-    for (int c = threadIdx.x; c < k.C; c += blockDim.x) {
-        for (int j = 0; j + 2 < k.taps; ++j) hist[(size_t)j * k.C + c] = hist[(size_t)(j + 1) * k.C + c];
-        hist[(size_t)(k.taps - 2) * k.C + c] = to_f32(zrow[I + c]);
-    }
+    const int c = ((int)blockIdx.y - k.parts) * blockDim.x + threadIdx.x;
+    if (c >= k.C) return;
+    const float own = to_f32(zrow[I + c]);
+    for (int j = 0; j + 2 < k.taps; ++j) hist[(size_t)j * k.C + c] = hist[(size_t)(j + 1) * k.C + c];
+    hist[(size_t)(k.taps - 2) * k.C + c] = own;
 }
 
-// grid (tokens, parts).  VPT = 0: any sizes, the values made twice; else 8 VPT neighbouring values a thread, kept in registers.
+// grid (tokens, parts (+ blocks that move the inputs)).  VPT = 0: any sizes, the values made twice; else 8 VPT neighbouring values a thread, kept in registers.
 template <typename T, int VPT>
 __global__ void __launch_bounds__(256) gated_part_norm_kernel(const float* __restrict__ y, const T* __restrict__ x, int ldx, const float* __restrict__ Dv, int V,
                                                               const T* __restrict__ z, int ldz, const float* __restrict__ w, T* __restrict__ out, int I, int gs,
                                                               float eps, const Tail tail) {
     __shared__ float scratch[32];
     const size_t t = blockIdx.x;
+    const T* zr = z + t * ldz;
+    if ((int)blockIdx.y >= tail.parts) { shift_inputs(zr, I, tail); return; }
     const int c0 = blockIdx.y * gs;
     const float* yr = y + t * I + c0;
-    const T* zr = z + t * ldz;
     const T* xr = x ? x + t * ldx + c0 : nullptr;
-    if (tail.state && blockIdx.y == gridDim.y - 1) shift_inputs(zr, I, tail);
     if constexpr (VPT == 0) {
         auto value = [&](int i) { return (yr[i] + (xr ? Dv[(c0 + i) / V] * to_f32(xr[i]) : 0.f)) * silu(to_f32(zr[c0 + i])); };
         float ss = 0.f;
@@ -475,10 +485,12 @@ MI_EXPORT int mi_ssd_step(const void* p, int ldp, const float* conv, const float
     const size_t smem = (size_t)(V + 2 * N + rows * V) * sizeof(float);
     if (smem > 48 * 1024) return -2;
     const dim3 grid(num_segs, H);
-#define GO(T, VEC) ssd_step_kernel<T, VEC><<<grid, 256, smem, stream>>>((const T*)p, ldp, conv, conv_b, taps, dt_bias, A, Dv, state, state_stride, out, \
-                                                                        seg_q_start, seg_slot, H, V, N, G)
+#define STEP(T, VEC, TAPS) ssd_step_kernel<T, VEC, TAPS><<<grid, 256, smem, stream>>>((const T*)p, ldp, conv, conv_b, taps, dt_bias, A, Dv, state, state_stride, out, \
+                                                                                 seg_q_start, seg_slot, H, V, N, G)
+#define GO(T, VEC) do { if (taps == 4) STEP(T, VEC, 4); else if (taps == 3) STEP(T, VEC, 3); else STEP(T, VEC, 0); } while (0)
     if (dtype == MI_BF16) { if (vec) GO(__nv_bfloat16, 4); else GO(__nv_bfloat16, 1); }
     else { if (vec) GO(float, 4); else GO(float, 1); }
+#undef STEP
 #undef GO
     return (int)cudaGetLastError();
 }
@@ -492,8 +504,8 @@ MI_EXPORT int mi_gated_part_norm(const float* y, const void* x, int ldx, const f
     if (T_ == 0) return 0;
     if (I % parts || parts > 65535) return -2;
     const int gs = I / parts;
-    const Tail tail{taps > 1 ? state : nullptr, state_stride, off, seg_slot, C, taps};
-    const dim3 grid(T_, parts);
+    const Tail tail{taps > 1 ? state : nullptr, state_stride, off, seg_slot, C, taps, parts};
+    const dim3 grid(T_, parts + (tail.state ? (C + 255) / 256 : 0));
     const bool vec = dtype == MI_BF16 && gs % 8 == 0 && gs <= 8192 && I % 8 == 0 && ldz % 8 == 0 && (!x || (ldx % 8 == 0 && V % 8 == 0)) &&
                      ((uintptr_t)y | (uintptr_t)x | (uintptr_t)z | (uintptr_t)w | (uintptr_t)out) % 16 == 0;
 #define GO(T, VPT) gated_part_norm_kernel<T, VPT><<<grid, 256, 0, stream>>>(y, (const T*)x, ldx, Dv, V, (const T*)z, ldz, w, (T*)out, I, gs, eps, tail)
