@@ -47,7 +47,7 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
 }
 __device__ __forceinline__ float rest(float x) { return x - __bfloat162float(__float2bfloat16_rn(x)); }      // what the rounding leaves
 
-constexpr int Q = 64, VB = 32, CH_THREADS = 256;
+constexpr int Q = 64, VB = 32, CH_WARPS = 16, CH_THREADS = 32 * CH_WARPS;
 
 // byte offset of the 16-byte piece `ch` of row `row`: rows of N entries (a multiple of 128 bytes), and rows of 32 entries (64 bytes)
 template <int N> __device__ __forceinline__ uint32_t at_n(int row, int ch) { return (uint32_t)(row * N * 2 + ((ch ^ (row & 7)) << 4)); }
@@ -56,23 +56,23 @@ __device__ __forceinline__ uint32_t at_v(int row, int ch) { return (uint32_t)(ro
 template <int N>
 struct ChunkSmem {
     static constexpr int BC = Q * N * 2, X = Q * VB * 2, STAGE = 2 * BC + X, S = N * VB * 2;
-    static constexpr int XW = 2 * STAGE, SH = XW + 2 * X, YP = SH + 2 * S, CUM = YP + Q * (VB + 2) * 4, TOTAL = CUM + 4 * Q * 4;
+    static constexpr int XW = 2 * STAGE, SH = XW + 2 * X, YP = SH + 2 * S, CUM = YP + 4 * Q * (VB + 2) * 4, TOTAL = CUM + 4 * Q * 4;
 };
 
 // grid (entries, heads, V / 32)
 template <int N>
-__global__ void __launch_bounds__(CH_THREADS, 2) ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, int ldx, const __nv_bfloat16* __restrict__ dt_in, int ld_dt,
+__global__ void __launch_bounds__(CH_THREADS, 1) ssd_chunk_kernel(const __nv_bfloat16* __restrict__ xbc, int ldx, const __nv_bfloat16* __restrict__ dt_in, int ld_dt,
                                                                   const float* __restrict__ dt_bias, const float* __restrict__ A, float* __restrict__ state,
                                                                   long long state_stride, float* __restrict__ out, const int* __restrict__ seg_q_start,
                                                                   const int* __restrict__ seg_slot, int H, int V, int G) {
     using L = ChunkSmem<N>;
     extern __shared__ __align__(128) unsigned char smem[];
     const uint32_t base = (uint32_t)__cvta_generic_to_shared(smem);
-    float* ypart = reinterpret_cast<float*>(smem + L::YP);         // [Q][VB + 2]
+    float* ypart = reinterpret_cast<float*>(smem + L::YP);         // [4][Q][VB + 2]
     float* dts = reinterpret_cast<float*>(smem + L::CUM);          // [2][Q]
     float* cums = dts + 2 * Q;                                     // [2][Q], base 2
     constexpr int CHN = N / 8, KN = N / 16;                        // 16-byte pieces of a row, k-steps over the state rows
-    constexpr int NTS = N == 128 ? 4 : 2;                          // the state's tiles of 8 columns a warp owns
+    constexpr int NTS = N == 128 ? 2 : 1;                          // the state's tiles of 8 columns a warp owns
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, c = lane & 3, mi_ = lane >> 3;
     const int seg = blockIdx.x, h = blockIdx.y, v0 = blockIdx.z * VB, grp = h / (H / G), I = H * V;
     const int qs = seg_q_start[seg], n = seg_q_start[seg + 1] - qs;
@@ -92,9 +92,11 @@ __global__ void __launch_bounds__(CH_THREADS, 2) ssd_chunk_kernel(const __nv_bfl
             cp16(st + at_n<N>(row, ch), bg + off, ok);
             cp16(st + L::BC + at_n<N>(row, ch), cg + off, ok);
         }
-        const int row = tid >> 2, ch = tid & 3;                    // Q * 4 pieces of x: one a thread
-        const bool ok = r0 + row < n;
-        cp16(st + 2 * L::BC + at_v(row, ch), xg + (ok ? (size_t)(r0 + row) * ldx + ch * 8 : 0), ok);
+        if (tid < Q * 4) {                                         // the pieces of x
+            const int row = tid >> 2, ch = tid & 3;
+            const bool ok = r0 + row < n;
+            cp16(st + 2 * L::BC + at_v(row, ch), xg + (ok ? (size_t)(r0 + row) * ldx + ch * 8 : 0), ok);
+        }
         asm volatile("cp.async.commit_group;\n" ::: "memory");
     };
     // warp 0: two tokens a lane; the raw steps are fetched a chunk ahead
@@ -120,7 +122,7 @@ __global__ void __launch_bounds__(CH_THREADS, 2) ssd_chunk_kernel(const __nv_bfl
     };
 
     // this warp's piece of the state: rows sn .. sn + 15, columns 8 (st0 + nt)
-    const int sn = (N == 128 ? warp : warp & 3) * 16, st0 = N == 128 ? 0 : (warp >> 2) * 2;
+    const int sn = (warp & (N / 16 - 1)) * 16, st0 = warp / (N / 16) * NTS;
     float* S = state + (long long)seg_slot[seg] * state_stride + (long long)h * N * V + v0;
     float s[NTS][4];
     auto spread_state = [&]() {                                    // the state as two bfloat16 numbers each, for the next chunk's read-out
@@ -146,7 +148,9 @@ __global__ void __launch_bounds__(CH_THREADS, 2) ssd_chunk_kernel(const __nv_bfl
     spread_state();
     if (warp == 0) sum_dt(0);
 
-    const int m0 = (warp & 3) * 16, hf = warp >> 2;                // the warp's 16 tokens; its half of the state rows and of the chunk's tokens
+    // the warp's 16 tokens, its quarter of the state rows and of the chunk's tokens (token tiles turned from quarter to quarter: late tiles have
+    // more tokens before them, and a scheduler's four warps should not all own late ones)
+    const int qd = warp >> 2, m0 = ((warp + qd) & 3) * 16;
     for (int ck = 0; ck < chunks; ++ck) {
         asm volatile("cp.async.wait_group 0;\n" ::: "memory");
         __syncthreads();                                           // the chunk, its decays and the spread state are there; the other stage is free
@@ -156,30 +160,22 @@ __global__ void __launch_bounds__(CH_THREADS, 2) ssd_chunk_kernel(const __nv_bfl
         const float* cum = cums + (ck & 1) * Q;
         const float end = cum[Q - 1];
         {   // the decayed x of the state's update
-            const int row = tid >> 2, ch = tid & 3;
-            const uint32_t off = at_v(row, ch);
+            const int row = tid >> 3, part = tid & 7;              // four entries a thread
+            const uint32_t off = at_v(row, part >> 1) + (part & 1) * 8;
             const float w = exp2f(end - cum[row]) * dt[row];
-            float xv[8];
-            load16<__nv_bfloat16>(reinterpret_cast<const __nv_bfloat16*>(smem + (xt - base) + off), xv);
-            uint4 hi, lo;
-            uint32_t* ph = reinterpret_cast<uint32_t*>(&hi);
-            uint32_t* pl = reinterpret_cast<uint32_t*>(&lo);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const float a = w * xv[2 * e], b = w * xv[2 * e + 1];
-                ph[e] = pack2(a, b);
-                pl[e] = pack2(rest(a), rest(b));
-            }
-            *reinterpret_cast<uint4*>(smem + L::XW + off) = hi;
-            *reinterpret_cast<uint4*>(smem + L::XW + L::X + off) = lo;
+            const uint2 raw = *reinterpret_cast<const uint2*>(smem + (xt - base) + off);
+            const float x0 = w * __uint_as_float(raw.x << 16), x1 = w * __uint_as_float(raw.x & 0xffff0000u);
+            const float x2 = w * __uint_as_float(raw.y << 16), x3 = w * __uint_as_float(raw.y & 0xffff0000u);
+            *reinterpret_cast<uint2*>(smem + L::XW + off) = make_uint2(pack2(x0, x1), pack2(x2, x3));
+            *reinterpret_cast<uint2*>(smem + L::XW + L::X + off) = make_uint2(pack2(rest(x0), rest(x1)), pack2(rest(x2), rest(x3)));
         }
-        // ---- what the state of before the chunk gives to the outputs: this warp's half of its rows
+        // ---- what the state of before the chunk gives to the outputs: this warp's quarter of its rows
         float y[4][4];
 #pragma unroll
         for (int nt = 0; nt < 4; ++nt) y[nt][0] = y[nt][1] = y[nt][2] = y[nt][3] = 0.f;
 #pragma unroll
-        for (int k = 0; k < KN / 2; ++k) {
-            const int ks = hf * (KN / 2) + k;
+        for (int k = 0; k < KN / 4; ++k) {
+            const int ks = qd * (KN / 4) + k;
             uint32_t a[4], b[4];
             ldsm4(a, ct + at_n<N>(m0 + (lane & 7) + (mi_ & 1) * 8, ks * 2 + (mi_ >> 1)));
 #pragma unroll
@@ -197,70 +193,63 @@ __global__ void __launch_bounds__(CH_THREADS, 2) ssd_chunk_kernel(const __nv_bfl
 #pragma unroll
             for (int nt = 0; nt < 4; ++nt) { y[nt][0] *= e0; y[nt][1] *= e0; y[nt][2] *= e1; y[nt][3] *= e1; }
         }
-        // ---- the chunk's own tokens: this warp's half of them, as far as they are not behind its rows
-        if (32 * hf <= m0 + 15) {
-            float sc[4][4];
+        // ---- the chunk's own tokens: this warp's quarter of them, unless they all come after its rows
+        if (16 * qd <= m0) {
+            float sc[2][4];
 #pragma unroll
-            for (int nt = 0; nt < 4; ++nt) sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f;
+            for (int nt = 0; nt < 2; ++nt) sc[nt][0] = sc[nt][1] = sc[nt][2] = sc[nt][3] = 0.f;
 #pragma unroll
             for (int ks = 0; ks < KN; ++ks) {
                 uint32_t a[4], b[4];
                 ldsm4(a, ct + at_n<N>(m0 + (lane & 7) + (mi_ & 1) * 8, ks * 2 + (mi_ >> 1)));
-#pragma unroll
-                for (int np = 0; np < 2; ++np) {
-                    ldsm4(b, bt + at_n<N>(32 * hf + (2 * np + (mi_ >> 1)) * 8 + (lane & 7), ks * 2 + (mi_ & 1)));
-                    mma16816(sc[2 * np], a, b[0], b[1]);
-                    mma16816(sc[2 * np + 1], a, b[2], b[3]);
-                }
+                ldsm4(b, bt + at_n<N>(16 * qd + (mi_ >> 1) * 8 + (lane & 7), ks * 2 + (mi_ & 1)));
+                mma16816(sc[0], a, b[0], b[1]);
+                mma16816(sc[1], a, b[2], b[3]);
             }
 #pragma unroll
-            for (int nt = 0; nt < 4; ++nt)
+            for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
                 for (int e = 0; e < 2; ++e) {
-                    const int j = 32 * hf + nt * 8 + 2 * c + e;
+                    const int j = 16 * qd + nt * 8 + 2 * c + e;
                     const float cj = cum[j], dj = dt[j];
                     sc[nt][e] = j <= m0 + g ? sc[nt][e] * exp2f(ct0 - cj) * dj : 0.f;
                     sc[nt][2 + e] = j <= m0 + g + 8 ? sc[nt][2 + e] * exp2f(ct1 - cj) * dj : 0.f;
                 }
+            uint32_t pa[4], pr[4], b[4];
 #pragma unroll
-            for (int kk = 0; kk < 2; ++kk) {
-                uint32_t pa[4], pr[4], b[4];
+            for (int q = 0; q < 4; ++q) {
+                const float lo = sc[q >> 1][2 * (q & 1)], hi = sc[q >> 1][2 * (q & 1) + 1];
+                pa[q] = pack2(lo, hi);
+                pr[q] = pack2(rest(lo), rest(hi));
+            }
 #pragma unroll
-                for (int q = 0; q < 4; ++q) {
-                    const float lo = sc[2 * kk + (q >> 1)][2 * (q & 1)], hi = sc[2 * kk + (q >> 1)][2 * (q & 1) + 1];
-                    pa[q] = pack2(lo, hi);
-                    pr[q] = pack2(rest(lo), rest(hi));
-                }
-#pragma unroll
-                for (int dp = 0; dp < 2; ++dp) {
-                    ldsm4t(b, xt + at_v(32 * hf + kk * 16 + (mi_ & 1) * 8 + (lane & 7), 2 * dp + (mi_ >> 1)));
-                    mma16816(y[2 * dp], pa, b[0], b[1]);
-                    mma16816(y[2 * dp + 1], pa, b[2], b[3]);
-                    mma16816(y[2 * dp], pr, b[0], b[1]);
-                    mma16816(y[2 * dp + 1], pr, b[2], b[3]);
-                }
+            for (int dp = 0; dp < 2; ++dp) {
+                ldsm4t(b, xt + at_v(16 * qd + (mi_ & 1) * 8 + (lane & 7), 2 * dp + (mi_ >> 1)));
+                mma16816(y[2 * dp], pa, b[0], b[1]);
+                mma16816(y[2 * dp + 1], pa, b[2], b[3]);
+                mma16816(y[2 * dp], pr, b[0], b[1]);
+                mma16816(y[2 * dp + 1], pr, b[2], b[3]);
             }
         }
-        if (hf == 1) {
+        {
+            float* yp = ypart + (qd * Q + m0 + g) * (VB + 2) + 2 * c;
 #pragma unroll
             for (int nt = 0; nt < 4; ++nt) {
-                *reinterpret_cast<float2*>(ypart + (m0 + g) * (VB + 2) + nt * 8 + 2 * c) = make_float2(y[nt][0], y[nt][1]);
-                *reinterpret_cast<float2*>(ypart + (m0 + g + 8) * (VB + 2) + nt * 8 + 2 * c) = make_float2(y[nt][2], y[nt][3]);
+                *reinterpret_cast<float2*>(yp + nt * 8) = make_float2(y[nt][0], y[nt][1]);
+                *reinterpret_cast<float2*>(yp + 8 * (VB + 2) + nt * 8) = make_float2(y[nt][2], y[nt][3]);
             }
         }
         __syncthreads();                                           // partial outputs and the decayed x are there; nobody reads the spread state any more
-        if (hf == 0) {
 #pragma unroll
-            for (int half = 0; half < 2; ++half) {
-                const int row = m0 + g + 8 * half, t = ck * Q + row;
-                if (t >= n) continue;
-                float* o = out + (size_t)(qs + t) * I + (size_t)h * V + v0;
+        for (int i = tid; i < Q * VB / 2; i += CH_THREADS) {       // the four quarters, added in order; a row's 32 columns leave together
+            const int row = i / (VB / 2), col = i % (VB / 2) * 2, t = ck * Q + row;
+            float2 sum = make_float2(0.f, 0.f);
 #pragma unroll
-                for (int nt = 0; nt < 4; ++nt) {
-                    const float2 other = *reinterpret_cast<const float2*>(ypart + row * (VB + 2) + nt * 8 + 2 * c);
-                    *reinterpret_cast<float2*>(o + nt * 8 + 2 * c) = make_float2(y[nt][2 * half] + other.x, y[nt][2 * half + 1] + other.y);
-                }
+            for (int q = 0; q < 4; ++q) {
+                const float2 v = *reinterpret_cast<const float2*>(ypart + (q * Q + row) * (VB + 2) + col);
+                sum.x += v.x; sum.y += v.y;
             }
+            if (t < n) *reinterpret_cast<float2*>(out + (size_t)(qs + t) * I + (size_t)h * V + v0 + col) = sum;
         }
         // ---- the state after the chunk
         const float keep = exp2f(end);
@@ -270,14 +259,18 @@ __global__ void __launch_bounds__(CH_THREADS, 2) ssd_chunk_kernel(const __nv_bfl
         for (int kt = 0; kt < Q / 16; ++kt) {
             uint32_t a[4], b[4];
             ldsm4t(a, bt + at_n<N>(kt * 16 + (lane & 7) + (mi_ >> 1) * 8, (sn >> 3) + (mi_ & 1)));
+            if constexpr (NTS == 2) {
 #pragma unroll
-            for (int part = 0; part < 2; ++part)
-#pragma unroll
-                for (int dp = 0; dp < NTS / 2; ++dp) {
-                    ldsm4t(b, base + L::XW + part * L::X + at_v(kt * 16 + (mi_ & 1) * 8 + (lane & 7), st0 + 2 * dp + (mi_ >> 1)));
-                    mma16816(s[2 * dp], a, b[0], b[1]);
-                    mma16816(s[2 * dp + 1], a, b[2], b[3]);
+                for (int part = 0; part < 2; ++part) {
+                    ldsm4t(b, base + L::XW + part * L::X + at_v(kt * 16 + (mi_ & 1) * 8 + (lane & 7), st0 + (mi_ >> 1)));
+                    mma16816(s[0], a, b[0], b[1]);
+                    mma16816(s[1], a, b[2], b[3]);
                 }
+            } else {                                               // one tile of columns: its two parts in one load
+                ldsm4t(b, base + L::XW + (mi_ >> 1) * L::X + at_v(kt * 16 + (mi_ & 1) * 8 + (lane & 7), st0));
+                mma16816(s[0], a, b[0], b[1]);
+                mma16816(s[0], a, b[2], b[3]);
+            }
         }
         if (ck + 1 < chunks) {
             spread_state();
