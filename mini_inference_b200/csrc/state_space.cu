@@ -41,6 +41,11 @@ __device__ __forceinline__ void cp16(uint32_t dst, const void* src, bool valid) 
     const int bytes = valid ? 16 : 0;                              // 0: the 16 bytes are filled with zeros
     asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" :: "r"(dst), "l"(src), "r"(bytes) : "memory");
 }
+__device__ __forceinline__ float fast_exp2(float x) {              // ex2.approx: 2 ulp
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
+    return y;
+}
 __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
     __nv_bfloat162 v = __floats2bfloat162_rn(lo, hi);
     return *reinterpret_cast<uint32_t*>(&v);
@@ -66,7 +71,7 @@ __global__ void __launch_bounds__(CH_THREADS, 1) ssd_chunk_kernel(const __nv_bfl
                                                                   long long state_stride, float* __restrict__ out, const int* __restrict__ seg_q_start,
                                                                   const int* __restrict__ seg_slot, int H, int V, int G) {
     using L = ChunkSmem<N>;
-    extern __shared__ __align__(128) unsigned char smem[];
+    extern __shared__ __align__(1024) unsigned char smem[];         // rows of up to 256 bytes start on 256: pieces are chosen by XOR below
     const uint32_t base = (uint32_t)__cvta_generic_to_shared(smem);
     float* ypart = reinterpret_cast<float*>(smem + L::YP);         // [4][Q][VB + 2]
     float* dts = reinterpret_cast<float*>(smem + L::CUM);          // [2][Q]
@@ -99,7 +104,7 @@ __global__ void __launch_bounds__(CH_THREADS, 1) ssd_chunk_kernel(const __nv_bfl
         }
         asm volatile("cp.async.commit_group;\n" ::: "memory");
     };
-    // warp 0: two tokens a lane; the raw steps are fetched a chunk ahead
+    // one warp, two tokens a lane; the raw steps are fetched a chunk before they are summed
     float raw0 = 0.f, raw1 = 0.f;
     auto fetch_dt = [&](int chunk) {
         const int t = chunk * Q + 2 * lane;
@@ -136,8 +141,10 @@ __global__ void __launch_bounds__(CH_THREADS, 1) ssd_chunk_kernel(const __nv_bfl
                 *reinterpret_cast<uint32_t*>(smem + L::SH + L::S + off) = pack2(rest(s[nt][2 * half]), rest(s[nt][2 * half + 1]));
             }
     };
+    // one warp sums the steps a chunk ahead: one whose tokens have none of its quarter before them, so that it has the time
+    const bool steps_warp = warp == 13;
     load(0);
-    if (warp == 0) fetch_dt(0);
+    if (steps_warp) fetch_dt(0);
 #pragma unroll
     for (int nt = 0; nt < NTS; ++nt)
 #pragma unroll
@@ -146,15 +153,19 @@ __global__ void __launch_bounds__(CH_THREADS, 1) ssd_chunk_kernel(const __nv_bfl
             s[nt][2 * half] = t.x; s[nt][2 * half + 1] = t.y;
         }
     spread_state();
-    if (warp == 0) sum_dt(0);
+    if (steps_warp) { sum_dt(0); fetch_dt(1); }
 
     // the warp's 16 tokens, its quarter of the state rows and of the chunk's tokens (token tiles turned from quarter to quarter: late tiles have
     // more tokens before them, and a scheduler's four warps should not all own late ones)
     const int qd = warp >> 2, m0 = ((warp + qd) & 3) * 16;
+    // this lane's ldmatrix rows: of C (its tokens), of B (its quarter), of a 32-column tile, of B transposed.  The 16-byte piece is XOR-ed with the
+    // row, and a k-step moves it by two: one XOR with 32 times the step
+    const uint32_t o_c = at_n<N>(m0 + (lane & 7) + (mi_ & 1) * 8, mi_ >> 1), o_b = at_n<N>(16 * qd + (mi_ >> 1) * 8 + (lane & 7), mi_ & 1);
+    const uint32_t o_v = at_v((mi_ & 1) * 8 + (lane & 7), mi_ >> 1), o_t = at_n<N>((lane & 7) + (mi_ >> 1) * 8, (sn >> 3) + (mi_ & 1));
     for (int ck = 0; ck < chunks; ++ck) {
         asm volatile("cp.async.wait_group 0;\n" ::: "memory");
         __syncthreads();                                           // the chunk, its decays and the spread state are there; the other stage is free
-        if (ck + 1 < chunks) { load(ck + 1); if (warp == 0) fetch_dt(ck + 1); }
+        if (ck + 1 < chunks) load(ck + 1);
         const uint32_t bt = base + (ck & 1) * L::STAGE, ct = bt + L::BC, xt = bt + 2 * L::BC;
         const float* dt = dts + (ck & 1) * Q;
         const float* cum = cums + (ck & 1) * Q;
@@ -162,7 +173,7 @@ __global__ void __launch_bounds__(CH_THREADS, 1) ssd_chunk_kernel(const __nv_bfl
         {   // the decayed x of the state's update
             const int row = tid >> 3, part = tid & 7;              // four entries a thread
             const uint32_t off = at_v(row, part >> 1) + (part & 1) * 8;
-            const float w = exp2f(end - cum[row]) * dt[row];
+            const float w = fast_exp2(end - cum[row]) * dt[row];
             const uint2 raw = *reinterpret_cast<const uint2*>(smem + (xt - base) + off);
             const float x0 = w * __uint_as_float(raw.x << 16), x1 = w * __uint_as_float(raw.x & 0xffff0000u);
             const float x2 = w * __uint_as_float(raw.y << 16), x3 = w * __uint_as_float(raw.y & 0xffff0000u);
@@ -177,19 +188,19 @@ __global__ void __launch_bounds__(CH_THREADS, 1) ssd_chunk_kernel(const __nv_bfl
         for (int k = 0; k < KN / 4; ++k) {
             const int ks = qd * (KN / 4) + k;
             uint32_t a[4], b[4];
-            ldsm4(a, ct + at_n<N>(m0 + (lane & 7) + (mi_ & 1) * 8, ks * 2 + (mi_ >> 1)));
+            ldsm4(a, (ct + o_c) ^ (32 * ks));
 #pragma unroll
             for (int part = 0; part < 2; ++part)
 #pragma unroll
                 for (int dp = 0; dp < 2; ++dp) {
-                    ldsm4t(b, base + L::SH + part * L::S + at_v(ks * 16 + (mi_ & 1) * 8 + (lane & 7), 2 * dp + (mi_ >> 1)));
+                    ldsm4t(b, (base + L::SH + part * L::S + ks * 16 * 64 + o_v) ^ (32 * dp));
                     mma16816(y[2 * dp], a, b[0], b[1]);
                     mma16816(y[2 * dp + 1], a, b[2], b[3]);
                 }
         }
         const float ct0 = cum[m0 + g], ct1 = cum[m0 + g + 8];
         {
-            const float e0 = exp2f(ct0), e1 = exp2f(ct1);
+            const float e0 = fast_exp2(ct0), e1 = fast_exp2(ct1);
 #pragma unroll
             for (int nt = 0; nt < 4; ++nt) { y[nt][0] *= e0; y[nt][1] *= e0; y[nt][2] *= e1; y[nt][3] *= e1; }
         }
@@ -201,8 +212,8 @@ __global__ void __launch_bounds__(CH_THREADS, 1) ssd_chunk_kernel(const __nv_bfl
 #pragma unroll
             for (int ks = 0; ks < KN; ++ks) {
                 uint32_t a[4], b[4];
-                ldsm4(a, ct + at_n<N>(m0 + (lane & 7) + (mi_ & 1) * 8, ks * 2 + (mi_ >> 1)));
-                ldsm4(b, bt + at_n<N>(16 * qd + (mi_ >> 1) * 8 + (lane & 7), ks * 2 + (mi_ & 1)));
+                ldsm4(a, (ct + o_c) ^ (32 * ks));
+                ldsm4(b, (bt + o_b) ^ (32 * ks));
                 mma16816(sc[0], a, b[0], b[1]);
                 mma16816(sc[1], a, b[2], b[3]);
             }
@@ -212,8 +223,8 @@ __global__ void __launch_bounds__(CH_THREADS, 1) ssd_chunk_kernel(const __nv_bfl
                 for (int e = 0; e < 2; ++e) {
                     const int j = 16 * qd + nt * 8 + 2 * c + e;
                     const float cj = cum[j], dj = dt[j];
-                    sc[nt][e] = j <= m0 + g ? sc[nt][e] * exp2f(ct0 - cj) * dj : 0.f;
-                    sc[nt][2 + e] = j <= m0 + g + 8 ? sc[nt][2 + e] * exp2f(ct1 - cj) * dj : 0.f;
+                    sc[nt][e] = j <= m0 + g ? sc[nt][e] * fast_exp2(ct0 - cj) * dj : 0.f;
+                    sc[nt][2 + e] = j <= m0 + g + 8 ? sc[nt][2 + e] * fast_exp2(ct1 - cj) * dj : 0.f;
                 }
             uint32_t pa[4], pr[4], b[4];
 #pragma unroll
@@ -224,13 +235,14 @@ __global__ void __launch_bounds__(CH_THREADS, 1) ssd_chunk_kernel(const __nv_bfl
             }
 #pragma unroll
             for (int dp = 0; dp < 2; ++dp) {
-                ldsm4t(b, xt + at_v(16 * qd + (mi_ & 1) * 8 + (lane & 7), 2 * dp + (mi_ >> 1)));
+                ldsm4t(b, (xt + qd * 16 * 64 + o_v) ^ (32 * dp));
                 mma16816(y[2 * dp], pa, b[0], b[1]);
                 mma16816(y[2 * dp + 1], pa, b[2], b[3]);
                 mma16816(y[2 * dp], pr, b[0], b[1]);
                 mma16816(y[2 * dp + 1], pr, b[2], b[3]);
             }
         }
+        if (steps_warp && ck + 1 < chunks) { sum_dt(ck + 1); fetch_dt(ck + 2); }
         {
             float* yp = ypart + (qd * Q + m0 + g) * (VB + 2) + 2 * c;
 #pragma unroll
@@ -252,17 +264,17 @@ __global__ void __launch_bounds__(CH_THREADS, 1) ssd_chunk_kernel(const __nv_bfl
             if (t < n) *reinterpret_cast<float2*>(out + (size_t)(qs + t) * I + (size_t)h * V + v0 + col) = sum;
         }
         // ---- the state after the chunk
-        const float keep = exp2f(end);
+        const float keep = fast_exp2(end);
 #pragma unroll
         for (int nt = 0; nt < NTS; ++nt) { s[nt][0] *= keep; s[nt][1] *= keep; s[nt][2] *= keep; s[nt][3] *= keep; }
 #pragma unroll
         for (int kt = 0; kt < Q / 16; ++kt) {
             uint32_t a[4], b[4];
-            ldsm4t(a, bt + at_n<N>(kt * 16 + (lane & 7) + (mi_ >> 1) * 8, (sn >> 3) + (mi_ & 1)));
+            ldsm4t(a, bt + kt * 16 * N * 2 + o_t);
             if constexpr (NTS == 2) {
 #pragma unroll
                 for (int part = 0; part < 2; ++part) {
-                    ldsm4t(b, base + L::XW + part * L::X + at_v(kt * 16 + (mi_ & 1) * 8 + (lane & 7), st0 + (mi_ >> 1)));
+                    ldsm4t(b, (base + L::XW + part * L::X + kt * 16 * 64 + o_v) ^ (16 * st0));
                     mma16816(s[0], a, b[0], b[1]);
                     mma16816(s[1], a, b[2], b[3]);
                 }
@@ -274,7 +286,6 @@ __global__ void __launch_bounds__(CH_THREADS, 1) ssd_chunk_kernel(const __nv_bfl
         }
         if (ck + 1 < chunks) {
             spread_state();
-            if (warp == 0) sum_dt(ck + 1);
         }
     }
 #pragma unroll
