@@ -18,6 +18,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Optional, Tuple
 
+from .json_keys import frozen, need, positive, thawed
 from .model_config import ConfigError
 
 MIXER_KEYS = {
@@ -25,26 +26,6 @@ MIXER_KEYS = {
     "mamba2": ("heads", "vdim", "state", "groups", "norm_groups", "conv"),
 }
 SHARED_SIZES = ("heads", "kv_heads", "dim", "vdim", "rot")      # what a layer must have in common with the one whose keys it reads
-
-
-def _need(d, keys, where: str):
-    if not isinstance(d, dict):
-        raise ConfigError(f"config.json: {where} must be an object")
-    missing = [k for k in keys if d.get(k) is None]
-    if missing:
-        raise ConfigError(f"config.json: {where} lacks {', '.join(missing)}")
-
-
-def _frozen(value):
-    if isinstance(value, dict):
-        return tuple(sorted((k, _frozen(v)) for k, v in value.items()))
-    return value
-
-
-def _thawed(value):
-    if isinstance(value, tuple):
-        return {k: _thawed(v) for k, v in value}
-    return value
 
 
 @dataclass(frozen=True)
@@ -60,24 +41,18 @@ class FetodraLayer:
     mlp: Optional[FetodraMLP]
 
     def mixer_dict(self) -> dict:
-        return _thawed(self.mixer)
-
-
-def _positive(m: dict, keys, where: str):
-    for k in keys:
-        if int(m[k]) < 1:
-            raise ConfigError(f"config.json: {where}.{k} must be at least 1")
+        return thawed(self.mixer)
 
 
 def _read_attention(mx: dict, where: str, index: int, before) -> dict:
-    _positive(mx, ("heads", "kv_heads", "dim", "vdim", "conv"), where)
+    positive(mx, ("heads", "kv_heads", "dim", "vdim", "conv"), where)
     if int(mx["heads"]) % int(mx["kv_heads"]):
         raise ConfigError(f"config.json: {where}: {mx['heads']} heads are not a multiple of {mx['kv_heads']} kv_heads")
-    _need(mx["rot"], ("base", "dims"), f"{where}.rot")
+    need(mx["rot"], ("base", "dims"), f"{where}.rot")
     if int(mx["rot"]["dims"]) % 2 or not 0 <= int(mx["rot"]["dims"]) <= int(mx["dim"]):
         raise ConfigError(f"config.json: {where}.rot.dims must be an even number up to dim")
     if mx.get("mask") is not None:
-        _need(mx["mask"], ("size",), f"{where}.mask")
+        need(mx["mask"], ("size",), f"{where}.mask")
         mask = {"size": int(mx["mask"]["size"]), "keep_first": int(mx["mask"].get("keep_first") or 0)}
         if mask["size"] < 1 or mask["keep_first"] < 0:
             raise ConfigError(f"config.json: {where}.mask: a window of {mask['size']} keys with the first {mask['keep_first']} kept")
@@ -99,7 +74,7 @@ def _read_attention(mx: dict, where: str, index: int, before) -> dict:
 
 
 def _read_mamba2(mx: dict, where: str) -> dict:
-    _positive(mx, MIXER_KEYS["mamba2"], where)
+    positive(mx, MIXER_KEYS["mamba2"], where)
     if int(mx["heads"]) % int(mx["groups"]):
         raise ConfigError(f"config.json: {where}: {mx['heads']} heads are not a multiple of {mx['groups']} groups")
     if int(mx["heads"]) * int(mx["vdim"]) % int(mx["norm_groups"]):
@@ -119,27 +94,27 @@ class FetodraConfig:
 
     @classmethod
     def from_dict(cls, raw: dict) -> "FetodraConfig":
-        _need(raw, ("vocab", "width", "layers", "norm", "postln_alpha"), "the top level")
-        _need(raw["norm"], ("eps",), "'norm'")
+        need(raw, ("vocab", "width", "layers", "norm", "postln_alpha"), "the top level")
+        need(raw["norm"], ("eps",), "'norm'")
         if not isinstance(raw["layers"], list) or not raw["layers"]:
             raise ConfigError("config.json: 'layers' must be a non-empty list")
         layers = []
         for i, entry in enumerate(raw["layers"]):
             where = f"layers[{i}]"
-            _need(entry, ("type", "mixer"), where)
+            need(entry, ("type", "mixer"), where)
             kind = entry["type"]
             if kind not in MIXER_KEYS:
                 raise ConfigError(f"config.json: {where} has type '{kind}' (known: {', '.join(sorted(MIXER_KEYS))})")
             mx = dict(entry["mixer"])
-            _need(mx, MIXER_KEYS[kind], f"{where}.mixer")
+            need(mx, MIXER_KEYS[kind], f"{where}.mixer")
             mx = _read_attention(mx, f"{where}.mixer", i, layers) if kind == "attention" else _read_mamba2(mx, f"{where}.mixer")
             mlp = entry.get("mlp")
             if mlp is not None:
-                _need(mlp, ("kind", "ff", "limit"), f"{where}.mlp")
+                need(mlp, ("kind", "ff", "limit"), f"{where}.mlp")
                 if mlp["kind"] != "dense":
                     raise ConfigError(f"config.json: {where}.mlp.kind '{mlp['kind']}' is not dense")
                 mlp = FetodraMLP(int(mlp["ff"]), float(mlp["limit"]))
-            layers.append(FetodraLayer(kind, _frozen(mx), mlp))
+            layers.append(FetodraLayer(kind, frozen(mx), mlp))
         return cls(architecture=raw.get("architecture") or (raw.get("architectures") or ["Fetodra"])[0],
                    vocab=int(raw["vocab"]), width=int(raw["width"]), norm_eps=float(raw["norm"]["eps"]),
                    postln_alpha=float(raw["postln_alpha"]), layers=tuple(layers), max_position=int(raw.get("max_position", 1 << 20)))

@@ -21,6 +21,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Optional, Tuple
 
+from .json_keys import frozen, need, thawed
 from .model_config import ConfigError
 
 MIXER_KEYS = {
@@ -28,28 +29,6 @@ MIXER_KEYS = {
     "latent_attention_2": ("heads", "dim", "vdim", "kv_rank", "q_rank", "scale"),
     "attention": ("heads", "kv_heads", "dim", "vdim", "scale"),
 }
-
-
-def _need(d, keys, where: str):
-    if not isinstance(d, dict):
-        raise ConfigError(f"config.json: {where} must be an object")
-    missing = [k for k in keys if d.get(k) is None]
-    if missing:
-        raise ConfigError(f"config.json: {where} lacks {', '.join(missing)}")
-
-
-def _frozen(value):
-    if isinstance(value, dict):
-        return tuple(sorted((k, _frozen(v)) for k, v in value.items()))
-    if isinstance(value, list):
-        return tuple(_frozen(v) for v in value)
-    return value
-
-
-def _thawed(value):
-    if isinstance(value, tuple) and all(isinstance(v, tuple) and len(v) == 2 and isinstance(v[0], str) for v in value):
-        return {k: _thawed(v) for k, v in value}
-    return value
 
 
 @dataclass(frozen=True)
@@ -77,28 +56,28 @@ class MegovikLayer:
     mlp: Optional[MegovikMLP]
 
     def mixer_dict(self) -> dict:
-        return _thawed(self.mixer)
+        return thawed(self.mixer)
 
 
 def _read_mlp(mlp, where: str) -> Optional[MegovikMLP]:
     if mlp is None:
         return None
-    _need(mlp, ("kind",), where)
+    need(mlp, ("kind",), where)
     if mlp["kind"] == "dense":
-        _need(mlp, ("ff",), where)
+        need(mlp, ("ff",), where)
         return MegovikMLP("dense", int(mlp["ff"]))
     if mlp["kind"] != "moe":
         raise ConfigError(f"config.json: {where}.kind '{mlp['kind']}' is not one of dense, moe")
-    _need(mlp, ("router", "expert"), where)
-    _need(mlp["router"], ("experts", "top"), f"{where}.router")
-    _need(mlp["expert"], ("ff",), f"{where}.expert")
+    need(mlp, ("router", "expert"), where)
+    need(mlp["router"], ("experts", "top"), f"{where}.router")
+    need(mlp["expert"], ("ff",), f"{where}.expert")
     r = mlp["router"]
     experts, top = int(r["experts"]), int(r["top"])
     if not 1 <= top <= experts:
         raise ConfigError(f"config.json: {where}.router.top is {top}; {experts} experts can be chosen")
     groups = None
     if r.get("groups") is not None:
-        _need(r["groups"], ("count", "keep"), f"{where}.router.groups")
+        need(r["groups"], ("count", "keep"), f"{where}.router.groups")
         count, keep = int(r["groups"]["count"]), int(r["groups"]["keep"])
         if count < 1 or experts % count or not 1 <= keep <= count:
             raise ConfigError(f"config.json: {where}.router.groups: {experts} experts in {count} groups of which {keep} are kept")
@@ -122,34 +101,34 @@ class MegovikConfig:
 
     @classmethod
     def from_dict(cls, raw: dict) -> "MegovikConfig":
-        _need(raw, ("vocab", "width", "layers", "norm", "max_positions"), "the top level")
-        _need(raw["norm"], ("eps",), "'norm'")
+        need(raw, ("vocab", "width", "layers", "norm", "max_positions"), "the top level")
+        need(raw["norm"], ("eps",), "'norm'")
         if not isinstance(raw["layers"], list) or not raw["layers"]:
             raise ConfigError("config.json: 'layers' must be a non-empty list")
         layers = []
         for i, entry in enumerate(raw["layers"]):
             where = f"layers[{i}]"
-            _need(entry, ("type", "mixer"), where)
+            need(entry, ("type", "mixer"), where)
             kind = entry["type"]
             if kind not in MIXER_KEYS:
                 raise ConfigError(f"config.json: {where} has type '{kind}' (known: {', '.join(sorted(MIXER_KEYS))})")
             mx = dict(entry["mixer"])
-            _need(mx, MIXER_KEYS[kind], f"{where}.mixer")
+            need(mx, MIXER_KEYS[kind], f"{where}.mixer")
             if kind == "attention":
                 if int(mx["heads"]) % int(mx["kv_heads"]):
                     raise ConfigError(f"config.json: {where}: {mx['heads']} heads are not a multiple of {mx['kv_heads']} kv_heads")
                 if int(mx["vdim"]) != int(mx["dim"]):
                     raise ConfigError(f"config.json: {where}: the values are the keys, so vdim ({mx['vdim']}) must equal dim ({mx['dim']})")
                 if mx.get("q_temp") is not None:
-                    _need(mx["q_temp"], ("coef", "every"), f"{where}.mixer.q_temp")
+                    need(mx["q_temp"], ("coef", "every"), f"{where}.mixer.q_temp")
                     if int(mx["q_temp"]["every"]) < 1:
                         raise ConfigError(f"config.json: {where}.mixer.q_temp.every must be at least 1")
                 else:
                     mx.pop("q_temp", None)
-            layers.append(MegovikLayer(kind, _frozen(mx), _read_mlp(entry.get("mlp"), f"{where}.mlp")))
+            layers.append(MegovikLayer(kind, frozen(mx), _read_mlp(entry.get("mlp"), f"{where}.mlp")))
         loop = raw.get("loop")
         if loop is not None:
-            _need(loop, ("start", "stop", "times"), "'loop'")
+            need(loop, ("start", "stop", "times"), "'loop'")
             loop = (int(loop["start"]), int(loop["stop"]), int(loop["times"]))
             if not (0 <= loop[0] <= loop[1] <= len(layers)) or loop[2] < 1:
                 raise ConfigError(f"config.json: loop {loop} does not fit {len(layers)} layers")

@@ -18,20 +18,13 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Optional, Tuple
 
+from .json_keys import need
 from .model_config import ConfigError
 
 MIXER_KEYS = {
     "attention": ("heads", "kv_heads", "dim", "vdim", "scale"),
     "retention": ("heads", "dim", "vdim", "decay", "rot"),
 }
-
-
-def _need(d, keys, where: str):
-    if not isinstance(d, dict):
-        raise ConfigError(f"config.json: {where} must be an object")
-    missing = [k for k in keys if d.get(k) is None]
-    if missing:
-        raise ConfigError(f"config.json: {where} lacks {', '.join(missing)}")
 
 
 @dataclass(frozen=True)
@@ -75,19 +68,19 @@ class NamesunLayer:
 def _read_mlp(mlp, where: str) -> Optional[NamesunMLP]:
     if mlp is None:
         return None
-    _need(mlp, ("kind",), where)
+    need(mlp, ("kind",), where)
     if mlp["kind"] == "dense":
-        _need(mlp, ("ff",), where)
+        need(mlp, ("ff",), where)
         return NamesunMLP("dense", int(mlp["ff"]))
     if mlp["kind"] != "moe":
         raise ConfigError(f"config.json: {where}.kind '{mlp['kind']}' is not one of dense, moe")
-    _need(mlp, ("router", "expert"), where)
-    _need(mlp["router"], ("experts", "top"), f"{where}.router")
-    _need(mlp["expert"], ("ff", "limit"), f"{where}.expert")
+    need(mlp, ("router", "expert"), where)
+    need(mlp["router"], ("experts", "top"), f"{where}.router")
+    need(mlp["expert"], ("ff", "limit"), f"{where}.expert")
     experts, top = int(mlp["router"]["experts"]), int(mlp["router"]["top"])
     groups = mlp["router"].get("groups")
     if groups is not None:
-        _need(groups, ("count", "keep"), f"{where}.router.groups")
+        need(groups, ("count", "keep"), f"{where}.router.groups")
         groups = (int(groups["count"]), int(groups["keep"]))
         if groups[0] < 1 or experts % groups[0] or not 1 <= groups[1] <= groups[0]:
             raise ConfigError(f"config.json: {where}.router.groups {groups} do not cut {experts} experts into equal groups of which some are kept")
@@ -96,7 +89,7 @@ def _read_mlp(mlp, where: str) -> Optional[NamesunMLP]:
         raise ConfigError(f"config.json: {where}.router.top is {top}; {allowed} experts can be chosen")
     shared = mlp.get("shared")
     if shared is not None:
-        _need(shared, ("ff", "limit"), f"{where}.shared")
+        need(shared, ("ff", "limit"), f"{where}.shared")
         shared = (int(shared["ff"]), float(shared["limit"]))
     return NamesunMLP("moe", int(mlp["expert"]["ff"]), experts, top, groups, float(mlp["expert"]["limit"]), shared)
 
@@ -113,25 +106,25 @@ class NamesunConfig:
 
     @classmethod
     def from_dict(cls, raw: dict) -> "NamesunConfig":
-        _need(raw, ("vocab", "width", "layers", "norm", "residual_mult"), "the top level")
-        _need(raw["norm"], ("eps",), "'norm'")
+        need(raw, ("vocab", "width", "layers", "norm", "residual_mult"), "the top level")
+        need(raw["norm"], ("eps",), "'norm'")
         if not isinstance(raw["layers"], list) or not raw["layers"]:
             raise ConfigError("config.json: 'layers' must be a non-empty list")
         layers = []
         for i, entry in enumerate(raw["layers"]):
             where = f"layers[{i}]"
-            _need(entry, ("type", "mixer"), where)
+            need(entry, ("type", "mixer"), where)
             kind = entry["type"]
             if kind not in MIXER_KEYS:
                 raise ConfigError(f"config.json: {where} has type '{kind}' (known: {', '.join(sorted(MIXER_KEYS))})")
             mx = dict(entry["mixer"])
-            _need(mx, MIXER_KEYS[kind], f"{where}.mixer")
+            need(mx, MIXER_KEYS[kind], f"{where}.mixer")
             if kind == "attention":
                 if int(mx["heads"]) % int(mx["kv_heads"]):
                     raise ConfigError(f"config.json: {where}: {mx['heads']} heads are not a multiple of {mx['kv_heads']} kv_heads")
                 mask = mx.get("mask")
                 if mask is not None:
-                    _need(mask, ("size",), f"{where}.mixer.mask")
+                    need(mask, ("size",), f"{where}.mixer.mask")
                     if int(mask["size"]) < 1:
                         raise ConfigError(f"config.json: {where}.mixer.mask.size must be at least 1")
                     mask = (("size", int(mask["size"])),)
@@ -142,7 +135,7 @@ class NamesunConfig:
                 mx["decay"] = tuple(float(v) for v in mx["decay"])
                 if len(mx["decay"]) != int(mx["heads"]):
                     raise ConfigError(f"config.json: {where}.mixer.decay has {len(mx['decay'])} entries for {mx['heads']} heads")
-                _need(mx["rot"], ("base", "dims"), f"{where}.mixer.rot")
+                need(mx["rot"], ("base", "dims"), f"{where}.mixer.rot")
                 rot = {"base": float(mx["rot"]["base"]), "dims": int(mx["rot"]["dims"])}
                 if rot["dims"] % 2 or not 0 <= rot["dims"] <= int(mx["dim"]):
                     raise ConfigError(f"config.json: {where}.mixer.rot.dims must be even and at most dim")

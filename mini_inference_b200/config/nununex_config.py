@@ -22,6 +22,7 @@ from __future__ import annotations
 from dataclasses import dataclass
 from typing import Optional, Tuple
 
+from .json_keys import frozen, need, thawed
 from .model_config import ConfigError
 
 MIXER_KEYS = {
@@ -31,28 +32,6 @@ MIXER_KEYS = {
 }
 LEFT_KEYS = ("heads", "kv_heads", "dim", "vdim", "scale", "bias_max")
 RIGHT_KEYS = ("heads", "dim", "vdim", "gate_cap")
-
-
-def _need(d, keys, where: str):
-    if not isinstance(d, dict):
-        raise ConfigError(f"config.json: {where} must be an object")
-    missing = [k for k in keys if d.get(k) is None]
-    if missing:
-        raise ConfigError(f"config.json: {where} lacks {', '.join(missing)}")
-
-
-def _frozen(value):
-    if isinstance(value, dict):
-        return tuple(sorted((k, _frozen(v)) for k, v in value.items()))
-    if isinstance(value, list):
-        return tuple(_frozen(v) for v in value)
-    return value
-
-
-def _thawed(value):
-    if isinstance(value, tuple) and all(isinstance(v, tuple) and len(v) == 2 and isinstance(v[0], str) for v in value):
-        return {k: _thawed(v) for k, v in value}
-    return value
 
 
 @dataclass(frozen=True)
@@ -79,27 +58,27 @@ class NununexLayer:
     mlp: Optional[NununexMLP]
 
     def mixer_dict(self) -> dict:
-        return _thawed(self.mixer)
+        return thawed(self.mixer)
 
 
 def _read_mlp(mlp, where: str) -> Optional[NununexMLP]:
     if mlp is None:
         return None
-    _need(mlp, ("kind",), where)
+    need(mlp, ("kind",), where)
     if mlp["kind"] == "dense":
-        _need(mlp, ("ff",), where)
+        need(mlp, ("ff",), where)
         return NununexMLP("dense", int(mlp["ff"]))
     if mlp["kind"] != "moe":
         raise ConfigError(f"config.json: {where}.kind '{mlp['kind']}' is not one of dense, moe")
-    _need(mlp, ("router", "expert"), where)
-    _need(mlp["router"], ("experts", "top"), f"{where}.router")
-    _need(mlp["expert"], ("ff",), f"{where}.expert")
+    need(mlp, ("router", "expert"), where)
+    need(mlp["router"], ("experts", "top"), f"{where}.router")
+    need(mlp["expert"], ("ff",), f"{where}.expert")
     experts, top = int(mlp["router"]["experts"]), int(mlp["router"]["top"])
     if not 1 <= top <= experts:
         raise ConfigError(f"config.json: {where}.router.top is {top}; {experts} experts can be chosen")
     shared = mlp.get("shared")
     if shared is not None:
-        _need(shared, ("ff",), f"{where}.shared")
+        need(shared, ("ff",), f"{where}.shared")
         shared = int(shared["ff"])
     return NununexMLP("moe", int(mlp["expert"]["ff"]), experts, top, shared)
 
@@ -118,11 +97,11 @@ class NununexConfig:
 
     @classmethod
     def from_dict(cls, raw: dict) -> "NununexConfig":
-        _need(raw, ("vocab", "width", "layers", "norm", "canon", "embedding"), "the top level")
-        _need(raw["norm"], ("eps",), "'norm'")
-        _need(raw["canon"], ("taps",), "'canon'")
-        _need(raw["embedding"], ("bigram",), "'embedding'")
-        _need(raw["embedding"]["bigram"], ("buckets", "mul_prev", "mul_cur"), "'embedding.bigram'")
+        need(raw, ("vocab", "width", "layers", "norm", "canon", "embedding"), "the top level")
+        need(raw["norm"], ("eps",), "'norm'")
+        need(raw["canon"], ("taps",), "'canon'")
+        need(raw["embedding"], ("bigram",), "'embedding'")
+        need(raw["embedding"]["bigram"], ("buckets", "mul_prev", "mul_cur"), "'embedding.bigram'")
         if int(raw["canon"]["taps"]) < 1:
             raise ConfigError("config.json: canon.taps must be at least 1")
         if not isinstance(raw["layers"], list) or not raw["layers"]:
@@ -130,20 +109,20 @@ class NununexConfig:
         layers = []
         for i, entry in enumerate(raw["layers"]):
             where = f"layers[{i}]"
-            _need(entry, ("type", "mixer"), where)
+            need(entry, ("type", "mixer"), where)
             kind = entry["type"]
             if kind not in MIXER_KEYS:
                 raise ConfigError(f"config.json: {where} has type '{kind}' (known: {', '.join(sorted(MIXER_KEYS))})")
             mx = dict(entry["mixer"])
-            _need(mx, MIXER_KEYS[kind], f"{where}.mixer")
+            need(mx, MIXER_KEYS[kind], f"{where}.mixer")
             if kind == "parallel":
                 left, right = dict(mx["left"]), dict(mx["right"])
-                _need(left, LEFT_KEYS, f"{where}.mixer.left")
-                _need(right, RIGHT_KEYS, f"{where}.mixer.right")
+                need(left, LEFT_KEYS, f"{where}.mixer.left")
+                need(right, RIGHT_KEYS, f"{where}.mixer.right")
                 if int(left["heads"]) % int(left["kv_heads"]):
                     raise ConfigError(f"config.json: {where}: {left['heads']} heads are not a multiple of {left['kv_heads']} kv_heads")
                 if left.get("mask") is not None:
-                    _need(left["mask"], ("size",), f"{where}.mixer.left.mask")
+                    need(left["mask"], ("size",), f"{where}.mixer.left.mask")
                     if int(left["mask"]["size"]) < 1:
                         raise ConfigError(f"config.json: {where}.mixer.left.mask.size must be at least 1")
                 else:
@@ -151,7 +130,7 @@ class NununexConfig:
                 mx["left"], mx["right"] = left, right
             if kind == "mamba1" and int(mx["conv"]) < 1:
                 raise ConfigError(f"config.json: {where}.mixer.conv must be at least 1")
-            layers.append(NununexLayer(kind, _frozen(mx), _read_mlp(entry.get("mlp"), f"{where}.mlp")))
+            layers.append(NununexLayer(kind, frozen(mx), _read_mlp(entry.get("mlp"), f"{where}.mlp")))
         b = raw["embedding"]["bigram"]
         cap = raw.get("logit_softcap")
         return cls(architecture=raw.get("architecture") or (raw.get("architectures") or ["Nununex"])[0],
