@@ -67,11 +67,14 @@ class ExecStep:
     table of pass vectors (ModelSpec.pass_vectors_name) that is added to the residual stream
     right before this step's layer runs (a model that repeats a span of layers marks each
     repetition this way).  add_embedding: the embedded tokens, as they entered the stream before the first
-    layer, are added to the stream right before this step's layer runs (row by row, in the stream's precision)."""
+    layer, are added to the stream right before this step's layer runs (row by row, in the stream's precision).
+    join_embedding: right before this step's layer runs the stream becomes W [stream; embedded tokens], W being the model's
+    [hidden, 2 hidden] tensor ModelSpec.join_name."""
     layer: int
     cache_from: Optional[int] = None
     add_row: Optional[int] = None
     add_embedding: bool = False
+    join_embedding: bool = False
 
 
 @dataclass(frozen=True)
@@ -105,6 +108,8 @@ class ModelSpec:
     # the embedded token is multiplied by embedding_scale as it enters a float32 stream; the head's product by logit_scale
     embedding_scale: float = 1.0
     logit_scale: float = 1.0
+    # the [hidden, 2 hidden] tensor of the steps that set ExecStep.join_embedding (stream columns first)
+    join_name: Optional[str] = None
 
     def __post_init__(self):
         for i, step in enumerate(self.order):
@@ -119,5 +124,7 @@ class ModelSpec:
                 raise ValueError(f"order[{i}] adds pass vector {step.add_row}; the model has {self.pass_vectors_rows}")
             if step.add_row is not None and step.add_embedding:
                 raise ValueError(f"order[{i}] adds both a pass vector and the embedded tokens")
+            if step.join_embedding and (self.join_name is None or self.residual != "float32" or step.add_row is not None or step.add_embedding):
+                raise ValueError(f"order[{i}] joins the stream with the embedded tokens: that takes ModelSpec.join_name and a float32 stream, and excludes other additions")
         if self.residual not in ("compute", "float32"):
             raise ValueError(f"residual '{self.residual}' is not one of compute, float32")

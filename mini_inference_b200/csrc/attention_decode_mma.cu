@@ -678,7 +678,7 @@ MI_EXPORT int mi_attn_decode_mma_rows_biased(const void* q, int q_stride, const 
                                              float scale, int window, int* merge_counters, int* error_word, int cache_pages,
                                              int cluster_merge, int block, int sink, const float* sink_values, const float* bias_t,
                                              int bias_last, cudaStream_t stream) {
-    if (!bias_t) return -2;
+    if (!bias_t && !sink_values) return -2;                // bias_t may be null: a learned sink alone
     return decode_mma_rows_launch<true, true>(DECODE_ROWS_ARGS, block, sink, sink_values, bias_t, bias_last);
 }
 

@@ -1,9 +1,10 @@
 // Latent attention over a one-plane paged cache: every token caches ONE row [c (C entries) | kr (R entries)]; all H
 // query heads attend over these shared rows with queries of size C + R (the key up-projection absorbed into the
 // query) and the weighted sum is taken over the first C entries of the same rows (the value up-projection is
-// applied afterwards, per head).  Any C and R; float32 or bfloat16 storage; scores, softmax and sums in float32 on
-// the CUDA cores in an order that depends only on the request's own positions.  Sizes that the tensor-core paged
-// attention kernels take (C + R of 64 or 128, bfloat16) are sent there by the kernel namespace instead.
+// applied afterwards, per head).  sink (float32 [H] or null): the softmax has one more term exp(sink[h]), which carries no value.
+// Any C and R; float32 or bfloat16 storage; scores, softmax and sums in float32 on the CUDA cores in an order that depends only on
+// the request's own positions.  Sizes that the tensor-core paged attention kernels take (C + R of 64 or 128, bfloat16) are sent
+// there by the kernel namespace instead.
 //
 // Cache layout: [pages, 1, page_size, C + R]; the row of key j of a request is at (table[j / ps] * ps + j % ps) * (C + R).
 // Output: element d of head h of token t goes to out[h * out_hs + t * out_ts + d] ([H, T, C]: out_hs = T C, out_ts = C, what the
@@ -20,18 +21,29 @@ constexpr int WARPS = 4;
 // ------------------------------------------------------------------ per token: latent norm, rotations, cache write, query assembly
 // p [T, ldp]: q heads [H, D + R] | dkv [C + R] | ...;  q_abs [H, T, C] (the absorbed unrotated queries).
 // q_out [T, H, C + R] = [q_abs | rotate(q rot part)];  cache row = [rmsnorm(dkv[:C]) * w | rotate(dkv[C:])].
-// Interleaved rotation: pairs (2i, 2i+1), i < nf, by the angle pos * inv_freq[i]; entries from 2 nf on pass unchanged.
+// Rotation by the angle pos * inv_freq[i], i < nf: the pairs (2i, 2i+1), or with half_pairs (i, i + nf); entries from 2 nf on pass
+// unchanged.  The token's cosines and sines are made once, in shared memory (2 nf floats).
+__device__ __forceinline__ float rotated(float own, float other, int j, int nf, int half_pairs, const float* cs, const float* sn) {
+    const int i = half_pairs ? (j < nf ? j : j - nf) : j >> 1;
+    const bool second = half_pairs ? j >= nf : j & 1;
+    return second ? own * cs[i] + other * sn[i] : own * cs[i] - other * sn[i];
+}
+__device__ __forceinline__ int partner(int j, int nf, int half_pairs) { return half_pairs ? (j < nf ? j + nf : j - nf) : j ^ 1; }
+
 template <typename T>
 __global__ void latent_prepare_kernel(const T* __restrict__ p, int ldp, const T* __restrict__ q_rows, int ldq, int dkv_col,
                                       const T* __restrict__ q_abs, T* __restrict__ q_out,
                                       T* __restrict__ cache, const float* __restrict__ norm_w, const float* __restrict__ inv_freq,
                                       int nf, const int* __restrict__ positions, const int* __restrict__ slots, int T_, int H,
-                                      int D, int R, int C, float eps) {
+                                      int D, int R, int C, float eps, int half_pairs) {
     __shared__ float scratch[32];
+    extern __shared__ float turn[];                        // cos [nf] | sin [nf]
     const int t = blockIdx.x;
     const T* row = p + (size_t)t * ldp;
     const T* qrow = q_rows + (size_t)t * ldq;              // the query heads as projected: p itself, or a tensor of their own
     const float pos = (float)positions[t];
+    for (int i = threadIdx.x; i < nf; i += blockDim.x) sincosf(pos * inv_freq[i], turn + nf + i, turn + i);
+    __syncthreads();
     T* qo = q_out + (size_t)t * H * (C + R);
     for (int idx = threadIdx.x; idx < H * C; idx += blockDim.x) {
         const int h = idx / C, i = idx - h * C;
@@ -41,12 +53,7 @@ __global__ void latent_prepare_kernel(const T* __restrict__ p, int ldp, const T*
         const int h = idx / R, j = idx - h * R;
         const T* src = qrow + (size_t)h * (D + R) + D;
         float val = to_f32(src[j]);
-        if (j < 2 * nf) {
-            float sn, cs;
-            sincosf(pos * inv_freq[j >> 1], &sn, &cs);
-            const float other = to_f32(src[j ^ 1]);
-            val = (j & 1) ? val * cs + other * sn : val * cs - other * sn;
-        }
+        if (j < 2 * nf) val = rotated(val, to_f32(src[partner(j, nf, half_pairs)]), j, nf, half_pairs, turn, turn + nf);
         qo[(size_t)h * (C + R) + C + j] = from_f32<T>(val);
     }
     if (cache == nullptr) return;
@@ -58,12 +65,7 @@ __global__ void latent_prepare_kernel(const T* __restrict__ p, int ldp, const T*
     for (int i = threadIdx.x; i < C; i += blockDim.x) crow[i] = from_f32<T>(to_f32(dkv[i]) * r * norm_w[i]);
     for (int j = threadIdx.x; j < R; j += blockDim.x) {
         float val = to_f32(dkv[C + j]);
-        if (j < 2 * nf) {
-            float sn, cs;
-            sincosf(pos * inv_freq[j >> 1], &sn, &cs);
-            const float other = to_f32(dkv[C + (j ^ 1)]);
-            val = (j & 1) ? val * cs + other * sn : val * cs - other * sn;
-        }
+        if (j < 2 * nf) val = rotated(val, to_f32(dkv[C + partner(j, nf, half_pairs)]), j, nf, half_pairs, turn, turn + nf);
         crow[C + j] = from_f32<T>(val);
     }
 }
@@ -123,7 +125,7 @@ __global__ void latent_prefill_kernel(const T* __restrict__ q, const T* __restri
                                       const int* __restrict__ tiles, const int* __restrict__ seg_q_start,
                                       const int* __restrict__ seg_pos0, const int* __restrict__ block_table,
                                       const int* __restrict__ table_rows, int table_stride, long long out_hs, long long out_ts, int H, int Dk, int Dv, int ps,
-                                      int tile_rows, float scale, int vec) {
+                                      int tile_rows, float scale, int vec, const float* __restrict__ sink) {
     extern __shared__ float q_sm[];                      // [WARPS, Dk]
     const int seg = tiles[2 * blockIdx.x], r0 = tiles[2 * blockIdx.x + 1];
     const int h = blockIdx.y;
@@ -137,7 +139,7 @@ __global__ void latent_prefill_kernel(const T* __restrict__ q, const T* __restri
         const T* qr = q + ((size_t)tok * H + h) * Dk;
         for (int d = lane; d < Dk; d += 32) q_s[d] = to_f32(qr[d]) * scale;
         __syncwarp();
-        float m = -INFINITY, l = 0.f, acc[NV];
+        float m = sink ? sink[h] : -INFINITY, l = sink ? 1.f : 0.f, acc[NV];       // the sink's term e^(sink - m) = 1
 #pragma unroll
         for (int k = 0; k < NV; ++k) acc[k] = 0.f;
         attend_rows<T, NV>(q_s, cache, table_row, Dk, Dv, ps, vec != 0, 0, pq + 1, m, l, acc);
@@ -158,7 +160,8 @@ __global__ void latent_decode_kernel(const T* __restrict__ q, const T* __restric
                                      float* __restrict__ o_part, float* __restrict__ lse_part, const int* __restrict__ decode_segs,
                                      const int* __restrict__ seg_q_start, const int* __restrict__ seg_kv_len,
                                      const int* __restrict__ block_table, const int* __restrict__ table_rows, int table_stride,
-                                     long long out_hs, long long out_ts, int H, int Dk, int Dv, int ps, float scale, int vec) {
+                                     long long out_hs, long long out_ts, int H, int Dk, int Dv, int ps, float scale, int vec,
+                                     const float* __restrict__ sink) {
     extern __shared__ float q_sm[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int h = blockIdx.y * WARPS + warp;
@@ -172,7 +175,8 @@ __global__ void latent_decode_kernel(const T* __restrict__ q, const T* __restric
     const T* qr = q + ((size_t)tok * H + h) * Dk;
     for (int d = lane; d < Dk; d += 32) q_s[d] = to_f32(qr[d]) * scale;
     __syncwarp();
-    float m = -INFINITY, l = 0.f, acc[NV];
+    const bool own_sink = sink && S == 1;                       // several pieces: the merge adds the sink's term
+    float m = own_sink ? sink[h] : -INFINITY, l = own_sink ? 1.f : 0.f, acc[NV];
 #pragma unroll
     for (int k = 0; k < NV; ++k) acc[k] = 0.f;
     if (lo < hi)
@@ -191,16 +195,17 @@ __global__ void latent_decode_kernel(const T* __restrict__ q, const T* __restric
     }
 }
 
-// out = sum_s e^(lse_s - max) o_s / sum_s e^(lse_s - max), in split order
+// out = sum_s e^(lse_s - max) o_s / (sum_s e^(lse_s - max) + [sink] e^(sink - max)), in split order
 template <typename T>
 __global__ void latent_merge_kernel(const float* __restrict__ o_part, const float* __restrict__ lse_part, T* __restrict__ out,
-                                    const int* __restrict__ decode_segs, const int* __restrict__ seg_q_start, long long out_hs, long long out_ts, int H, int Dv, int S) {
+                                    const int* __restrict__ decode_segs, const int* __restrict__ seg_q_start, long long out_hs, long long out_ts, int H, int Dv, int S,
+                                    const float* __restrict__ sink) {
     const int i = blockIdx.x, h = blockIdx.y;
     const int tok = seg_q_start[decode_segs[i]];
     const size_t base = ((size_t)i * H + h) * S;
-    float mx = -INFINITY;
+    float mx = sink ? sink[h] : -INFINITY;
     for (int s = 0; s < S; ++s) mx = fmaxf(mx, lse_part[base + s]);
-    float den = 0.f;
+    float den = sink ? expf(sink[h] - mx) : 0.f;
     for (int s = 0; s < S; ++s) den += expf(lse_part[base + s] - mx);
     for (int d = threadIdx.x; d < Dv; d += blockDim.x) {
         float num = 0.f;
@@ -215,17 +220,19 @@ __global__ void latent_merge_kernel(const float* __restrict__ o_part, const floa
 // at which [c as projected | kr] starts (negative: behind the query heads, H (D + R)).
 MI_EXPORT int mi_latent_prepare(const void* p, int ldp, const void* q_rows, int ldq, int dkv_col, const void* q_abs, void* q_out, void* cache,
                                 const float* norm_w, const float* inv_freq, int nf, const int* positions, const int* slots, int T_, int H,
-                                int D, int R, int C, float eps, int dtype, cudaStream_t stream) {
+                                int D, int R, int C, float eps, int half_pairs, int dtype, cudaStream_t stream) {
     if (T_ == 0) return 0;
+    if (nf > 4096) return -2;
+    const size_t smem = 2 * (size_t)nf * sizeof(float);
     if (!q_rows) { q_rows = p; ldq = ldp; }
     if (dkv_col < 0) dkv_col = H * (D + R);
     if (dtype == MI_BF16)
-        latent_prepare_kernel<__nv_bfloat16><<<T_, 128, 0, stream>>>((const __nv_bfloat16*)p, ldp, (const __nv_bfloat16*)q_rows, ldq, dkv_col,
+        latent_prepare_kernel<__nv_bfloat16><<<T_, 128, smem, stream>>>((const __nv_bfloat16*)p, ldp, (const __nv_bfloat16*)q_rows, ldq, dkv_col,
                                                                      (const __nv_bfloat16*)q_abs, (__nv_bfloat16*)q_out,
-                                                                     (__nv_bfloat16*)cache, norm_w, inv_freq, nf, positions, slots, T_, H, D, R, C, eps);
+                                                                     (__nv_bfloat16*)cache, norm_w, inv_freq, nf, positions, slots, T_, H, D, R, C, eps, half_pairs);
     else
-        latent_prepare_kernel<float><<<T_, 128, 0, stream>>>((const float*)p, ldp, (const float*)q_rows, ldq, dkv_col, (const float*)q_abs,
-                                                             (float*)q_out, (float*)cache, norm_w, inv_freq, nf, positions, slots, T_, H, D, R, C, eps);
+        latent_prepare_kernel<float><<<T_, 128, smem, stream>>>((const float*)p, ldp, (const float*)q_rows, ldq, dkv_col, (const float*)q_abs,
+                                                             (float*)q_out, (float*)cache, norm_w, inv_freq, nf, positions, slots, T_, H, D, R, C, eps, half_pairs);
     return (int)cudaGetLastError();
 }
 
@@ -233,7 +240,7 @@ MI_EXPORT int mi_latent_prepare(const void* p, int ldp, const void* q_rows, int 
 
 MI_EXPORT int mi_latent_prefill(const void* q, const void* cache, void* out, const int* tiles, int num_tiles, const int* seg_q_start,
                                 const int* seg_pos0, const int* block_table, const int* table_rows, int table_stride, long long out_hs,
-                                long long out_ts, int H, int C, int R, int ps, int tile_rows, float scale, int dtype, cudaStream_t stream) {
+                                long long out_ts, int H, int C, int R, int ps, int tile_rows, float scale, const float* sink, int dtype, cudaStream_t stream) {
     if (num_tiles == 0) return 0;
     const int Dk = C + R, Dv = C;
     if (Dv > 512 || Dk > 2048 || H > 65535) return -2;
@@ -243,9 +250,9 @@ MI_EXPORT int mi_latent_prefill(const void* q, const void* cache, void* out, con
     dim3 grid(num_tiles, H);
 #define CALL(NV) do { \
         if (dtype == MI_BF16) latent_prefill_kernel<__nv_bfloat16, NV><<<grid, WARPS * 32, smem, stream>>>((const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, \
-            (__nv_bfloat16*)out, tiles, seg_q_start, seg_pos0, block_table, table_rows, table_stride, out_hs, out_ts, H, Dk, Dv, ps, tile_rows, scale, vec); \
+            (__nv_bfloat16*)out, tiles, seg_q_start, seg_pos0, block_table, table_rows, table_stride, out_hs, out_ts, H, Dk, Dv, ps, tile_rows, scale, vec, sink); \
         else latent_prefill_kernel<float, NV><<<grid, WARPS * 32, smem, stream>>>((const float*)q, (const float*)cache, (float*)out, tiles, seg_q_start, \
-            seg_pos0, block_table, table_rows, table_stride, out_hs, out_ts, H, Dk, Dv, ps, tile_rows, scale, vec); } while (0)
+            seg_pos0, block_table, table_rows, table_stride, out_hs, out_ts, H, Dk, Dv, ps, tile_rows, scale, vec, sink); } while (0)
     LATENT_PICK_NV(CALL);
 #undef CALL
     return (int)cudaGetLastError();
@@ -254,7 +261,7 @@ MI_EXPORT int mi_latent_prefill(const void* q, const void* cache, void* out, con
 MI_EXPORT int mi_latent_decode(const void* q, const void* cache, void* out, float* o_part, float* lse_part, const int* decode_segs,
                                int num_decode, const int* seg_q_start, const int* seg_kv_len, const int* block_table,
                                const int* table_rows, int table_stride, long long out_hs, long long out_ts, int H, int C, int R, int ps, int splits,
-                               float scale, int dtype, cudaStream_t stream) {
+                               float scale, const float* sink, int dtype, cudaStream_t stream) {
     if (num_decode == 0) return 0;
     const int Dk = C + R, Dv = C;
     if (Dv > 512 || Dk > 2048 || H > 65535 * WARPS) return -2;
@@ -264,17 +271,17 @@ MI_EXPORT int mi_latent_decode(const void* q, const void* cache, void* out, floa
     dim3 grid(num_decode, (H + WARPS - 1) / WARPS, splits);
 #define CALL(NV) do { \
         if (dtype == MI_BF16) latent_decode_kernel<__nv_bfloat16, NV><<<grid, WARPS * 32, smem, stream>>>((const __nv_bfloat16*)q, (const __nv_bfloat16*)cache, \
-            (__nv_bfloat16*)out, o_part, lse_part, decode_segs, seg_q_start, seg_kv_len, block_table, table_rows, table_stride, out_hs, out_ts, H, Dk, Dv, ps, scale, vec); \
+            (__nv_bfloat16*)out, o_part, lse_part, decode_segs, seg_q_start, seg_kv_len, block_table, table_rows, table_stride, out_hs, out_ts, H, Dk, Dv, ps, scale, vec, sink); \
         else latent_decode_kernel<float, NV><<<grid, WARPS * 32, smem, stream>>>((const float*)q, (const float*)cache, (float*)out, o_part, lse_part, \
-            decode_segs, seg_q_start, seg_kv_len, block_table, table_rows, table_stride, out_hs, out_ts, H, Dk, Dv, ps, scale, vec); } while (0)
+            decode_segs, seg_q_start, seg_kv_len, block_table, table_rows, table_stride, out_hs, out_ts, H, Dk, Dv, ps, scale, vec, sink); } while (0)
     LATENT_PICK_NV(CALL);
 #undef CALL
     int err = (int)cudaGetLastError();
     if (err || splits == 1) return err;
     dim3 mgrid(num_decode, H);
     if (dtype == MI_BF16)
-        latent_merge_kernel<__nv_bfloat16><<<mgrid, 128, 0, stream>>>(o_part, lse_part, (__nv_bfloat16*)out, decode_segs, seg_q_start, out_hs, out_ts, H, Dv, splits);
+        latent_merge_kernel<__nv_bfloat16><<<mgrid, 128, 0, stream>>>(o_part, lse_part, (__nv_bfloat16*)out, decode_segs, seg_q_start, out_hs, out_ts, H, Dv, splits, sink);
     else
-        latent_merge_kernel<float><<<mgrid, 128, 0, stream>>>(o_part, lse_part, (float*)out, decode_segs, seg_q_start, out_hs, out_ts, H, Dv, splits);
+        latent_merge_kernel<float><<<mgrid, 128, 0, stream>>>(o_part, lse_part, (float*)out, decode_segs, seg_q_start, out_hs, out_ts, H, Dv, splits, sink);
     return (int)cudaGetLastError();
 }

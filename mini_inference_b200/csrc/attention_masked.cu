@@ -19,7 +19,8 @@
 // (visible) keys of a request cut into `splits` pieces, one warp per (head, piece), merged by a second kernel.
 //
 // Prepare kernel, one block per token: q and k divided by their root mean square per head (eps > 0) and, when given, multiplied by
-// a weight of D entries that all heads share (one for q, one for k); q then multiplied by the temperature
+// a weight of D entries that all heads share (one for q, one for k) and, when frequencies are given, rotated (rotate-half: coordinate i < half
+// with i + half, by the angle position * inv_freq[i]; the token's cosines and sines are made once, in shared memory); q then multiplied by the temperature
 // 1 + coef * ln(floor((p + 1) / every) + 1) of its position p (every > 0); v blended with another layer's values of the same
 // token ((1 - lambda) v + lambda v_src), or, with v_is_k, taken from the keys AS PROJECTED (before the norm; there are no v
 // columns then); k and v written to the token's slot of the pages, q written back in place.
@@ -210,17 +211,36 @@ __global__ void masked_merge_kernel(const float* __restrict__ o_part, const floa
 
 // ------------------------------------------------------------------ unit norms, value blend, cache write
 // p [T, ldp] = q [H D] | k [KV D] | v [KV Dv].  One block per token, a warp per head in turn.
+// dst = rotate(x * r * w) for one head by one warp; dst may be x (a lane reads both coordinates of a pair before it writes them)
+template <typename T>
+__device__ __forceinline__ void put_head(const T* x, T* dst, int D, float r, const float* __restrict__ w, int half, const float* turn, int lane) {
+    for (int d = lane; d < D; d += 32) {
+        if (d >= half && d < 2 * half) continue;                // the lane of its partner d - half writes it
+        const float a = to_f32(x[d]) * r * (w ? w[d] : 1.f);
+        if (d >= half) { dst[d] = from_f32<T>(a); continue; }
+        const float b = to_f32(x[d + half]) * r * (w ? w[d + half] : 1.f), cs = turn[d], sn = turn[half + d];
+        dst[d] = from_f32<T>(a * cs - b * sn);
+        dst[d + half] = from_f32<T>(b * cs + a * sn);
+    }
+}
+
 template <typename T>
 __global__ void unit_qk_cache_kernel(T* __restrict__ p, int ldp, const T* __restrict__ v_src, int ld_src, const float* __restrict__ lam,
                                      const int* __restrict__ slots, T* __restrict__ k_cache, T* __restrict__ v_cache,
                                      int H, int KV, int D, int Dv, int ps, float eps, int unit, const float* __restrict__ q_w,
                                      const float* __restrict__ k_w, const int* __restrict__ positions, float temp_coef, int temp_every,
-                                     int v_is_k) {
+                                     int v_is_k, const float* __restrict__ inv_freq, int half) {
+    extern __shared__ float turn[];                             // cos [half] | sin [half]
     const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
     T* row = p + (size_t)t * ldp;
     const int slot = slots[t];
     const long long page = slot / ps, off = slot % ps;
     const float temp = temp_every > 0 ? 1.f + temp_coef * logf((float)((positions[t] + 1) / temp_every + 1)) : 1.f;
+    if (half > 0) {
+        const float pos = (float)positions[t];
+        for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * inv_freq[i], turn + half + i, turn + i);
+        __syncthreads();
+    }
     for (int u = warp; u < H + KV; u += nw) {                   // q heads, then k heads
         T* x = row + (size_t)u * D;
         float r = 1.f;
@@ -230,11 +250,11 @@ __global__ void unit_qk_cache_kernel(T* __restrict__ p, int ldp, const T* __rest
             r = rsqrtf(warp_sum(ss) / D + eps);
         }
         if (u < H) {
-            if (unit || q_w || temp_every > 0)
-                for (int d = lane; d < D; d += 32) x[d] = from_f32<T>(to_f32(x[d]) * r * (q_w ? q_w[d] : 1.f) * temp);
+            if (unit || q_w || temp_every > 0 || half > 0)
+                put_head<T>(x, x, D, r * temp, q_w, half, turn, lane);
         } else if (k_cache) {
             T* dst = k_cache + ((page * KV + (u - H)) * ps + off) * D;
-            for (int d = lane; d < D; d += 32) dst[d] = from_f32<T>(to_f32(x[d]) * r * (k_w ? k_w[d] : 1.f));
+            put_head<T>(x, dst, D, r, k_w, half, turn, lane);
             if (v_is_k && v_cache) {                           // the values are these keys as projected
                 T* vd = v_cache + ((page * KV + (u - H)) * ps + off) * D;
                 for (int d = lane; d < D; d += 32) vd[d] = x[d];
@@ -254,23 +274,26 @@ __global__ void unit_qk_cache_kernel(T* __restrict__ p, int ldp, const T* __rest
 
 }  // namespace
 
-// q_w, k_w: float32 [D] or null; positions with temp_every > 0: the query temperature; v_is_k: p has no v columns, Dv == D
+// q_w, k_w: float32 [D] or null; positions with temp_every > 0: the query temperature; v_is_k: p has no v columns, Dv == D;
+// inv_freq [half] with half > 0: the first 2 half coordinates of every q and k head are rotated by the token's position
 MI_EXPORT int mi_normed_qk_cache(void* p, int ldp, const void* v_src, int ld_src, const float* lam, const int* slots, void* k_cache,
                                  void* v_cache, int T_, int H, int KV, int D, int Dv, int ps, float eps, int unit, const float* q_w,
-                                 const float* k_w, const int* positions, float temp_coef, int temp_every, int v_is_k, int dtype,
-                                 cudaStream_t stream) {
+                                 const float* k_w, const int* positions, float temp_coef, int temp_every, int v_is_k, const float* inv_freq,
+                                 int half, int dtype, cudaStream_t stream) {
     if (T_ == 0) return 0;
-    if ((v_is_k && (Dv != D || v_src)) || (temp_every > 0 && !positions) || ((q_w == nullptr) != (k_w == nullptr))) return -2;
+    if ((v_is_k && (Dv != D || v_src)) || (temp_every > 0 && !positions) || ((q_w == nullptr) != (k_w == nullptr)) ||
+        (half > 0 && (!positions || !inv_freq || 2 * half > D || half > 4096))) return -2;
+    const size_t turn = half > 0 ? 2 * (size_t)half * sizeof(float) : 0;
     // few tokens (decode steps): a warp per head, so that no warp walks several heads one after the other
     const int nt = T_ >= 256 ? 128 : min(1024, max(128, 32 * (H + KV)));
     if (dtype == MI_BF16)
-        unit_qk_cache_kernel<__nv_bfloat16><<<T_, nt, 0, stream>>>((__nv_bfloat16*)p, ldp, (const __nv_bfloat16*)v_src, ld_src, lam, slots,
+        unit_qk_cache_kernel<__nv_bfloat16><<<T_, nt, turn, stream>>>((__nv_bfloat16*)p, ldp, (const __nv_bfloat16*)v_src, ld_src, lam, slots,
                                                                     (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, H, KV, D, Dv, ps, eps, unit,
-                                                                    q_w, k_w, positions, temp_coef, temp_every, v_is_k);
+                                                                    q_w, k_w, positions, temp_coef, temp_every, v_is_k, inv_freq, half);
     else
-        unit_qk_cache_kernel<float><<<T_, nt, 0, stream>>>((float*)p, ldp, (const float*)v_src, ld_src, lam, slots, (float*)k_cache,
+        unit_qk_cache_kernel<float><<<T_, nt, turn, stream>>>((float*)p, ldp, (const float*)v_src, ld_src, lam, slots, (float*)k_cache,
                                                            (float*)v_cache, H, KV, D, Dv, ps, eps, unit, q_w, k_w, positions, temp_coef,
-                                                            temp_every, v_is_k);
+                                                            temp_every, v_is_k, inv_freq, half);
     return (int)cudaGetLastError();
 }
 
@@ -278,7 +301,7 @@ MI_EXPORT int mi_unit_qk_cache(void* p, int ldp, const void* v_src, int ld_src, 
                                void* v_cache, int T_, int H, int KV, int D, int Dv, int ps, float eps, int unit, int dtype,
                                cudaStream_t stream) {
     return mi_normed_qk_cache(p, ldp, v_src, ld_src, lam, slots, k_cache, v_cache, T_, H, KV, D, Dv, ps, eps, unit, nullptr, nullptr, nullptr,
-                              0.f, 0, 0, dtype, stream);
+                              0.f, 0, 0, nullptr, 0, dtype, stream);
 }
 
 MI_EXPORT int mi_masked_prefill(const void* q, int q_stride, const void* k_cache, const void* v_cache, void* out, const int* tiles,

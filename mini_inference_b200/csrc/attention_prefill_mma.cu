@@ -339,7 +339,7 @@ MI_EXPORT int mi_attn_prefill_mma_biased(const void* q, int q_stride, const void
                                          const int* block_table, const int* table_rows, int table_stride, int H, int KV, int D, int ps,
                                          int tile_rows, float scale, int window, int block, int sink, const float* sink_values,
                                          const float* bias_t, int bias_last, cudaStream_t stream) {
-    if (!bias_t) return -2;
+    if (!bias_t && !sink_values) return -2;                // bias_t may be null: a learned sink alone
     return prefill_mma_launch<true, true>(q, q_stride, k_cache, v_cache, out, tiles, num_tiles, seg_q_start, seg_pos0, block_table, table_rows,
                                           table_stride, H, KV, D, ps, tile_rows, scale, window, block, sink, stream, sink_values, bias_t, bias_last);
 }

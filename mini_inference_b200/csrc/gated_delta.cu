@@ -1,0 +1,273 @@
+// Gated delta rule with one decay per head and token, around the state scan of recurrent.cu:
+//
+//     q, k, v = silu(conv(.));  q, k <- x / sqrt(sum x^2 + unit_eps), q also * key_dim^-1/2;  beta = sigmoid(b);  f = exp(-rate softplus(a + dt_bias))
+//     S <- f S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q;     rows: o / rms(o) * weight * silu(gate) per head
+//
+// p [T, ldp] as projected: q [KV D] | k [KV D] | v [H V] (the C channels that pass the convolution) | gate [H V] | b [H] | a [H] | ..
+// conv float32 [C, taps], the last tap multiplies the current token.  A request's slot holds S (float32 [H, D, V]) and behind it a ring
+// of the convolution's inputs, [taps, C]: position p has row p mod taps, positions before 0 count as zeros.
+//
+// Prompts: delta_ready_kernel makes what the scan stages (float32 rows q | k | v | beta | f), the scan runs (recurrent.cu), then
+// delta_ring_kernel writes the entry's newest inputs into the ring.  Decode steps (every entry one token): delta_step_kernel does all of
+// it in one pass over the state, one block per (entry, head).  The ring has one row more than a token looks back on, so the block that
+// writes a token's inputs overwrites none that the other heads' blocks (which share a q and k head) still read.
+// Everything is float32; the decay is rounded once from a double-precision exponential, since it acts on a state hundreds of times in a row.
+#include "common.cuh"
+#include <math.h>
+
+using namespace mi;
+
+namespace {
+
+__device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
+__device__ __forceinline__ float head_decay(float a, float dt_bias, float rate) {
+    const double z = (double)a + (double)dt_bias;
+    return (float)exp(-(double)rate * (z > 30.0 ? z : log1p(exp(z))));
+}
+
+// ------------------------------------------------------------------ prompts: what the scan stages
+// grid (token groups of TOK, units / 4), four warps, a warp per unit: the KV q heads, the KV k heads, then the value channels in pieces of
+// 32 NI, then one unit for the gates of all heads.  A lane owns the channels c0 + lane + 32 i of its unit (i < NI) with their taps in
+// registers and walks the group's tokens, its last taps - 1 inputs held in registers from token to token inside an entry.
+template <typename T, int TAPS, int NI, int TOK>
+__global__ void __launch_bounds__(128) delta_ready_kernel(const T* __restrict__ p, int ldp, const float* __restrict__ conv, const float* __restrict__ rate,
+                                                          const float* __restrict__ dt_bias, const float* __restrict__ state, long long state_stride,
+                                                          long long ring_off, float* __restrict__ out, int ldo, const int* __restrict__ positions,
+                                                          const int* __restrict__ token_seg, const int* __restrict__ seg_q_start,
+                                                          const int* __restrict__ seg_slot, int T_, int H, int KV, int D, int V, int taps_, float unit_eps,
+                                                          float q_scale) {
+    constexpr int W = TAPS > 0 ? TAPS : 1;                     // TAPS 0: any number of taps, read again for every token
+    const int taps = TAPS > 0 ? TAPS : taps_;
+    const int lane = threadIdx.x & 31, unit = blockIdx.y * 4 + (threadIdx.x >> 5);
+    const int C = 2 * KV * D + H * V, pieces = (H * V + 32 * NI - 1) / (32 * NI);
+    const int t0 = blockIdx.x * TOK, t1 = min(T_, t0 + TOK);
+    if (unit > 2 * KV + pieces) return;
+    if (unit == 2 * KV + pieces) {                             // beta and f of every head
+        for (int i = lane; i < (t1 - t0) * H; i += 32) {
+            const int t = t0 + i / H, h = i % H;
+            const T* row = p + (size_t)t * ldp + C + H * V;
+            float* o = out + (size_t)t * ldo + C;
+            o[h] = 1.f / (1.f + expf(-to_f32(row[h])));
+            o[H + h] = head_decay(to_f32(row[H + h]), dt_bias[h], rate[h]);
+        }
+        return;
+    }
+    const bool head = unit < 2 * KV;
+    const int c0 = head ? unit * D : 2 * KV * D + (unit - 2 * KV) * 32 * NI;
+    const int n = head ? D : min(32 * NI, C - c0);
+    float w[NI][W], x[NI][W];
+#pragma unroll
+    for (int i = 0; i < NI; ++i)
+#pragma unroll
+        for (int j = 0; j < W; ++j) { w[i][j] = TAPS > 0 && lane + 32 * i < n ? conv[(size_t)(c0 + lane + 32 * i) * TAPS + j] : 0.f; x[i][j] = 0.f; }
+    int last = -1;                                             // the entry whose inputs the registers hold
+    for (int t = t0; t < t1; ++t) {
+        const int seg = token_seg[t], qs = seg_q_start[seg], r = t - qs, pos = positions[t];
+        const float* ring = state + (long long)seg_slot[seg] * state_stride + ring_off;
+        auto input = [&](int c, int back) {                    // the input `back` tokens before t
+            if (back <= r) return to_f32(p[(size_t)(t - back) * ldp + c]);
+            return back <= pos ? ring[(size_t)((pos - back) % taps) * C + c] : 0.f;
+        };
+        float y[NI], ss = 0.f;
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            y[i] = 0.f;
+            const int c = c0 + lane + 32 * i;
+            if (lane + 32 * i >= n) continue;
+            float acc = 0.f;
+            if constexpr (TAPS > 0) {
+                if (seg == last) {
+#pragma unroll
+                    for (int j = 0; j + 1 < TAPS; ++j) x[i][j] = x[i][j + 1];
+                } else {
+#pragma unroll
+                    for (int j = 0; j + 1 < TAPS; ++j) x[i][j] = input(c, TAPS - 1 - j);
+                }
+                x[i][TAPS - 1] = to_f32(p[(size_t)t * ldp + c]);
+#pragma unroll
+                for (int j = 0; j < TAPS; ++j) acc = fmaf(w[i][j], x[i][j], acc);
+            } else {
+                for (int j = 0; j < taps; ++j) acc = fmaf(conv[(size_t)c * taps + j], input(c, taps - 1 - j), acc);
+            }
+            y[i] = silu(acc);
+            ss = fmaf(y[i], y[i], ss);
+        }
+        last = seg;
+        float s = 1.f;
+        if (head) s = (unit < KV ? q_scale : 1.f) / sqrtf(warp_sum(ss) + unit_eps);
+        float* o = out + (size_t)t * ldo + c0;
+#pragma unroll
+        for (int i = 0; i < NI; ++i)
+            if (lane + 32 * i < n) o[lane + 32 * i] = y[i] * s;
+    }
+}
+
+// the entry's inputs of its last min(n, taps - 1) positions -> their ring rows; grid (entries, channel groups)
+template <typename T>
+__global__ void delta_ring_kernel(const T* __restrict__ p, int ldp, float* __restrict__ state, long long state_stride, long long ring_off,
+                                  const int* __restrict__ positions, const int* __restrict__ seg_q_start, const int* __restrict__ seg_slot, int C, int taps) {
+    const int seg = blockIdx.x, q1 = seg_q_start[seg + 1], n = q1 - seg_q_start[seg], c = blockIdx.y * blockDim.x + threadIdx.x;
+    if (c >= C) return;
+    float* ring = state + (long long)seg_slot[seg] * state_stride + ring_off;
+    for (int t = q1 - min(n, taps - 1); t < q1; ++t) ring[(size_t)(positions[t] % taps) * C + c] = to_f32(p[(size_t)t * ldp + c]);
+}
+
+// ------------------------------------------------------------------ decode steps: everything in one pass over the state
+// grid (entries, H).  Thread (rg, cv) of a block holds four neighbouring columns 4 cv .. of the rows rg + RG i (i < NR), cv < V / 4,
+// RG = blockDim / (V / 4): the state is read once and written once, in 16-byte pieces, its loads issued before anything else.
+template <typename T, int NR>
+__global__ void __launch_bounds__(256) delta_step_kernel(const T* __restrict__ p, int ldp, const float* __restrict__ conv, int taps,
+                                                         const float* __restrict__ rate, const float* __restrict__ dt_bias, float* __restrict__ state,
+                                                         long long state_stride, long long ring_off, const float* __restrict__ norm, T* __restrict__ rows,
+                                                         const int* __restrict__ positions, const int* __restrict__ seg_q_start,
+                                                         const int* __restrict__ seg_slot, int H, int KV, int D, int V, float unit_eps, float q_scale, float eps) {
+    extern __shared__ __align__(16) float sm[];
+    __shared__ float scratch[32];
+    float* qs = sm;                                            // [D]
+    float* ks = qs + D;                                        // [D]
+    float* vs = ks + D;                                        // [V]: the values, then u
+    float* red = sm + ((2 * D + V + 3) & ~3);                  // [RG, V]
+    const int seg = blockIdx.x, h = blockIdx.y, rep = H / KV, kvh = h / rep, tid = threadIdx.x;
+    const int t = seg_q_start[seg], pos = positions[t];
+    float* slot = state + (long long)seg_slot[seg] * state_stride;
+    float* ring = slot + ring_off;
+    float* S = slot + (long long)h * D * V;
+    const int CV = V >> 2, RG = 256 / CV, cv = tid % CV, rg = tid / CV;
+    float4 s[NR];
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+        const int r = rg + RG * i;
+        s[i] = rg < RG && r < D ? *reinterpret_cast<const float4*>(S + (size_t)r * V + 4 * cv) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    const T* row = p + (size_t)t * ldp;
+    const int C = 2 * KV * D + H * V;
+    float sq = 0.f, sk = 0.f;
+    for (int i = tid; i < 2 * D + V; i += 256) {               // this head's q, k and v channels
+        const int c = i < D ? kvh * D + i : i < 2 * D ? KV * D + kvh * D + i - D : 2 * KV * D + h * V + i - 2 * D;
+        const float own = to_f32(row[c]);
+        float acc = 0.f;
+        for (int j = 0; j + 1 < taps; ++j) {
+            const int back = taps - 1 - j;
+            if (back <= pos) acc = fmaf(conv[(size_t)c * taps + j], ring[(size_t)((pos - back) % taps) * C + c], acc);
+        }
+        const float y = silu(fmaf(conv[(size_t)c * taps + taps - 1], own, acc));
+        sm[i] = y;
+        if (i < D) sq = fmaf(y, y, sq); else if (i < 2 * D) sk = fmaf(y, y, sk);
+        if (taps > 1 && (i >= 2 * D || h % rep == 0)) ring[(size_t)(pos % taps) * C + c] = own;      // one writer a channel
+    }
+    const float beta = 1.f / (1.f + expf(-to_f32(row[C + H * V + h])));
+    const float f = head_decay(to_f32(row[C + H * V + H + h]), dt_bias[h], rate[h]);
+    const float rq = q_scale / sqrtf(block_sum<256>(sq, scratch) + unit_eps), rk = 1.f / sqrtf(block_sum<256>(sk, scratch) + unit_eps);
+    // (block_sum's barriers also make qs, ks and vs visible)
+    float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < NR; ++i) {
+        const int r = rg + RG * i;
+        const float kr = rg < RG && r < D ? ks[r] * rk : 0.f;
+        a.x = fmaf(s[i].x, kr, a.x); a.y = fmaf(s[i].y, kr, a.y); a.z = fmaf(s[i].z, kr, a.z); a.w = fmaf(s[i].w, kr, a.w);
+    }
+    if (rg < RG) *reinterpret_cast<float4*>(red + rg * V + 4 * cv) = a;
+    __syncthreads();
+    for (int c = tid; c < V; c += 256) {
+        float dot = 0.f;
+        for (int g = 0; g < RG; ++g) dot += red[g * V + c];
+        vs[c] = beta * (vs[c] - f * dot);
+    }
+    __syncthreads();
+    if (rg < RG) {
+        const float4 u = make_float4(vs[4 * cv], vs[4 * cv + 1], vs[4 * cv + 2], vs[4 * cv + 3]);
+        float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int i = 0; i < NR; ++i) {
+            const int r = rg + RG * i;
+            if (r >= D) continue;
+            const float kr = ks[r] * rk, qr = qs[r] * rq;
+            s[i].x = fmaf(kr, u.x, f * s[i].x); s[i].y = fmaf(kr, u.y, f * s[i].y);
+            s[i].z = fmaf(kr, u.z, f * s[i].z); s[i].w = fmaf(kr, u.w, f * s[i].w);
+            o.x = fmaf(s[i].x, qr, o.x); o.y = fmaf(s[i].y, qr, o.y); o.z = fmaf(s[i].z, qr, o.z); o.w = fmaf(s[i].w, qr, o.w);
+            *reinterpret_cast<float4*>(S + (size_t)r * V + 4 * cv) = s[i];
+        }
+        *reinterpret_cast<float4*>(red + rg * V + 4 * cv) = o;
+    }
+    __syncthreads();
+    float ss = 0.f;
+    for (int c = tid; c < V; c += 256) {
+        float o = 0.f;
+        for (int g = 0; g < RG; ++g) o += red[g * V + c];
+        vs[c] = o;                                             // read again below by the same thread
+        ss = fmaf(o, o, ss);
+    }
+    const float r = rsqrtf(block_sum<256>(ss, scratch) / V + eps);
+    for (int c = tid; c < V; c += 256)
+        rows[(size_t)t * H * V + (size_t)h * V + c] = from_f32<T>(vs[c] * r * norm[c] * silu(to_f32(row[C + h * V + c])));
+}
+
+template <typename T>
+int launch_ready(const T* p, int ldp, const float* conv, const float* rate, const float* dt_bias, const float* state, long long state_stride,
+                 long long ring_off, float* out, int ldo, const int* positions, const int* token_seg, const int* seg_q_start, const int* seg_slot,
+                 int T_, int H, int KV, int D, int V, int taps, float unit_eps, cudaStream_t stream) {
+    const int NI = D <= 32 ? 1 : D <= 64 ? 2 : D <= 128 ? 4 : 8;
+    const int units = 2 * KV + (H * V + 32 * NI - 1) / (32 * NI) + 1;
+    const int TOK = T_ >= 1024 ? 16 : T_ >= 128 ? 4 : 1;
+    dim3 grid((T_ + TOK - 1) / TOK, (units + 3) / 4);
+    if (grid.y > 65535) return -2;
+    const float q_scale = 1.f / sqrtf((float)D);
+#define GO(TAPS, N, TK) delta_ready_kernel<T, TAPS, N, TK><<<grid, 128, 0, stream>>>(p, ldp, conv, rate, dt_bias, state, state_stride, ring_off, out, ldo, \
+                            positions, token_seg, seg_q_start, seg_slot, T_, H, KV, D, V, taps, unit_eps, q_scale)
+#define TOKENS(TAPS, N) do { if (TOK == 16) GO(TAPS, N, 16); else if (TOK == 4) GO(TAPS, N, 4); else GO(TAPS, N, 1); } while (0)
+#define CHANNELS(TAPS) do { if (NI == 1) TOKENS(TAPS, 1); else if (NI == 2) TOKENS(TAPS, 2); else if (NI == 4) TOKENS(TAPS, 4); else TOKENS(TAPS, 8); } while (0)
+    if (taps == 4) CHANNELS(4); else if (taps == 3) CHANNELS(3); else if (taps == 2) CHANNELS(2); else CHANNELS(0);
+#undef CHANNELS
+#undef TOKENS
+#undef GO
+    return (int)cudaGetLastError();
+}
+
+}  // namespace
+
+// out [T, ldo] float32 = q | k | v | beta [H] | f [H] (ldo may pad)
+MI_EXPORT int mi_gated_delta_ready(const void* p, int ldp, const float* conv, const float* rate, const float* dt_bias, const float* state,
+                                   long long state_stride, long long ring_off, float* out, int ldo, const int* positions, const int* token_seg,
+                                   const int* seg_q_start, const int* seg_slot, int T_, int H, int KV, int D, int V, int taps, float unit_eps, int dtype,
+                                   cudaStream_t stream) {
+    if (T_ == 0) return 0;
+    if (H % KV || D > 256 || taps < 1) return -2;
+    if (dtype == MI_BF16)
+        return launch_ready<__nv_bfloat16>((const __nv_bfloat16*)p, ldp, conv, rate, dt_bias, state, state_stride, ring_off, out, ldo, positions, token_seg,
+                                           seg_q_start, seg_slot, T_, H, KV, D, V, taps, unit_eps, stream);
+    return launch_ready<float>((const float*)p, ldp, conv, rate, dt_bias, state, state_stride, ring_off, out, ldo, positions, token_seg, seg_q_start, seg_slot,
+                               T_, H, KV, D, V, taps, unit_eps, stream);
+}
+
+MI_EXPORT int mi_gated_delta_ring(const void* p, int ldp, float* state, long long state_stride, long long ring_off, const int* positions,
+                                  const int* seg_q_start, const int* seg_slot, int num_segs, int C, int taps, int dtype, cudaStream_t stream) {
+    if (num_segs == 0 || taps <= 1) return 0;
+    dim3 grid(num_segs, (C + 255) / 256);
+    if (grid.y > 65535) return -2;
+    if (dtype == MI_BF16)
+        delta_ring_kernel<__nv_bfloat16><<<grid, 256, 0, stream>>>((const __nv_bfloat16*)p, ldp, state, state_stride, ring_off, positions, seg_q_start, seg_slot, C, taps);
+    else
+        delta_ring_kernel<float><<<grid, 256, 0, stream>>>((const float*)p, ldp, state, state_stride, ring_off, positions, seg_q_start, seg_slot, C, taps);
+    return (int)cudaGetLastError();
+}
+
+// Every entry brings one token.  rows [entries, H V] in the type of p.  -2: sizes that this form does not take (V not a multiple of four, or
+// more than 16 K state entries a head); the caller then runs the prompt form.
+MI_EXPORT int mi_gated_delta_step(const void* p, int ldp, const float* conv, int taps, const float* rate, const float* dt_bias, float* state,
+                                  long long state_stride, long long ring_off, const float* norm, void* rows, const int* positions, const int* seg_q_start,
+                                  const int* seg_slot, int num_segs, int H, int KV, int D, int V, float unit_eps, float eps, int dtype, cudaStream_t stream) {
+    if (num_segs == 0) return 0;
+    if (H % KV || H > 65535 || V % 4 || V > 1024 || D > 1024 || state_stride % 4 || (uintptr_t)state % 16) return -2;
+    const int RG = 256 / (V / 4), need = (D + RG - 1) / RG;
+    if (need > 32) return -2;
+    const size_t smem = (size_t)(((2 * D + V + 3) & ~3) + RG * V) * sizeof(float);
+    const float q_scale = 1.f / sqrtf((float)D);
+    dim3 grid(num_segs, H);
+#define GO(T, NR) delta_step_kernel<T, NR><<<grid, 256, smem, stream>>>((const T*)p, ldp, conv, taps, rate, dt_bias, state, state_stride, ring_off, norm, (T*)rows, \
+                      positions, seg_q_start, seg_slot, H, KV, D, V, unit_eps, q_scale, eps)
+#define PICK(T) do { if (need <= 4) GO(T, 4); else if (need <= 8) GO(T, 8); else if (need <= 16) GO(T, 16); else GO(T, 32); } while (0)
+    if (dtype == MI_BF16) PICK(__nv_bfloat16); else PICK(float);
+#undef PICK
+#undef GO
+    return (int)cudaGetLastError();
+}

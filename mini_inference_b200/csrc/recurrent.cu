@@ -48,14 +48,16 @@ template <int N> __device__ __forceinline__ void cp_wait() { asm volatile("cp.as
 //   1  S <- diag(g) S; u = beta (v - S^T k); S <- S + k u^T       (rows q, k, g; one number beta per token and head)
 //   2  S <- diag(g) S - c (u^T S) + k v^T, both terms reading the old S   (rows q, k, g, u, c = removal rate times u)
 //   3  S <- f S + k v^T with one number f per token and head      (rows q, k; k arrives already multiplied by its input gate)
+//   4  S <- f S; u = beta (v - S^T k); S <- S + k u^T             (rows q, k; two numbers beta and f per token and head)
 // always followed by o = S^T q.
 __host__ __device__ constexpr int rows_of(int MODE) { return MODE == 1 ? 3 : MODE == 2 ? 5 : 2; }
-__host__ __device__ constexpr bool scalar_of(int MODE) { return MODE == 1 || MODE == 3; }
+__host__ __device__ constexpr int scalars_of(int MODE) { return MODE == 4 ? 2 : MODE == 1 || MODE == 3 ? 1 : 0; }
 
 // Where the scan finds a token's numbers in its float32 row (ld floats per token).
 struct ScanLayout {
     int ld, q_off, k_off, v_off, g_off, b_off;      // q/k: + kv_head * D; v: + head * V; g: + head * D; the per-token number (beta or f): + head
     int u_off, c_off;                               // MODE 2: + head * D
+    int f_off = 0;                                  // MODE 4: + head
 };
 
 // One chunk of nt tokens into a buffer: rows of Dp floats (D copied, the rest stays zero), v [COLS], the per-token number.
@@ -69,7 +71,7 @@ __device__ __forceinline__ void stage_chunk(float* buf, int Dp, int TC, const fl
     float* usm = gsm + TC * Dp;                               // MODE 2
     float* csm = usm + TC * Dp;                               // MODE 2
     float* vsm = buf + NR * TC * Dp;                          // [TC, COLS]
-    float* bsm = vsm + TC * COLS;                             // [TC] (MODE 1, 3)
+    float* bsm = vsm + TC * COLS;                             // [TC] (MODE 1, 3, 4), behind it [TC] (MODE 4: f)
     const int ncol = min(COLS, V - col0);
     if (vec) {
         const int dq = D >> 2, vq = ncol >> 2;
@@ -99,8 +101,12 @@ __device__ __forceinline__ void stage_chunk(float* buf, int Dp, int TC, const fl
             vsm[tt * COLS + c] = prep[(size_t)(tok0 + tt) * L.ld + L.v_off + h * V + col0 + c];
         }
     }
-    if (scalar_of(MODE))
-        for (int tt = threadIdx.x; tt < nt; tt += SCAN_THREADS) bsm[tt] = prep[(size_t)(tok0 + tt) * L.ld + L.b_off + h];
+    if (scalars_of(MODE))
+        for (int tt = threadIdx.x; tt < nt; tt += SCAN_THREADS) {
+            const float* row = prep + (size_t)(tok0 + tt) * L.ld;
+            bsm[tt] = row[L.b_off + h];
+            if (MODE == 4) bsm[TC + tt] = row[L.f_off + h];
+        }
 }
 
 // Sums a0 and a1 over the LN row lanes of a column pair (the low lane bits) with log2(LN) + 1 shuffles; every lane gets both.
@@ -124,7 +130,7 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(
     extern __shared__ __align__(16) float sm[];
     constexpr int LANES = LN, COLS = cols_of(LN), Dp = 4 * LN * NG, NR = rows_of(MODE);
     constexpr bool DELTA = MODE == 1;
-    const int buf_floats = TC * (NR * Dp + COLS + (scalar_of(MODE) ? 1 : 0));
+    const int buf_floats = TC * (NR * Dp + COLS + scalars_of(MODE));
     const int buf_stride = (buf_floats + 3) & ~3;
     float* part = sm + 2 * buf_stride;                         // [TC, COLS, LN + 1] partial sums of the read-out
     const int seg = blockIdx.x, h = blockIdx.y, kvh = h / (H / KV);
@@ -194,6 +200,35 @@ __global__ void __launch_bounds__(SCAN_THREADS) state_scan_kernel(
                 const float2 dot = reduce_pair<LN>(d0 + d1, e0 + e1, l);
                 const float beta = bsm[tt];
                 const float u0 = beta * (vv.x - dot.x), u1 = beta * (vv.y - dot.y);
+#pragma unroll
+                for (int g = 0; g < NG; ++g) {
+                    const float4 kv = kk[LANES * g], qv = qq[LANES * g];
+                    s0[4 * g] = fmaf(kv.x, u0, s0[4 * g]); s0[4 * g + 1] = fmaf(kv.y, u0, s0[4 * g + 1]);
+                    s0[4 * g + 2] = fmaf(kv.z, u0, s0[4 * g + 2]); s0[4 * g + 3] = fmaf(kv.w, u0, s0[4 * g + 3]);
+                    s1[4 * g] = fmaf(kv.x, u1, s1[4 * g]); s1[4 * g + 1] = fmaf(kv.y, u1, s1[4 * g + 1]);
+                    s1[4 * g + 2] = fmaf(kv.z, u1, s1[4 * g + 2]); s1[4 * g + 3] = fmaf(kv.w, u1, s1[4 * g + 3]);
+                    a0 = fmaf(s0[4 * g], qv.x, a0); a1 = fmaf(s0[4 * g + 1], qv.y, a1);
+                    a0 = fmaf(s0[4 * g + 2], qv.z, a0); a1 = fmaf(s0[4 * g + 3], qv.w, a1);
+                    b0 = fmaf(s1[4 * g], qv.x, b0); b1 = fmaf(s1[4 * g + 1], qv.y, b1);
+                    b0 = fmaf(s1[4 * g + 2], qv.z, b0); b1 = fmaf(s1[4 * g + 3], qv.w, b1);
+                }
+            } else if (MODE == 4) {
+                // S^T k of the decayed state is f times that of the old one: the decay's products fill the wait for the sum
+                float d0 = 0.f, d1 = 0.f, e0 = 0.f, e1 = 0.f;
+                const float f = bsm[TC + tt];
+#pragma unroll
+                for (int g = 0; g < NG; ++g) {
+                    const float4 kv = kk[LANES * g];
+                    d0 = fmaf(s0[4 * g], kv.x, d0); d1 = fmaf(s0[4 * g + 1], kv.y, d1);
+                    d0 = fmaf(s0[4 * g + 2], kv.z, d0); d1 = fmaf(s0[4 * g + 3], kv.w, d1);
+                    e0 = fmaf(s1[4 * g], kv.x, e0); e1 = fmaf(s1[4 * g + 1], kv.y, e1);
+                    e0 = fmaf(s1[4 * g + 2], kv.z, e0); e1 = fmaf(s1[4 * g + 3], kv.w, e1);
+                }
+                const float2 dot = reduce_pair<LN>(d0 + d1, e0 + e1, l);
+#pragma unroll
+                for (int i = 0; i < 4 * NG; ++i) { s0[i] *= f; s1[i] *= f; }
+                const float beta = bsm[tt];
+                const float u0 = beta * (vv.x - f * dot.x), u1 = beta * (vv.y - f * dot.y);
 #pragma unroll
                 for (int g = 0; g < NG; ++g) {
                     const float4 kv = kk[LANES * g], qv = qq[LANES * g];
@@ -288,7 +323,7 @@ int launch_scan(const float* prep, ScanLayout L, const float* decay, float* stat
     int NG = (D + 4 * LN - 1) / (4 * LN);
     if (LN == 8) NG = NG <= 2 ? NG : NG <= 4 ? 4 : 8;                      // the forms that exist: the kernel's rows have 4 LN NG floats
     const int COLS = cols_of(LN);
-    const int per_token = NR * 4 * LN * NG + COLS + 1;
+    const int per_token = NR * 4 * LN * NG + COLS + (scalars_of(MODE) > 1 ? scalars_of(MODE) : 1);
     const int per_chunk_token = 2 * per_token + COLS * (LN + 1);          // two staging buffers and the partial sums
     const int TC = T_ <= 4 * num_segs ? 4 : per_chunk_token * 16 * 4 <= 96 * 1024 ? 16 : per_chunk_token * 8 * 4 <= 96 * 1024 ? 8 : 4;   // decode steps: small buffers, more blocks per SM
     const size_t smem = (2 * (size_t)((TC * per_token + 3) & ~3) + (size_t)TC * COLS * (LN + 1)) * sizeof(float);
@@ -1080,4 +1115,13 @@ MI_EXPORT int mi_state_space_scan(const void* xbc, int ldx, const void* dt_in, i
     if (err) return err;
     const ScanLayout L{ldprep, 0, GN, 2 * GN, 0, 2 * GN + H * V, 0, 0};
     return launch_scan<3>(prep, L, nullptr, state, state_stride, out, seg_q_start, seg_slot, T_, num_segs, H, G, N, V, stream);
+}
+
+// prep [T, ld] float32 = q [KV D] | k [KV D] | v [H V] | beta [H] | f [H]: S <- f S; u = beta (v - S^T k); S <- S + k u^T; out = S^T q, float32 [T, H V]
+MI_EXPORT int mi_gated_delta_scan(const float* prep, int ld, float* state, long long state_stride, float* out, const int* seg_q_start,
+                                  const int* seg_slot, int T_, int num_segs, int H, int KV, int D, int V, cudaStream_t stream) {
+    if (T_ == 0) return 0;
+    const int KD = KV * D, C = 2 * KD + H * V;
+    const ScanLayout L{ld, 0, KD, 2 * KD, 0, C, 0, 0, C + H};
+    return launch_scan<4>(prep, L, nullptr, state, state_stride, out, seg_q_start, seg_slot, T_, num_segs, H, KV, D, V, stream);
 }

@@ -113,6 +113,25 @@ __global__ void head_gate_kernel(const T* __restrict__ o, const T* __restrict__ 
     for (int i = threadIdx.x; i < V; i += blockDim.x) dst[i] = from_f32<T>(to_f32(src[i]) * sg);
 }
 
+// ------------------------------------------------------------------ rows[t, i] *= sigmoid(gate[t, i]), in place
+// grid (tokens, pieces of the row); VN neighbouring entries per thread and step (1, or 16 bytes of T)
+template <typename T, int VN>
+__global__ void sigmoid_gate_kernel(T* __restrict__ rows, const T* __restrict__ gate, int gate_stride, int n) {
+    T* r = rows + (size_t)blockIdx.x * n;
+    const T* g = gate + (size_t)blockIdx.x * gate_stride;
+    for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * VN; i < n; i += gridDim.y * blockDim.x * VN) {
+        if constexpr (VN == 1) {
+            r[i] = from_f32<T>(to_f32(r[i]) / (1.f + expf(-to_f32(g[i]))));
+        } else {
+            float a[VN], b[VN];
+            load16(r + i, a);
+            load16(g + i, b);
+#pragma unroll
+            for (int e = 0; e < VN; e += 2) store2(r + i + e, a[e] / (1.f + expf(-b[e])), a[e + 1] / (1.f + expf(-b[e + 1])));
+        }
+    }
+}
+
 // ------------------------------------------------------------------ embedding -> float32 stream (+ its rows in the table's type)
 template <typename T>
 __global__ void embed_stream_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ x, T* __restrict__ rows,
@@ -270,5 +289,20 @@ MI_EXPORT int mi_head_gate(const void* o, const void* gate, int gate_stride, voi
         head_gate_kernel<__nv_bfloat16><<<grid, nt, 0, stream>>>((const __nv_bfloat16*)o, (const __nv_bfloat16*)gate, gate_stride, (__nv_bfloat16*)y, T_, H, V);
     else
         head_gate_kernel<float><<<grid, nt, 0, stream>>>((const float*)o, (const float*)gate, gate_stride, (float*)y, T_, H, V);
+    return (int)cudaGetLastError();
+}
+
+// rows [T, n] contiguous and gate (rows gate_stride apart) in one type
+MI_EXPORT int mi_sigmoid_gate(void* rows, const void* gate, int gate_stride, int T_, int n, int dtype, cudaStream_t stream) {
+    if (T_ == 0) return 0;
+    const int vn = dtype == MI_BF16 ? 8 : 4;
+    const bool vec = n % vn == 0 && gate_stride % vn == 0 && ((uintptr_t)rows | (uintptr_t)gate) % 16 == 0;
+    const int per = vec ? vn : 1, nt = n / per >= 256 ? 256 : 128;
+    const int pieces = (n + nt * per - 1) / (nt * per);
+    dim3 grid(T_, pieces < 65535 ? pieces : 65535);
+#define GO(T, VN) sigmoid_gate_kernel<T, VN><<<grid, nt, 0, stream>>>((T*)rows, (const T*)gate, gate_stride, n)
+    if (dtype == MI_BF16) { if (vec) GO(__nv_bfloat16, 8); else GO(__nv_bfloat16, 1); }
+    else { if (vec) GO(float, 4); else GO(float, 1); }
+#undef GO
     return (int)cudaGetLastError();
 }

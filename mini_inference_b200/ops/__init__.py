@@ -128,7 +128,7 @@ class CudaOps:
         self.skinny_max_rows, self.skinny_max_cols = 16, 4096    # ... where it is at least as fast as the library's
         self.fast_attention = True           # tests clear this to run the generic attention kernels in bfloat16
         self.biased_attention_tc = True      # prompts of attention with a distance table or a learned sink on the tensor cores (bfloat16)
-        self._zero_bias = {}
+        self.fused_delta_step = True         # decode steps of the delta rule with one decay per head in one kernel (tests clear this)
         self.chunked_scan = True             # prompts of a state space with one decay per head in chunks on the tensor cores (tests clear this)
         # Latent attention whose cached rows have 64 or 128 entries can run on the tensor-core paged attention kernels.  Those
         # round the softmax weights to bfloat16 before the weighted sum; a design that asks for float32 weights gets the
@@ -730,26 +730,29 @@ class CudaOps:
         self.launches += H
         return rows if side_by_side else out
 
-    def latent_prepare(self, p, q_abs, H, D, R, C, norm_w, eps, inv_freq, meta, cache, q_rows=None, dkv_col=None):
+    def latent_prepare(self, p, q_abs, H, D, R, C, norm_w, eps, inv_freq, meta, cache, q_rows=None, dkv_col=None, half_pairs=False):
         """p [T, ..] = q heads [H, D + R] | dkv [C + R] | ..; q_abs [H, T, C].  Returns q [T, H, C + R] = [q_abs | rotated
         q part]; writes the token's cache row [rmsnorm(dkv[:C]) * norm_w | rotated dkv[C:]] at its slot (cache None: no write).
-        q_rows [T, H (D + R)]: the query heads lie in a tensor of their own; dkv_col: the column of p at which dkv starts."""
+        q_rows [T, H (D + R)]: the query heads lie in a tensor of their own; dkv_col: the column of p at which dkv starts; half_pairs: the
+        rotated pairs are (i, i + n) of the first 2 n = 2 len(inv_freq) entries instead of (2i, 2i + 1)."""
         T = p.shape[0]
         assert p.stride(1) == 1 and q_abs.is_contiguous() and (q_rows is None or (q_rows.stride(1) == 1 and q_rows.dtype == p.dtype))
         q = torch.empty((T, H, C + R), dtype=p.dtype, device=p.device)
         nf = 0 if inv_freq is None else inv_freq.numel()
         _check(self.lib.mi_latent_prepare(_p(p), p.stride(0), _p(q_rows), 0 if q_rows is None else q_rows.stride(0),
                                           -1 if dkv_col is None else int(dkv_col), _p(q_abs), _p(q), _p(cache), _p(norm_w), _p(inv_freq), nf,
-                                          _p(meta.positions), _p(meta.slots), T, H, D, R, C, _c.c_float(eps), _code(p.dtype),
+                                          _p(meta.positions), _p(meta.slots), T, H, D, R, C, _c.c_float(eps), int(bool(half_pairs)), _code(p.dtype),
                                           self._stream()), "latent_prepare")
         self.launches += 1
         return q
 
-    def latent_attention(self, q, cache, meta, H, C, R, scale):
+    def latent_attention(self, q, cache, meta, H, C, R, scale, sink_values=None):
         """q [T, H, C + R] over the cached rows [c | kr] (cache [pages, 1, page, C + R]); causal softmax; the weighted
-        sum is over the rows' first C entries.  Returns [H, T, C]."""
+        sum is over the rows' first C entries.  sink_values float32 [H]: the softmax has one more term exp(sink_values[h]) without a
+        value.  Returns [H, T, C]."""
         T = q.shape[0]
-        if self.latent_tc and q.dtype == torch.bfloat16 and (C + R) in (64, 128) and meta.page_size % 16 == 0:
+        assert sink_values is None or (sink_values.dtype == torch.float32 and sink_values.numel() == H)
+        if self.latent_tc and sink_values is None and q.dtype == torch.bfloat16 and (C + R) in (64, 128) and meta.page_size % 16 == 0:
             # one shared key head of size C + R whose rows are also the values: the paged attention kernels on the tensor cores
             # take it as it is (the pool given as keys AND values); the last R columns of each head's output are dropped
             o = self.paged_attention(q.view(T, H * (C + R)), cache, cache, meta, H, 1, C + R, scale, None)
@@ -761,14 +764,18 @@ class CudaOps:
         # weights' precision where the design wants it; their output has C + R columns per head, of which the first C count.
         if (q.dtype == torch.bfloat16 and Dk in (64, 128) and meta.tile == 64 and self.fast_attention and meta.page_size % 16 == 0
                 and q.data_ptr() % 16 == 0):
-            if H <= 16 or not num_decode:
-                o = self.paged_attention(q.view(T, H * Dk), cache, cache, meta, H, 1, Dk, scale, None, split_weights=True)
-            else:
-                # the decode kernel takes up to 16 query heads per key head as the rows of its tile: more heads go in groups of 16
-                # (each group reads the cached rows once; the rows are small next to what the heads' weights cost)
-                qv = q.view(T, H * Dk)
-                o = torch.cat([self.paged_attention(qv[:, h0 * Dk:min(h0 + 16, H) * Dk], cache, cache, meta, min(16, H - h0), 1, Dk, scale, None,
-                                                    split_weights=True) for h0 in range(0, H, 16)], dim=1)
+            qv = q.view(T, H * Dk)
+            # the decode kernel takes up to 16 query heads per key head as the rows of its tile: more heads go in groups of 16
+            # (each group reads the cached rows once; the rows are small next to what the heads' weights cost)
+            step = H if H <= 16 or not num_decode else 16
+            parts = []
+            for h0 in range(0, H, step):
+                n, part = min(step, H - h0), qv[:, h0 * Dk:min(h0 + step, H) * Dk]
+                if sink_values is None:
+                    parts.append(self.paged_attention(part, cache, cache, meta, n, 1, Dk, scale, None, split_weights=True))
+                else:
+                    parts.append(self.masked_attention(part, cache, cache, meta, n, 1, Dk, Dk, scale, None, None, True, sink_values=sink_values[h0:h0 + n]))
+            o = parts[0] if len(parts) == 1 else torch.cat(parts, dim=1)
             return o.view(T, H, Dk)[:, :, :C].permute(1, 0, 2)
         out = torch.empty((H, T, C), dtype=q.dtype, device=q.device)
         buf, hs, ts = out, T * C, C
@@ -776,7 +783,7 @@ class CudaOps:
             _check(self.lib.mi_latent_prefill(_p(q), _p(cache), _p(buf), _p(meta.prefill_tiles), num_tiles, _p(meta.seg_q_start),
                                               _p(meta.seg_pos0), _p(meta.block_table), _p(meta.table_rows), meta.max_pages,
                                               _c.c_longlong(hs), _c.c_longlong(ts), H, C, R, meta.page_size, meta.tile,
-                                              _c.c_float(scale), code, self._stream()), "latent_prefill")
+                                              _c.c_float(scale), _p(sink_values), code, self._stream()), "latent_prefill")
             self.launches += 1
         if num_decode:
             S = self.choose_splits(num_decode * math.ceil(H / 4), meta.max_kv_len, 2)
@@ -787,7 +794,7 @@ class CudaOps:
             _check(self.lib.mi_latent_decode(_p(q), _p(cache), _p(buf), _p(o_part), _p(lse), _p(meta.decode_segs), num_decode,
                                              _p(meta.seg_q_start), _p(meta.seg_kv_len), _p(meta.block_table), _p(meta.table_rows),
                                              meta.max_pages, _c.c_longlong(hs), _c.c_longlong(ts), H, C, R, meta.page_size, S,
-                                             _c.c_float(scale), code, self._stream()), "latent_decode")
+                                             _c.c_float(scale), _p(sink_values), code, self._stream()), "latent_decode")
             self.launches += 2 if S > 1 else 1
         return out
 
@@ -844,13 +851,14 @@ class CudaOps:
 
     # ---------------------------------------------------------------- attention with a block mask, a sink and unit-norm q, k
     def unit_qk_cache(self, p, H, KV, D, V, eps, lam, source, meta, k_cache, v_cache, q_weight=None, k_weight=None, q_temp=None,
-                      values_are_keys=False):
+                      values_are_keys=False, inv_freq=None):
         """p [T, H D + KV D + KV V] = q | k | v.  q and k are divided by their root mean square per head (eps None: left as they
         are), q in place; v becomes (1 - lam) v + lam source when source [T, KV V] (another layer's values, a view is allowed) is
         given; k and v go to the rows' slots of the caches (None: this layer writes none).  Returns the q view.
         q_weight, k_weight float32 [D]: multiplied in after the division (shared by all heads); q_temp (coef, every): q at position p
         is multiplied by 1 + coef * ln(floor((p + 1) / every) + 1); values_are_keys: p has no v columns and the cached values are
-        the keys as projected, before the norm."""
+        the keys as projected, before the norm; inv_freq float32 [n]: the first 2 n coordinates of every q and k head are then turned by
+        the token's position (rotate-half)."""
         T = p.shape[0]
         assert p.is_contiguous() and p.shape[1] == (H + KV) * D + (0 if values_are_keys else KV * V)
         assert source is None or (source.stride(1) == 1 and source.dtype == p.dtype and lam is not None)
@@ -858,8 +866,9 @@ class CudaOps:
         coef, every = q_temp if q_temp else (0.0, 0)
         _check(self.lib.mi_normed_qk_cache(_p(p), p.stride(0), _p(source), 0 if source is None else source.stride(0), _p(lam if source is not None else None),
                                            _p(meta.slots), _p(k_cache), _p(v_cache), T, H, KV, D, V, meta.page_size,
-                                           _c.c_float(eps or 0.0), int(eps is not None), _p(q_weight), _p(k_weight), _p(meta.positions if q_temp else None),
-                                           _c.c_float(coef), int(every), int(bool(values_are_keys)), _code(p.dtype), self._stream()), "unit_qk_cache")
+                                           _c.c_float(eps or 0.0), int(eps is not None), _p(q_weight), _p(k_weight),
+                                           _p(meta.positions if q_temp or inv_freq is not None else None), _c.c_float(coef), int(every),
+                                           int(bool(values_are_keys)), _p(inv_freq), 0 if inv_freq is None else inv_freq.numel(), _code(p.dtype), self._stream()), "unit_qk_cache")
         self.launches += 1
         return p[:, :H * D]
 
@@ -910,8 +919,8 @@ class CudaOps:
         elif (num_tiles and not extended and self.fast_attention and self.biased_attention_tc and q.dtype == torch.bfloat16 and D == V and D in (64, 128)
                 and meta.tile == 64 and q.stride(0) % 8 == 0 and q.data_ptr() % 16 == 0):
             # the same kernel with the learned sink's score and the distance table (one row per head) in its softmax
-            no_table = slopes is not None and distance_bias is None and distance_bias_by_head is None        # slopes alone: the kernel reads no table
-            bias_t = None if no_table else self._bias_rows_by_head(distance_bias, distance_bias_by_head, H, q.device)
+            no_table = distance_bias is None and distance_bias_by_head is None        # slopes or a learned sink alone: the kernel reads no table
+            bias_t = None if no_table else self._bias_rows_by_head(distance_bias, distance_bias_by_head)
             args = (_p(q), q.stride(0), _p(k_cache), _p(v_cache), _p(out), _p(meta.prefill_tiles), num_tiles, _p(meta.seg_q_start),
                     _p(meta.seg_pos0), _p(meta.block_table), _p(rows), meta.max_pages, H, KV, D, meta.page_size, meta.tile,
                     _c.c_float(scale), win, blk, int(bool(sink)), _p(sink_values), _p(bias_t), 0 if no_table else bias_t.shape[1] - 1)
@@ -954,16 +963,13 @@ class CudaOps:
             elif plain:
                 _check(self.lib.mi_attn_decode_mma_rows_masked(*args, self._stream()), "attn_decode_mma_masked")
             else:                                          # the learned sink's score and the distance table (one row per head) in the softmax
+                no_table = distance_bias is None and distance_bias_by_head is None             # slopes or a learned sink alone: the kernel reads no table
+                bias_t = None if no_table else self._bias_rows_by_head(distance_bias, distance_bias_by_head)
+                args += (_p(sink_values), _p(bias_t), 0 if no_table else bias_t.shape[1] - 1)
                 if slopes is None:
-                    bias_t = self._bias_rows_by_head(distance_bias, distance_bias_by_head, H, q.device)
-                    _check(self.lib.mi_attn_decode_mma_rows_biased(*args, _p(sink_values), _p(bias_t), bias_t.shape[1] - 1, self._stream()),
-                           "attn_decode_mma_biased")
-                elif distance_bias is None and distance_bias_by_head is None:                 # slopes alone: the kernel reads no table
-                    _check(self.lib.mi_attn_decode_mma_rows_sloped(*args, _p(sink_values), _p(None), 0, _p(slopes), self._stream()), "attn_decode_mma_sloped")
+                    _check(self.lib.mi_attn_decode_mma_rows_biased(*args, self._stream()), "attn_decode_mma_biased")
                 else:
-                    bias_t = self._bias_rows_by_head(distance_bias, distance_bias_by_head, H, q.device)
-                    _check(self.lib.mi_attn_decode_mma_rows_sloped(*args, _p(sink_values), _p(bias_t), bias_t.shape[1] - 1, _p(slopes), self._stream()),
-                           "attn_decode_mma_sloped")
+                    _check(self.lib.mi_attn_decode_mma_rows_sloped(*args, _p(slopes), self._stream()), "attn_decode_mma_sloped")
             self.launches += 1
             if S > 1 and counters is None:
                 _check(self.lib.mi_attn_decode_merge(_p(o_part), _p(lse), _p(out), _p(meta.decode_segs), num_decode,
@@ -984,18 +990,13 @@ class CudaOps:
             self.launches += 2 if S > 1 else 1
         return out
 
-    def _bias_rows_by_head(self, distance_bias, by_head, H, device):
-        """The distance table [far + 1, H] one row per head, [H, far + 1]: the caller's own copy if it keeps one, else made here;
-        no table at all (a learned sink alone): one zero a head."""
+    @staticmethod
+    def _bias_rows_by_head(distance_bias, by_head):
+        """The distance table [far + 1, H] one row per head, [H, far + 1]: the caller's own copy if it keeps one, else made here."""
         if by_head is not None:
-            assert by_head.dtype == torch.float32 and by_head.is_contiguous() and by_head.shape[0] == H
+            assert by_head.dtype == torch.float32 and by_head.is_contiguous()
             return by_head
-        if distance_bias is not None:
-            return distance_bias.t().contiguous()
-        zero = self._zero_bias.get(H)
-        if zero is None:
-            zero = self._zero_bias[H] = torch.zeros((H, 1), dtype=torch.float32, device=device)
-        return zero
+        return distance_bias.t().contiguous()
 
     # ---------------------------------------------------------------- retention
     def retention_scan(self, p, H, D, V, inv_freq, k_scale, decay, state, batch):
@@ -1364,6 +1365,72 @@ class CudaOps:
                "state_space_scan")
         self.launches += 2
         return y
+
+    # ---------------------------------------------------------------- layer norms on both sides, element gate, delta rule with one decay per head
+    def stream_layernorm(self, x, delta, pre_add, weight, eps, rows, out_dtype):
+        """v = x + pre_add + L(y) * w_y with delta = NormedDelta(y, w_y, ..), each of the two may be None; L(z) = (z - mean) / sqrt(var + eps).
+        Returns L(v) * weight in out_dtype and leaves v in x (float32 stream); weight None: returns v itself in out_dtype and leaves x as it
+        is.  rows: only these rows are normed and the stream is left as it is.  pre_add: float32 [T, hidden].  One kernel."""
+        hidden = x.shape[-1]
+        n = x.shape[0] if rows is None else rows.shape[0]
+        out = torch.empty((n, hidden), dtype=out_dtype, device=x.device)
+        assert x.dtype == torch.float32 and x.is_contiguous()
+        assert pre_add is None or (pre_add.dtype == torch.float32 and pre_add.is_contiguous() and pre_add.shape == x.shape)
+        y = wy = None
+        eps_y = 0.0
+        if delta is not None:
+            y, wy, eps_y = delta.y, delta.weight, delta.eps
+            assert y.is_contiguous() and y.shape == x.shape and y.dtype == out_dtype and wy.dtype == torch.float32
+        _check(self.lib.mi_stream_layernorm(_p(x), _p(y), _p(wy), _c.c_float(eps_y), _p(pre_add), _p(weight), _p(out), _p(rows), n, hidden, _c.c_float(eps),
+                                            int(weight is None), _code(out_dtype), _code(out_dtype), self._stream()), "stream_layernorm")
+        self.launches += 1
+        return out
+
+    def sigmoid_gate(self, rows, gate):
+        """rows [T, n] *= sigmoid(gate), in place; gate [T, n] may be a strided view."""
+        assert rows.is_contiguous() and gate.shape == rows.shape and gate.stride(1) == 1 and gate.dtype == rows.dtype
+        _check(self.lib.mi_sigmoid_gate(_p(rows), _p(gate), gate.stride(0), rows.shape[0], rows.shape[1], _code(rows.dtype), self._stream()), "sigmoid_gate")
+        self.launches += 1
+        return rows
+
+    def gated_delta_mix(self, p, conv, taps, rate, dt_bias, H, KV, D, V, unit_eps, norm, eps, state, batch):
+        """p [T, >= C + H V + 2 H] = q | k | v | gate | b | a as projected (C = 2 KV D + H V).  q, k, v pass the convolution and silu, q and k
+        become unit vectors (q * D^-1/2); beta = sigmoid(b), f = exp(-rate softplus(a + dt_bias)); S <- f S, u = beta (v - S^T k),
+        S <- S + k u^T, o = S^T q from the slot's state (float32 H D V; behind it the ring of inputs [taps, C]).  Returns the rows
+        o / rms(o) * norm * silu(gate) per head in p's dtype."""
+        T, C, ring = p.shape[0], 2 * KV * D + H * V, H * D * V
+        assert p.stride(1) == 1 and p.shape[1] >= C + H * V + 2 * H and conv.dtype == torch.float32 and conv.is_contiguous() and conv.shape == (C, taps)
+        assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] >= ring + (taps * C if taps > 1 else 0)
+        code, stride = _code(p.dtype), (_c.c_longlong(state.stride(0)), _c.c_longlong(ring))
+        if T == batch.num_segs and self.fused_delta_step:   # every entry brings one token
+            rows = torch.empty((T, H * V), dtype=p.dtype, device=p.device)
+            rc = self.lib.mi_gated_delta_step(_p(p), p.stride(0), _p(conv), taps, _p(rate), _p(dt_bias), _p(state), *stride, _p(norm), _p(rows), _p(batch.positions),
+                                              _p(batch.seg_q_start), _p(batch.seg_slot), T, H, KV, D, V, _c.c_float(unit_eps), _c.c_float(eps), code, self._stream())
+            if rc == 0:
+                self.launches += 1
+                return rows
+            if rc != -2:
+                _check(rc, "gated_delta_step")
+        prep = torch.empty((T, (C + 2 * H + 3) // 4 * 4), dtype=torch.float32, device=p.device)
+        _check(self.lib.mi_gated_delta_ready(_p(p), p.stride(0), _p(conv), _p(rate), _p(dt_bias), _p(state), *stride, _p(prep), prep.stride(0), _p(batch.positions),
+                                             _p(batch.token_seg), _p(batch.seg_q_start), _p(batch.seg_slot), T, H, KV, D, V, taps, _c.c_float(unit_eps), code,
+                                             self._stream()), "gated_delta_ready")
+        o = self.gated_delta_scan(prep, H, KV, D, V, state, batch)
+        if taps > 1:
+            _check(self.lib.mi_gated_delta_ring(_p(p), p.stride(0), _p(state), *stride, _p(batch.positions), _p(batch.seg_q_start), _p(batch.seg_slot), batch.num_segs,
+                                                C, taps, code, self._stream()), "gated_delta_ring")
+        self.launches += 2 if taps > 1 else 1
+        return self.group_rmsnorm_gate(o, norm, p[:, C:C + H * V], eps, H, V, p.dtype, act="silu")
+
+    def gated_delta_scan(self, prep, H, KV, D, V, state, batch):
+        """prep float32 [T, ..] = q [KV D] | k [KV D] | v [H V] | beta [H] | f [H]; S <- f S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q
+        token by token.  float32 [T, H V]."""
+        T = prep.shape[0]
+        out = torch.empty((T, H * V), dtype=torch.float32, device=prep.device)
+        _check(self.lib.mi_gated_delta_scan(_p(prep), prep.stride(0), _p(state), _c.c_longlong(state.stride(0)), _p(out), _p(batch.seg_q_start), _p(batch.seg_slot),
+                                            T, batch.num_segs, H, KV, D, V, self._stream()), "gated_delta_scan")
+        self.launches += 1
+        return out
 
     # ---------------------------------------------------------------- sampling
     def argmax(self, logits):

@@ -64,6 +64,10 @@ a block reads the attributes, it never probes with hasattr:
                                with residual="float32" needs it of all its norms
   takes_pair_delta = True  Norm: forward accepts a PairDelta as `delta` (two sublayers' outputs and a bias vector, added to the
                                stream in float32 inside the norm's kernel) and pre_add=<float32 [T, hidden]> (added row by row)
+  takes_normed_delta = True
+                           Norm: forward accepts a NormedDelta as `delta` (a sublayer's output that is normed itself before it is added
+                               to the stream, all in the norm's kernel) and pre_add=<float32 [T, hidden]>; output_delta(y) makes one of
+                               this norm's weights; stream_rows(x, delta, ctx) gives the rows of x + delta in the run's dtype, not normed
   absolute_table           Position: a learned [rows, hidden] table; the kernel that starts a float32 stream adds row p to the token
                                at position p (on_embedding then has nothing left to do)
   takes_next_weight = True Norm: forward accepts next_weight=<tensor> and passes it to ctx.ops.add_rmsnorm: the block
@@ -157,6 +161,16 @@ class PairDelta:
         self.a, self.b, self.bias = a, b, bias
 
 
+class NormedDelta:
+    """A sublayer's output y that passes a norm of its own before it joins the residual stream: the stream receives norm(y) with the
+    given float32 weight and epsilon.  Only norms that declare takes_normed_delta understand it; a block hands it to the next norm,
+    whose kernel norms y, adds it to the stream in float32 and norms the sum."""
+    __slots__ = ("y", "weight", "eps")
+
+    def __init__(self, y, weight, eps):
+        self.y, self.weight, self.eps = y, weight, eps
+
+
 class LayerCache:
     """What one execution step's mixer gets from the cache manager: for pages, the step's key
     and value pools [pages, kv_heads, page_size, head_dim] and the index of the cache group
@@ -208,7 +222,9 @@ class Part:
     keeps_float32_stream = False     # Norm: reads and writes a float32 residual stream whatever the run's dtype, takes pre_add=
     takes_gated_delta = False        # Norm: `delta` may be a GatedDelta, applied to the stream in the norm's kernel
     takes_pair_delta = False         # Norm: `delta` may be a PairDelta; pre_add may be a [T, hidden] float32 tensor added row by row
+    takes_normed_delta = False       # Norm: `delta` may be a NormedDelta; offers output_delta(y) and stream_rows(x, delta, ctx)
     adds_to_embedding = False        # Position: owns an absolute_table (known before the weights are loaded)
+    interleaved = False              # Position: coordinates 2i and 2i+1 are rotated together (otherwise i and i + half the rotated ones)
     absolute_table = None            # Position: a [rows, hidden] table whose row p the embedding kernel adds to the token at position p
     # Mixer: a step that reads an earlier step's pages (ExecStep.cache_from) still keeps the states its cache_need() declares for itself;
     # the pages are kept long enough for the windows of all who read them

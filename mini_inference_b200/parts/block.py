@@ -220,3 +220,37 @@ class ParallelPreNormBlock(Part):
 class ParallelPreNormMixerOnly(ParallelPreNormBlock):
     """A layer without feed-forward: x <- x + mixer(norm1(x)), in the same float32 arithmetic."""
     roles = {"mixer": "mixer", "norm1": "norm", "position": "position"}
+
+
+@register_block("sandwich")
+class SandwichBlock(Part):
+    """A norm before and behind each sublayer:  x <- x + norm1b(mixer(norm1(x)));  x <- x + norm2b(feed_forward(norm2(x))).
+    The stream is float32.  Each output travels as a NormedDelta to the next norm, whose kernel norms it, adds it to the stream in
+    float32 and norms the sum.  pre_add: float32 rows added to the stream before this layer, in the first norm's kernel."""
+    roles = {"mixer": "mixer", "feed_forward": "feed_forward", "norm1": "norm", "norm1b": "norm", "norm2": "norm", "norm2b": "norm",
+             "position": "position"}
+
+    def __init__(self, spec, parts):
+        super().__init__(spec)
+        self.parts = dict(parts)
+        self.mixer, self.feed_forward, self.position = parts["mixer"], parts.get("feed_forward"), parts["position"]
+        self.norm1, self.norm1b, self.norm2, self.norm2b = parts["norm1"], parts["norm1b"], parts.get("norm2"), parts.get("norm2b")
+        if not all(n.takes_normed_delta for n in (self.norm1, self.norm1b, self.norm2, self.norm2b) if n is not None):
+            raise ValueError("the arrangement with norms on both sides needs norms that add a normed output (takes_normed_delta)")
+
+    def norms(self):
+        return [n for n in (self.norm1, self.norm2) if n is not None]
+
+    def forward(self, x, delta, ctx, cache, owns_cache=True, pre_add=None):
+        n = self.norm1.forward(x, delta, ctx, pre_add=pre_add)
+        a = self.norm1b.output_delta(self.mixer.forward(n, ctx, cache, self.position, owns_cache))
+        if self.feed_forward is None:
+            return x, a
+        n = self.norm2.forward(x, a, ctx)
+        return x, self.norm2b.output_delta(self.feed_forward.forward(n, ctx))
+
+
+@register_block("sandwich_mixer")
+class SandwichMixerOnly(SandwichBlock):
+    """A layer without feed-forward: x <- x + norm1b(mixer(norm1(x)))."""
+    roles = {"mixer": "mixer", "norm1": "norm", "norm1b": "norm", "position": "position"}

@@ -13,14 +13,17 @@ for prompt portions and decoded tokens alike; neither keys nor values of a head 
 
 Options: rot_dim=0 (no rotated part: the cached row is the latent alone and positions do not enter); gate=False (no
 per-head output gate, no tensor `g`); q_rank=n (the queries pass a latent of their own: c_q = rmsnorm(W_dq h) * w with the
-tensor `dq.norm`, q = W_uq c_q; tensors `dq`, `dq.norm`, `uq` instead of `q`).
+tensor `dq.norm`, q = W_uq c_q; tensors `dq`, `dq.norm`, `uq` instead of `q`); gate="elements" (the concatenated heads are multiplied
+element by element with sigmoid(W_g h), `g` [H value_dim, hidden]); sink=True (the softmax has one more term exp(sink_h), a learned
+number per head, which carries no value and is not scaled).  The position part chooses the pairs that are rotated (interleaved or
+rotate-half).
 """
 from __future__ import annotations
 
 import torch
 
 from .attention import paged_attention_step_arrays
-from .base import KVCacheNeed, Part, WeightSpec, register_mixer
+from .base import KVCacheNeed, Part, WeightSpec, pad_rows, register_mixer
 
 
 @register_mixer("latent_attention")
@@ -34,9 +37,12 @@ class LatentAttention(Part):
         self.hidden, self.H = int(g("hidden_size")), int(g("num_heads"))
         self.D, self.R, self.V, self.C = int(g("nope_dim")), int(g("rot_dim")), int(g("value_dim")), int(g("kv_rank"))
         self.scale, self.eps = float(g("scale")), float(g("latent_norm_eps"))
-        self.gate = bool(g("gate", True))
+        self.gate = {True: "heads", False: None}.get(g("gate", True), g("gate", True))       # "heads" | "elements" | None
+        if self.gate not in (None, "heads", "elements"):
+            raise ValueError("latent_attention: gate is heads, elements or none")
+        self.sink = bool(g("sink", False))
         self.q_rank = int(g("q_rank")) if g("q_rank") else None
-        self.proj = self.uk_t = self.uv = self.o = self.latent_norm = self.uq = self.q_norm = None
+        self.proj = self.uk_t = self.uv = self.o = self.latent_norm = self.uq = self.q_norm = self.sink_values = None
 
     def weight_specs(self):
         H, D, R, V, C, hid = self.H, self.D, self.R, self.V, self.C, self.hidden
@@ -47,8 +53,10 @@ class LatentAttention(Part):
             specs = [WeightSpec("q", (H * (D + R), hid))]
         specs += [WeightSpec("dkv", (C + R, hid)), WeightSpec("dkv.norm", (C,), kind="vector", init="norm"),
                   WeightSpec("uk", (H * D, C)), WeightSpec("uv", (H * V, C))]
+        if self.sink:
+            specs.append(WeightSpec("sink", (H,), kind="vector"))
         if self.gate:
-            specs.append(WeightSpec("g", (H, hid)))
+            specs.append(WeightSpec("g", (H * V if self.gate == "elements" else H, hid)))
         return specs + [WeightSpec("o", (hid, H * V))]
 
     def cache_need(self):
@@ -58,6 +66,10 @@ class LatentAttention(Part):
         H, D, V, C = self.H, self.D, self.V, self.C
         first = [tensors.pop("dq")] if self.q_rank else [tensors.pop("q")]                                     # q (or its latent) | c, kr | gate
         self.proj = torch.cat(first + [tensors.pop("dkv")] + ([tensors.pop("g")] if self.gate else []), dim=0).contiguous()
+        if self.gate == "elements":
+            self.proj = pad_rows(self.proj, 8)                                         # the rows of the product start on 16 bytes
+        if self.sink:
+            self.sink_values = tensors.pop("sink").float().contiguous()
         if self.q_rank:
             self.uq, self.q_norm = tensors.pop("uq"), tensors.pop("dq.norm").float().contiguous()
         self.uk_t = tensors.pop("uk").view(H, D, C).transpose(1, 2).contiguous()       # [H, C, D]: q_abs_h = uk_t_h q_u
@@ -86,21 +98,24 @@ class LatentAttention(Part):
     def forward_open(self, h, ctx, cache, position, owns_cache=True):
         ops, H, D, R, V, C = ctx.ops, self.H, self.D, self.R, self.V, self.C
         meta = ctx.batch.group_view(cache.group, self.step_arrays_key)
-        p = ops.linear(h, self.proj)                                               # [T, H (D + R) + C + R + H]
-        if self.q_rank:                                                            # p = c_q as projected | c, kr | gate
+        p = ops.linear(h, self.proj)                                               # q [H (D + R)], or c_q as projected | c, kr | gate
+        turn = dict(half_pairs=not position.interleaved)
+        pages = cache.k if owns_cache else None
+        if self.q_rank:
             qp = ops.linear(ops.rows_rmsnorm(p[:, :self.q_rank], self.q_norm, self.eps), self.uq)
             q_abs = ops.batched_linear(qp, 0, D + R, D, self.uk_t)
-            q = ops.latent_prepare(p, q_abs, H, D, R, C, self.latent_norm, self.eps, position.rotary_inv_freq(), meta,
-                                   cache.k if owns_cache else None, q_rows=qp, dkv_col=self.q_rank)
+            q = ops.latent_prepare(p, q_abs, H, D, R, C, self.latent_norm, self.eps, position.rotary_inv_freq(), meta, pages, q_rows=qp,
+                                   dkv_col=self.q_rank, **turn)
             gate_col = self.q_rank + C + R
         else:
             q_abs = ops.batched_linear(p, 0, D + R, D, self.uk_t)                  # [H, T, C]
-            q = ops.latent_prepare(p, q_abs, H, D, R, C, self.latent_norm, self.eps, position.rotary_inv_freq(), meta,
-                                   cache.k if owns_cache else None)                # [T, H, C + R]; [c | kr] -> the pages
+            q = ops.latent_prepare(p, q_abs, H, D, R, C, self.latent_norm, self.eps, position.rotary_inv_freq(), meta, pages,
+                                   **turn)                                         # [T, H, C + R]; [c | kr] -> the pages
             gate_col = H * (D + R) + C + R
-        o_lat = ops.latent_attention(q, cache.k, meta, H, C, R, self.scale)        # [H, T, C]
-        if not self.gate:                                                          # no gate: the products write the heads side by side
-            return ops.batched_linear(o_lat, None, None, C, self.uv, side_by_side=True), self.o
-        o = ops.batched_linear(o_lat, None, None, C, self.uv)                      # [H, T, V]
-        rows = ops.head_gate(o, p[:, gate_col:], ctx.dtype)                        # [T, H V]
-        return rows, self.o
+        term = dict(sink_values=self.sink_values) if self.sink else {}
+        o_lat = ops.latent_attention(q, cache.k, meta, H, C, R, self.scale, **term)     # [H, T, C]
+        if self.gate == "heads":
+            o = ops.batched_linear(o_lat, None, None, C, self.uv)                  # [H, T, V]
+            return ops.head_gate(o, p[:, gate_col:], ctx.dtype), self.o            # [T, H V]
+        rows = ops.batched_linear(o_lat, None, None, C, self.uv, side_by_side=True)     # the products write the heads side by side
+        return (ops.sigmoid_gate(rows, p[:, gate_col:gate_col + H * V]) if self.gate else rows), self.o

@@ -68,11 +68,17 @@ class DecoderModel:
                                  (spec.residual != "float32" or spec.embedding_norm is not None or spec.embedding_part is not None)):
             raise ValueError("a position table and an embedding scale belong to the plain start of a float32 stream, one table at most")
         self._adds_embedding = any(step.add_embedding for step in spec.order)
+        self._joins = any(step.join_embedding for step in spec.order)
+        if self._joins and (spec.embedding_part is not None or spec.embedding_norm is not None or self._absolute is not None or spec.embedding_scale != 1.0):
+            raise ValueError("a stream that is joined with the embedded tokens starts as the plain rows of the embedding table")
+        if self._joins and not all(lookup("norm", spec.layers[s.layer].part("norm1").kind).takes_normed_delta for s in spec.order if s.join_embedding):
+            raise ValueError("a layer behind a join needs a first norm that hands out the stream's own rows (takes_normed_delta)")
         for ws in self.final_norm.weight_specs():
             self._owned.append((spec.final_norm_name, ws, self.final_norm))
         self.embedding = None
         self.lm_head = None
         self.pass_vectors = None
+        self.join_stream = self.join_embedded = None           # the two halves of the joining product's weight
         self.dtype = None
         self.device = None
 
@@ -90,6 +96,8 @@ class DecoderModel:
         if self.spec.pass_vectors_name is not None:
             table.append((self.spec.pass_vectors_name, WeightSpec("pass_vectors", (self.spec.pass_vectors_rows, self.spec.hidden_size),
                                                                   kind="vector")))
+        if self.spec.join_name is not None:
+            table.append((self.spec.join_name, WeightSpec("join", (self.spec.hidden_size, 2 * self.spec.hidden_size))))
         if self.spec.lm_head_name is not None:
             table.append((self.spec.lm_head_name, WeightSpec("lm_head", (self.spec.vocab_size, self.spec.hidden_size))))
         return table
@@ -116,6 +124,9 @@ class DecoderModel:
         if self.spec.pass_vectors_name is not None:            # added to a float32 stream or to one of the run's dtype
             pv = tensors[self.spec.pass_vectors_name]
             self.pass_vectors = (pv.float() if self.spec.residual == "float32" else pv.to(dtype)).contiguous()
+        if self.spec.join_name is not None:
+            joint, W = tensors[self.spec.join_name], self.spec.hidden_size
+            self.join_stream, self.join_embedded = joint[:, :W].contiguous(), joint[:, W:].contiguous()
         self.lm_head = self.embedding if self.spec.lm_head_name is None else tensors[self.spec.lm_head_name]
 
     def matrix_weights(self):
@@ -124,6 +135,8 @@ class DecoderModel:
         for block in self.blocks:
             for part in self._parts_of(block):
                 out += [v for v in vars(part).values() if isinstance(v, torch.Tensor) and v.dim() == 2 and v.is_floating_point()]
+        if self.join_stream is not None:
+            out += [self.join_stream, self.join_embedded]
         out.append(self.lm_head)
         return out
 
@@ -165,7 +178,11 @@ class DecoderModel:
         """Floating-point operations of a step that feeds `rows` tokens which see `pairs` (query, key) pairs in all and
         wants logits for `logit_rows` of them: 2 per weight element and row, plus what the mixers report."""
         total = 2 * logit_rows * self.lm_head.numel()
+        if self._joins:
+            total += 2 * rows * self.join_embedded.numel()
         for step in self.spec.order:
+            if step.join_embedding:
+                total += 2 * rows * self.join_stream.numel()
             for part in self._parts_of(self.blocks[step.layer]):
                 total += 2 * rows * sum(v.numel() for v in vars(part).values()
                                         if isinstance(v, torch.Tensor) and v.dim() == 2 and v.is_floating_point())
@@ -228,12 +245,18 @@ class DecoderModel:
             x = position.on_embedding(x, ctx)
         delta = None
         entered = x.clone() if self._adds_embedding else None  # the stream is rewritten in place; the passes add what entered it
+        # W [x; x0] = W_x x + W_0 x0: the second half is the same for every pass, so it is made once, in float32, and the norm that
+        # opens a pass adds it to the new stream
+        joined = ops.linear(ctx.rows_of(x), self.join_embedded, out_dtype=torch.float32) if self._joins else None
         for i, step in enumerate(self.spec.order):
             block = self.blocks[step.layer]
             cache = caches[i if step.cache_from is None else step.cache_from]
             if step.cache_from is not None and block.mixer.keeps_states_when_borrowing:
                 cache = cache.with_states(caches[i])
-            if step.add_embedding:
+            if step.join_embedding:
+                x = ops.linear(block.parts["norm1"].stream_rows(x, delta, ctx), self.join_stream, out_dtype=torch.float32)
+                x, delta = block.forward(x, None, ctx, cache, step.cache_from is None, pre_add=joined)
+            elif step.add_embedding:
                 x, delta = block.forward(x, delta, ctx, cache, step.cache_from is None, pre_add=entered)
             elif step.add_row is None:
                 x, delta = block.forward(x, delta, ctx, cache, step.cache_from is None)

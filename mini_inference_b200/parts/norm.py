@@ -5,7 +5,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import PairDelta, Part, WeightSpec, register_norm
+from .base import NormedDelta, PairDelta, Part, WeightSpec, register_norm
 
 
 @register_norm("rmsnorm")
@@ -147,3 +147,33 @@ class SumRMSNorm(Part):
 
     def forward(self, x, delta, ctx, rows=None, pre_add=None):
         raise TypeError("sum_rmsnorm norms the sum of the stream and a sublayer's output (norm_sum); it hands out no rows of its own")
+
+
+@register_norm("stream_layernorm")
+class StreamLayerNorm(Part):
+    """Layer norm without a bias on a float32 residual stream: y = (x - mean) / sqrt(variance + eps) * w, the variance being the mean of
+    the squared deviations; rows handed out in the run's dtype.  It stands before a sublayer (forward) or behind one (output_delta: the
+    sublayer's output travels as a NormedDelta to the next norm before a sublayer, whose kernel norms it, adds it and norms the sum)."""
+    keeps_float32_stream = True
+    takes_normed_delta = True
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        self.size, self.eps = int(spec.get("size")), float(spec.get("eps"))
+        self.weight = None
+
+    def weight_specs(self):
+        return [WeightSpec("weight", (self.size,), kind="vector", init="norm")]
+
+    def load(self, tensors, dtype, device):
+        self.weight = tensors["weight"].float().contiguous()
+
+    def output_delta(self, y):
+        return NormedDelta(y, self.weight, self.eps)
+
+    def forward(self, x, delta, ctx, rows=None, pre_add=None):
+        return ctx.ops.stream_layernorm(x, delta, pre_add, self.weight, self.eps, rows, ctx.dtype)
+
+    def stream_rows(self, x, delta, ctx):
+        """The rows of x + delta in the run's dtype, not normed; x itself is left as it is (whoever asks replaces the stream)."""
+        return ctx.rows_of(x) if delta is None else ctx.ops.stream_layernorm(x, delta, None, None, self.eps, None, ctx.dtype)

@@ -401,3 +401,62 @@ class Mamba2(Part):
         rows = ops.mamba2_mix(p, self.conv, self.conv_b, self.taps, self.dt_bias, self.A, self.Dv, self.H, self.V, self.N, self.G,
                               self.norm, self.parts, self.eps, cache.state, ctx.batch)
         return ops.linear(rows, self.o)
+
+
+@register_mixer("gated_delta")
+class GatedDeltaRule(Part):
+    """The gated delta rule with ONE decay per head and token (head h reads the q and k of group floor(h / (heads / kv_heads))):
+        q, k, v = silu(conv(W h)) (causal, per channel, conv_taps taps);  q, k <- x / sqrt(sum x^2 + unit_eps), q also * key_dim^-1/2;
+        beta = sigmoid(W_b h),  g = exp(-exp(A_log) softplus(W_a h + dt_bias))   (one of each per head);
+        S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q;
+    rows: per head o / rms(o) * weight [value_dim], * silu(W_g h); then W_o.
+    The state slot holds S (float32 [heads, key_dim, value_dim]) and behind it the convolution's inputs of the last conv_taps positions,
+    a ring in which position p has row p mod conv_taps (one more than a token looks back on, so that the kernel which appends a token's
+    own inputs overwrites nothing that its other blocks read).  A decode step is one kernel; prompts are made ready (convolution, norms,
+    gates) by one kernel and scanned by another."""
+
+    def __init__(self, spec):
+        super().__init__(spec)
+        g = spec.get
+        self.hidden, self.H, self.KV = int(g("hidden_size")), int(g("num_heads")), int(g("num_kv_heads"))
+        self.D, self.V, self.taps = int(g("key_dim")), int(g("value_dim")), int(g("conv_taps"))
+        self.eps, self.unit_eps = float(g("out_norm_eps")), float(g("unit_eps"))
+        if self.H % self.KV or self.taps < 1:
+            raise ValueError(f"gated_delta: {self.H} heads on {self.KV} key heads, {self.taps} taps")
+        self.C = 2 * self.KV * self.D + self.H * self.V             # channels that pass the short convolution
+        self.proj = self.conv = self.rate = self.dt_bias = self.norm = self.o = None
+
+    def weight_specs(self):
+        H, KV, D, V, hid, taps = self.H, self.KV, self.D, self.V, self.hidden, self.taps
+        specs = []
+        for n, rows in (("q", KV * D), ("k", KV * D), ("v", H * V)):
+            specs += [WeightSpec(n, (rows, hid)), WeightSpec(n + ".conv", (rows, taps), kind="vector")]
+        return specs + [WeightSpec("b", (H, hid)), WeightSpec("A_log", (H,), kind="vector", init="zeros"),
+                        WeightSpec("norm", (V,), kind="vector", init="norm"), WeightSpec("a", (H, hid)),
+                        WeightSpec("dt_bias", (H,), kind="vector", init="zeros"), WeightSpec("g", (H * V, hid)), WeightSpec("o", (hid, H * V))]
+
+    def cache_need(self):
+        floats = self.H * self.D * self.V + (self.taps * self.C if self.taps > 1 else 0)
+        return StateNeed(((floats + 3) // 4 * 4,), "float32")              # whole 16-byte pieces a slot
+
+    def load(self, tensors, dtype, device):
+        # one product for everything that reads the mixer's input: q | k | v | gate | b | a (| unused)
+        self.proj = pad_rows(torch.cat([tensors.pop(n) for n in ("q", "k", "v", "g", "b", "a")], dim=0), 8)
+        self.conv = torch.cat([tensors.pop(n + ".conv") for n in ("q", "k", "v")], dim=0).float().contiguous()
+        self.rate = torch.exp(tensors.pop("A_log").double()).float().contiguous()
+        self.dt_bias, self.norm = tensors.pop("dt_bias").float().contiguous(), tensors.pop("norm").float().contiguous()
+        self.o = tensors.pop("o")
+
+    @property
+    def first_weight(self):
+        return self.proj
+
+    def step_flops(self, rows, pairs):
+        return 8 * self.H * self.D * self.V * rows                 # decay, S^T k, rank-one update, read-out
+
+    def forward(self, h, ctx, cache, position, owns_cache=True):
+        ops = ctx.ops
+        p = ops.linear(h, self.proj)
+        rows = ops.gated_delta_mix(p, self.conv, self.taps, self.rate, self.dt_bias, self.H, self.KV, self.D, self.V, self.unit_eps, self.norm,
+                                   self.eps, cache.state, ctx.batch)
+        return ops.linear(rows, self.o)

@@ -1,7 +1,8 @@
 """Softmax attention over the paged cache whose mask, softmax and inputs are chosen by constants:
 
-  unit norm    q and k are divided by their root mean square per head (no weight) instead of being rotated;
+  unit norm    q and k are divided by their root mean square per head (no weight); without rotate=True they are not rotated and
                positions do not enter the scores
+  rotate       True: after the norm, the position part's rotate-half frequencies turn the first coordinates of every q and k head
   block_size   B: position i sees j <= i only inside its own block of B positions, floor(i / B) = floor(j / B),
                blocks counted from position 0 of the sequence (None: every j <= i); window: the last W keys (None: all)
   sink         the softmax has one more term whose score is 0 and which carries no value:
@@ -53,6 +54,7 @@ class SinkAttention(Part):
         self.value_mix = g("value_mix")
         self.mix_key = g("value_mix_key", "values")
         self.norm_weights, self.values_are_keys = bool(g("norm_weights", False)), g("values", "projected") == "keys"
+        self.rotate = bool(g("rotate", False))
         self.q_temp = tuple(g("q_temp")) if g("q_temp") else None                               # (coef, every)
         self.slope_exponent = float(g("slope_exponent")) if g("slope_exponent") is not None else None
         if g("values", "projected") not in ("projected", "keys"):
@@ -133,10 +135,11 @@ class SinkAttention(Part):
                 raise ValueError("a layer that blends values in runs before the layer that lends them, or their sizes differ")
         elif self.value_mix == "source":
             ctx.shared[("value_mix", self.mix_key)] = p[:, (H + KV) * D:]      # a view: the kernel below leaves these columns alone
-        if self.norm_weights or self.values_are_keys or self.q_temp:
+        if self.norm_weights or self.values_are_keys or self.q_temp or self.rotate:
+            turn = dict(inv_freq=position.rotary_inv_freq()) if self.rotate else {}
             q = ops.unit_qk_cache(p, H, KV, D, V, self.eps, self.lam, source, meta, cache.k if owns_cache else None,
                                   cache.v if owns_cache else None, q_weight=self.q_norm, k_weight=self.k_norm, q_temp=self.q_temp,
-                                  values_are_keys=self.values_are_keys)
+                                  values_are_keys=self.values_are_keys, **turn)
         else:
             q = ops.unit_qk_cache(p, H, KV, D, V, self.eps, self.lam, source, meta,
                                   cache.k if owns_cache else None, cache.v if owns_cache else None)

@@ -226,15 +226,18 @@ def _batched_linear(self, x, col0, head_stride, K, w, side_by_side=False):
     return out.transpose(0, 1).reshape(out.shape[1], -1).contiguous() if side_by_side else out
 
 
-def _rotate_pairs(v, positions, inv_freq):
-    n = inv_freq.numel()
+def _rotate_pairs(v, positions, inv_freq, half=False):
+    n = 0 if inv_freq is None else inv_freq.numel()
+    if n == 0:
+        return v.clone()
     ang = positions.float()[:, None] * inv_freq.float()[None, :]
     shape = (v.shape[0],) + (1,) * (v.dim() - 2) + (n,)
     c, s = ang.cos().view(shape), ang.sin().view(shape)
     out = v.clone()
-    a, b = v[..., 0:2 * n:2], v[..., 1:2 * n:2]
-    out[..., 0:2 * n:2] = a * c - b * s
-    out[..., 1:2 * n:2] = b * c + a * s
+    first, second = (slice(0, n), slice(n, 2 * n)) if half else (slice(0, 2 * n, 2), slice(1, 2 * n, 2))
+    a, b = v[..., first], v[..., second]
+    out[..., first] = a * c - b * s
+    out[..., second] = b * c + a * s
     return out
 
 
@@ -250,7 +253,7 @@ def _latent_prepare(self, p, q_abs, H, D, R, C, norm_w, eps, inv_freq, meta, cac
     return q.contiguous()
 
 
-def _latent_attention(self, q, cache, meta, H, C, R, scale):
+def _latent_attention(self, q, cache, meta, H, C, R, scale, sink_values=None):
     T = q.shape[0]
     out = torch.zeros(H, T, C, dtype=q.dtype, device=q.device)
     q_start, pos0, kv_len = meta.seg_q_start.tolist(), meta.seg_pos0.tolist(), meta.seg_kv_len.tolist()
@@ -263,7 +266,9 @@ def _latent_attention(self, q, cache, meta, H, C, R, scale):
         pq = pos0[s] + torch.arange(b - a, device=q.device)
         sc = torch.einsum("phd,jd->hpj", q[a:b].float(), kv) * scale
         sc = sc.masked_fill(~(j[None, :] <= pq[:, None])[None], float("-inf"))
-        out[:, a:b] = torch.einsum("hpj,jc->hpc", torch.softmax(sc, dim=-1), kv[:, :C]).to(q.dtype)
+        if sink_values is not None:
+            sc = torch.cat([sc, sink_values.float()[:, None, None].expand(-1, b - a, 1)], dim=-1)
+        out[:, a:b] = torch.einsum("hpj,jc->hpc", torch.softmax(sc, dim=-1)[..., :L], kv[:, :C]).to(q.dtype)
     return out
 
 
@@ -660,21 +665,21 @@ def _scale_logits(self, logits, s):
 _latent_prepare_plain = _latent_prepare
 
 
-def _latent_prepare_general(self, p, q_abs, H, D, R, C, norm_w, eps, inv_freq, meta, cache, q_rows=None, dkv_col=None):
-    if q_rows is None and dkv_col is None and R:
+def _latent_prepare_general(self, p, q_abs, H, D, R, C, norm_w, eps, inv_freq, meta, cache, q_rows=None, dkv_col=None, half_pairs=False):
+    if q_rows is None and dkv_col is None and R and not half_pairs:
         return _latent_prepare_plain(self, p, q_abs, H, D, R, C, norm_w, eps, inv_freq, meta, cache)
     T, dt = p.shape[0], p.dtype
     src = p if q_rows is None else q_rows
     col = H * (D + R) if dkv_col is None else dkv_col
     parts = [q_abs.transpose(0, 1).float()]
     if R:
-        parts.append(_rotate_pairs(src[:, :H * (D + R)].view(T, H, D + R)[:, :, D:].float(), meta.positions, inv_freq))
+        parts.append(_rotate_pairs(src[:, :H * (D + R)].view(T, H, D + R)[:, :, D:].float(), meta.positions, inv_freq, half_pairs))
     q = torch.cat(parts, dim=-1).to(dt)
     if cache is not None:
         dkv = p[:, col:col + C + R].float()
         row = _rms(dkv[:, :C], eps) * norm_w.float()
         if R:
-            row = torch.cat([row, _rotate_pairs(dkv[:, C:], meta.positions, inv_freq)], dim=-1)
+            row = torch.cat([row, _rotate_pairs(dkv[:, C:], meta.positions, inv_freq, half_pairs)], dim=-1)
         page, off = meta.slots.long() // meta.page_size, meta.slots.long() % meta.page_size
         cache[page, 0, off, :] = row.to(cache.dtype)
     return q.contiguous()
@@ -694,8 +699,8 @@ _unit_qk_cache_plain = _unit_qk_cache
 
 
 def _unit_qk_cache_general(self, p, H, KV, D, V, eps, lam, source, meta, k_cache, v_cache, q_weight=None, k_weight=None, q_temp=None,
-                           values_are_keys=False):
-    if q_weight is None and q_temp is None and not values_are_keys:
+                           values_are_keys=False, inv_freq=None):
+    if q_weight is None and q_temp is None and not values_are_keys and inv_freq is None:
         return _unit_qk_cache_plain(self, p, H, KV, D, V, eps, lam, source, meta, k_cache, v_cache)
     T, dt = p.shape[0], p.dtype
     q = p[:, :H * D].float().view(T, H, D)
@@ -706,6 +711,7 @@ def _unit_qk_cache_general(self, p, H, KV, D, V, eps, lam, source, meta, k_cache
         q, k = _rms(q, eps), _rms(k_raw, eps)
     if q_weight is not None:
         q, k = q * q_weight.float(), k * k_weight.float()
+    q, k = _rotate_pairs(q, meta.positions, inv_freq, True), _rotate_pairs(k, meta.positions, inv_freq, True)
     if q_temp is not None:
         coef, every = q_temp
         pos = meta.positions.long()
@@ -861,6 +867,60 @@ def _mamba2_mix(self, p, conv, conv_b, taps, dt_bias, A, Dv, H, V, N, G, norm, p
 _masked_attention = _masked_attention_capped
 
 
+# ---------------------------------------------------------------- layer norms on both sides, element gate, delta rule with one decay per head
+def _layer_norm(z, w, eps):
+    d = z - z.mean(-1, keepdim=True)
+    return d * torch.rsqrt(d.pow(2).mean(-1, keepdim=True) + eps) * w.float()
+
+
+def _stream_layernorm(self, x, delta, pre_add, weight, eps, rows, out_dtype):
+    assert x.dtype == torch.float32
+    v = x if pre_add is None else x + pre_add
+    if delta is not None:
+        v = v + _layer_norm(delta.y.float(), delta.weight, delta.eps)
+    if weight is None:
+        return v.to(out_dtype).clone()
+    if rows is not None:
+        v = v[rows.long()]
+    elif v is not x:
+        x.copy_(v)
+    return _layer_norm(v, weight, eps).to(out_dtype)
+
+
+def _sigmoid_gate(self, rows, gate):
+    rows.copy_((rows.float() * torch.sigmoid(gate.float())).to(rows.dtype))
+    return rows
+
+
+def _gated_delta_mix(self, p, conv, taps, rate, dt_bias, H, KV, D, V, unit_eps, norm, eps, state, batch):
+    T, C, base = p.shape[0], 2 * KV * D + H * V, H * D * V
+    x = p[:, :C].float()
+    out = torch.empty(T, H, V, device=p.device)
+    beta = torch.sigmoid(p[:, C + H * V:C + H * V + H].float())
+    f = torch.exp(-rate.double() * torch.nn.functional.softplus(p[:, C + H * V + H:C + H * V + 2 * H].double() + dt_bias.double())).float()
+    for a, b, slot in _segments(batch):
+        S = state[slot, :base].view(H, D, V).clone()
+        ring = state[slot, base:base + taps * C].view(taps, C) if taps > 1 else None
+        for t in range(a, b):
+            pos = int(batch.positions[t])
+            y = conv[:, taps - 1] * x[t]
+            for back in range(1, min(taps, pos + 1)):
+                y = y + conv[:, taps - 1 - back] * ring[(pos - back) % taps]
+            if taps > 1:
+                ring[pos % taps] = x[t]
+            y = torch.nn.functional.silu(y)
+            qk = y[:2 * KV * D].view(2 * KV, D)
+            qk = qk / torch.sqrt(qk.pow(2).sum(-1, keepdim=True) + unit_eps)
+            q, k = (qk[:KV] * D ** -0.5).repeat_interleave(H // KV, dim=0), qk[KV:].repeat_interleave(H // KV, dim=0)
+            S = f[t][:, None, None] * S
+            u = beta[t][:, None] * (y[2 * KV * D:].view(H, V) - torch.einsum("hdv,hd->hv", S, k))
+            S = S + k[:, :, None] * u[:, None, :]
+            out[t] = torch.einsum("hdv,hd->hv", S, q)
+        state[slot, :base] = S.reshape(-1)
+    rows = (_rms(out, eps) * norm.float()).reshape(T, H * V) * torch.nn.functional.silu(p[:, C:C + H * V].float())
+    return rows.to(p.dtype)
+
+
 for _name, _fn in list(globals().items()):
     if _name.startswith("_") and _name[1:] in ("embed_scaled_norm", "add_scaled_rmsnorm", "polynorm", "lightning_scan", "group_rmsnorm_gate",
                                                "delta_prepare", "delta_scan", "batched_linear", "latent_prepare", "latent_attention", "head_gate",
@@ -869,5 +929,6 @@ for _name, _fn in list(globals().items()):
                                                "embed_bigram_stream", "short_conv", "general_delta_prepare", "general_delta_scan", "matrix_memory",
                                                "selective_scan", "dual_rmsnorm_mix", "bias_act", "softcap",
                                                "embed_scaled_stream", "stream_rmsnorm_pair", "rows_rmsnorm", "bias_glu", "scale_logits",
-                                               "sum_rmsnorm", "conv_qkv_cache", "mamba2_mix"):
+                                               "sum_rmsnorm", "conv_qkv_cache", "mamba2_mix",
+                                               "stream_layernorm", "sigmoid_gate", "gated_delta_mix"):
         setattr(TorchRefOps, _name[1:], _fn)
