@@ -277,9 +277,9 @@ def reference_arm(args):
 
 
 def design_bench(args):
-    """--design naditar | namesun | nununex | megovik | fetodra: prompt and decode throughput of that design at layer sizes of real models (random weights),
-    beside Qwen3 dense of the same width, depth, vocabulary and feed-forward parameters, and every new kernel beside its
-    Qwen3 counterpart with its share of the bound it is up against.  One JSON line; the default workload is untouched."""
+    """--design naditar | namesun | nununex | megovik | fetodra | kofutar: prompt and decode throughput of that design at layer sizes of real models (random weights),
+    beside the closest design the engine had (Qwen3 dense unless microbench.BESIDE names another) of the same width, depth, vocabulary and feed-forward parameters, and every new kernel beside its
+    counterpart with its share of the bound it is up against.  One JSON line; the default workload is untouched."""
     import torch
 
     from mini_inference_b200.cli import microbench
@@ -293,7 +293,7 @@ def design_bench(args):
         res = {}
         for name, cfg in ((args.design, design_config(size, args.design_layers, vocab)),
                           (microbench.BESIDE.get(args.design, "qwen3"), qwen3_config(size, args.design_layers, vocab))):
-            for tc in ((False, True) if name == "naditar" else (False,)):
+            for tc in ((False, True) if name == args.design == "naditar" else (False,)):
                 llm = LLM(None, random_config=cfg, random_seed=0, dtype="bfloat16", device="cuda:0", kv_block_size=16,
                           kv_cache_tokens=64 * args.ctx + 4096, kv_watermark=0.0, max_num_seqs=64, max_model_len=args.ctx,
                           max_batched_tokens=4096, cuda_graphs=False)
@@ -321,8 +321,8 @@ def design_bench(args):
 
 def main():
     ap = argparse.ArgumentParser()
-    ap.add_argument("--design", default=None, choices=["naditar", "namesun", "nununex", "megovik", "fetodra"],
-                    help="instead of the default workload: this design beside the closest one the engine had (Qwen3; for nununex, megovik and fetodra: Namesun) at equal sizes")
+    ap.add_argument("--design", default=None, choices=["naditar", "namesun", "nununex", "megovik", "fetodra", "kofutar"],
+                    help="instead of the default workload: this design beside the closest one the engine had (Qwen3; for nununex, megovik and fetodra: Namesun; for kofutar: Naditar) at equal sizes")
     ap.add_argument("--design-sizes", default="2k,4k")
     ap.add_argument("--design-layers", type=int, default=8)
     ap.add_argument("--gpus", type=int, default=1)

@@ -974,16 +974,177 @@ def bench_fetodra(args, ops, peak, out=print):
     return rows
 
 
+def kofutar_config(size, layers, vocab=65536):
+    """Layers of the sizes of NADITAR_SIZES: delta rule, attention, delta rule, latent attention, .., the third and fourth run twice in a row
+    (`layers` layer runs in all); the three feed-forward matrices hold what Naditar's two do."""
+    z = NADITAR_SIZES[size]
+    ff = {"kind": "dense", "ff": z["ff"] * 2 // 3 // 128 * 128}
+    delta = {"type": "delta", "mlp": ff, "mixer": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "conv": z["conv"]}}
+    att = {"type": "attention", "mlp": ff, "mixer": {"heads": z["heads"], "kv_heads": z["kv_heads"], "dim": z["dim"], "vdim": z["vdim"], "scale": z["dim"] ** -0.5,
+                                                     "rot": {"base": 1e6, "dims": z["dim"] // 2, "scaling": {"factor": 4.0}}}}
+    lat = {"type": "latent_attention", "mlp": ff,
+           "mixer": {"heads": z["l_heads"], "dim": z["l_dim"], "rot_dim": z["l_rot"], "vdim": z["l_vdim"], "kv_rank": z["l_rank"], "q_rank": z["width"] * 3 // 8,
+                     "scale": (z["l_dim"] + z["l_rot"]) ** -0.5, "rot": {"base": 1e6, "dims": z["l_rot"]}}}
+    pattern = [delta, att, delta, lat]
+    return {"architecture": "Kofutar", "vocab": vocab, "width": z["width"], "norm": {"eps": 1e-6}, "layers": [pattern[i % 4] for i in range(layers - 2)],
+            "loop": {"start": 2, "stop": 4, "times": 2}}
+
+
+def naditar_config_like_kofutar(size, layers, vocab=65536):
+    """Naditar (float32 stream, delta rule with short convolutions, rotated and gated latent attention, a looped span) of the same width, depth,
+    vocabulary, heads and feed-forward parameters; it has no grouped attention, so latent attention stands there."""
+    cfg = naditar_config(size, 4, vocab)
+    delta, _, lat, _ = cfg["layers"]
+    cfg["layers"] = [delta if i % 2 == 0 else lat for i in range(layers - 2)]
+    cfg["loop"] = {"start": 2, "stop": 4, "times": 2}
+    return cfg
+
+
+def bench_kofutar(args, ops, peak, out=print):
+    """Each kernel that the Kofutar design added or widened, at the layer sizes of --design-size, beside the like kernel of Naditar (of Namesun
+    for grouped attention), with the bytes or operations it cannot avoid as a share of its bound: the measured copy bandwidth, the measured
+    bf16 peak, or (token-by-token scans) the float32 FMA rate of the CUDA cores."""
+    import numpy as np
+    z = NADITAR_SIZES[args.design_size]
+    here = os.path.dirname(os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
+    bf16_peak = 1590.0
+    if os.path.isfile(os.path.join(here, "MEASURED_PEAKS.json")):
+        with open(os.path.join(here, "MEASURED_PEAKS.json")) as f:
+            bf16_peak = json.load(f)["bf16_tflops"]
+    fma_peak = ops.NUM_SMS * 128 * 2 * 1.965e9 / 1e12
+    rows = []
+
+    def line(kernel, shape, us, amount, bound):
+        got, top, unit = {"hbm": (amount / us / 1e3, peak, "GB/s"), "bf16": (amount / us / 1e6, bf16_peak, "TFLOP/s"),
+                          "fma": (amount / us / 1e6, fma_peak, "TF(f32)")}[bound]
+        rows.append({"kernel": kernel, "shape": shape, "us": round(us, 2), "achieved": round(got, 2), "unit": unit, "frac": round(got / top, 3)})
+        out(f"{kernel:52s} {shape:46s} {us:9.2f} us {got:9.2f} {unit:10s} {100 * got / top:5.1f} % of bound", flush=True)
+
+    t = lambda a: torch.tensor(np.asarray(a, dtype=np.int32), device="cuda")       # noqa: E731
+    from ..parts.base import NormedDelta
+    bf = torch.bfloat16
+    W, T, it, F = z["width"], args.tokens, args.iters, z["ff"] * 2 // 3 // 128 * 128
+    rb = lambda *s: torch.randn(*s, device="cuda", dtype=bf)                       # noqa: E731
+    rf = lambda *s: torch.randn(*s, device="cuda")                                 # noqa: E731
+    # ---- the stream: norm of the output + add + norm of the sum; the stream's own rows for the joining product
+    wn, g1 = torch.ones(W, device="cuda"), torch.ones(1, device="cuda")
+    for n in (T, 64, 8):
+        reps = 4 if n > 64 else 2
+        x, a, pre = rf(reps, n, W), rb(reps, n, W), rf(n, W)
+        us = timed(lambda i: ops.stream_layernorm(x[i % reps], NormedDelta(a[i % reps], wn, 1e-6), None, wn, 1e-6, None, bf), it)
+        line("output norm + add + norm (layer norms)", f"T={n} width={W}", us, n * W * 12.0, "hbm")
+        us = timed(lambda i: ops.add_scaled_rmsnorm(x[i % reps], a[i % reps], g1, 1e-6, None, None, bf), it)
+        line("  Naditar: add + norm", f"T={n} width={W}", us, n * W * 12.0, "hbm")
+        if n == T:
+            us = timed(lambda i: ops.stream_layernorm(x[i % reps], NormedDelta(a[i % reps], wn, 1e-6), None, None, 1e-6, None, bf), it)
+            line("output norm + add -> rows for the join", f"T={n} width={W}", us, n * W * 8.0, "hbm")
+            us = timed(lambda i: ops.stream_layernorm(x[i % reps], None, pre, wn, 1e-6, None, bf), it)
+            line("joined half + norm", f"T={n} width={W}", us, n * W * 14.0, "hbm")
+    gu, zz, coef = rb(2, T, 2 * F), rb(2, T, z["ff"]), torch.tensor([0.5, 0.3, 0.2, 0.1], device="cuda")
+    us = timed(lambda i: ops.bias_glu(gu[i % 2], None, "gelu_tanh"), it)
+    line("gelu gate", f"T={T} ff={F}", us, T * F * 6.0, "hbm")
+    us = timed(lambda i: ops.polynorm(zz[i % 2], coef, 1e-6), it)
+    line("  Naditar: polynorm activation", f"T={T} ff={z['ff']}", us, T * z["ff"] * 4.0, "hbm")
+    del gu, zz
+    # ---- delta rule
+    H, KV, D, V, taps = z["heads"], z["kv_heads"], z["dim"], z["vdim"], z["conv"]
+    C = 2 * KV * D + H * V
+    conv, rate, dtb, norm = rf(C, taps) * 0.3, torch.ones(H, device="cuda"), rf(H) - 3.0, torch.ones(V, device="cuda")
+    A_log, dtb_c = torch.zeros(H, device="cuda"), torch.zeros(H * D, device="cuda")
+    for B, n in ((1, T), (8, T // 8), (8, 1), (64, 1)):
+        Tn = B * n
+        reps = 1 if n > 1 else max(2, (300 << 20) // (B * H * D * V * 4) + 1)       # decode: states rotated through more than the L2 holds
+        batch = types.SimpleNamespace(num_segs=B, seg_q_start=t(np.arange(B + 1) * n), seg_slot=t(np.arange(B) + 1), positions=t(np.tile(np.arange(n) + 5, B)),
+                                      token_seg=t(np.repeat(np.arange(B), n)))
+        state = torch.zeros(reps, B + 1, H * D * V + taps * C, device="cuda")
+        p = rb(2, Tn, (C + H * V + 2 * H + 7) // 8 * 8)
+        shape = f"{'prompt' if n > 1 else 'decode'} B={B} T={n} heads={H} {D}x{V}"
+        us = timed(lambda i: ops.gated_delta_mix(p[i % 2], conv, taps, rate, dtb, H, KV, D, V, 1e-6, norm, 1e-6, state[i % reps], batch), it)
+        moved = 2.0 * B * (H * D * V + (taps * C if n == 1 else 0)) * 4 + Tn * (C + 2 * H * V) * 2.0
+        if n > 1:
+            line("delta rule: filter, scan, gated norm", shape, us, 8.0 * H * D * V * Tn, "fma")
+            prep = torch.randn(Tn, C + 2 * H, device="cuda") * 0.1
+            us = timed(lambda i: ops.gated_delta_scan(prep, H, KV, D, V, state[0], batch), it)
+            line("  its scan", shape, us, 8.0 * H * D * V * Tn, "fma")
+        else:
+            line("delta rule: filter, state, gated norm (one kernel)", shape, us, moved, "hbm")
+        nstate = torch.zeros(reps, B + 1, H * D * V + (taps - 1) * C, device="cuda")
+        pd, ac, gate = rb(Tn, C + H + 2 * z["rank"]), rb(Tn, H * D), rb(Tn, H * V)
+
+        def channel(i):
+            pr = ops.delta_prepare(pd, ac, conv, A_log, dtb_c, H, KV, D, V, taps, 1e-6, nstate[i % reps], batch)
+            return ops.group_rmsnorm_gate(ops.delta_scan(pr, H, KV, D, V, nstate[i % reps], batch), norm, gate, 1e-6, H, V, bf)
+        us = timed(channel, it)
+        if n > 1:
+            line("  Naditar: delta rule, decay per channel", shape, us, 8.0 * H * D * V * Tn, "fma")
+            pr = ops.delta_prepare(pd, ac, conv, A_log, dtb_c, H, KV, D, V, taps, 1e-6, nstate[0], batch)
+            us = timed(lambda i: ops.delta_scan(pr, H, KV, D, V, nstate[0], batch), it)
+            line("  Naditar: its scan", shape, us, 8.0 * H * D * V * Tn, "fma")
+        else:
+            line("  Naditar: delta rule, decay per channel", shape, us, moved + Tn * H * D * 2.0, "hbm")
+        del state, nstate
+    # ---- attention: weighted norms and rotation; latent attention with a sink and an element gate
+    page, qw, inv = 16, torch.ones(D, device="cuda"), torch.full((D // 4,), 0.01, device="cuda")
+    LH, LD, R, LV, LC, QR = z["l_heads"], z["l_dim"], z["l_rot"], z["l_vdim"], z["l_rank"], W * 3 // 8
+    linv, lw, sink = torch.full((R // 2,), 0.01, device="cuda"), torch.ones(LC, device="cuda"), torch.zeros(LH, device="cuda")
+    for B, n, ctx in ((1, T, T), (8, 1, args.ctx), (64, 1, args.ctx)):
+        pages_per = -(-ctx // page)
+        n_pages = B * pages_per + 1
+        kc, vc, lc = rb(n_pages, KV, page, D), rb(n_pages, KV, page, V), rb(n_pages, 1, page, LC + R)
+        tiles = [(s, r) for s in range(B) for r in range(0, n, 64)] if n > 1 else []
+        meta = types.SimpleNamespace(seg_q_start=t(np.arange(B + 1) * n), seg_pos0=t([ctx - n] * B), seg_kv_len=t([ctx] * B), table_rows=t(np.arange(B)),
+                                     block_table=t(np.arange(1, n_pages).reshape(B, pages_per)), max_pages=pages_per, page_size=page,
+                                     decode_segs=t(np.arange(B) if n == 1 else []), prefill_tiles=t(tiles).view(-1, 2), tile=64, max_kv_len=ctx,
+                                     slots=t((np.arange(B)[:, None] * pages_per * page + page + ctx - n + np.arange(n)[None, :]).reshape(-1)),
+                                     positions=t(np.tile(np.arange(ctx - n, ctx), B)))
+        Tn, pairs = B * n, n * (n + 1) / 2 * B
+        p3 = rb(2, Tn, (H + 2 * KV) * D)
+        us = timed(lambda i: ops.unit_qk_cache(p3[i % 2], H, KV, D, V, 1e-6, None, None, meta, kc, vc, q_weight=qw, k_weight=qw, inv_freq=inv), it)
+        line("q/k norm * weight, rotation, k and v -> pools", f"rows={Tn} H={H} KV={KV} D={D}", us, Tn * (2 * H + 4 * KV) * D * 2.0, "hbm")
+        us = timed(lambda i: ops.unit_qk_cache(p3[i % 2], H, KV, D, V, 1e-6, None, None, meta, kc, vc), it)
+        line("  Namesun: unit q/k, k and v -> pools", f"rows={Tn} H={H} KV={KV} D={D}", us, Tn * (2 * H + 4 * KV) * D * 2.0, "hbm")
+        q = p3[0][:, :H * D]
+        amount, bound = (4.0 * H * D * pairs, "bf16") if n > 1 else (B * ctx * KV * D * 4.0, "hbm")
+        us = timed(lambda i: ops.masked_attention(q, kc, vc, meta, H, KV, D, V, D ** -0.5, None, None, False), it)
+        line("attention", f"B={B} rows={n} keys={ctx} H={H}/{KV} D={D}", us, amount, bound)
+        us = timed(lambda i: ops.masked_attention(q, kc, vc, meta, H, KV, D, V, D ** -0.5, None, None, True), it)
+        line("  Namesun: attention with a sink (no block)", f"B={B} rows={n} keys={ctx} H={H}/{KV} D={D}", us, amount, bound)
+        cq, qp, q_abs = rb(Tn, QR + LC + R + LH * LV), rb(Tn, LH * (LD + R)), rb(LH, Tn, LC)
+        us = timed(lambda i: ops.latent_prepare(cq, q_abs, LH, LD, R, LC, lw, 1e-6, linv, meta, lc, q_rows=qp, dkv_col=QR, half_pairs=True), it)
+        moved = Tn * (2 * LH * (LC + R) + 2 * (LC + R)) * 2.0
+        line("latent: norm, rotations, row -> pool, queries", f"rows={Tn} heads={LH} rows {LC}+{R}", us, moved, "hbm")
+        pn = rb(Tn, LH * (LD + R) + LC + R + LH)
+        us = timed(lambda i: ops.latent_prepare(pn, q_abs, LH, LD, R, LC, lw, 1e-6, linv, meta, lc), it)
+        line("  Naditar: the same, pairs (2i, 2i + 1)", f"rows={Tn} heads={LH} rows {LC}+{R}", us, moved, "hbm")
+        ql = rb(Tn, LH, LC + R)
+        amount, bound = (2.0 * LH * (2 * LC + R) * pairs, "bf16") if n > 1 else (B * ctx * (LC + R) * 2.0, "hbm")
+        us = timed(lambda i: ops.latent_attention(ql, lc, meta, LH, LC, R, 0.1, sink_values=sink), it)
+        line("latent attention with a sink", f"B={B} rows={n} keys={ctx} heads={LH} rows {LC}+{R}", us, amount, bound)
+        us = timed(lambda i: ops.latent_attention(ql, lc, meta, LH, LC, R, 0.1), it)
+        line("  Naditar: latent attention", f"B={B} rows={n} keys={ctx} heads={LH} rows {LC}+{R}", us, amount, bound)
+        ro, oh = rb(Tn, LH * LV), rb(LH, Tn, LV)
+        us = timed(lambda i: ops.sigmoid_gate(ro, cq[:, QR + LC + R:]), it)
+        line("latent: element gate", f"rows={Tn} heads={LH} V={LV}", us, Tn * LH * LV * 6.0, "hbm")
+        us = timed(lambda i: ops.head_gate(oh, pn[:, -LH:], bf), it)
+        line("  Naditar: head gate", f"rows={Tn} heads={LH} V={LV}", us, Tn * LH * LV * 4.0, "hbm")
+        us = timed(lambda i: ops.rows_rmsnorm(cq[:, :QR], rate.new_ones(QR), 1e-6), it)
+        line("norm of the query latent", f"rows={Tn} q_rank={QR}", us, Tn * QR * 4.0, "hbm")
+        del kc, vc, lc
+    ops.check_errors()
+    return rows
+
+
 DESIGNS = {"naditar": (naditar_config, qwen3_config_like, bench_design), "namesun": (namesun_config, qwen3_config_like_namesun, bench_namesun),
            "nununex": (nununex_config, namesun_config_like_nununex, bench_nununex),
            "megovik": (megovik_config, namesun_config_like_megovik, bench_megovik),
-           "fetodra": (fetodra_config, namesun_config_like_fetodra, bench_fetodra)}
-BESIDE = {"nununex": "namesun", "megovik": "namesun", "fetodra": "namesun"}            # the design an entry of DESIGNS is set beside (default: qwen3)
+           "fetodra": (fetodra_config, namesun_config_like_fetodra, bench_fetodra),
+           "kofutar": (kofutar_config, naditar_config_like_kofutar, bench_kofutar)}
+BESIDE = {"nununex": "namesun", "megovik": "namesun", "fetodra": "namesun", "kofutar": "naditar"}            # the design an entry of DESIGNS is set beside (default: qwen3)
 
 
 def main(argv=None):
     ap = argparse.ArgumentParser(description=__doc__.split("\n")[0])
-    ap.add_argument("what", choices=["gemm", "attention", "prefill", "design", "namesun", "nununex", "megovik", "fetodra"])
+    ap.add_argument("what", choices=["gemm", "attention", "prefill", "design", "namesun", "nununex", "megovik", "fetodra", "kofutar"])
     ap.add_argument("--design-size", default="2k", choices=sorted(NADITAR_SIZES), help="design: layer sizes of the Naditar kernels")
     ap.add_argument("--size", default="4b", choices=sorted(SIZES))
     ap.add_argument("--rows", default="1,8,64", type=lambda s: [int(v) for v in s.split(",")])
@@ -1002,7 +1163,7 @@ def main(argv=None):
     ops = get_ops("cuda:0")
     peak, src = peak_gbs()
     print(f"# peak {peak} GB/s ({src})")
-    {"gemm": bench_gemm, "attention": bench_attention, "prefill": bench_prefill_attention, "design": bench_design, "namesun": bench_namesun, "nununex": bench_nununex, "megovik": bench_megovik, "fetodra": bench_fetodra}[args.what](args, ops, peak)
+    {"gemm": bench_gemm, "attention": bench_attention, "prefill": bench_prefill_attention, "design": bench_design, "namesun": bench_namesun, "nununex": bench_nununex, "megovik": bench_megovik, "fetodra": bench_fetodra, "kofutar": bench_kofutar}[args.what](args, ops, peak)
     return 0
 
 

@@ -102,14 +102,14 @@ __global__ void __launch_bounds__(128) delta_ready_kernel(const T* __restrict__ 
     }
 }
 
-// the entry's inputs of its last min(n, taps - 1) positions -> their ring rows; grid (entries, channel groups)
+// the inputs of the entry's last min(n, taps) positions -> their ring rows; grid (entries, channel groups)
 template <typename T>
 __global__ void delta_ring_kernel(const T* __restrict__ p, int ldp, float* __restrict__ state, long long state_stride, long long ring_off,
                                   const int* __restrict__ positions, const int* __restrict__ seg_q_start, const int* __restrict__ seg_slot, int C, int taps) {
     const int seg = blockIdx.x, q1 = seg_q_start[seg + 1], n = q1 - seg_q_start[seg], c = blockIdx.y * blockDim.x + threadIdx.x;
     if (c >= C) return;
     float* ring = state + (long long)seg_slot[seg] * state_stride + ring_off;
-    for (int t = q1 - min(n, taps - 1); t < q1; ++t) ring[(size_t)(positions[t] % taps) * C + c] = to_f32(p[(size_t)t * ldp + c]);
+    for (int t = q1 - min(n, taps); t < q1; ++t) ring[(size_t)(positions[t] % taps) * C + c] = to_f32(p[(size_t)t * ldp + c]);
 }
 
 // ------------------------------------------------------------------ decode steps: everything in one pass over the state

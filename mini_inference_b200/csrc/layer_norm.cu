@@ -14,14 +14,15 @@ using namespace mi;
 
 namespace {
 
-constexpr int NT = 256, NW = NT / 32;
+constexpr int LOOP_NT = 256;
 
 struct Moments { float mean, rstd; };
 
 // what the warps found (sum of their entries, squared deviations from their own mean, entries) -> the row's mean and 1 / deviation
-__device__ __forceinline__ Moments combine(float sum, float m2, float count, float* scratch /* 3 NW */, int hidden, float eps) {
+// (scratch: 3 NW floats that no earlier call of the block has used)
+template <int NW>
+__device__ __forceinline__ Moments combine(float sum, float m2, float count, float* scratch, int hidden, float eps) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    __syncthreads();
     if (lane == 0) { scratch[warp] = sum; scratch[NW + warp] = m2; scratch[2 * NW + warp] = count; }
     __syncthreads();
     float total = 0.f;
@@ -55,7 +56,7 @@ template <typename TY> __device__ __forceinline__ void store4(TY* p, float4 v) {
 }
 
 // Mean and deviation of a row held as v[VPT] (thread t: quads t, t + NT, ..; entries beyond the row are zero and not counted)
-template <int VPT>
+template <int NT, int VPT>
 __device__ __forceinline__ Moments row_moments(const float4 (&v)[VPT], int quads, int hidden, float eps, float* scratch) {
     const int warp0 = threadIdx.x & ~31;
     float sum = 0.f, count = 0.f;
@@ -73,17 +74,27 @@ __device__ __forceinline__ Moments row_moments(const float4 (&v)[VPT], int quads
             const float a = v[k].x - m, b = v[k].y - m, c = v[k].z - m, d = v[k].w - m;
             m2 += (a * a + b * b) + (c * c + d * d);
         }
-    return combine(sum, warp_sum(m2), count, scratch, hidden, eps);
+    return combine<NT / 32>(sum, warp_sum(m2), count, scratch, hidden, eps);
 }
 
-template <typename TD, typename TY, int VPT>
+// NT threads a row (few for many rows, so that more rows are in flight; many for few rows), VPT quads a thread
+template <typename TD, typename TY, int NT, int VPT>
 __global__ void __launch_bounds__(NT) stream_layernorm_vec_kernel(float* __restrict__ x, const TD* __restrict__ y, const float* __restrict__ wy, float eps_y,
                                                                   const float* __restrict__ pre, const float* __restrict__ w, TY* __restrict__ out,
                                                                   const int* __restrict__ rows, int hidden, float eps, int keep) {
-    __shared__ float scratch[3 * NW];
+    __shared__ float scratch[2][3 * NT / 32];
     const size_t r = (rows ? (size_t)rows[blockIdx.x] : (size_t)blockIdx.x) * hidden;
     const int quads = hidden >> 2;
-    float4 v[VPT];
+    constexpr bool AHEAD = VPT <= 2;                          // the weights are fetched with the row, so that no wait for them follows a sum
+    float4 v[VPT], wv[AHEAD ? VPT : 1], wyv[AHEAD ? VPT : 1];
+    if constexpr (AHEAD) {
+#pragma unroll
+        for (int k = 0; k < VPT; ++k) {
+            const int q = threadIdx.x + k * NT;
+            wv[k] = w && q < quads ? *reinterpret_cast<const float4*>(w + 4 * q) : make_float4(1.f, 1.f, 1.f, 1.f);
+            wyv[k] = y && q < quads ? *reinterpret_cast<const float4*>(wy + 4 * q) : make_float4(0.f, 0.f, 0.f, 0.f);
+        }
+    }
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
         const int q = threadIdx.x + k * NT;
@@ -100,27 +111,27 @@ __global__ void __launch_bounds__(NT) stream_layernorm_vec_kernel(float* __restr
             const int q = threadIdx.x + k * NT;
             d[k] = q < quads ? load4<TD>(y + r + 4 * q) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
-        const Moments m = row_moments<VPT>(d, quads, hidden, eps_y, scratch);
+        const Moments m = row_moments<NT, VPT>(d, quads, hidden, eps_y, scratch[0]);
 #pragma unroll
         for (int k = 0; k < VPT; ++k) {
             const int q = threadIdx.x + k * NT;
             if (q < quads) {
-                const float4 a = *reinterpret_cast<const float4*>(wy + 4 * q);
+                const float4 a = AHEAD ? wyv[AHEAD ? k : 0] : *reinterpret_cast<const float4*>(wy + 4 * q);
                 v[k].x = fmaf((d[k].x - m.mean) * m.rstd, a.x, v[k].x); v[k].y = fmaf((d[k].y - m.mean) * m.rstd, a.y, v[k].y);
                 v[k].z = fmaf((d[k].z - m.mean) * m.rstd, a.z, v[k].z); v[k].w = fmaf((d[k].w - m.mean) * m.rstd, a.w, v[k].w);
             }
         }
     }
     Moments m{0.f, 1.f};
-    if (w) m = row_moments<VPT>(v, quads, hidden, eps, scratch);
+    if (w) m = row_moments<NT, VPT>(v, quads, hidden, eps, scratch[1]);
     TY* o = out + (size_t)blockIdx.x * hidden;
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
         const int q = threadIdx.x + k * NT;
         if (q >= quads) continue;
         if (!keep) *reinterpret_cast<float4*>(x + r + 4 * q) = v[k];
-        float4 a = make_float4(1.f, 1.f, 1.f, 1.f);
-        if (w) a = *reinterpret_cast<const float4*>(w + 4 * q);
+        float4 a = wv[AHEAD ? k : 0];
+        if (!AHEAD) a = w ? *reinterpret_cast<const float4*>(w + 4 * q) : make_float4(1.f, 1.f, 1.f, 1.f);
         store4<TY>(o + 4 * q, make_float4((v[k].x - m.mean) * m.rstd * a.x, (v[k].y - m.mean) * m.rstd * a.y, (v[k].z - m.mean) * m.rstd * a.z,
                                           (v[k].w - m.mean) * m.rstd * a.w));
     }
@@ -129,23 +140,23 @@ __global__ void __launch_bounds__(NT) stream_layernorm_vec_kernel(float* __restr
 // the statistics of a row whose entry i is at(i), i over the block's threads
 template <typename F> __device__ __forceinline__ Moments loop_moments(F at, int hidden, float eps, float* scratch) {
     float sum = 0.f, count = 0.f;
-    for (int i = threadIdx.x; i < hidden; i += NT) { sum += at(i); count += 1.f; }
+    for (int i = threadIdx.x; i < hidden; i += LOOP_NT) { sum += at(i); count += 1.f; }
     sum = warp_sum(sum);
     count = warp_sum(count);
     const float m = count > 0.f ? sum / count : 0.f;
     float m2 = 0.f;
-    for (int i = threadIdx.x; i < hidden; i += NT) { const float d = at(i) - m; m2 += d * d; }
-    return combine(sum, warp_sum(m2), count, scratch, hidden, eps);
+    for (int i = threadIdx.x; i < hidden; i += LOOP_NT) { const float d = at(i) - m; m2 += d * d; }
+    return combine<LOOP_NT / 32>(sum, warp_sum(m2), count, scratch, hidden, eps);
 }
 
 template <typename TD, typename TY>
-__global__ void __launch_bounds__(NT) stream_layernorm_kernel(float* __restrict__ x, const TD* __restrict__ y, const float* __restrict__ wy, float eps_y,
+__global__ void __launch_bounds__(LOOP_NT) stream_layernorm_kernel(float* __restrict__ x, const TD* __restrict__ y, const float* __restrict__ wy, float eps_y,
                                                               const float* __restrict__ pre, const float* __restrict__ w, TY* __restrict__ out,
                                                               const int* __restrict__ rows, int hidden, float eps, int keep) {
-    __shared__ float scratch[3 * NW];
+    __shared__ float scratch[2][3 * LOOP_NT / 32];
     const size_t r = (rows ? (size_t)rows[blockIdx.x] : (size_t)blockIdx.x) * hidden;
     Moments my{0.f, 0.f};
-    if (y) my = loop_moments([&](int i) { return to_f32(y[r + i]); }, hidden, eps_y, scratch);
+    if (y) my = loop_moments([&](int i) { return to_f32(y[r + i]); }, hidden, eps_y, scratch[0]);
     auto sum = [&](int i) {                                   // the row as it will be; x is written only after its last reading
         float v = x[r + i];
         if (pre) v += pre[r + i];
@@ -153,9 +164,9 @@ __global__ void __launch_bounds__(NT) stream_layernorm_kernel(float* __restrict_
         return v;
     };
     Moments m{0.f, 1.f};
-    if (w) m = loop_moments(sum, hidden, eps, scratch);
+    if (w) m = loop_moments(sum, hidden, eps, scratch[1]);
     TY* o = out + (size_t)blockIdx.x * hidden;
-    for (int i = threadIdx.x; i < hidden; i += NT) {
+    for (int i = threadIdx.x; i < hidden; i += LOOP_NT) {
         const float v = sum(i);
         if (!keep) x[r + i] = v;
         o[i] = from_f32<TY>((v - m.mean) * m.rstd * (w ? w[i] : 1.f));
@@ -172,17 +183,19 @@ MI_EXPORT int mi_stream_layernorm(float* x, const void* y, const float* wy, floa
     if (y && !wy) return -2;
     keep = keep || rows || (!y && !pre);
     const uintptr_t all = (uintptr_t)x | (uintptr_t)y | (uintptr_t)wy | (uintptr_t)pre | (uintptr_t)w | (uintptr_t)out;
-    const bool vec = hidden % 4 == 0 && hidden <= 8 * 4 * NT && all % 16 == 0;
+    const bool vec = hidden % 4 == 0 && hidden <= 8192 && all % 16 == 0;
     const int quads = hidden / 4;
+#define VEC(TD, TY, NT, VPT) stream_layernorm_vec_kernel<TD, TY, NT, VPT><<<n, NT, 0, stream>>>(x, (const TD*)y, wy, eps_y, pre, w, (TY*)out, rows, hidden, eps, keep)
 #define GO(TD, TY) do { \
-        if (!vec) stream_layernorm_kernel<TD, TY><<<n, NT, 0, stream>>>(x, (const TD*)y, wy, eps_y, pre, w, (TY*)out, rows, hidden, eps, keep); \
-        else if (quads <= NT) stream_layernorm_vec_kernel<TD, TY, 1><<<n, NT, 0, stream>>>(x, (const TD*)y, wy, eps_y, pre, w, (TY*)out, rows, hidden, eps, keep); \
-        else if (quads <= 2 * NT) stream_layernorm_vec_kernel<TD, TY, 2><<<n, NT, 0, stream>>>(x, (const TD*)y, wy, eps_y, pre, w, (TY*)out, rows, hidden, eps, keep); \
-        else if (quads <= 4 * NT) stream_layernorm_vec_kernel<TD, TY, 4><<<n, NT, 0, stream>>>(x, (const TD*)y, wy, eps_y, pre, w, (TY*)out, rows, hidden, eps, keep); \
-        else stream_layernorm_vec_kernel<TD, TY, 8><<<n, NT, 0, stream>>>(x, (const TD*)y, wy, eps_y, pre, w, (TY*)out, rows, hidden, eps, keep); } while (0)
+        if (!vec) stream_layernorm_kernel<TD, TY><<<n, LOOP_NT, 0, stream>>>(x, (const TD*)y, wy, eps_y, pre, w, (TY*)out, rows, hidden, eps, keep); \
+        else if (n >= 512) { if (quads <= 128) VEC(TD, TY, 128, 1); else if (quads <= 256) VEC(TD, TY, 128, 2); else if (quads <= 512) VEC(TD, TY, 128, 4); \
+                             else if (quads <= 1024) VEC(TD, TY, 256, 4); else VEC(TD, TY, 256, 8); } \
+        else { if (quads <= 256) VEC(TD, TY, 256, 1); else if (quads <= 512) VEC(TD, TY, 512, 1); else if (quads <= 1024) VEC(TD, TY, 512, 2); \
+               else VEC(TD, TY, 512, 4); } } while (0)
     if (y_dtype == MI_BF16 && out_dtype == MI_BF16) GO(__nv_bfloat16, __nv_bfloat16);
     else if (y_dtype == MI_F32 && out_dtype == MI_F32) GO(float, float);
     else return -1;
 #undef GO
+#undef VEC
     return (int)cudaGetLastError();
 }
