@@ -1059,13 +1059,19 @@ def bench_kofutar(args, ops, peak, out=print):
         state = torch.zeros(reps, B + 1, H * D * V + taps * C, device="cuda")
         p = rb(2, Tn, (C + H * V + 2 * H + 7) // 8 * 8)
         shape = f"{'prompt' if n > 1 else 'decode'} B={B} T={n} heads={H} {D}x{V}"
-        us = timed(lambda i: ops.gated_delta_mix(p[i % 2], conv, taps, rate, dtb, H, KV, D, V, 1e-6, norm, 1e-6, state[i % reps], batch), it)
+        cut = [(s, r) for s in range(B) for r in range(0, n, 64)]
+        lists = (t(cut).view(-1, 2), t(np.arange(B) * -(-n // 64))) if n > 1 else None
+        us = timed(lambda i: ops.gated_delta_mix(p[i % 2], conv, taps, rate, dtb, H, KV, D, V, 1e-6, norm, 1e-6, state[i % reps], batch, lists), it)
         moved = 2.0 * B * (H * D * V + (taps * C if n == 1 else 0)) * 4 + Tn * (C + 2 * H * V) * 2.0
         if n > 1:
             line("delta rule: filter, scan, gated norm", shape, us, 8.0 * H * D * V * Tn, "fma")
-            prep = torch.randn(Tn, C + 2 * H, device="cuda") * 0.1
+            prep = torch.randn(Tn, C + 3 * H, device="cuda") * 0.1
+            prep[:, C:] = 0.5
+            prep[:, C + 2 * H:] = -0.7
+            us = timed(lambda i: ops.gated_delta_scan(prep, H, KV, D, V, state[0], batch, lists), it)
+            line("  its scan in chunks on the tensor cores", shape, us, 8.0 * H * D * V * Tn, "fma")
             us = timed(lambda i: ops.gated_delta_scan(prep, H, KV, D, V, state[0], batch), it)
-            line("  its scan", shape, us, 8.0 * H * D * V * Tn, "fma")
+            line("  (the same token by token)", shape, us, 8.0 * H * D * V * Tn, "fma")
         else:
             line("delta rule: filter, state, gated norm (one kernel)", shape, us, moved, "hbm")
         nstate = torch.zeros(reps, B + 1, H * D * V + (taps - 1) * C, device="cuda")

@@ -7,8 +7,8 @@
 // conv float32 [C, taps], the last tap multiplies the current token.  A request's slot holds S (float32 [H, D, V]) and behind it a ring
 // of the convolution's inputs, [taps, C]: position p has row p mod taps, positions before 0 count as zeros.
 //
-// Prompts: delta_ready_kernel makes what the scan stages (float32 rows q | k | v | beta | f), the scan runs (recurrent.cu), then
-// delta_ring_kernel writes the entry's newest inputs into the ring.  Decode steps (every entry one token): delta_step_kernel does all of
+// Prompts: delta_ready_kernel makes what the scan reads (float32 rows q | k | v | beta | f | log f), the scan runs (gated_delta_chunk.cu, or
+// token by token in recurrent.cu), then delta_ring_kernel writes the entry's newest inputs into the ring.  Decode steps (every entry one token): delta_step_kernel does all of
 // it in one pass over the state, one block per (entry, head).  The ring has one row more than a token looks back on, so the block that
 // writes a token's inputs overwrites none that the other heads' blocks (which share a q and k head) still read.
 // Everything is float32; the decay is rounded once from a double-precision exponential, since it acts on a state hundreds of times in a row.
@@ -20,15 +20,15 @@ using namespace mi;
 namespace {
 
 __device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
-__device__ __forceinline__ float head_decay(float a, float dt_bias, float rate) {
+__device__ __forceinline__ double log_decay(float a, float dt_bias, float rate) {
     const double z = (double)a + (double)dt_bias;
-    return (float)exp(-(double)rate * (z > 30.0 ? z : log1p(exp(z))));
+    return -(double)rate * (z > 30.0 ? z : log1p(exp(z)));
 }
 
-// ------------------------------------------------------------------ prompts: what the scan stages
+// ------------------------------------------------------------------ prompts: what the scan reads
 // grid (token groups of TOK, units / 4), four warps, a warp per unit: the KV q heads, the KV k heads, then the value channels in pieces of
 // 32 NI, then one unit for the gates of all heads.  A lane owns the channels c0 + lane + 32 i of its unit (i < NI) with their taps in
-// registers and walks the group's tokens, its last taps - 1 inputs held in registers from token to token inside an entry.
+// registers.  A group inside one entry fetches its inputs all at once; a group that crosses entries goes token by token.
 template <typename T, int TAPS, int NI, int TOK>
 __global__ void __launch_bounds__(128) delta_ready_kernel(const T* __restrict__ p, int ldp, const float* __restrict__ conv, const float* __restrict__ rate,
                                                           const float* __restrict__ dt_bias, const float* __restrict__ state, long long state_stride,
@@ -42,63 +42,77 @@ __global__ void __launch_bounds__(128) delta_ready_kernel(const T* __restrict__ 
     const int C = 2 * KV * D + H * V, pieces = (H * V + 32 * NI - 1) / (32 * NI);
     const int t0 = blockIdx.x * TOK, t1 = min(T_, t0 + TOK);
     if (unit > 2 * KV + pieces) return;
-    if (unit == 2 * KV + pieces) {                             // beta and f of every head
+    if (unit == 2 * KV + pieces) {                             // beta, f and log f of every head
         for (int i = lane; i < (t1 - t0) * H; i += 32) {
             const int t = t0 + i / H, h = i % H;
             const T* row = p + (size_t)t * ldp + C + H * V;
             float* o = out + (size_t)t * ldo + C;
+            const double lf = log_decay(to_f32(row[H + h]), dt_bias[h], rate[h]);
             o[h] = 1.f / (1.f + expf(-to_f32(row[h])));
-            o[H + h] = head_decay(to_f32(row[H + h]), dt_bias[h], rate[h]);
+            o[H + h] = (float)exp(lf);
+            o[2 * H + h] = (float)lf;
         }
         return;
     }
     const bool head = unit < 2 * KV;
     const int c0 = head ? unit * D : 2 * KV * D + (unit - 2 * KV) * 32 * NI;
     const int n = head ? D : min(32 * NI, C - c0);
-    float w[NI][W], x[NI][W];
+    auto finish = [&](float (&y)[NI], int t) {                 // silu, the head's unit norm, out
+        float ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < NI; ++i)
-#pragma unroll
-        for (int j = 0; j < W; ++j) { w[i][j] = TAPS > 0 && lane + 32 * i < n ? conv[(size_t)(c0 + lane + 32 * i) * TAPS + j] : 0.f; x[i][j] = 0.f; }
-    int last = -1;                                             // the entry whose inputs the registers hold
-    for (int t = t0; t < t1; ++t) {
-        const int seg = token_seg[t], qs = seg_q_start[seg], r = t - qs, pos = positions[t];
-        const float* ring = state + (long long)seg_slot[seg] * state_stride + ring_off;
-        auto input = [&](int c, int back) {                    // the input `back` tokens before t
-            if (back <= r) return to_f32(p[(size_t)(t - back) * ldp + c]);
-            return back <= pos ? ring[(size_t)((pos - back) % taps) * C + c] : 0.f;
-        };
-        float y[NI], ss = 0.f;
-#pragma unroll
-        for (int i = 0; i < NI; ++i) {
-            y[i] = 0.f;
-            const int c = c0 + lane + 32 * i;
-            if (lane + 32 * i >= n) continue;
-            float acc = 0.f;
-            if constexpr (TAPS > 0) {
-                if (seg == last) {
-#pragma unroll
-                    for (int j = 0; j + 1 < TAPS; ++j) x[i][j] = x[i][j + 1];
-                } else {
-#pragma unroll
-                    for (int j = 0; j + 1 < TAPS; ++j) x[i][j] = input(c, TAPS - 1 - j);
-                }
-                x[i][TAPS - 1] = to_f32(p[(size_t)t * ldp + c]);
-#pragma unroll
-                for (int j = 0; j < TAPS; ++j) acc = fmaf(w[i][j], x[i][j], acc);
-            } else {
-                for (int j = 0; j < taps; ++j) acc = fmaf(conv[(size_t)c * taps + j], input(c, taps - 1 - j), acc);
-            }
-            y[i] = silu(acc);
-            ss = fmaf(y[i], y[i], ss);
-        }
-        last = seg;
+        for (int i = 0; i < NI; ++i) { y[i] = lane + 32 * i < n ? silu(y[i]) : 0.f; ss = fmaf(y[i], y[i], ss); }
         float s = 1.f;
         if (head) s = (unit < KV ? q_scale : 1.f) / sqrtf(warp_sum(ss) + unit_eps);
         float* o = out + (size_t)t * ldo + c0;
 #pragma unroll
         for (int i = 0; i < NI; ++i)
             if (lane + 32 * i < n) o[lane + 32 * i] = y[i] * s;
+    };
+    auto input = [&](int c, int back, int t, int r, int pos, const float* ring) {      // the input `back` tokens before t
+        if (back <= r) return to_f32(p[(size_t)(t - back) * ldp + c]);
+        return back <= pos ? ring[(size_t)((pos - back) % taps) * C + c] : 0.f;
+    };
+    const int seg0 = token_seg[t0];
+    if (TAPS > 0 && t1 - t0 == TOK && token_seg[t1 - 1] == seg0) {
+        const int qs = seg_q_start[seg0], r = t0 - qs, pos = positions[t0];
+        const float* ring = state + (long long)seg_slot[seg0] * state_stride + ring_off;
+        float w[NI][W], x[NI][TOK + W - 1];
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int c = c0 + lane + 32 * i;
+            const bool mine = lane + 32 * i < n;
+#pragma unroll
+            for (int j = 0; j < W; ++j) w[i][j] = mine ? conv[(size_t)c * W + j] : 0.f;
+#pragma unroll
+            for (int j = 0; j < W - 1; ++j) x[i][j] = mine ? input(c, W - 1 - j, t0, r, pos, ring) : 0.f;
+#pragma unroll
+            for (int k = 0; k < TOK; ++k) x[i][W - 1 + k] = mine ? to_f32(p[(size_t)(t0 + k) * ldp + c]) : 0.f;
+        }
+#pragma unroll
+        for (int k = 0; k < TOK; ++k) {
+            float y[NI];
+#pragma unroll
+            for (int i = 0; i < NI; ++i) {
+                y[i] = 0.f;
+#pragma unroll
+                for (int j = 0; j < W; ++j) y[i] = fmaf(w[i][j], x[i][k + j], y[i]);
+            }
+            finish(y, t0 + k);
+        }
+        return;
+    }
+    for (int t = t0; t < t1; ++t) {
+        const int seg = token_seg[t], r = t - seg_q_start[seg], pos = positions[t];
+        const float* ring = state + (long long)seg_slot[seg] * state_stride + ring_off;
+        float y[NI];
+#pragma unroll
+        for (int i = 0; i < NI; ++i) {
+            const int c = c0 + lane + 32 * i;
+            y[i] = 0.f;
+            if (lane + 32 * i < n)
+                for (int j = 0; j < taps; ++j) y[i] = fmaf(conv[(size_t)c * taps + j], input(c, taps - 1 - j, t, r, pos, ring), y[i]);
+        }
+        finish(y, t);
     }
 }
 
@@ -156,7 +170,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const T* __restrict__ p
         if (taps > 1 && (i >= 2 * D || h % rep == 0)) ring[(size_t)(pos % taps) * C + c] = own;      // one writer a channel
     }
     const float beta = 1.f / (1.f + expf(-to_f32(row[C + H * V + h])));
-    const float f = head_decay(to_f32(row[C + H * V + H + h]), dt_bias[h], rate[h]);
+    const float f = (float)exp(log_decay(to_f32(row[C + H * V + H + h]), dt_bias[h], rate[h]));
     const float rq = q_scale / sqrtf(block_sum<256>(sq, scratch) + unit_eps), rk = 1.f / sqrtf(block_sum<256>(sk, scratch) + unit_eps);
     // (block_sum's barriers also make qs, ks and vs visible)
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
@@ -208,13 +222,13 @@ int launch_ready(const T* p, int ldp, const float* conv, const float* rate, cons
                  int T_, int H, int KV, int D, int V, int taps, float unit_eps, cudaStream_t stream) {
     const int NI = D <= 32 ? 1 : D <= 64 ? 2 : D <= 128 ? 4 : 8;
     const int units = 2 * KV + (H * V + 32 * NI - 1) / (32 * NI) + 1;
-    const int TOK = T_ >= 1024 ? 16 : T_ >= 128 ? 4 : 1;
+    const int TOK = T_ >= 512 ? 8 : T_ >= 128 ? 4 : 1;
     dim3 grid((T_ + TOK - 1) / TOK, (units + 3) / 4);
     if (grid.y > 65535) return -2;
     const float q_scale = 1.f / sqrtf((float)D);
 #define GO(TAPS, N, TK) delta_ready_kernel<T, TAPS, N, TK><<<grid, 128, 0, stream>>>(p, ldp, conv, rate, dt_bias, state, state_stride, ring_off, out, ldo, \
                             positions, token_seg, seg_q_start, seg_slot, T_, H, KV, D, V, taps, unit_eps, q_scale)
-#define TOKENS(TAPS, N) do { if (TOK == 16) GO(TAPS, N, 16); else if (TOK == 4) GO(TAPS, N, 4); else GO(TAPS, N, 1); } while (0)
+#define TOKENS(TAPS, N) do { if (TOK == 8) GO(TAPS, N, 8); else if (TOK == 4) GO(TAPS, N, 4); else GO(TAPS, N, 1); } while (0)
 #define CHANNELS(TAPS) do { if (NI == 1) TOKENS(TAPS, 1); else if (NI == 2) TOKENS(TAPS, 2); else if (NI == 4) TOKENS(TAPS, 4); else TOKENS(TAPS, 8); } while (0)
     if (taps == 4) CHANNELS(4); else if (taps == 3) CHANNELS(3); else if (taps == 2) CHANNELS(2); else CHANNELS(0);
 #undef CHANNELS
@@ -225,7 +239,7 @@ int launch_ready(const T* p, int ldp, const float* conv, const float* rate, cons
 
 }  // namespace
 
-// out [T, ldo] float32 = q | k | v | beta [H] | f [H] (ldo may pad)
+// out [T, ldo] float32 = q | k | v | beta [H] | f [H] | log f [H] (ldo may pad)
 MI_EXPORT int mi_gated_delta_ready(const void* p, int ldp, const float* conv, const float* rate, const float* dt_bias, const float* state,
                                    long long state_stride, long long ring_off, float* out, int ldo, const int* positions, const int* token_seg,
                                    const int* seg_q_start, const int* seg_slot, int T_, int H, int KV, int D, int V, int taps, float unit_eps, int dtype,

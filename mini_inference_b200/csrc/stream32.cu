@@ -102,6 +102,43 @@ __global__ void group_rmsnorm_gate_kernel(const float* __restrict__ o, const flo
     }
 }
 
+// The same for groups of up to 512 entries in whole quads: a warp per group, four neighbouring entries a lane and step (NQ steps), the
+// group in registers between the statistic and the output.
+template <typename T> __device__ __forceinline__ float4 quad_of(const T* p) {
+    float a, b, c, d;
+    load2(p, a, b);
+    load2(p + 2, c, d);
+    return make_float4(a, b, c, d);
+}
+template <typename TG, typename TY, int NQ>
+__global__ void __launch_bounds__(NT) group_rmsnorm_gate_warp_kernel(const float* __restrict__ o, const float* __restrict__ w, int wlen, const TG* __restrict__ gate,
+                                                                     int gate_stride, TY* __restrict__ y, long long units, int groups, int gs, float eps, int act) {
+    const long long u = (long long)blockIdx.x * (NT / 32) + (threadIdx.x >> 5);
+    if (u >= units) return;
+    const int lane = threadIdx.x & 31, c0 = (int)(u % groups) * gs;
+    const size_t t = u / groups, base = t * groups * gs + c0;
+    float4 v[NQ], gv[NQ];
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < NQ; ++k) {
+        const int i = 4 * (lane + 32 * k);
+        v[k] = i < gs ? *reinterpret_cast<const float4*>(o + base + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        gv[k] = i < gs ? quad_of<TG>(gate + t * gate_stride + c0 + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+        ss += v[k].x * v[k].x + v[k].y * v[k].y + v[k].z * v[k].z + v[k].w * v[k].w;
+    }
+    const float r = rsqrtf(warp_sum(ss) / gs + eps);
+    auto gated = [&](float a, float g) { const float sg = 1.f / (1.f + expf(-g)); return a * r * (act == 1 ? sg * g : sg); };
+#pragma unroll
+    for (int k = 0; k < NQ; ++k) {
+        const int i = 4 * (lane + 32 * k);
+        if (i >= gs) continue;
+        float4 wv = make_float4(1.f, 1.f, 1.f, 1.f);
+        if (w) wv = *reinterpret_cast<const float4*>(w + (c0 + i) % wlen);
+        store2(y + base + i, gated(v[k].x, gv[k].x) * wv.x, gated(v[k].y, gv[k].y) * wv.y);
+        store2(y + base + i + 2, gated(v[k].z, gv[k].z) * wv.z, gated(v[k].w, gv[k].w) * wv.w);
+    }
+}
+
 // ------------------------------------------------------------------ rows[t, h V + v] = o[h, t, v] * sigmoid(gate[t, h])
 template <typename T>
 __global__ void head_gate_kernel(const T* __restrict__ o, const T* __restrict__ gate, int gate_stride, T* __restrict__ y, int T_, int H, int V) {
@@ -270,6 +307,17 @@ MI_EXPORT int mi_polynorm(const void* z, const float* coef, void* out, int rows,
 MI_EXPORT int mi_group_rmsnorm_gate(const float* o, const float* w, int wlen, const void* gate, int gate_stride, void* y,
                                     int T_, int groups, int gs, float eps, int dtype, int act, cudaStream_t stream) {
     if (T_ == 0) return 0;
+    const int pair = dtype == MI_BF16 ? 4 : 8;                 // bytes of two neighbouring entries
+    if (gs % 4 == 0 && gs <= 512 && wlen % 4 == 0 && gate_stride % 2 == 0 && (uintptr_t)gate % pair == 0 && ((uintptr_t)o | (uintptr_t)w) % 16 == 0 && (uintptr_t)y % pair == 0) {
+        const long long units = (long long)T_ * groups;
+        const int blocks = (int)((units + NT / 32 - 1) / (NT / 32));
+#define GO(TT, NQ) group_rmsnorm_gate_warp_kernel<TT, TT, NQ><<<blocks, NT, 0, stream>>>(o, w, wlen, (const TT*)gate, gate_stride, (TT*)y, units, groups, gs, eps, act)
+#define PICK(TT) do { if (gs <= 128) GO(TT, 1); else if (gs <= 256) GO(TT, 2); else GO(TT, 4); } while (0)
+        if (dtype == MI_BF16) PICK(__nv_bfloat16); else PICK(float);
+#undef PICK
+#undef GO
+        return (int)cudaGetLastError();
+    }
     if (groups > 65535) return -2;
     dim3 grid(T_, groups);
     if (dtype == MI_BF16)

@@ -128,8 +128,9 @@ class CudaOps:
         self.skinny_max_rows, self.skinny_max_cols = 16, 4096    # ... where it is at least as fast as the library's
         self.fast_attention = True           # tests clear this to run the generic attention kernels in bfloat16
         self.biased_attention_tc = True      # prompts of attention with a distance table or a learned sink on the tensor cores (bfloat16)
+        self.delta_work_bytes = 160 << 20    # scratch of the delta rule's chunks: as many heads at a time as fit
         self.fused_delta_step = True         # decode steps of the delta rule with one decay per head in one kernel (tests clear this)
-        self.chunked_scan = True             # prompts of a state space with one decay per head in chunks on the tensor cores (tests clear this)
+        self.chunked_scan = True             # prompts of a state space or delta rule with one decay per head in chunks on the tensor cores (tests clear this)
         # Latent attention whose cached rows have 64 or 128 entries can run on the tensor-core paged attention kernels.  Those
         # round the softmax weights to bfloat16 before the weighted sum; a design that asks for float32 weights gets the
         # float32 kernels of csrc/attention_latent.cu unless MI_LATENT_TC=1 (or this flag) says otherwise.
@@ -475,7 +476,7 @@ class CudaOps:
         if code != 0:
             self._stream_error.zero_()
             self._tc2_counters.zero_()
-            raise RuntimeError(f"a pipeline wait inside a kernel ran out (code {code}: 1-2 gemm_stream, 21+ attention, 51-55 gemm_tc2, 61-63 grouped expert product)")
+            raise RuntimeError(f"a pipeline wait inside a kernel ran out (code {code}: 1-2 gemm_stream, 21+ attention, 51-55 gemm_tc2, 61-63 grouped expert product, 71 delta-rule chunks)")
 
     # ---------------------------------------------------------------- q/k norm, rotation, cache write
     def qk_norm_rope_cache(self, qkv, H, KV, D, q_weight, k_weight, eps, inv_freq, meta, k_cache, v_cache):
@@ -1393,11 +1394,13 @@ class CudaOps:
         self.launches += 1
         return rows
 
-    def gated_delta_mix(self, p, conv, taps, rate, dt_bias, H, KV, D, V, unit_eps, norm, eps, state, batch):
+    def gated_delta_mix(self, p, conv, taps, rate, dt_bias, H, KV, D, V, unit_eps, norm, eps, state, batch, chunks=None):
         """p [T, >= C + H V + 2 H] = q | k | v | gate | b | a as projected (C = 2 KV D + H V).  q, k, v pass the convolution and silu, q and k
         become unit vectors (q * D^-1/2); beta = sigmoid(b), f = exp(-rate softplus(a + dt_bias)); S <- f S, u = beta (v - S^T k),
         S <- S + k u^T, o = S^T q from the slot's state (float32 H D V; behind it the ring of inputs [taps, C]).  Returns the rows
-        o / rms(o) * norm * silu(gate) per head in p's dtype."""
+        o / rms(o) * norm * silu(gate) per head in p's dtype.  chunks: (int32 [n, 2] of (entry, first row), every entry cut into chunks of 64
+        rows; int32 [entries], the number of each entry's first chunk), for the form that scans prompts in chunks on the tensor cores
+        (bfloat16, heads of 64 or 128); without them prompts are scanned token by token."""
         T, C, ring = p.shape[0], 2 * KV * D + H * V, H * D * V
         assert p.stride(1) == 1 and p.shape[1] >= C + H * V + 2 * H and conv.dtype == torch.float32 and conv.is_contiguous() and conv.shape == (C, taps)
         assert state.dtype == torch.float32 and state.is_contiguous() and state.shape[1] >= ring + (taps * C if taps > 1 else 0)
@@ -1411,23 +1414,37 @@ class CudaOps:
                 return rows
             if rc != -2:
                 _check(rc, "gated_delta_step")
-        prep = torch.empty((T, (C + 2 * H + 3) // 4 * 4), dtype=torch.float32, device=p.device)
+        prep = torch.empty((T, (C + 3 * H + 3) // 4 * 4), dtype=torch.float32, device=p.device)
         _check(self.lib.mi_gated_delta_ready(_p(p), p.stride(0), _p(conv), _p(rate), _p(dt_bias), _p(state), *stride, _p(prep), prep.stride(0), _p(batch.positions),
                                              _p(batch.token_seg), _p(batch.seg_q_start), _p(batch.seg_slot), T, H, KV, D, V, taps, _c.c_float(unit_eps), code,
                                              self._stream()), "gated_delta_ready")
-        o = self.gated_delta_scan(prep, H, KV, D, V, state, batch)
+        o = self.gated_delta_scan(prep, H, KV, D, V, state, batch, chunks if p.dtype == torch.bfloat16 else None)
         if taps > 1:
             _check(self.lib.mi_gated_delta_ring(_p(p), p.stride(0), _p(state), *stride, _p(batch.positions), _p(batch.seg_q_start), _p(batch.seg_slot), batch.num_segs,
                                                 C, taps, code, self._stream()), "gated_delta_ring")
         self.launches += 2 if taps > 1 else 1
         return self.group_rmsnorm_gate(o, norm, p[:, C:C + H * V], eps, H, V, p.dtype, act="silu")
 
-    def gated_delta_scan(self, prep, H, KV, D, V, state, batch):
-        """prep float32 [T, ..] = q [KV D] | k [KV D] | v [H V] | beta [H] | f [H]; S <- f S, u = beta (v - S^T k), S <- S + k u^T, o = S^T q
-        token by token.  float32 [T, H V]."""
+    def gated_delta_scan(self, prep, H, KV, D, V, state, batch, chunks=None):
+        """prep float32 [T, ..] = q [KV D] | k [KV D] | v [H V] | beta [H] | f [H] | log f [H]; S <- f S, u = beta (v - S^T k),
+        S <- S + k u^T, o = S^T q.  float32 [T, H V].  With chunks (see gated_delta_mix), sizes that have the form and more than a token or
+        two an entry: in chunks on the tensor cores, every float32 operand as two bfloat16 numbers; otherwise token by token in float32."""
         T = prep.shape[0]
         out = torch.empty((T, H * V), dtype=torch.float32, device=prep.device)
-        _check(self.lib.mi_gated_delta_scan(_p(prep), prep.stride(0), _p(state), _c.c_longlong(state.stride(0)), _p(out), _p(batch.seg_q_start), _p(batch.seg_slot),
+        stride = _c.c_longlong(state.stride(0))
+        per = int(self.lib.mi_delta_chunk_bytes(D, V)) if chunks is not None and self.chunked_scan and T > 4 * batch.num_segs else -2
+        if per > 0:
+            lists, first = chunks
+            heads = max(1, min(H, self.delta_work_bytes // (lists.shape[0] * per)))
+            work = torch.empty(lists.shape[0] * per * heads, dtype=torch.uint8, device=prep.device)
+            rc = self.lib.mi_gated_delta_chunks(_p(prep), prep.stride(0), _p(lists), lists.shape[0], _p(first), _p(work), _c.c_longlong(work.numel()), _p(state), stride,
+                                                _p(out), _p(batch.seg_q_start), _p(batch.seg_slot), batch.num_segs, H, KV, D, V, _p(self._stream_error), self._stream())
+            if rc == 0:
+                self.launches += 2 * -(-H // heads)
+                return out
+            if rc != -2:
+                _check(rc, "gated_delta_chunks")
+        _check(self.lib.mi_gated_delta_scan(_p(prep), prep.stride(0), _p(state), stride, _p(out), _p(batch.seg_q_start), _p(batch.seg_slot),
                                             T, batch.num_segs, H, KV, D, V, self._stream()), "gated_delta_scan")
         self.launches += 1
         return out

@@ -16,6 +16,7 @@ channel_delta   q, k, v = silu(causal_conv(W h)); q, k unit vectors per head (q 
 """
 from __future__ import annotations
 
+import numpy as np
 import torch
 
 from .base import Part, StateNeed, WeightSpec, pad_rows, register_mixer
@@ -413,7 +414,9 @@ class GatedDeltaRule(Part):
     The state slot holds S (float32 [heads, key_dim, value_dim]) and behind it the convolution's inputs of the last conv_taps positions,
     a ring in which position p has row p mod conv_taps (one more than a token looks back on, so that the kernel which appends a token's
     own inputs overwrites nothing that its other blocks read).  A decode step is one kernel; prompts are made ready (convolution, norms,
-    gates) by one kernel and scanned by another."""
+    gates) by one kernel and then scanned, in chunks of CHUNK tokens on the tensor cores where the sizes have that form."""
+    CHUNK = 64
+    step_arrays_key = "delta_chunks"
 
     def __init__(self, spec):
         super().__init__(spec)
@@ -454,9 +457,19 @@ class GatedDeltaRule(Part):
     def step_flops(self, rows, pairs):
         return 8 * self.H * self.D * self.V * rows                 # decay, S^T k, rank-one update, read-out
 
+    @staticmethod
+    def step_arrays(facts):
+        """Every entry cut into chunks: (entry, first row) of each, and the number of an entry's first chunk (empty when no entry brings
+        more than one token: such a step is one kernel that needs neither)."""
+        lens = facts.lens if any(n > 1 for n in facts.lens) else []
+        cut = [(i, r) for i, n in enumerate(lens) for r in range(0, n, GatedDeltaRule.CHUNK)]
+        first = np.cumsum([0] + [-(-n // GatedDeltaRule.CHUNK) for n in lens])[:len(lens)]
+        return {"chunks": np.asarray(cut, dtype=np.int32).reshape(-1, 2), "first": np.asarray(first, dtype=np.int32).reshape(-1)}
+
     def forward(self, h, ctx, cache, position, owns_cache=True):
         ops = ctx.ops
         p = ops.linear(h, self.proj)
+        lists = ctx.batch.extras[self.step_arrays_key]
         rows = ops.gated_delta_mix(p, self.conv, self.taps, self.rate, self.dt_bias, self.H, self.KV, self.D, self.V, self.unit_eps, self.norm,
-                                   self.eps, cache.state, ctx.batch)
+                                   self.eps, cache.state, ctx.batch, chunks=(lists["chunks"], lists["first"]))
         return ops.linear(rows, self.o)

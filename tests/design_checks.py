@@ -55,12 +55,12 @@ def err(got, want):
 
 def assert_close(got, want, tol, what=""):
     """float32 (tol < 1e-2): every logit within tol of the largest.  bfloat16: the root mean square over the vocabulary within tol at
-    every position and within a quarter of it at the median one."""
+    every position and within a third of it at the median one."""
     if tol < 1e-2:
         assert err(got, want) < tol, (what, err(got, want))
         return
     per = (got - want).pow(2).mean(-1).sqrt() / want.pow(2).mean(-1).sqrt()
-    assert per.max().item() < tol and per.median().item() < tol / 4, (what, per.median().item(), per.max().item())
+    assert per.max().item() < tol and per.median().item() < tol / 3, (what, per.median().item(), per.max().item())
 
 
 def engine(d, page, pages, dtype="float32", device="cpu", max_seqs=4):

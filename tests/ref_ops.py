@@ -892,7 +892,7 @@ def _sigmoid_gate(self, rows, gate):
     return rows
 
 
-def _gated_delta_mix(self, p, conv, taps, rate, dt_bias, H, KV, D, V, unit_eps, norm, eps, state, batch):
+def _gated_delta_mix(self, p, conv, taps, rate, dt_bias, H, KV, D, V, unit_eps, norm, eps, state, batch, chunks=None):
     T, C, base = p.shape[0], 2 * KV * D + H * V, H * D * V
     x = p[:, :C].float()
     out = torch.empty(T, H, V, device=p.device)

@@ -22,7 +22,7 @@ from mini_inference_b200.config.kofutar_config import KofutarConfig
 from mini_inference_b200.engine.batch import StepEntry
 from mini_inference_b200.engine.factory import make_runner
 from mini_inference_b200.parts.base import KVCacheNeed, NormedDelta, StateNeed, build_part
-from mini_inference_b200.parts.model import DecoderModel
+from mini_inference_b200.parts.recurrent import GatedDeltaRule
 from mini_inference_b200.weights import write_random_model
 from tests.design_checks import Judge, assert_close, check_cuts, check_mixed, engine, err, feed, rewrite_weights, tokens
 from tests.plain import kofutar_plain as plain
@@ -439,6 +439,18 @@ def test_far_keys_and_the_sink_on_cpu(L, hot, kind):
             assert (out - want).abs().max() < 1e-4 * want.abs().max() + 1e-6
 
 
+def chunk_lists(lens, device):
+    lists = GatedDeltaRule.step_arrays(SimpleNamespace(lens=lens))
+    return torch.from_numpy(lists["chunks"]).to(device), torch.from_numpy(lists["first"]).to(device)
+
+
+def test_chunk_lists():
+    a, first = chunk_lists([1, 130, 64, 2], "cpu")
+    assert a.tolist() == [[0, 0], [1, 0], [1, 64], [1, 128], [2, 0], [3, 0]] and first.tolist() == [0, 1, 4, 5]
+    a, first = chunk_lists([1, 1, 1], "cpu")                       # a decode step needs none (and their number depends on the lengths alone)
+    assert a.shape == (0, 2) and first.shape == (0,)
+
+
 def remembering_case(ops, device, dtype, cuts, H=4, KV=2, D=16, V=12, taps=3, T=301):
     """A state that must remember: token 0 alone writes (beta near 1 at it, next to nothing behind it), 300 quiet tokens with keys
     orthogonal to the first follow, and the last one asks with the first one's key.  What is read is known: f^300 D^-1/2 beta_0 v_0 -- a
@@ -468,7 +480,7 @@ def remembering_case(ops, device, dtype, cuts, H=4, KV=2, D=16, V=12, taps=3, T=
         batch = SimpleNamespace(num_segs=1, host={"seg_q_start": [0, n], "seg_slot": [1]}, seg_q_start=_i32([0, n], device), seg_slot=_i32([1], device),
                                 token_seg=_i32([0] * n, device), positions=_i32(list(range(at, at + n)), device))
         out = ops.gated_delta_mix(p[at:at + n].to(device), conv.to(device), taps, rate.to(device), dt_bias.to(device), H, KV, D, V, 1e-6, norm.to(device), 1e-12,
-                                  st, batch)
+                                  st, batch, chunks=chunk_lists([n], device) if n > 1 else None)
         at += n
     assert at == T
     silu = torch.nn.functional.silu
@@ -565,13 +577,13 @@ def test_far_keys_and_the_sink_on_gpu(L, hot, dtype):
 @pytest.mark.parametrize("cuts", CUTS_301, ids=lambda c: f"{len(c)}cuts")
 def test_a_state_that_must_remember_on_gpu(cuts, dtype):
     ops = cuda_ops()
-    for H, KV, D, V, taps in ((4, 2, 16, 12, 3), (2, 1, 128, 128, 4), (4, 4, 64, 32, 1), (3, 1, 20, 7, 2), (2, 2, 64, 128, 4)):
-        for fused in (True, False):
-            ops.fused_delta_step = fused
+    for H, KV, D, V, taps in ((4, 2, 16, 12, 3), (2, 1, 128, 128, 4), (4, 4, 64, 32, 1), (3, 1, 20, 7, 2), (2, 2, 64, 128, 4), (3, 1, 64, 64, 2), (2, 1, 128, 64, 3)):
+        for fused in (True, False):                                # decode steps in one kernel; prompts in chunks where the sizes have the form
+            ops.fused_delta_step = ops.chunked_scan = fused
             try:
                 out, want, state, S = remembering_case(ops, "cuda:0", dtype, cuts, H, KV, D, V, taps)
             finally:
-                ops.fused_delta_step = True
+                ops.fused_delta_step = ops.chunked_scan = True
             assert (out - want).abs().max() < (1e-4 if dtype == torch.float32 else 2e-2) * want.abs().max(), (H, KV, D, V, taps, fused)
             assert (state - S).abs().max() < (1e-4 if dtype == torch.float32 else 2e-3) * S.abs().max(), (H, KV, D, V, taps, fused)
     ops.check_errors()
@@ -646,7 +658,8 @@ def test_kernels_against_the_stand_ins(dtype, lens, starts):
             want = ref.latent_prepare(p, q_abs, H, D, R, C, nw, 1e-5, inv, ca, pa, q_rows=qp, dkv_col=q_rank, half_pairs=half)
             got = ops.latent_prepare(mv(p), mv(q_abs), H, D, R, C, mv(nw), 1e-5, mv(inv), cg, pb, q_rows=mv(qp), dkv_col=q_rank, half_pairs=half)
             assert close(got, want) and close(pb, pa), (H, D, R, C, nf, half)
-    for H, KV, D, V, taps in ((4, 2, 6, 8, 3), (3, 1, 7, 5, 2), (2, 2, 32, 64, 4), (6, 2, 64, 36, 1), (4, 1, 128, 128, 4), (1, 1, 200, 96, 5), (2, 1, 256, 132, 4), (16, 8, 128, 128, 4)):
+    for H, KV, D, V, taps in ((4, 2, 6, 8, 3), (3, 1, 7, 5, 2), (2, 2, 32, 64, 4), (6, 2, 64, 36, 1), (4, 1, 128, 128, 4), (2, 2, 64, 64, 3), (3, 1, 64, 128, 2), (2, 1, 128, 64, 4),
+                              (1, 1, 200, 96, 5), (2, 1, 256, 132, 4), (16, 8, 128, 128, 4)):
         C, rows = 2 * KV * D + H * V, (2 * KV * D + 2 * H * V + 2 * H + 7) // 8 * 8
         p = rnd(T, rows)
         conv, rate, dtb, norm = f32(C, taps) * 0.5, torch.exp(f32(H) - 1.0), f32(H) - 2.0, f32(V)
@@ -659,10 +672,54 @@ def test_kernels_against_the_stand_ins(dtype, lens, starts):
         for fused in (True, False):
             ops.fused_delta_step, sb = fused, state.to(dev)
             try:
-                got = ops.gated_delta_mix(mv(p), mv(conv), taps, mv(rate), mv(dtb), H, KV, D, V, 1e-6, mv(norm), 1e-5, sb, gpu_b)
+                got = ops.gated_delta_mix(mv(p), mv(conv), taps, mv(rate), mv(dtb), H, KV, D, V, 1e-6, mv(norm), 1e-5, sb, gpu_b,
+                                          chunks=chunk_lists(lens, dev) if fused else None)
             finally:
                 ops.fused_delta_step = True
             assert close(got, want) and close(sb, sa, 1e-4 if dtype == torch.float32 else 5e-3), (H, KV, D, V, taps, fused)
+    ops.check_errors()
+
+
+@gpu
+@pytest.mark.parametrize("D,V", [(64, 64), (64, 128), (128, 64), (128, 128)])
+def test_chunks_against_token_by_token(D, V):
+    """The scan in chunks on the tensor cores against the float32 scan of the same rows: entries that end inside a chunk, at its edge and one
+    behind it, single tokens among them; decays that forget at once, hardly ever, and per head; keys that repeat (I + A far from the unit
+    matrix); states that earlier steps left; scratch that holds one head, two heads or all."""
+    ops, dev = cuda_ops(), "cuda:0"
+    g = torch.Generator().manual_seed(D + V)
+    lens, H, KV = [64, 1, 65, 63, 200, 2, 129], 6, 2
+    T, S, C = sum(lens), len(lens), 2 * KV * D + H * V
+    starts = [sum(lens[:i]) for i in range(S + 1)]
+    batch = SimpleNamespace(num_segs=S, seg_q_start=_i32(starts, dev), seg_slot=_i32([3, 1, 7, 2, 5, 6, 4], dev))
+    prep = torch.zeros(T, (C + 3 * H + 3) // 4 * 4)
+    unit = torch.nn.functional.normalize
+    few = unit(torch.randn(5, D, generator=g), dim=-1)                                     # keys that come again and again
+    k = torch.where(torch.rand(T, KV, 1, generator=g) < 0.5, few[torch.randint(0, 5, (T, KV), generator=g)], unit(torch.randn(T, KV, D, generator=g), dim=-1))
+    prep[:, :KV * D] = (unit(torch.randn(T, KV, D, generator=g), dim=-1) * D ** -0.5).reshape(T, -1)
+    prep[:, KV * D:2 * KV * D] = k.reshape(T, -1)
+    prep[:, 2 * KV * D:C] = torch.randn(T, H * V, generator=g)
+    prep[:, C:C + H] = torch.rand(T, H, generator=g) * 0.98 + 0.01
+    lf = -torch.tensor([1e-6, 1e-3, 0.03, 0.5, 6.0, 60.0]) * (torch.rand(T, H, generator=g) + 0.5)
+    prep[:, C + H:C + 2 * H], prep[:, C + 2 * H:C + 3 * H] = lf.exp(), lf
+    prep, state = prep.to(dev), torch.randn(9, H * D * V + 8, generator=g).to(dev) * 0.2
+    want_state, lists = state.clone(), chunk_lists(lens, dev)
+    want = ops.gated_delta_scan(prep, H, KV, D, V, want_state, batch)
+    kept = ops.delta_work_bytes
+    for heads in (1, 4, 6):
+        got_state = state.clone()
+        ops.delta_work_bytes = heads * lists[0].shape[0] * int(ops.lib.mi_delta_chunk_bytes(D, V))
+        try:
+            before = ops.launches
+            got = ops.gated_delta_scan(prep, H, KV, D, V, got_state, batch, lists)
+            assert ops.launches - before == 2 * -(-H // heads)                             # the chunked form ran
+        finally:
+            ops.delta_work_bytes = kept
+        for h in range(H):
+            a, b = got.view(T, H, V)[:, h], want.view(T, H, V)[:, h]
+            assert (a - b).abs().max() < 2e-4 * b.abs().max(), (heads, h)
+        assert (got_state - want_state).abs().max() < 2e-4 * want_state.abs().max()
+        assert torch.equal(got_state[0], state[0]) and torch.equal(got_state[8], state[8])      # slots of nobody
     ops.check_errors()
 
 
