@@ -23,6 +23,8 @@ def main(argv=None) -> int:
     ap.add_argument("kind", choices=["decode", "prefill"])
     ap.add_argument("--size", default="4b", choices=sorted(SIZES))
     ap.add_argument("--layers", type=int, default=None)
+    ap.add_argument("--design", default=None, help="a design of the microbenchmarks (naditar, .., kofutar) at its size --design-size instead of --size")
+    ap.add_argument("--design-size", default="2k")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--ctx", type=int, default=4096)
     ap.add_argument("--tokens", type=int, default=2048, help="prefill: tokens of the prompt")
@@ -41,7 +43,10 @@ def main(argv=None) -> int:
     cfg = dict(dict(architectures=["Qwen3ForCausalLM"], rms_norm_eps=1e-6, max_position_embeddings=40960), **SIZES[a.size])
     if a.layers:
         cfg["num_hidden_layers"] = a.layers
-    vocab = cfg["vocab_size"]
+    if a.design:
+        from .microbench import DESIGNS
+        cfg = DESIGNS[a.design][0](a.design_size, a.layers or 8)
+    vocab = cfg["vocab"] if a.design else cfg["vocab_size"]
     llm = LLM(None, random_config=cfg, random_seed=0, dtype="bfloat16", device="cuda:0", kv_block_size=a.page_size,
               kv_cache_tokens=a.batch * a.ctx + 4096, kv_watermark=0.0, max_num_seqs=a.batch, max_model_len=a.ctx,
               max_batched_tokens=max(4096, a.tokens), cuda_graphs=False)

@@ -22,7 +22,8 @@ constexpr int WARPS = 4;
 // p [T, ldp]: q heads [H, D + R] | dkv [C + R] | ...;  q_abs [H, T, C] (the absorbed unrotated queries).
 // q_out [T, H, C + R] = [q_abs | rotate(q rot part)];  cache row = [rmsnorm(dkv[:C]) * w | rotate(dkv[C:])].
 // Rotation by the angle pos * inv_freq[i], i < nf: the pairs (2i, 2i+1), or with half_pairs (i, i + nf); entries from 2 nf on pass
-// unchanged.  The token's cosines and sines are made once, in shared memory (2 nf floats).
+// unchanged.  The token's cosines and sines are made once a block, in shared memory (2 nf floats).  grid (tokens, parts): part y takes the
+// query heads h = y, y + parts, .., the last part the cache row too; with VEC the absorbed queries move in 16-byte pieces.
 __device__ __forceinline__ float rotated(float own, float other, int j, int nf, int half_pairs, const float* cs, const float* sn) {
     const int i = half_pairs ? (j < nf ? j : j - nf) : j >> 1;
     const bool second = half_pairs ? j >= nf : j & 1;
@@ -30,7 +31,7 @@ __device__ __forceinline__ float rotated(float own, float other, int j, int nf, 
 }
 __device__ __forceinline__ int partner(int j, int nf, int half_pairs) { return half_pairs ? (j < nf ? j + nf : j - nf) : j ^ 1; }
 
-template <typename T>
+template <typename T, bool VEC>
 __global__ void latent_prepare_kernel(const T* __restrict__ p, int ldp, const T* __restrict__ q_rows, int ldq, int dkv_col,
                                       const T* __restrict__ q_abs, T* __restrict__ q_out,
                                       T* __restrict__ cache, const float* __restrict__ norm_w, const float* __restrict__ inv_freq,
@@ -45,18 +46,23 @@ __global__ void latent_prepare_kernel(const T* __restrict__ p, int ldp, const T*
     for (int i = threadIdx.x; i < nf; i += blockDim.x) sincosf(pos * inv_freq[i], turn + nf + i, turn + i);
     __syncthreads();
     T* qo = q_out + (size_t)t * H * (C + R);
-    for (int idx = threadIdx.x; idx < H * C; idx += blockDim.x) {
-        const int h = idx / C, i = idx - h * C;
-        qo[(size_t)h * (C + R) + i] = q_abs[((size_t)h * T_ + t) * C + i];
+    const int parts = gridDim.y, mine = (H - (int)blockIdx.y + parts - 1) / parts;        // this part's heads
+    constexpr int VN = VEC ? Vec16<T>::N : 1;
+    for (int idx = threadIdx.x; idx < mine * (C / VN); idx += blockDim.x) {
+        const int hh = idx / (C / VN), i = (idx - hh * (C / VN)) * VN, h = blockIdx.y + hh * parts;
+        const T* from = q_abs + ((size_t)h * T_ + t) * C + i;
+        T* to = qo + (size_t)h * (C + R) + i;
+        if constexpr (VEC) *reinterpret_cast<uint4*>(to) = *reinterpret_cast<const uint4*>(from);
+        else *to = *from;
     }
-    for (int idx = threadIdx.x; idx < H * R; idx += blockDim.x) {
-        const int h = idx / R, j = idx - h * R;
+    for (int idx = threadIdx.x; idx < mine * R; idx += blockDim.x) {
+        const int hh = idx / R, j = idx - hh * R, h = blockIdx.y + hh * parts;
         const T* src = qrow + (size_t)h * (D + R) + D;
         float val = to_f32(src[j]);
         if (j < 2 * nf) val = rotated(val, to_f32(src[partner(j, nf, half_pairs)]), j, nf, half_pairs, turn, turn + nf);
         qo[(size_t)h * (C + R) + C + j] = from_f32<T>(val);
     }
-    if (cache == nullptr) return;
+    if (cache == nullptr || blockIdx.y + 1 != parts) return;
     const T* dkv = row + dkv_col;
     float ss = 0.f;
     for (int i = threadIdx.x; i < C; i += blockDim.x) { const float v = to_f32(dkv[i]); ss += v * v; }
@@ -226,13 +232,14 @@ MI_EXPORT int mi_latent_prepare(const void* p, int ldp, const void* q_rows, int 
     const size_t smem = 2 * (size_t)nf * sizeof(float);
     if (!q_rows) { q_rows = p; ldq = ldp; }
     if (dkv_col < 0) dkv_col = H * (D + R);
-    if (dtype == MI_BF16)
-        latent_prepare_kernel<__nv_bfloat16><<<T_, 128, smem, stream>>>((const __nv_bfloat16*)p, ldp, (const __nv_bfloat16*)q_rows, ldq, dkv_col,
-                                                                     (const __nv_bfloat16*)q_abs, (__nv_bfloat16*)q_out,
-                                                                     (__nv_bfloat16*)cache, norm_w, inv_freq, nf, positions, slots, T_, H, D, R, C, eps, half_pairs);
-    else
-        latent_prepare_kernel<float><<<T_, 128, smem, stream>>>((const float*)p, ldp, (const float*)q_rows, ldq, dkv_col, (const float*)q_abs,
-                                                             (float*)q_out, (float*)cache, norm_w, inv_freq, nf, positions, slots, T_, H, D, R, C, eps, half_pairs);
+    const int per = dtype == MI_BF16 ? 8 : 4;
+    const bool vec = C % per == 0 && (C + R) % per == 0 && ((uintptr_t)q_abs | (uintptr_t)q_out) % 16 == 0;
+    dim3 grid(T_, T_ >= 256 ? 1 : min(H, 8));
+#define GO(T, VEC) latent_prepare_kernel<T, VEC><<<grid, 128, smem, stream>>>((const T*)p, ldp, (const T*)q_rows, ldq, dkv_col, (const T*)q_abs, (T*)q_out, (T*)cache, \
+                       norm_w, inv_freq, nf, positions, slots, T_, H, D, R, C, eps, half_pairs)
+    if (dtype == MI_BF16) { if (vec) GO(__nv_bfloat16, true); else GO(__nv_bfloat16, false); }
+    else { if (vec) GO(float, true); else GO(float, false); }
+#undef GO
     return (int)cudaGetLastError();
 }
 

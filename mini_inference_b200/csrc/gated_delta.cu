@@ -20,6 +20,11 @@ using namespace mi;
 namespace {
 
 __device__ __forceinline__ float silu(float x) { return x / (1.f + expf(-x)); }
+// behind a convolution of bfloat16 inputs the fast exponential and quotient (a few units in the last place of float32) are as good
+template <typename T> __device__ __forceinline__ float conv_silu(float x) {
+    if constexpr (sizeof(T) == 2) return __fdividef(x, 1.f + __expf(-x));
+    else return silu(x);
+}
 __device__ __forceinline__ double log_decay(float a, float dt_bias, float rate) {
     const double z = (double)a + (double)dt_bias;
     return -(double)rate * (z > 30.0 ? z : log1p(exp(z)));
@@ -60,7 +65,7 @@ __global__ void __launch_bounds__(128) delta_ready_kernel(const T* __restrict__ 
     auto finish = [&](float (&y)[NI], int t) {                 // silu, the head's unit norm, out
         float ss = 0.f;
 #pragma unroll
-        for (int i = 0; i < NI; ++i) { y[i] = lane + 32 * i < n ? silu(y[i]) : 0.f; ss = fmaf(y[i], y[i], ss); }
+        for (int i = 0; i < NI; ++i) { y[i] = lane + 32 * i < n ? conv_silu<T>(y[i]) : 0.f; ss = fmaf(y[i], y[i], ss); }
         float s = 1.f;
         if (head) s = (unit < KV ? q_scale : 1.f) / sqrtf(warp_sum(ss) + unit_eps);
         float* o = out + (size_t)t * ldo + c0;
@@ -129,22 +134,22 @@ __global__ void delta_ring_kernel(const T* __restrict__ p, int ldp, float* __res
 // ------------------------------------------------------------------ decode steps: everything in one pass over the state
 // grid (entries, H).  Thread (rg, cv) of a block holds four neighbouring columns 4 cv .. of the rows rg + RG i (i < NR), cv < V / 4,
 // RG = blockDim / (V / 4): the state is read once and written once, in 16-byte pieces, its loads issued before anything else.
-template <typename T, int NR>
-__global__ void __launch_bounds__(256) delta_step_kernel(const T* __restrict__ p, int ldp, const float* __restrict__ conv, int taps,
+template <typename T, int NR, int TAPS>
+__global__ void __launch_bounds__(256, NR <= 16 ? 2 : 1) delta_step_kernel(const T* __restrict__ p, int ldp, const float* __restrict__ conv, int taps_,
                                                          const float* __restrict__ rate, const float* __restrict__ dt_bias, float* __restrict__ state,
                                                          long long state_stride, long long ring_off, const float* __restrict__ norm, T* __restrict__ rows,
                                                          const int* __restrict__ positions, const int* __restrict__ seg_q_start,
                                                          const int* __restrict__ seg_slot, int H, int KV, int D, int V, float unit_eps, float q_scale, float eps) {
     extern __shared__ __align__(16) float sm[];
-    __shared__ float scratch[32];
+    __shared__ float2 squares[8];
+    __shared__ float outs[8], gates[2];
+    const int taps = TAPS > 0 ? TAPS : taps_;
     float* qs = sm;                                            // [D]
     float* ks = qs + D;                                        // [D]
     float* vs = ks + D;                                        // [V]: the values, then u
     float* red = sm + ((2 * D + V + 3) & ~3);                  // [RG, V]
-    const int seg = blockIdx.x, h = blockIdx.y, rep = H / KV, kvh = h / rep, tid = threadIdx.x;
-    const int t = seg_q_start[seg], pos = positions[t];
+    const int seg = blockIdx.x, h = blockIdx.y, rep = H / KV, kvh = h / rep, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     float* slot = state + (long long)seg_slot[seg] * state_stride;
-    float* ring = slot + ring_off;
     float* S = slot + (long long)h * D * V;
     const int CV = V >> 2, RG = 256 / CV, cv = tid % CV, rg = tid / CV;
     float4 s[NR];
@@ -153,26 +158,43 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const T* __restrict__ p
         const int r = rg + RG * i;
         s[i] = rg < RG && r < D ? *reinterpret_cast<const float4*>(S + (size_t)r * V + 4 * cv) : make_float4(0.f, 0.f, 0.f, 0.f);
     }
+    const int t = seg_q_start[seg], pos = positions[t];
+    float* ring = slot + ring_off;
     const T* row = p + (size_t)t * ldp;
     const int C = 2 * KV * D + H * V;
+    if (tid == 255) {                                          // one thread: beta and the decay (double-precision exponentials)
+        gates[0] = 1.f / (1.f + expf(-to_f32(row[C + H * V + h])));
+        gates[1] = (float)exp(log_decay(to_f32(row[C + H * V + H + h]), dt_bias[h], rate[h]));
+    }
     float sq = 0.f, sk = 0.f;
+#pragma unroll 2
     for (int i = tid; i < 2 * D + V; i += 256) {               // this head's q, k and v channels
         const int c = i < D ? kvh * D + i : i < 2 * D ? KV * D + kvh * D + i - D : 2 * KV * D + h * V + i - 2 * D;
         const float own = to_f32(row[c]);
         float acc = 0.f;
-        for (int j = 0; j + 1 < taps; ++j) {
+        auto tap = [&](int j) {
             const int back = taps - 1 - j;
             if (back <= pos) acc = fmaf(conv[(size_t)c * taps + j], ring[(size_t)((pos - back) % taps) * C + c], acc);
+        };
+        if constexpr (TAPS > 0) {
+#pragma unroll
+            for (int j = 0; j + 1 < TAPS; ++j) tap(j);
+        } else {
+            for (int j = 0; j + 1 < taps; ++j) tap(j);
         }
         const float y = silu(fmaf(conv[(size_t)c * taps + taps - 1], own, acc));
         sm[i] = y;
         if (i < D) sq = fmaf(y, y, sq); else if (i < 2 * D) sk = fmaf(y, y, sk);
         if (taps > 1 && (i >= 2 * D || h % rep == 0)) ring[(size_t)(pos % taps) * C + c] = own;      // one writer a channel
     }
-    const float beta = 1.f / (1.f + expf(-to_f32(row[C + H * V + h])));
-    const float f = (float)exp(log_decay(to_f32(row[C + H * V + H + h]), dt_bias[h], rate[h]));
-    const float rq = q_scale / sqrtf(block_sum<256>(sq, scratch) + unit_eps), rk = 1.f / sqrtf(block_sum<256>(sk, scratch) + unit_eps);
-    // (block_sum's barriers also make qs, ks and vs visible)
+    sq = warp_sum(sq);
+    sk = warp_sum(sk);
+    if (lane == 0) squares[warp] = make_float2(sq, sk);
+    __syncthreads();
+    sq = sk = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) { sq += squares[w].x; sk += squares[w].y; }
+    const float beta = gates[0], f = gates[1], rq = q_scale / sqrtf(sq + unit_eps), rk = 1.f / sqrtf(sk + unit_eps);
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
 #pragma unroll
     for (int i = 0; i < NR; ++i) {
@@ -184,6 +206,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const T* __restrict__ p
     __syncthreads();
     for (int c = tid; c < V; c += 256) {
         float dot = 0.f;
+#pragma unroll 8
         for (int g = 0; g < RG; ++g) dot += red[g * V + c];
         vs[c] = beta * (vs[c] - f * dot);
     }
@@ -207,11 +230,18 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const T* __restrict__ p
     float ss = 0.f;
     for (int c = tid; c < V; c += 256) {
         float o = 0.f;
+#pragma unroll 8
         for (int g = 0; g < RG; ++g) o += red[g * V + c];
         vs[c] = o;                                             // read again below by the same thread
         ss = fmaf(o, o, ss);
     }
-    const float r = rsqrtf(block_sum<256>(ss, scratch) / V + eps);
+    ss = warp_sum(ss);
+    if (lane == 0) outs[warp] = ss;
+    __syncthreads();
+    ss = 0.f;
+#pragma unroll
+    for (int w = 0; w < 8; ++w) ss += outs[w];
+    const float r = rsqrtf(ss / V + eps);
     for (int c = tid; c < V; c += 256)
         rows[(size_t)t * H * V + (size_t)h * V + c] = from_f32<T>(vs[c] * r * norm[c] * silu(to_f32(row[C + h * V + c])));
 }
@@ -277,11 +307,13 @@ MI_EXPORT int mi_gated_delta_step(const void* p, int ldp, const float* conv, int
     const size_t smem = (size_t)(((2 * D + V + 3) & ~3) + RG * V) * sizeof(float);
     const float q_scale = 1.f / sqrtf((float)D);
     dim3 grid(num_segs, H);
-#define GO(T, NR) delta_step_kernel<T, NR><<<grid, 256, smem, stream>>>((const T*)p, ldp, conv, taps, rate, dt_bias, state, state_stride, ring_off, norm, (T*)rows, \
+#define GO(T, NR, TAPS) delta_step_kernel<T, NR, TAPS><<<grid, 256, smem, stream>>>((const T*)p, ldp, conv, taps, rate, dt_bias, state, state_stride, ring_off, norm, (T*)rows, \
                       positions, seg_q_start, seg_slot, H, KV, D, V, unit_eps, q_scale, eps)
-#define PICK(T) do { if (need <= 4) GO(T, 4); else if (need <= 8) GO(T, 8); else if (need <= 16) GO(T, 16); else GO(T, 32); } while (0)
+#define ROWS(T, TAPS) do { if (need <= 4) GO(T, 4, TAPS); else if (need <= 8) GO(T, 8, TAPS); else if (need <= 16) GO(T, 16, TAPS); else GO(T, 32, TAPS); } while (0)
+#define PICK(T) do { if (taps == 4) ROWS(T, 4); else ROWS(T, 0); } while (0)
     if (dtype == MI_BF16) PICK(__nv_bfloat16); else PICK(float);
 #undef PICK
+#undef ROWS
 #undef GO
     return (int)cudaGetLastError();
 }

@@ -158,11 +158,17 @@ __device__ __forceinline__ float4 block_product(const float* A, const float* T, 
     const float* a = A + (ib * 16 + (e >> 2)) * lda;
     const float* t = T + jb * 16 + (e & 3) * 4;
     float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
-    for (int k = kb0 * 16; k < kb1 * 16; ++k) {
-        const float av = a[k];
-        const float4 tv = *reinterpret_cast<const float4*>(t + k * lda);
-        s.x = fmaf(av, tv.x, s.x); s.y = fmaf(av, tv.y, s.y); s.z = fmaf(av, tv.z, s.z); s.w = fmaf(av, tv.w, s.w);
-    }
+    for (int kb = kb0; kb < kb1; ++kb)
+#pragma unroll
+        for (int kk = 0; kk < 16; kk += 4) {
+            const float4 av = *reinterpret_cast<const float4*>(a + kb * 16 + kk);
+            const float ae[4] = {av.x, av.y, av.z, av.w};
+#pragma unroll
+            for (int e4 = 0; e4 < 4; ++e4) {
+                const float4 tv = *reinterpret_cast<const float4*>(t + (kb * 16 + kk + e4) * lda);
+                s.x = fmaf(ae[e4], tv.x, s.x); s.y = fmaf(ae[e4], tv.y, s.y); s.z = fmaf(ae[e4], tv.z, s.z); s.w = fmaf(ae[e4], tv.w, s.w);
+            }
+        }
     return s;
 }
 
@@ -214,11 +220,12 @@ __global__ void __launch_bounds__(NTH, 2) delta_chunk_kernel(const float* __rest
     for (int i = tid; i < Q * L::LDA; i += NTH) { A[i] = 0.f; T[i] = 0.f; }
     __syncthreads();
     // the six 16 x 32 tiles that reach below the diagonal: (0,0) (1,0) (2,0) (2,1) (3,0) (3,1)
-    const int task_rb[6] = {0, 1, 2, 2, 3, 3}, task_ch[6] = {0, 0, 0, 1, 0, 1};
+    auto task_rb = [](int i) { return i < 2 ? i : i < 4 ? 2 : 3; };
+    auto task_ch = [](int i) { return i == 3 || i == 5 ? 1 : 0; };
     const uint32_t kh = base + L::K, kl = kh + Q * D * 2, qh = base + L::QV, ql = qh + Q * D * 2;
     if (warp < 6) {
         float s[4][4];
-        const int rb = task_rb[warp], ch = task_ch[warp];
+        const int rb = task_rb(warp), ch = task_ch(warp);
         scores<D>(s, kh, kl, kh, kl, rb, ch, lane);
 #pragma unroll
         for (int nt = 0; nt < 4; ++nt)
@@ -231,7 +238,7 @@ __global__ void __launch_bounds__(NTH, 2) delta_chunk_kernel(const float* __rest
     __syncthreads();
     if (warp >= 2) {                                               // P, while two warps invert the diagonal blocks of I + A
         float s[4][4];
-        const int rb = task_rb[warp - 2], ch = task_ch[warp - 2];
+        const int rb = task_rb(warp - 2), ch = task_ch(warp - 2);
         scores<D>(s, qh, ql, kh, kl, rb, ch, lane);
 #pragma unroll
         for (int nt = 0; nt < 4; ++nt)
@@ -249,9 +256,13 @@ __global__ void __launch_bounds__(NTH, 2) delta_chunk_kernel(const float* __rest
         float x[16];
 #pragma unroll
         for (int i = 0; i < 16; ++i) {
-            float s = 0.f;
+            float s = 0.f, s2 = 0.f;
 #pragma unroll
-            for (int k = 0; k < i; ++k) s = fmaf(a[i * L::LDA + k], x[k], s);
+            for (int k = 0; k < i; k += 2) {
+                s = fmaf(a[i * L::LDA + k], x[k], s);
+                if (k + 1 < i) s2 = fmaf(a[i * L::LDA + k + 1], x[k + 1], s2);
+            }
+            s += s2;
             x[i] = i < j ? 0.f : i == j ? 1.f : -s;
             T[(b * 16 + i) * L::LDA + b * 16 + j] = x[i];
         }

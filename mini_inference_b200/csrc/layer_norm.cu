@@ -18,24 +18,21 @@ constexpr int LOOP_NT = 256;
 
 struct Moments { float mean, rstd; };
 
-// what the warps found (sum of their entries, squared deviations from their own mean, entries) -> the row's mean and 1 / deviation
-// (scratch: 3 NW floats that no earlier call of the block has used)
+// what the warps found (mean of their entries, squared deviations from it, entries) -> the row's mean and 1 / deviation
+// (scratch: a float4 per warp that no earlier call of the block has used)
 template <int NW>
-__device__ __forceinline__ Moments combine(float sum, float m2, float count, float* scratch, int hidden, float eps) {
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    if (lane == 0) { scratch[warp] = sum; scratch[NW + warp] = m2; scratch[2 * NW + warp] = count; }
+__device__ __forceinline__ Moments combine(float mean_w, float m2, float count, float4* scratch, int hidden, float eps) {
+    if ((threadIdx.x & 31) == 0) scratch[threadIdx.x >> 5] = make_float4(mean_w, m2, count, 0.f);
     __syncthreads();
-    float total = 0.f;
+    const float inv = 1.f / hidden;
+    float4 p[NW];
+    float total = 0.f, sq = 0.f;
 #pragma unroll
-    for (int w = 0; w < NW; ++w) total += scratch[w];
-    const float mean = total / hidden;
-    float sq = 0.f;
+    for (int w = 0; w < NW; ++w) { p[w] = scratch[w]; total = fmaf(p[w].x, p[w].z, total); }
+    const float mean = total * inv;
 #pragma unroll
-    for (int w = 0; w < NW; ++w) {
-        const float n = scratch[2 * NW + w], d = n > 0.f ? scratch[w] / n - mean : 0.f;
-        sq += fmaf(n * d, d, scratch[NW + w]);
-    }
-    return Moments{mean, rsqrtf(sq / hidden + eps)};
+    for (int w = 0; w < NW; ++w) { const float d = p[w].x - mean; sq += fmaf(p[w].z * d, d, p[w].y); }
+    return Moments{mean, rsqrtf(sq * inv + eps)};
 }
 
 template <typename TD> __device__ __forceinline__ float4 load4(const TD* p) {
@@ -57,7 +54,7 @@ template <typename TY> __device__ __forceinline__ void store4(TY* p, float4 v) {
 
 // Mean and deviation of a row held as v[VPT] (thread t: quads t, t + NT, ..; entries beyond the row are zero and not counted)
 template <int NT, int VPT>
-__device__ __forceinline__ Moments row_moments(const float4 (&v)[VPT], int quads, int hidden, float eps, float* scratch) {
+__device__ __forceinline__ Moments row_moments(const float4 (&v)[VPT], int quads, int hidden, float eps, float4* scratch) {
     const int warp0 = threadIdx.x & ~31;
     float sum = 0.f, count = 0.f;
 #pragma unroll
@@ -74,7 +71,7 @@ __device__ __forceinline__ Moments row_moments(const float4 (&v)[VPT], int quads
             const float a = v[k].x - m, b = v[k].y - m, c = v[k].z - m, d = v[k].w - m;
             m2 += (a * a + b * b) + (c * c + d * d);
         }
-    return combine<NT / 32>(sum, warp_sum(m2), count, scratch, hidden, eps);
+    return combine<NT / 32>(m, warp_sum(m2), count, scratch, hidden, eps);
 }
 
 // NT threads a row (few for many rows, so that more rows are in flight; many for few rows), VPT quads a thread
@@ -82,7 +79,7 @@ template <typename TD, typename TY, int NT, int VPT>
 __global__ void __launch_bounds__(NT) stream_layernorm_vec_kernel(float* __restrict__ x, const TD* __restrict__ y, const float* __restrict__ wy, float eps_y,
                                                                   const float* __restrict__ pre, const float* __restrict__ w, TY* __restrict__ out,
                                                                   const int* __restrict__ rows, int hidden, float eps, int keep) {
-    __shared__ float scratch[2][3 * NT / 32];
+    __shared__ float4 scratch[2][NT / 32];
     const size_t r = (rows ? (size_t)rows[blockIdx.x] : (size_t)blockIdx.x) * hidden;
     const int quads = hidden >> 2;
     constexpr bool AHEAD = VPT <= 2;                          // the weights are fetched with the row, so that no wait for them follows a sum
@@ -138,7 +135,7 @@ __global__ void __launch_bounds__(NT) stream_layernorm_vec_kernel(float* __restr
 }
 
 // the statistics of a row whose entry i is at(i), i over the block's threads
-template <typename F> __device__ __forceinline__ Moments loop_moments(F at, int hidden, float eps, float* scratch) {
+template <typename F> __device__ __forceinline__ Moments loop_moments(F at, int hidden, float eps, float4* scratch) {
     float sum = 0.f, count = 0.f;
     for (int i = threadIdx.x; i < hidden; i += LOOP_NT) { sum += at(i); count += 1.f; }
     sum = warp_sum(sum);
@@ -146,14 +143,14 @@ template <typename F> __device__ __forceinline__ Moments loop_moments(F at, int 
     const float m = count > 0.f ? sum / count : 0.f;
     float m2 = 0.f;
     for (int i = threadIdx.x; i < hidden; i += LOOP_NT) { const float d = at(i) - m; m2 += d * d; }
-    return combine<LOOP_NT / 32>(sum, warp_sum(m2), count, scratch, hidden, eps);
+    return combine<LOOP_NT / 32>(m, warp_sum(m2), count, scratch, hidden, eps);
 }
 
 template <typename TD, typename TY>
 __global__ void __launch_bounds__(LOOP_NT) stream_layernorm_kernel(float* __restrict__ x, const TD* __restrict__ y, const float* __restrict__ wy, float eps_y,
                                                               const float* __restrict__ pre, const float* __restrict__ w, TY* __restrict__ out,
                                                               const int* __restrict__ rows, int hidden, float eps, int keep) {
-    __shared__ float scratch[2][3 * LOOP_NT / 32];
+    __shared__ float4 scratch[2][LOOP_NT / 32];
     const size_t r = (rows ? (size_t)rows[blockIdx.x] : (size_t)blockIdx.x) * hidden;
     Moments my{0.f, 0.f};
     if (y) my = loop_moments([&](int i) { return to_f32(y[r + i]); }, hidden, eps_y, scratch[0]);
@@ -190,7 +187,7 @@ MI_EXPORT int mi_stream_layernorm(float* x, const void* y, const float* wy, floa
         if (!vec) stream_layernorm_kernel<TD, TY><<<n, LOOP_NT, 0, stream>>>(x, (const TD*)y, wy, eps_y, pre, w, (TY*)out, rows, hidden, eps, keep); \
         else if (n >= 512) { if (quads <= 128) VEC(TD, TY, 128, 1); else if (quads <= 256) VEC(TD, TY, 128, 2); else if (quads <= 512) VEC(TD, TY, 128, 4); \
                              else if (quads <= 1024) VEC(TD, TY, 256, 4); else VEC(TD, TY, 256, 8); } \
-        else { if (quads <= 256) VEC(TD, TY, 256, 1); else if (quads <= 512) VEC(TD, TY, 512, 1); else if (quads <= 1024) VEC(TD, TY, 512, 2); \
+        else { if (quads <= 256) VEC(TD, TY, 256, 1); else if (quads <= 512) VEC(TD, TY, 256, 2); else if (quads <= 1024) VEC(TD, TY, 512, 2); \
                else VEC(TD, TY, 512, 4); } } while (0)
     if (y_dtype == MI_BF16 && out_dtype == MI_BF16) GO(__nv_bfloat16, __nv_bfloat16);
     else if (y_dtype == MI_F32 && out_dtype == MI_F32) GO(float, float);
