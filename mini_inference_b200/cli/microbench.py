@@ -1129,6 +1129,7 @@ def bench_kofutar(args, ops, peak, out=print):
         us = timed(lambda i: ops.latent_attention(ql, lc, meta, LH, LC, R, 0.1), it)
         line("  Naditar: latent attention", f"B={B} rows={n} keys={ctx} heads={LH} rows {LC}+{R}", us, amount, bound)
         ro, oh = rb(Tn, LH * LV), rb(LH, Tn, LV)
+        cq[:, QR + LC + R:] = 20.0                                  # an open gate: it is applied in place, time after time
         us = timed(lambda i: ops.sigmoid_gate(ro, cq[:, QR + LC + R:]), it)
         line("latent: element gate", f"rows={Tn} heads={LH} V={LV}", us, Tn * LH * LV * 6.0, "hbm")
         us = timed(lambda i: ops.head_gate(oh, pn[:, -LH:], bf), it)

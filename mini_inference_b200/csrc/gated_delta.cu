@@ -11,11 +11,13 @@
 // token by token in recurrent.cu), then delta_ring_kernel writes the entry's newest inputs into the ring.  Decode steps (every entry one token): delta_step_kernel does all of
 // it in one pass over the state, one block per (entry, head).  The ring has one row more than a token looks back on, so the block that
 // writes a token's inputs overwrites none that the other heads' blocks (which share a q and k head) still read.
-// Everything is float32; the decay is rounded once from a double-precision exponential, since it acts on a state hundreds of times in a row.
-#include "common.cuh"
+// Everything is float32.  The decay acts on a state hundreds of times in a row, so it is made as 1 + expm1(.) where it is near one: rounded
+// once, not one-sided.
+#include "sm100.cuh"
 #include <math.h>
 
 using namespace mi;
+using namespace mi::sm100;
 
 namespace {
 
@@ -25,10 +27,11 @@ template <typename T> __device__ __forceinline__ float conv_silu(float x) {
     if constexpr (sizeof(T) == 2) return __fdividef(x, 1.f + __expf(-x));
     else return silu(x);
 }
-__device__ __forceinline__ double log_decay(float a, float dt_bias, float rate) {
-    const double z = (double)a + (double)dt_bias;
-    return -(double)rate * (z > 30.0 ? z : log1p(exp(z)));
+__device__ __forceinline__ float log_decay(float a, float dt_bias, float rate) {
+    const float z = a + dt_bias;
+    return -rate * (z > 20.f ? z : log1pf(expf(z)));
 }
+__device__ __forceinline__ float decay_of(float log_f) { return log_f > -0.7f ? 1.f + expm1f(log_f) : expf(log_f); }
 
 // ------------------------------------------------------------------ prompts: what the scan reads
 // grid (token groups of TOK, units / 4), four warps, a warp per unit: the KV q heads, the KV k heads, then the value channels in pieces of
@@ -52,10 +55,10 @@ __global__ void __launch_bounds__(128) delta_ready_kernel(const T* __restrict__ 
             const int t = t0 + i / H, h = i % H;
             const T* row = p + (size_t)t * ldp + C + H * V;
             float* o = out + (size_t)t * ldo + C;
-            const double lf = log_decay(to_f32(row[H + h]), dt_bias[h], rate[h]);
+            const float lf = log_decay(to_f32(row[H + h]), dt_bias[h], rate[h]);
             o[h] = 1.f / (1.f + expf(-to_f32(row[h])));
-            o[H + h] = (float)exp(lf);
-            o[2 * H + h] = (float)lf;
+            o[H + h] = decay_of(lf);
+            o[2 * H + h] = lf;
         }
         return;
     }
@@ -132,39 +135,46 @@ __global__ void delta_ring_kernel(const T* __restrict__ p, int ldp, float* __res
 }
 
 // ------------------------------------------------------------------ decode steps: everything in one pass over the state
-// grid (entries, H).  Thread (rg, cv) of a block holds four neighbouring columns 4 cv .. of the rows rg + RG i (i < NR), cv < V / 4,
-// RG = blockDim / (V / 4): the state is read once and written once, in 16-byte pieces, its loads issued before anything else.
-template <typename T, int NR, int TAPS>
-__global__ void __launch_bounds__(256, NR <= 16 ? 2 : 1) delta_step_kernel(const T* __restrict__ p, int ldp, const float* __restrict__ conv, int taps_,
+// grid (entries, H).  The head's state (D V contiguous floats) comes into shared memory as one bulk copy, under which the convolution, the
+// norms and the gates are made; thread (rg, cv) then owns the columns 4 cv .. of the rows rg + RG i, cv < V / 4, RG = 256 / (V / 4), in
+// both passes over it (S^T k; update, read-out and the way back to memory).
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(256) delta_step_kernel(const T* __restrict__ p, int ldp, const float* __restrict__ conv, int taps_,
                                                          const float* __restrict__ rate, const float* __restrict__ dt_bias, float* __restrict__ state,
                                                          long long state_stride, long long ring_off, const float* __restrict__ norm, T* __restrict__ rows,
                                                          const int* __restrict__ positions, const int* __restrict__ seg_q_start,
-                                                         const int* __restrict__ seg_slot, int H, int KV, int D, int V, float unit_eps, float q_scale, float eps) {
-    extern __shared__ __align__(16) float sm[];
+                                                         const int* __restrict__ seg_slot, int H, int KV, int D, int V, float unit_eps, float q_scale, float eps,
+                                                         int* __restrict__ error) {
+    extern __shared__ __align__(128) float sm[];
+    __shared__ __align__(8) uint64_t arrived;
     __shared__ float2 squares[8];
     __shared__ float outs[8], gates[2];
     const int taps = TAPS > 0 ? TAPS : taps_;
-    float* qs = sm;                                            // [D]
+    float* Ss = sm;                                            // [D, V]
+    float* qs = Ss + D * V;                                    // [D]
     float* ks = qs + D;                                        // [D]
     float* vs = ks + D;                                        // [V]: the values, then u
-    float* red = sm + ((2 * D + V + 3) & ~3);                  // [RG, V]
+    float* red = qs + ((2 * D + V + 3) & ~3);                  // [RG, V]
     const int seg = blockIdx.x, h = blockIdx.y, rep = H / KV, kvh = h / rep, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     float* slot = state + (long long)seg_slot[seg] * state_stride;
     float* S = slot + (long long)h * D * V;
-    const int CV = V >> 2, RG = 256 / CV, cv = tid % CV, rg = tid / CV;
-    float4 s[NR];
-#pragma unroll
-    for (int i = 0; i < NR; ++i) {
-        const int r = rg + RG * i;
-        s[i] = rg < RG && r < D ? *reinterpret_cast<const float4*>(S + (size_t)r * V + 4 * cv) : make_float4(0.f, 0.f, 0.f, 0.f);
+    const uint32_t bar = smem_u32(&arrived);
+    if (tid == 0) {
+        const uint32_t bytes = (uint32_t)(D * V) * 4;
+        mbar_init(bar, 1);
+        mbar_init_fence();
+        mbar_expect_tx(bar, bytes);
+        asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];\n"
+                     :: "r"(smem_u32(Ss)), "l"(S), "r"(bytes), "r"(bar) : "memory");
     }
+    const int CV = V >> 2, RG = 256 / CV, cv = tid % CV, rg = tid / CV;
     const int t = seg_q_start[seg], pos = positions[t];
     float* ring = slot + ring_off;
     const T* row = p + (size_t)t * ldp;
     const int C = 2 * KV * D + H * V;
-    if (tid == 255) {                                          // one thread: beta and the decay (double-precision exponentials)
+    if (tid == 255) {
         gates[0] = 1.f / (1.f + expf(-to_f32(row[C + H * V + h])));
-        gates[1] = (float)exp(log_decay(to_f32(row[C + H * V + H + h]), dt_bias[h], rate[h]));
+        gates[1] = decay_of(log_decay(to_f32(row[C + H * V + H + h]), dt_bias[h], rate[h]));
     }
     float sq = 0.f, sk = 0.f;
 #pragma unroll 2
@@ -183,46 +193,50 @@ __global__ void __launch_bounds__(256, NR <= 16 ? 2 : 1) delta_step_kernel(const
             for (int j = 0; j + 1 < taps; ++j) tap(j);
         }
         const float y = silu(fmaf(conv[(size_t)c * taps + taps - 1], own, acc));
-        sm[i] = y;
+        qs[i] = y;
         if (i < D) sq = fmaf(y, y, sq); else if (i < 2 * D) sk = fmaf(y, y, sk);
         if (taps > 1 && (i >= 2 * D || h % rep == 0)) ring[(size_t)(pos % taps) * C + c] = own;      // one writer a channel
     }
     sq = warp_sum(sq);
     sk = warp_sum(sk);
     if (lane == 0) squares[warp] = make_float2(sq, sk);
-    __syncthreads();
+    __syncthreads();                                           // also: the barrier's word is ready for every thread
     sq = sk = 0.f;
 #pragma unroll
     for (int w = 0; w < 8; ++w) { sq += squares[w].x; sk += squares[w].y; }
     const float beta = gates[0], f = gates[1], rq = q_scale / sqrtf(sq + unit_eps), rk = 1.f / sqrtf(sk + unit_eps);
+    const bool here = mbar_wait(bar, 0);
+    if (!here) atomicExch(error, 72);
+    if (__syncthreads_or(!here)) return;                       // the state did not arrive: nothing of it is changed
     float4 a = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-    for (int i = 0; i < NR; ++i) {
-        const int r = rg + RG * i;
-        const float kr = rg < RG && r < D ? ks[r] * rk : 0.f;
-        a.x = fmaf(s[i].x, kr, a.x); a.y = fmaf(s[i].y, kr, a.y); a.z = fmaf(s[i].z, kr, a.z); a.w = fmaf(s[i].w, kr, a.w);
+    if (rg < RG) {
+#pragma unroll 8
+        for (int r = rg; r < D; r += RG) {
+            const float4 s = *reinterpret_cast<const float4*>(Ss + r * V + 4 * cv);
+            const float kr = ks[r];
+            a.x = fmaf(s.x, kr, a.x); a.y = fmaf(s.y, kr, a.y); a.z = fmaf(s.z, kr, a.z); a.w = fmaf(s.w, kr, a.w);
+        }
+        *reinterpret_cast<float4*>(red + rg * V + 4 * cv) = a;
     }
-    if (rg < RG) *reinterpret_cast<float4*>(red + rg * V + 4 * cv) = a;
     __syncthreads();
     for (int c = tid; c < V; c += 256) {
         float dot = 0.f;
 #pragma unroll 8
         for (int g = 0; g < RG; ++g) dot += red[g * V + c];
-        vs[c] = beta * (vs[c] - f * dot);
+        vs[c] = beta * (vs[c] - f * (rk * dot));
     }
     __syncthreads();
     if (rg < RG) {
-        const float4 u = make_float4(vs[4 * cv], vs[4 * cv + 1], vs[4 * cv + 2], vs[4 * cv + 3]);
+        const float4 u = *reinterpret_cast<const float4*>(vs + 4 * cv);
+        const float4 ku = make_float4(rk * u.x, rk * u.y, rk * u.z, rk * u.w);
         float4 o = make_float4(0.f, 0.f, 0.f, 0.f);
-#pragma unroll
-        for (int i = 0; i < NR; ++i) {
-            const int r = rg + RG * i;
-            if (r >= D) continue;
-            const float kr = ks[r] * rk, qr = qs[r] * rq;
-            s[i].x = fmaf(kr, u.x, f * s[i].x); s[i].y = fmaf(kr, u.y, f * s[i].y);
-            s[i].z = fmaf(kr, u.z, f * s[i].z); s[i].w = fmaf(kr, u.w, f * s[i].w);
-            o.x = fmaf(s[i].x, qr, o.x); o.y = fmaf(s[i].y, qr, o.y); o.z = fmaf(s[i].z, qr, o.z); o.w = fmaf(s[i].w, qr, o.w);
-            *reinterpret_cast<float4*>(S + (size_t)r * V + 4 * cv) = s[i];
+#pragma unroll 8
+        for (int r = rg; r < D; r += RG) {
+            float4 s = *reinterpret_cast<const float4*>(Ss + r * V + 4 * cv);
+            const float kr = ks[r], qr = qs[r];
+            s.x = fmaf(kr, ku.x, f * s.x); s.y = fmaf(kr, ku.y, f * s.y); s.z = fmaf(kr, ku.z, f * s.z); s.w = fmaf(kr, ku.w, f * s.w);
+            o.x = fmaf(s.x, qr, o.x); o.y = fmaf(s.y, qr, o.y); o.z = fmaf(s.z, qr, o.z); o.w = fmaf(s.w, qr, o.w);
+            *reinterpret_cast<float4*>(S + (size_t)r * V + 4 * cv) = s;
         }
         *reinterpret_cast<float4*>(red + rg * V + 4 * cv) = o;
     }
@@ -232,6 +246,7 @@ __global__ void __launch_bounds__(256, NR <= 16 ? 2 : 1) delta_step_kernel(const
         float o = 0.f;
 #pragma unroll 8
         for (int g = 0; g < RG; ++g) o += red[g * V + c];
+        o *= rq;
         vs[c] = o;                                             // read again below by the same thread
         ss = fmaf(o, o, ss);
     }
@@ -295,25 +310,31 @@ MI_EXPORT int mi_gated_delta_ring(const void* p, int ldp, float* state, long lon
     return (int)cudaGetLastError();
 }
 
-// Every entry brings one token.  rows [entries, H V] in the type of p.  -2: sizes that this form does not take (V not a multiple of four, or
-// more than 16 K state entries a head); the caller then runs the prompt form.
+// Every entry brings one token.  rows [entries, H V] in the type of p.  -2: sizes that this form does not take (V or D not a multiple of
+// four, or a head's state larger than shared memory); the caller then runs the prompt form.  error: receives 72 when a head's state did
+// not arrive in time (the entry is then left as it is).
 MI_EXPORT int mi_gated_delta_step(const void* p, int ldp, const float* conv, int taps, const float* rate, const float* dt_bias, float* state,
                                   long long state_stride, long long ring_off, const float* norm, void* rows, const int* positions, const int* seg_q_start,
-                                  const int* seg_slot, int num_segs, int H, int KV, int D, int V, float unit_eps, float eps, int dtype, cudaStream_t stream) {
+                                  const int* seg_slot, int num_segs, int H, int KV, int D, int V, float unit_eps, float eps, int* error, int dtype,
+                                  cudaStream_t stream) {
     if (num_segs == 0) return 0;
-    if (H % KV || H > 65535 || V % 4 || V > 1024 || D > 1024 || state_stride % 4 || (uintptr_t)state % 16) return -2;
-    const int RG = 256 / (V / 4), need = (D + RG - 1) / RG;
-    if (need > 32) return -2;
-    const size_t smem = (size_t)(((2 * D + V + 3) & ~3) + RG * V) * sizeof(float);
+    if (H % KV || H > 65535 || V % 4 || D % 2 || V > 1024 || state_stride % 4 || (uintptr_t)state % 16) return -2;
+    const int RG = 256 / (V / 4);
+    const size_t smem = ((size_t)D * V + ((2 * D + V + 3) & ~3) + RG * V) * sizeof(float);
+    if (smem > 220 * 1024) return -2;
     const float q_scale = 1.f / sqrtf((float)D);
     dim3 grid(num_segs, H);
-#define GO(T, NR, TAPS) delta_step_kernel<T, NR, TAPS><<<grid, 256, smem, stream>>>((const T*)p, ldp, conv, taps, rate, dt_bias, state, state_stride, ring_off, norm, (T*)rows, \
-                      positions, seg_q_start, seg_slot, H, KV, D, V, unit_eps, q_scale, eps)
-#define ROWS(T, TAPS) do { if (need <= 4) GO(T, 4, TAPS); else if (need <= 8) GO(T, 8, TAPS); else if (need <= 16) GO(T, 16, TAPS); else GO(T, 32, TAPS); } while (0)
-#define PICK(T) do { if (taps == 4) ROWS(T, 4); else ROWS(T, 0); } while (0)
-    if (dtype == MI_BF16) PICK(__nv_bfloat16); else PICK(float);
-#undef PICK
-#undef ROWS
+#define GO(T, TAPS) do { \
+        static bool configured = false; \
+        if (!configured) { \
+            const cudaError_t e = cudaFuncSetAttribute(delta_step_kernel<T, TAPS>, cudaFuncAttributeMaxDynamicSharedMemorySize, 220 * 1024); \
+            if (e != cudaSuccess) return (int)e; \
+            configured = true; \
+        } \
+        delta_step_kernel<T, TAPS><<<grid, 256, smem, stream>>>((const T*)p, ldp, conv, taps, rate, dt_bias, state, state_stride, ring_off, norm, (T*)rows, positions, \
+                                                                seg_q_start, seg_slot, H, KV, D, V, unit_eps, q_scale, eps, error); } while (0)
+    if (dtype == MI_BF16) { if (taps == 4) GO(__nv_bfloat16, 4); else GO(__nv_bfloat16, 0); }
+    else { if (taps == 4) GO(float, 4); else GO(float, 0); }
 #undef GO
     return (int)cudaGetLastError();
 }

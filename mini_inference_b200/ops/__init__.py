@@ -476,7 +476,7 @@ class CudaOps:
         if code != 0:
             self._stream_error.zero_()
             self._tc2_counters.zero_()
-            raise RuntimeError(f"a pipeline wait inside a kernel ran out (code {code}: 1-2 gemm_stream, 21+ attention, 51-55 gemm_tc2, 61-63 grouped expert product, 71 delta-rule chunks)")
+            raise RuntimeError(f"a pipeline wait inside a kernel ran out (code {code}: 1-2 gemm_stream, 21+ attention, 51-55 gemm_tc2, 61-63 grouped expert product, 71-72 delta rule)")
 
     # ---------------------------------------------------------------- q/k norm, rotation, cache write
     def qk_norm_rope_cache(self, qkv, H, KV, D, q_weight, k_weight, eps, inv_freq, meta, k_cache, v_cache):
@@ -1408,7 +1408,7 @@ class CudaOps:
         if T == batch.num_segs and self.fused_delta_step:   # every entry brings one token
             rows = torch.empty((T, H * V), dtype=p.dtype, device=p.device)
             rc = self.lib.mi_gated_delta_step(_p(p), p.stride(0), _p(conv), taps, _p(rate), _p(dt_bias), _p(state), *stride, _p(norm), _p(rows), _p(batch.positions),
-                                              _p(batch.seg_q_start), _p(batch.seg_slot), T, H, KV, D, V, _c.c_float(unit_eps), _c.c_float(eps), code, self._stream())
+                                              _p(batch.seg_q_start), _p(batch.seg_slot), T, H, KV, D, V, _c.c_float(unit_eps), _c.c_float(eps), _p(self._stream_error), code, self._stream())
             if rc == 0:
                 self.launches += 1
                 return rows
