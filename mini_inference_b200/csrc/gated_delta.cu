@@ -80,21 +80,33 @@ __global__ void __launch_bounds__(128) delta_ready_kernel(const T* __restrict__ 
         if (back <= r) return to_f32(p[(size_t)(t - back) * ldp + c]);
         return back <= pos ? ring[(size_t)((pos - back) % taps) * C + c] : 0.f;
     };
-    const int seg0 = token_seg[t0];
-    if (TAPS > 0 && t1 - t0 == TOK && token_seg[t1 - 1] == seg0) {
-        const int qs = seg_q_start[seg0], r = t0 - qs, pos = positions[t0];
-        const float* ring = state + (long long)seg_slot[seg0] * state_stride + ring_off;
+    if (TAPS > 0 && t1 - t0 == TOK) {
+        // the rows are fetched before it is known where the tokens stand in their entry; what lies before the entry is replaced then
         float w[NI][W], x[NI][TOK + W - 1];
 #pragma unroll
         for (int i = 0; i < NI; ++i) {
             const int c = c0 + lane + 32 * i;
             const bool mine = lane + 32 * i < n;
 #pragma unroll
-            for (int j = 0; j < W; ++j) w[i][j] = mine ? conv[(size_t)c * W + j] : 0.f;
+            for (int j = 0; j < TOK + W - 1; ++j) x[i][j] = mine && t0 + j >= W - 1 ? to_f32(p[(size_t)(t0 + j - (W - 1)) * ldp + c]) : 0.f;
+            if constexpr (W == 4) {
+                const float4 t = mine ? *reinterpret_cast<const float4*>(conv + (size_t)c * 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+                w[i][0] = t.x; w[i][1] = t.y; w[i][2] = t.z; w[i][3] = t.w;
+            } else {
 #pragma unroll
-            for (int j = 0; j < W - 1; ++j) x[i][j] = mine ? input(c, W - 1 - j, t0, r, pos, ring) : 0.f;
+                for (int j = 0; j < W; ++j) w[i][j] = mine ? conv[(size_t)c * W + j] : 0.f;
+            }
+        }
+        const int seg0 = token_seg[t0], pos = positions[t0];
+        if (token_seg[t1 - 1] == seg0) {
+        const int r = t0 - seg_q_start[seg0];
+        if (r < W - 1) {
+            const float* ring = state + (long long)seg_slot[seg0] * state_stride + ring_off;
 #pragma unroll
-            for (int k = 0; k < TOK; ++k) x[i][W - 1 + k] = mine ? to_f32(p[(size_t)(t0 + k) * ldp + c]) : 0.f;
+            for (int i = 0; i < NI; ++i)
+#pragma unroll
+                for (int j = 0; j < W - 1; ++j)
+                    if (W - 1 - j > r) x[i][j] = lane + 32 * i < n ? input(c0 + lane + 32 * i, W - 1 - j, t0, r, pos, ring) : 0.f;
         }
 #pragma unroll
         for (int k = 0; k < TOK; ++k) {
@@ -108,6 +120,7 @@ __global__ void __launch_bounds__(128) delta_ready_kernel(const T* __restrict__ 
             finish(y, t0 + k);
         }
         return;
+        }
     }
     for (int t = t0; t < t1; ++t) {
         const int seg = token_seg[t], r = t - seg_q_start[seg], pos = positions[t];

@@ -40,11 +40,16 @@ __device__ __forceinline__ uint32_t pack2(float lo, float hi) {
 __device__ __forceinline__ float rest(float x) { return x - __bfloat162float(__float2bfloat16_rn(x)); }
 __device__ __forceinline__ float low_of(uint32_t w) { return __uint_as_float(w << 16); }
 __device__ __forceinline__ float high_of(uint32_t w) { return __uint_as_float(w & 0xffff0000u); }
-// c += (ah + al) (bh + bl) without al bl
-__device__ __forceinline__ void mma3(float (&c)[4], const uint32_t (&ah)[4], const uint32_t (&al)[4], uint32_t bh0, uint32_t bh1, uint32_t bl0, uint32_t bl1) {
-    mma16816(c, ah, bh0, bh1);
-    mma16816(c, ah, bl0, bl1);
-    mma16816(c, al, bh0, bh1);
+// c[t] += (ah + al) (bh_t + bl_t) without al bl_t for N neighbouring tiles of 8 columns, their two halves each as ldmatrix left them (two
+// tiles a register group).  Product by product over all tiles, so that a tile's three sums do not wait for one another.
+template <int N>
+__device__ __forceinline__ void mma3(float (&c)[N][4], const uint32_t (&ah)[4], const uint32_t (&al)[4], const uint32_t (&bh)[(N + 1) / 2][4], const uint32_t (&bl)[(N + 1) / 2][4]) {
+#pragma unroll
+    for (int t = 0; t < N; ++t) mma16816(c[t], ah, bh[t / 2][2 * (t % 2)], bh[t / 2][2 * (t % 2) + 1]);
+#pragma unroll
+    for (int t = 0; t < N; ++t) mma16816(c[t], ah, bl[t / 2][2 * (t % 2)], bl[t / 2][2 * (t % 2) + 1]);
+#pragma unroll
+    for (int t = 0; t < N; ++t) mma16816(c[t], al, bh[t / 2][2 * (t % 2)], bh[t / 2][2 * (t % 2) + 1]);
 }
 
 // byte offset of the 16-byte piece `ch` of row `row` in a tile of rows of N bfloat16 (N a multiple of 64; pieces XOR-ed with the row so that
@@ -70,14 +75,24 @@ template <int D, int V> struct PrepareSmem {
 };
 
 // rows of N floats, ld apart (rows beyond n: zeros), -> two bfloat16 tiles
-template <int N> __device__ __forceinline__ void split_rows(unsigned char* hi, unsigned char* lo, const float* __restrict__ src, int ld, int n) {
-    for (int id = threadIdx.x; id < Q * (N / 8); id += NTH) {
-        const int row = id / (N / 8), ch = id % (N / 8);
-        float4 a = make_float4(0.f, 0.f, 0.f, 0.f), b = a;
-        if (row < n) {
-            a = *reinterpret_cast<const float4*>(src + (size_t)row * ld + ch * 8);
-            b = *reinterpret_cast<const float4*>(src + (size_t)row * ld + ch * 8 + 4);
-        }
+// (fetch: all of a thread's pieces at once, into registers; store: what they hold)
+template <int N> struct Pieces { float4 v[2 * Q * (N / 8) / NTH]; };
+template <int N> __device__ __forceinline__ Pieces<N> fetch_rows(const float* __restrict__ src, int ld, int n) {
+    Pieces<N> p;
+#pragma unroll
+    for (int i = 0; i < Q * (N / 8) / NTH; ++i) {
+        const int id = threadIdx.x + i * NTH, row = id / (N / 8), ch = id % (N / 8);
+        const float* s = src + (size_t)row * ld + ch * 8;
+        p.v[2 * i] = row < n ? *reinterpret_cast<const float4*>(s) : make_float4(0.f, 0.f, 0.f, 0.f);
+        p.v[2 * i + 1] = row < n ? *reinterpret_cast<const float4*>(s + 4) : make_float4(0.f, 0.f, 0.f, 0.f);
+    }
+    return p;
+}
+template <int N> __device__ __forceinline__ void store_rows(unsigned char* hi, unsigned char* lo, const Pieces<N>& p) {
+#pragma unroll
+    for (int i = 0; i < Q * (N / 8) / NTH; ++i) {
+        const int id = threadIdx.x + i * NTH, row = id / (N / 8), ch = id % (N / 8);
+        const float4 a = p.v[2 * i], b = p.v[2 * i + 1];
         *reinterpret_cast<uint4*>(hi + at<N>(row, ch)) = make_uint4(pack2(a.x, a.y), pack2(a.z, a.w), pack2(b.x, b.y), pack2(b.z, b.w));
         *reinterpret_cast<uint4*>(lo + at<N>(row, ch)) = make_uint4(pack2(rest(a.x), rest(a.y)), pack2(rest(a.z), rest(a.w)), pack2(rest(b.x), rest(b.y)), pack2(rest(b.z), rest(b.w)));
     }
@@ -110,28 +125,26 @@ template <int D> __device__ __forceinline__ void scores(float (&s)[4][4], uint32
     for (int nt = 0; nt < 4; ++nt) { s[nt][0] = s[nt][1] = s[nt][2] = s[nt][3] = 0.f; }
 #pragma unroll
     for (int ks = 0; ks < D / 16; ++ks) {
-        uint32_t ah[4], al[4];
+        uint32_t ah[4], al[4], bh[2][4], bl[2][4];
         const uint32_t ao = at<D>(rb * 16 + (lane & 7) + (m & 1) * 8, ks * 2 + (m >> 1));
         ldsm4(ah, xh + ao);
         ldsm4(al, xl + ao);
 #pragma unroll
         for (int np = 0; np < 2; ++np) {
-            uint32_t bh[4], bl[4];
             const uint32_t bo = at<D>(ch * 32 + (2 * np + (m >> 1)) * 8 + (lane & 7), ks * 2 + (m & 1));
-            ldsm4(bh, kh + bo);
-            ldsm4(bl, kl + bo);
-            mma3(s[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
-            mma3(s[2 * np + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+            ldsm4(bh[np], kh + bo);
+            ldsm4(bl[np], kl + bo);
         }
+        mma3<4>(s, ah, al, bh, bl);
     }
 }
 
 // the rows rb * 16 .. of T D(scale) X for the N / 2 columns of half `half`; T float32 lower triangular in shared memory, X a split tile of N columns
-template <int N> __device__ __forceinline__ void apply_inverse(float (&acc)[N / 16][4], const float* T, int lda, const float* scale, uint32_t xh, uint32_t xl,
+template <int N> __device__ __forceinline__ void apply_inverse(float (&acc)[N / 64][4][4], const float* T, int lda, const float* scale, uint32_t xh, uint32_t xl,
                                                                int rb, int half, int lane) {
     const int g = lane >> 2, c = lane & 3, m = lane >> 3;
 #pragma unroll
-    for (int nt = 0; nt < N / 16; ++nt) { acc[nt][0] = acc[nt][1] = acc[nt][2] = acc[nt][3] = 0.f; }
+    for (int i = 0; i < N / 4; ++i) acc[i / 16][i / 4 % 4][i % 4] = 0.f;
     for (int kb = 0; kb <= rb; ++kb) {
         uint32_t ah[4], al[4];
 #pragma unroll
@@ -142,13 +155,15 @@ template <int N> __device__ __forceinline__ void apply_inverse(float (&acc)[N / 
             al[i] = pack2(rest(t.x * s.x), rest(t.y * s.y));
         }
 #pragma unroll
-        for (int np = 0; np < N / 32; ++np) {
-            uint32_t bh[4], bl[4];
-            const uint32_t bo = at<N>(kb * 16 + (m & 1) * 8 + (lane & 7), half * (N / 16) + 2 * np + (m >> 1));
-            ldsm4t(bh, xh + bo);
-            ldsm4t(bl, xl + bo);
-            mma3(acc[2 * np], ah, al, bh[0], bh[1], bl[0], bl[1]);
-            mma3(acc[2 * np + 1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+        for (int q4 = 0; q4 < N / 64; ++q4) {                      // four tiles of 8 columns at a time
+            uint32_t bh[2][4], bl[2][4];
+#pragma unroll
+            for (int np = 0; np < 2; ++np) {
+                const uint32_t bo = at<N>(kb * 16 + (m & 1) * 8 + (lane & 7), half * (N / 16) + 4 * q4 + 2 * np + (m >> 1));
+                ldsm4t(bh[np], xh + bo);
+                ldsm4t(bl[np], xl + bo);
+            }
+            mma3<4>(acc[q4], ah, al, bh, bl);
         }
     }
 }
@@ -196,6 +211,8 @@ __global__ void __launch_bounds__(NTH, 2) delta_chunk_kernel(const float* __rest
     unsigned char* kp = wq + W::WQ;
     float* u0 = reinterpret_cast<float*>(kp + W::KP);
 
+    const Pieces<D> kp_in = fetch_rows<D>(rows + KV * D + kvh * D, ld, n), qp_in = fetch_rows<D>(rows + kvh * D, ld, n);
+    for (int i = tid; i < Q * L::LDA; i += NTH) { A[i] = 0.f; T[i] = 0.f; }
     if (warp == 0) {                                               // two tokens a lane: beta, sums of the decays' logarithms
         const int i = 2 * lane;
         const float* ra = rows + (size_t)i * ld + C + h;
@@ -215,9 +232,8 @@ __global__ void __launch_bounds__(NTH, 2) delta_chunk_kernel(const float* __rest
         tail[i] = exp2f(last - (incl - l1)); tail[i + 1] = exp2f(last - incl);
         if (lane == 31) *reinterpret_cast<float*>(kp + W::KP + W::U0) = exp2f(last);
     }
-    split_rows<D>(smem + L::K, smem + L::K + Q * D * 2, rows + KV * D + kvh * D, ld, n);
-    split_rows<D>(smem + L::QV, smem + L::QV + Q * D * 2, rows + kvh * D, ld, n);
-    for (int i = tid; i < Q * L::LDA; i += NTH) { A[i] = 0.f; T[i] = 0.f; }
+    store_rows<D>(smem + L::K, smem + L::K + Q * D * 2, kp_in);
+    store_rows<D>(smem + L::QV, smem + L::QV + Q * D * 2, qp_in);
     __syncthreads();
     // the six 16 x 32 tiles that reach below the diagonal: (0,0) (1,0) (2,0) (2,1) (3,0) (3,1)
     auto task_rb = [](int i) { return i < 2 ? i : i < 4 ? 2 : 3; };
@@ -286,6 +302,7 @@ __global__ void __launch_bounds__(NTH, 2) delta_chunk_kernel(const float* __rest
         *reinterpret_cast<uint4*>(wq + 3 * W::KD + off) = make_uint4(ol[0], ol[1], ol[2], ol[3]);
     }
     scale_rows<D>(kp, smem + L::K, smem + L::K + Q * D * 2, tail);                 // K'
+    const Pieces<V> v_in = fetch_rows<V>(rows + 2 * KV * D + h * V, ld, n);
     // the blocks of T below the diagonal, by distance d from it: T_ij = -T_ii sum_{j <= k < i} A_ik T_kj
     for (int d = 1; d < 4; ++d) {
         const int blk = tid >> 6, e = tid & 63, ib = blk + d, jb = blk;
@@ -300,30 +317,30 @@ __global__ void __launch_bounds__(NTH, 2) delta_chunk_kernel(const float* __rest
         if (ib < 4) *reinterpret_cast<float4*>(at_ij) = make_float4(-y.x, -y.y, -y.z, -y.w);
         __syncthreads();
     }
-    split_rows<V>(smem + L::QV, smem + L::QV + Q * V * 2, rows + 2 * KV * D + h * V, ld, n);      // Q is no longer needed
+    store_rows<V>(smem + L::QV, smem + L::QV + Q * V * 2, v_in);      // Q is no longer needed
     __syncthreads();
     const int rb = warp >> 1, half = warp & 1;
     {
-        float acc[D / 16][4];
+        float acc[D / 64][4][4];
         apply_inverse<D>(acc, T, L::LDA, bg, kh, kl, rb, half, lane);
 #pragma unroll
         for (int nt = 0; nt < D / 16; ++nt)
 #pragma unroll
             for (int hf = 0; hf < 2; ++hf) {
                 const uint32_t off = at<D>(rb * 16 + g + hf * 8, half * (D / 16) + nt) + 4 * c;
-                const float a = -acc[nt][2 * hf], b = -acc[nt][2 * hf + 1];
+                const float a = -acc[nt / 4][nt % 4][2 * hf], b = -acc[nt / 4][nt % 4][2 * hf + 1];
                 *reinterpret_cast<uint32_t*>(wq + off) = pack2(a, b);
                 *reinterpret_cast<uint32_t*>(wq + W::KD + off) = pack2(rest(a), rest(b));
             }
     }
     {
-        float acc[V / 16][4];
+        float acc[V / 64][4][4];
         apply_inverse<V>(acc, T, L::LDA, beta, base + L::QV, base + L::QV + Q * V * 2, rb, half, lane);
 #pragma unroll
         for (int nt = 0; nt < V / 16; ++nt)
 #pragma unroll
             for (int hf = 0; hf < 2; ++hf)
-                *reinterpret_cast<float2*>(u0 + (rb * 16 + g + hf * 8) * V + half * (V / 2) + nt * 8 + 2 * c) = make_float2(acc[nt][2 * hf], acc[nt][2 * hf + 1]);
+                *reinterpret_cast<float2*>(u0 + (rb * 16 + g + hf * 8) * V + half * (V / 2) + nt * 8 + 2 * c) = make_float2(acc[nt / 4][nt % 4][2 * hf], acc[nt / 4][nt % 4][2 * hf + 1]);
     }
 }
 
@@ -375,9 +392,12 @@ __global__ void __launch_bounds__(NTH, 1) delta_pass_kernel(const unsigned char*
         if (alive && !mbar_wait(bar, k & 1)) { alive = false; atomicExch(error, 71); }
     };
 
-    // rows of U and O: row block rb, columns nc0 .. of the block's NC; of the state: row block sb, columns sc0 ..
-    constexpr int NT = NC / 16, SB = D / 16, SW = 8 / SB, SNT = NC / 8 / SW;      // tiles of 8 columns a warp has of U and O; of the state
-    const int rb = warp & 3, nc0 = (warp >> 2) * (NC / 2), sb = warp % SB, sc0 = warp / SB * (NC / SW);
+    // Of U and O a warp has either the same 16 rows and half the columns of both, or (NC = 16, where the reads of W and Q' from shared memory
+    // are what counts) 16 rows and all columns of one of them: warps 0 .. 3 of U, 4 .. 7 of O.  Of the state: row block sb, columns sc0 ..
+    constexpr bool ROLES = NC == 16;
+    constexpr int NT = 2, SB = D / 16, SW = 8 / SB, SNT = NC / 8 / SW;      // tiles of 8 columns a warp has of U and O; of the state
+    const int rb = warp & 3, nc0 = ROLES ? 0 : (warp >> 2) * (NC / 2), sb = warp % SB, sc0 = warp / SB * (NC / SW);
+    const bool has_u = !ROLES || warp < 4, has_o = !ROLES || warp >= 4;
     float* S = state + (long long)seg_slot[seg] * state_stride + (long long)h * D * V + v0;
     float s[SNT][4];
     auto spread_state = [&]() {
@@ -401,6 +421,7 @@ __global__ void __launch_bounds__(NTH, 1) delta_pass_kernel(const unsigned char*
     spread_state();
     float next_u[NT][4], next_decay = 0.f;
     auto fetch_u = [&](int k) {
+        if (!has_u) { next_decay = reinterpret_cast<const float*>(first + k * step + W::WQ + W::KP)[Q * V]; return; }
         const float* u0 = reinterpret_cast<const float*>(first + k * step + W::WQ + W::KP);
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt)
@@ -414,42 +435,53 @@ __global__ void __launch_bounds__(NTH, 1) delta_pass_kernel(const unsigned char*
     };
     fetch_u(0);
     __syncthreads();
-    // the B operand's registers for 16 rows k0 .. and the NTILES tiles of 8 columns at col of a tile of NC columns: b[2 t], b[2 t + 1] of tile t
     for (int k = 0; k < chunks; ++k) {
         float u[NT][4], o[NT][4];
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) { u[nt][e] = next_u[nt][e]; o[nt][e] = 0.f; }
+            for (int e = 0; e < 4; ++e) { u[nt][e] = has_u ? next_u[nt][e] : 0.f; o[nt][e] = 0.f; }
         const float decay = next_decay;
         if (k + 1 < chunks) fetch_u(k + 1);
         await(bar_wq, k);
+        const uint32_t mine = base + L::WQ + (has_u ? 0 : 2 * W::KD);
 #pragma unroll
         for (int ks = 0; ks < D / 16; ++ks) {                      // U = U_0 - W S;  O = Q' S
-            uint32_t wh[4], wl[4], qh[4], ql[4], bh[4], bl[4];
+            uint32_t ah[4], al[4], bh[1][4], bl[1][4];
             const uint32_t ao = at<D>(rb * 16 + (lane & 7) + (m & 1) * 8, ks * 2 + (m >> 1));
-            ldsm4(wh, base + L::WQ + ao);
-            ldsm4(wl, base + L::WQ + W::KD + ao);
-            ldsm4(qh, base + L::WQ + 2 * W::KD + ao);
-            ldsm4(ql, base + L::WQ + 3 * W::KD + ao);
-            // NC = 16: the upper two matrices would be another warp's columns; they are read all the same and left unused
-            const uint32_t bo = at<NC>(ks * 16 + (m & 1) * 8 + (lane & 7), NT == 2 ? nc0 / 8 + (m >> 1) : nc0 / 8);
-            ldsm4t(bh, base + L::S + bo);
-            ldsm4t(bl, base + L::S + D * NC * 2 + bo);
-#pragma unroll
-            for (int nt = 0; nt < NT; ++nt) {
-                mma3(u[nt], wh, wl, bh[2 * nt], bh[2 * nt + 1], bl[2 * nt], bl[2 * nt + 1]);
-                mma3(o[nt], qh, ql, bh[2 * nt], bh[2 * nt + 1], bl[2 * nt], bl[2 * nt + 1]);
+            const uint32_t bo = at<NC>(ks * 16 + (m & 1) * 8 + (lane & 7), nc0 / 8 + (m >> 1));
+            ldsm4t(bh[0], base + L::S + bo);
+            ldsm4t(bl[0], base + L::S + D * NC * 2 + bo);
+            if constexpr (ROLES) {
+                ldsm4(ah, mine + ao);
+                ldsm4(al, mine + W::KD + ao);
+                mma3<NT>(u, ah, al, bh, bl);                       // U, or O held in u
+            } else {
+                uint32_t qh[4], ql[4];
+                ldsm4(ah, base + L::WQ + ao);
+                ldsm4(al, base + L::WQ + W::KD + ao);
+                ldsm4(qh, base + L::WQ + 2 * W::KD + ao);
+                ldsm4(ql, base + L::WQ + 3 * W::KD + ao);
+                mma3<NT>(u, ah, al, bh, bl);
+                mma3<NT>(o, qh, ql, bh, bl);
             }
         }
+        if constexpr (ROLES) {
 #pragma unroll
-        for (int nt = 0; nt < NT; ++nt)
+            for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-            for (int hf = 0; hf < 2; ++hf) {
-                const uint32_t off = at<NC>(rb * 16 + g + hf * 8, nc0 / 8 + nt) + 4 * c;
-                *reinterpret_cast<uint32_t*>(smem + L::U + off) = pack2(u[nt][2 * hf], u[nt][2 * hf + 1]);
-                *reinterpret_cast<uint32_t*>(smem + L::U + Q * NC * 2 + off) = pack2(rest(u[nt][2 * hf]), rest(u[nt][2 * hf + 1]));
-            }
+                for (int e = 0; e < 4; ++e) o[nt][e] = u[nt][e];
+        }
+        if (has_u) {
+#pragma unroll
+            for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+                for (int hf = 0; hf < 2; ++hf) {
+                    const uint32_t off = at<NC>(rb * 16 + g + hf * 8, nc0 / 8 + nt) + 4 * c;
+                    *reinterpret_cast<uint32_t*>(smem + L::U + off) = pack2(u[nt][2 * hf], u[nt][2 * hf + 1]);
+                    *reinterpret_cast<uint32_t*>(smem + L::U + Q * NC * 2 + off) = pack2(rest(u[nt][2 * hf]), rest(u[nt][2 * hf + 1]));
+                }
+        }
         __syncthreads();                                           // U is complete; W and Q' have been read
         if (tid == 0 && k + 1 < chunks) fetch_wq(k + 1);
         await(bar_kp, k);
@@ -459,32 +491,31 @@ __global__ void __launch_bounds__(NTH, 1) delta_pass_kernel(const unsigned char*
             for (int e = 0; e < 4; ++e) s[nt][e] *= decay;
 #pragma unroll
         for (int kb = 0; kb < Q / 16; ++kb) {
-            uint32_t uh[4], ul[4];
-            if (kb <= rb) {                                        // O += P U
-                uint32_t ph[4], pl[4];
+            if (has_o && kb <= rb) {                               // O += P U
+                uint32_t ph[4], pl[4], uh[1][4], ul[1][4];
                 const uint32_t ao = at<Q>(rb * 16 + (lane & 7) + (m & 1) * 8, kb * 2 + (m >> 1));
                 ldsm4(ph, base + L::KP + 2 * W::KD + ao);
                 ldsm4(pl, base + L::KP + 2 * W::KD + W::PP + ao);
-                const uint32_t bo = at<NC>(kb * 16 + (m & 1) * 8 + (lane & 7), NT == 2 ? nc0 / 8 + (m >> 1) : nc0 / 8);
-                ldsm4t(uh, base + L::U + bo);
-                ldsm4t(ul, base + L::U + Q * NC * 2 + bo);
-#pragma unroll
-                for (int nt = 0; nt < NT; ++nt) mma3(o[nt], ph, pl, uh[2 * nt], uh[2 * nt + 1], ul[2 * nt], ul[2 * nt + 1]);
+                const uint32_t bo = at<NC>(kb * 16 + (m & 1) * 8 + (lane & 7), nc0 / 8 + (m >> 1));
+                ldsm4t(uh[0], base + L::U + bo);
+                ldsm4t(ul[0], base + L::U + Q * NC * 2 + bo);
+                mma3<NT>(o, ph, pl, uh, ul);
             }
-            uint32_t ah[4], al[4];                                 // S += K'^T U
+            uint32_t ah[4], al[4], uh[(SNT + 1) / 2][4], ul[(SNT + 1) / 2][4];      // S += K'^T U
             const uint32_t ao = at<D>(kb * 16 + (m >> 1) * 8 + (lane & 7), sb * 2 + (m & 1));
             ldsm4t(ah, base + L::KP + ao);
             ldsm4t(al, base + L::KP + W::KD + ao);
 #pragma unroll
             for (int np = 0; np < (SNT + 1) / 2; ++np) {
+                // (one tile a warp: the upper two matrices are read all the same and left unused)
                 const uint32_t bo = at<NC>(kb * 16 + (m & 1) * 8 + (lane & 7), SNT > 1 ? sc0 / 8 + 2 * np + (m >> 1) : sc0 / 8);
-                ldsm4t(uh, base + L::U + bo);
-                ldsm4t(ul, base + L::U + Q * NC * 2 + bo);
-                mma3(s[2 * np], ah, al, uh[0], uh[1], ul[0], ul[1]);
-                if constexpr (SNT > 1) mma3(s[2 * np + 1], ah, al, uh[2], uh[3], ul[2], ul[3]);
+                ldsm4t(uh[np], base + L::U + bo);
+                ldsm4t(ul[np], base + L::U + Q * NC * 2 + bo);
             }
+            mma3<SNT>(s, ah, al, uh, ul);
         }
         spread_state();
+        if (has_o)
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
