@@ -43,6 +43,15 @@ __device__ __forceinline__ float warp_max(float v) {
     return v;
 }
 
+// The gates of a feed-forward: act(g) * u.  The tanh form of gelu, 0.5 g (1 + tanh(y)) with y = sqrt(2 / pi) (g + 0.044715 g^3), is
+// g / (1 + e^(-2 y)).
+constexpr int GATE_RELU = 0, GATE_SILU = 1, GATE_GELU_TANH = 2;
+__device__ __forceinline__ float gate_act(float g, int act) {
+    if (act == GATE_RELU) return fmaxf(g, 0.f);
+    if (act == GATE_SILU) return g / (1.f + expf(-g));
+    return g / (1.f + expf(-1.5957691216057308f * (g + 0.044715f * g * g * g)));
+}
+
 // Sum over a block of NT threads (NT a multiple of 32, at most 1024); every thread gets the
 // same value, added in a fixed order so the result does not depend on what else runs.
 template <int NT> __device__ __forceinline__ float block_sum(float v, float* scratch /* >= 32 floats */) {

@@ -108,16 +108,32 @@ __global__ void __launch_bounds__(128) delta_ready_kernel(const T* __restrict__ 
                 for (int j = 0; j < W - 1; ++j)
                     if (W - 1 - j > r) x[i][j] = lane + 32 * i < n ? input(c0 + lane + 32 * i, W - 1 - j, t0, r, pos, ring) : 0.f;
         }
+        float y[TOK][NI], ss[TOK];                              // all tokens side by side: their sums over the warp do not wait for one another
 #pragma unroll
         for (int k = 0; k < TOK; ++k) {
-            float y[NI];
+            ss[k] = 0.f;
 #pragma unroll
             for (int i = 0; i < NI; ++i) {
-                y[i] = 0.f;
+                float a = 0.f;
 #pragma unroll
-                for (int j = 0; j < W; ++j) y[i] = fmaf(w[i][j], x[i][k + j], y[i]);
+                for (int j = 0; j < W; ++j) a = fmaf(w[i][j], x[i][k + j], a);
+                y[k][i] = lane + 32 * i < n ? conv_silu<T>(a) : 0.f;
+                ss[k] = fmaf(y[k][i], y[k][i], ss[k]);
             }
-            finish(y, t0 + k);
+        }
+        if (head) {
+#pragma unroll
+            for (int o = 16; o > 0; o >>= 1)
+#pragma unroll
+                for (int k = 0; k < TOK; ++k) ss[k] += __shfl_xor_sync(0xffffffffu, ss[k], o);
+        }
+#pragma unroll
+        for (int k = 0; k < TOK; ++k) {
+            const float s = head ? (unit < KV ? q_scale : 1.f) / sqrtf(ss[k] + unit_eps) : 1.f;
+            float* o = out + (size_t)(t0 + k) * ldo + c0;
+#pragma unroll
+            for (int i = 0; i < NI; ++i)
+                if (lane + 32 * i < n) o[lane + 32 * i] = y[k][i] * s;
         }
         return;
         }

@@ -18,7 +18,7 @@
 //            write [32 x 64] swizzled boxes to shared memory and store them with TMA; then tell the even
 //            block's accumulator-empty barrier (the odd block's warps arrive there remotely).
 // Gated mode: the tile's BN weight rows are BN/2 gate rows (loaded by the even block) and the matching BN/2
-// up rows (loaded by the odd block); the epilogue writes silu(gate) * up.
+// up rows (loaded by the odd block); the epilogue writes act(gate) * up (silu, or the tanh form of gelu).
 // Two accumulators of 256 columns fill the 512 columns of tensor memory, so a tile's epilogue overlaps
 // the next tile's products.  Every mbarrier wait is bounded; a wait that runs out raises the error word and
 // every role leaves its loop; both blocks always reach the closing cluster barrier.
@@ -126,11 +126,13 @@ __device__ __forceinline__ bool t2_work(const T2Shape& sh, int pair, int w, int 
     return true;
 }
 
-template <bool GATED>
+// ACT: -1 the product itself; a gate code of common.cuh: act(gate) * up
+template <int ACT>
 __global__ void __launch_bounds__(T2_THREADS, 1)
 gemm_tc2_kernel(const __grid_constant__ CUtensorMap amap, const __grid_constant__ CUtensorMap bmap,
                 const __grid_constant__ CUtensorMap omap, const T2Shape sh, __nv_bfloat16* __restrict__ out, int ldo, float* __restrict__ ws,
                 int* __restrict__ counters, int* __restrict__ error_word) {
+    constexpr bool GATED = ACT >= 0;
     extern __shared__ unsigned char smem_raw[];
     unsigned char* base = (unsigned char*)(((uintptr_t)smem_raw + 1023) & ~(uintptr_t)1023);
     const int BN = sh.BN, NS = sh.NS, HALF = BN / 2;
@@ -253,7 +255,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap amap, const __grid_constant_
         };
         auto activate = [](float gate, float up) {
             const float gt = round_to<__nv_bfloat16>(gate), u = round_to<__nv_bfloat16>(up);
-            return gt / (1.f + expf(-gt)) * u;
+            return gate_act(gt, ACT) * u;
         };
         for (int t = 0; !abort_flag && t2_work(sh, pair, t, nk, wk); ++t) {
             const int b = t & 1;
@@ -388,16 +390,17 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap amap, const __grid_constant_
 std::mutex t2_mutex;
 std::map<std::tuple<const void*, int, int, int>, CUtensorMap> t2_weight_maps;
 
-template <bool GATED>
+template <int ACT>
 int launch_tc2(const void* X, int ldx, const void* W, void* out, int ldo, int M, int N, int K, float* ws, long long ws_bytes,
                int* counters, int num_counters, int* error_word, cudaStream_t stream) {
+    constexpr bool GATED = ACT >= 0;
     const int n_cols = GATED ? N / 2 : N;
     if (ldo % 8 || ((uintptr_t)out % 16)) return -2;
     T2Shape sh;
     sh.M = M; sh.N = N; sh.K = K;
     sh.m_tiles = (M + 2 * BM - 1) / (2 * BM);
     static int pairs_max = 0;
-    auto kern = gemm_tc2_kernel<GATED>;
+    auto kern = gemm_tc2_kernel<ACT>;
     const size_t smem_max = 226 * 1024;
     static bool configured = false;
     if (!configured) {
@@ -481,13 +484,16 @@ MI_EXPORT int mi_gemm_tc2(const void* X, int ldx, const void* W, void* out, int 
                           long long ws_bytes, int* counters, int num_counters, int* error_word, cudaStream_t stream) {
     if (M == 0 || N == 0) return 0;
     if (K % BK || K < BK || ldx % 8 || ((uintptr_t)X % 16) || ((uintptr_t)W % 16)) return -2;
-    return launch_tc2<false>(X, ldx, W, out, ldo, M, N, K, ws, ws_bytes, counters, num_counters, error_word, stream);
+    return launch_tc2<-1>(X, ldx, W, out, ldo, M, N, K, ws, ws_bytes, counters, num_counters, error_word, stream);
 }
 
-// act[M, I] = silu(g) * u with [g | u] = X[M, K] * W[2 I, K]^T (both rounded to bfloat16 first, as the separate kernels do).
-MI_EXPORT int mi_gemm_tc2_swiglu(const void* X, int ldx, const void* W, void* act, int M, int inter, int K, float* ws,
-                                 long long ws_bytes, int* counters, int num_counters, int* error_word, cudaStream_t stream) {
+// act[M, I] = gate(g) * u with [g | u] = X[M, K] * W[2 I, K]^T (both rounded to bfloat16 first, as the separate kernels do); gate: a
+// gate code of common.cuh, silu or the tanh form of gelu.
+MI_EXPORT int mi_gemm_tc2_glu(const void* X, int ldx, const void* W, void* act, int M, int inter, int K, int gate, float* ws,
+                              long long ws_bytes, int* counters, int num_counters, int* error_word, cudaStream_t stream) {
     if (M == 0 || inter == 0) return 0;
     if (K % BK || K < BK || ldx % 8 || inter % 8 || ((uintptr_t)X % 16) || ((uintptr_t)W % 16) || ((uintptr_t)act % 16)) return -2;
-    return launch_tc2<true>(X, ldx, W, act, inter, M, 2 * inter, K, ws, ws_bytes, counters, num_counters, error_word, stream);
+    if (gate == GATE_SILU) return launch_tc2<GATE_SILU>(X, ldx, W, act, inter, M, 2 * inter, K, ws, ws_bytes, counters, num_counters, error_word, stream);
+    if (gate == GATE_GELU_TANH) return launch_tc2<GATE_GELU_TANH>(X, ldx, W, act, inter, M, 2 * inter, K, ws, ws_bytes, counters, num_counters, error_word, stream);
+    return -2;
 }

@@ -158,12 +158,6 @@ template <typename T> __device__ __forceinline__ void store16v(T* p, const float
     }
 }
 
-__device__ __forceinline__ float glu_act(float g, int act) {
-    if (act == 0) return fmaxf(g, 0.f);
-    if (act == 1) return g / (1.f + expf(-g));
-    return 0.5f * g * (1.f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g)));
-}
-
 // grid (rows, pieces of the row)
 template <typename T>
 __global__ void bias_glu_kernel(const T* __restrict__ gu, const float* __restrict__ bias, T* __restrict__ out, int inter, int act) {
@@ -172,7 +166,7 @@ __global__ void bias_glu_kernel(const T* __restrict__ gu, const float* __restric
     for (int i = blockIdx.y * NT + threadIdx.x; i < inter; i += gridDim.y * NT) {
         float gv = to_f32(g[i]), uv = to_f32(g[inter + i]);
         if (bias) { gv += bias[i]; uv += bias[inter + i]; }
-        o[i] = from_f32<T>(glu_act(gv, act) * uv);
+        o[i] = from_f32<T>(gate_act(gv, act) * uv);
     }
 }
 
@@ -195,7 +189,7 @@ __global__ void bias_glu_vec_kernel(const T* __restrict__ gu, const float* __res
             }
         }
 #pragma unroll
-        for (int e = 0; e < VN; ++e) r[e] = glu_act(gv[e], act) * uv[e];
+        for (int e = 0; e < VN; ++e) r[e] = gate_act(gv[e], act) * uv[e];
         store16v(o + i, r);
     }
 }

@@ -191,32 +191,34 @@ class CudaOps:
         self.launches += 1
         return y
 
-    def gated_linear(self, x, w):
-        """silu(g) * u with [g | u] = x @ w.T (w = [gate rows | up rows]).  Many rows with the own tcgen05 GEMM chosen for this shape:
+    GATES = {"relu": 0, "silu": 1, "gelu_tanh": 2}
+
+    def gated_linear(self, x, w, act="silu"):
+        """act(g) * u with [g | u] = x @ w.T (w = [gate rows | up rows]), act silu or gelu_tanh.  Many rows with the own tcgen05 GEMM chosen for this shape:
         one kernel whose epilogue applies the activation (csrc/gemm_tc2.cu), so the [M, 2 I] product is never written;
-        otherwise product, then swiglu (or, for a few rows, the activation kernel that adds the product's partial sums)."""
+        otherwise product, then the activation (or, for a few rows, the activation kernel that adds the product's partial sums)."""
         M, K = x.shape
         inter = w.shape[0] // 2
         if (self._use_tc(M, w.shape[0], K) and K % 64 == 0 and inter % 8 == 0 and x.stride(1) == 1 and x.stride(0) % 8 == 0
                 and w.is_contiguous() and x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16):
-            act = torch.empty((M, inter), dtype=torch.bfloat16, device=x.device)
-            rc = self.lib.mi_gemm_tc2_swiglu(_p(x), x.stride(0), _p(w), _p(act), M, inter, K, *self._tc2_scratch(), _p(self._stream_error), self._stream())
+            out = torch.empty((M, inter), dtype=torch.bfloat16, device=x.device)
+            rc = self.lib.mi_gemm_tc2_glu(_p(x), x.stride(0), _p(w), _p(out), M, inter, K, self.GATES[act], *self._tc2_scratch(), _p(self._stream_error), self._stream())
             if rc == 0:
                 self.launches += 1
-                return act
+                return out
             if rc != -2:
-                _check(rc, "gemm_tc2_swiglu")
+                _check(rc, "gemm_tc2_glu")
         gu = self.linear(x, w, defer=True)
         if isinstance(gu, DeferredSum):          # the few-row product left its partial sums: the activation kernel adds them
-            act = torch.empty((M, inter), dtype=torch.bfloat16, device=x.device)
-            rc = self.lib.mi_deferred_swiglu(_p(gu.ws), _p(act), M, inter, gu.K, gu.grid, gu.max_contrib, gu.tok, self._stream())
+            out = torch.empty((M, inter), dtype=torch.bfloat16, device=x.device)
+            rc = self.lib.mi_deferred_glu(_p(gu.ws), _p(out), M, inter, gu.K, gu.grid, gu.max_contrib, gu.tok, self.GATES[act], self._stream())
             if rc == 0:
                 self.launches += 1
-                return act
+                return out
             if rc != -2:
-                _check(rc, "deferred_swiglu")
+                _check(rc, "deferred_glu")
             gu = self.materialize(gu)
-        return self.swiglu(gu)
+        return self.swiglu(gu) if act == "silu" else self.bias_glu(gu, None, act)
 
     def materialize(self, value):
         """The bfloat16 tensor behind a DeferredSum (anything else is returned as it is)."""
@@ -1198,7 +1200,7 @@ class CudaOps:
         rows, inter = gu.shape[0], gu.shape[1] // 2
         assert gu.is_contiguous() and (bias is None or (bias.dtype == torch.float32 and bias.numel() == 2 * inter))
         out = torch.empty((rows, inter), dtype=gu.dtype, device=gu.device)
-        _check(self.lib.mi_bias_glu(_p(gu), _p(bias), _p(out), rows, inter, {"relu": 0, "silu": 1, "gelu_tanh": 2}[act], _code(gu.dtype),
+        _check(self.lib.mi_bias_glu(_p(gu), _p(bias), _p(out), rows, inter, self.GATES[act], _code(gu.dtype),
                                     self._stream()), "bias_glu")
         self.launches += 1
         return out

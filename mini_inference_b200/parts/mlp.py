@@ -217,7 +217,8 @@ class GatedMLP(Part):
     """W_down (act(W_gate h + b_gate) * (W_up h + b_up)) + b_down with act one of relu, silu, gelu_tanh; biases=False: no bias
     anywhere.  gate and up are one [2 I, hidden] product; the first biases, the activation and the product of the two halves are
     one kernel (float32 arithmetic on the product's values); the last bias is left to whoever adds the output to the stream
-    (forward_unbiased), or added here."""
+    (forward_unbiased), or added here.  Without biases, silu and gelu_tanh go to ctx.ops.gated_linear, which may apply them in the
+    product's epilogue (many rows) or in the kernel that adds the product's partial sums (few rows)."""
 
     def __init__(self, spec):
         super().__init__(spec)
@@ -226,6 +227,7 @@ class GatedMLP(Part):
         if self.act not in ("relu", "silu", "gelu_tanh"):
             raise ValueError("gated_mlp: act is relu, silu or gelu_tanh")
         self.offers_unbiased = self.biases
+        self.fused = not self.biases and self.act in ("silu", "gelu_tanh")
         self.gate_up = self.down = self.gate_up_b = self.down_b = None
 
     def weight_specs(self):
@@ -247,8 +249,20 @@ class GatedMLP(Part):
     def first_weight(self):
         return self.gate_up
 
+    @property
+    def gated_weight(self):
+        return self.gate_up if self.fused else None
+
+    def first_product_probe(self, ops, rows):
+        if not self.fused:
+            return None
+        x = torch.randn(rows, self.hidden, device=self.gate_up.device, dtype=self.gate_up.dtype)
+        return lambda w: ops.gated_linear(x, w, self.act)
+
     def forward_unbiased(self, h, ctx):
         ops = ctx.ops
+        if self.fused:
+            return ops.linear(ops.gated_linear(h, self.gate_up, self.act), self.down), None
         return ops.linear(ops.bias_glu(ops.linear(h, self.gate_up), self.gate_up_b, self.act), self.down), self.down_b
 
     def forward(self, h, ctx):

@@ -33,8 +33,8 @@ class TorchRefOps:
     def linear(self, x, w, out_dtype=None, defer=False):
         return (x.float() @ w.float().T).to(out_dtype or x.dtype)
 
-    def gated_linear(self, x, w):
-        return self.swiglu(self.linear(x, w))
+    def gated_linear(self, x, w, act="silu"):
+        return self.swiglu(self.linear(x, w)) if act == "silu" else self.bias_glu(self.linear(x, w), None, act)
 
     def swiglu(self, gate_up):
         g, u = gate_up.float().chunk(2, dim=-1)
