@@ -43,7 +43,9 @@ __global__ void latent_prepare_kernel(const T* __restrict__ p, int ldp, const T*
     const T* row = p + (size_t)t * ldp;
     const T* qrow = q_rows + (size_t)t * ldq;              // the query heads as projected: p itself, or a tensor of their own
     const float pos = (float)positions[t];
+    pdl_trigger();
     for (int i = threadIdx.x; i < nf; i += blockDim.x) sincosf(pos * inv_freq[i], turn + nf + i, turn + i);
+    pdl_wait();                                            // positions and frequencies were there before the step began
     __syncthreads();
     T* qo = q_out + (size_t)t * H * (C + R);
     const int parts = gridDim.y, mine = (H - (int)blockIdx.y + parts - 1) / parts;        // this part's heads
@@ -235,12 +237,12 @@ MI_EXPORT int mi_latent_prepare(const void* p, int ldp, const void* q_rows, int 
     const int per = dtype == MI_BF16 ? 8 : 4;
     const bool vec = C % per == 0 && (C + R) % per == 0 && ((uintptr_t)q_abs | (uintptr_t)q_out) % 16 == 0;
     dim3 grid(T_, T_ >= 256 ? 1 : min(H, 8));
-#define GO(T, VEC) latent_prepare_kernel<T, VEC><<<grid, 128, smem, stream>>>((const T*)p, ldp, (const T*)q_rows, ldq, dkv_col, (const T*)q_abs, (T*)q_out, (T*)cache, \
-                       norm_w, inv_freq, nf, positions, slots, T_, H, D, R, C, eps, half_pairs)
-    if (dtype == MI_BF16) { if (vec) GO(__nv_bfloat16, true); else GO(__nv_bfloat16, false); }
-    else { if (vec) GO(float, true); else GO(float, false); }
+#define GO(T, VEC) return (int)launch_pdl(latent_prepare_kernel<T, VEC>, grid, dim3(128), smem, stream, (const T*)p, ldp, (const T*)q_rows, ldq, dkv_col, (const T*)q_abs, \
+                       (T*)q_out, (T*)cache, norm_w, inv_freq, nf, positions, slots, T_, H, D, R, C, eps, half_pairs)
+    if (dtype == MI_BF16) { if (vec) GO(__nv_bfloat16, true); GO(__nv_bfloat16, false); }
+    if (vec) GO(float, true);
+    GO(float, false);
 #undef GO
-    return (int)cudaGetLastError();
 }
 
 #define LATENT_PICK_NV(CALL) do { if (Dv <= 64) { CALL(2); } else if (Dv <= 128) { CALL(4); } else if (Dv <= 256) { CALL(8); } else { CALL(16); } } while (0)

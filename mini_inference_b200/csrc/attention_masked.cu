@@ -236,11 +236,13 @@ __global__ void unit_qk_cache_kernel(T* __restrict__ p, int ldp, const T* __rest
     const int slot = slots[t];
     const long long page = slot / ps, off = slot % ps;
     const float temp = temp_every > 0 ? 1.f + temp_coef * logf((float)((positions[t] + 1) / temp_every + 1)) : 1.f;
+    pdl_trigger();
     if (half > 0) {
         const float pos = (float)positions[t];
         for (int i = threadIdx.x; i < half; i += blockDim.x) sincosf(pos * inv_freq[i], turn + half + i, turn + i);
-        __syncthreads();
     }
+    pdl_wait();                                                 // positions and frequencies were there before the step began
+    if (half > 0) __syncthreads();
     for (int u = warp; u < H + KV; u += nw) {                   // q heads, then k heads
         T* x = row + (size_t)u * D;
         float r = 1.f;
@@ -286,15 +288,11 @@ MI_EXPORT int mi_normed_qk_cache(void* p, int ldp, const void* v_src, int ld_src
     const size_t turn = half > 0 ? 2 * (size_t)half * sizeof(float) : 0;
     // few tokens (decode steps): a warp per head, so that no warp walks several heads one after the other
     const int nt = T_ >= 256 ? 128 : min(1024, max(128, 32 * (H + KV)));
-    if (dtype == MI_BF16)
-        unit_qk_cache_kernel<__nv_bfloat16><<<T_, nt, turn, stream>>>((__nv_bfloat16*)p, ldp, (const __nv_bfloat16*)v_src, ld_src, lam, slots,
-                                                                    (__nv_bfloat16*)k_cache, (__nv_bfloat16*)v_cache, H, KV, D, Dv, ps, eps, unit,
-                                                                    q_w, k_w, positions, temp_coef, temp_every, v_is_k, inv_freq, half);
-    else
-        unit_qk_cache_kernel<float><<<T_, nt, turn, stream>>>((float*)p, ldp, (const float*)v_src, ld_src, lam, slots, (float*)k_cache,
-                                                           (float*)v_cache, H, KV, D, Dv, ps, eps, unit, q_w, k_w, positions, temp_coef,
-                                                            temp_every, v_is_k, inv_freq, half);
-    return (int)cudaGetLastError();
+#define GO(T) return (int)launch_pdl(unit_qk_cache_kernel<T>, dim3(T_), dim3(nt), turn, stream, (T*)p, ldp, (const T*)v_src, ld_src, lam, slots, (T*)k_cache, (T*)v_cache, \
+                  H, KV, D, Dv, ps, eps, unit, q_w, k_w, positions, temp_coef, temp_every, v_is_k, inv_freq, half)
+    if (dtype == MI_BF16) GO(__nv_bfloat16);
+    GO(float);
+#undef GO
 }
 
 MI_EXPORT int mi_unit_qk_cache(void* p, int ldp, const void* v_src, int ld_src, const float* lam, const int* slots, void* k_cache,

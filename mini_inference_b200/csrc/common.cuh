@@ -52,6 +52,13 @@ __device__ __forceinline__ float gate_act(float g, int act) {
     return g / (1.f + expf(-1.5957691216057308f * (g + 0.044715f * g * g * g)));
 }
 
+// The same with the fast exponential and quotient (a few units in the last place of float32), for results that are rounded to bfloat16
+__device__ __forceinline__ float gate_act_fast(float g, int act) {
+    if (act == GATE_RELU) return fmaxf(g, 0.f);
+    const float y = act == GATE_SILU ? g : 1.5957691216057308f * fmaf(0.044715f * g * g, g, g);
+    return __fdividef(g, 1.f + __expf(-y));
+}
+
 // Sum over a block of NT threads (NT a multiple of 32, at most 1024); every thread gets the
 // same value, added in a fixed order so the result does not depend on what else runs.
 template <int NT> __device__ __forceinline__ float block_sum(float v, float* scratch /* >= 32 floats */) {

@@ -165,7 +165,8 @@ __global__ void delta_ring_kernel(const T* __restrict__ p, int ldp, float* __res
 
 // ------------------------------------------------------------------ decode steps: everything in one pass over the state
 // grid (entries, H).  The head's state (D V contiguous floats) comes into shared memory as one bulk copy, under which the convolution, the
-// norms and the gates are made; thread (rg, cv) then owns the columns 4 cv .. of the rows rg + RG i, cv < V / 4, RG = 256 / (V / 4), in
+// norms and the gates are made.  The copy, and the filter's sums over earlier inputs, start before the kernel ahead (which makes p) is
+// done: the state and the ring were last written in the step before.  Thread (rg, cv) then owns the columns 4 cv .. of the rows rg + RG i, cv < V / 4, RG = 256 / (V / 4), in
 // both passes over it (S^T k; update, read-out and the way back to memory).
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(256) delta_step_kernel(const T* __restrict__ p, int ldp, const float* __restrict__ conv, int taps_,
@@ -188,6 +189,7 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const T* __restrict__ p
     float* slot = state + (long long)seg_slot[seg] * state_stride;
     float* S = slot + (long long)h * D * V;
     const uint32_t bar = smem_u32(&arrived);
+    pdl_trigger();
     if (tid == 0) {
         const uint32_t bytes = (uint32_t)(D * V) * 4;
         mbar_init(bar, 1);
@@ -201,15 +203,9 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const T* __restrict__ p
     float* ring = slot + ring_off;
     const T* row = p + (size_t)t * ldp;
     const int C = 2 * KV * D + H * V;
-    if (tid == 255) {
-        gates[0] = 1.f / (1.f + expf(-to_f32(row[C + H * V + h])));
-        gates[1] = decay_of(log_decay(to_f32(row[C + H * V + H + h]), dt_bias[h], rate[h]));
-    }
-    float sq = 0.f, sk = 0.f;
-#pragma unroll 2
-    for (int i = tid; i < 2 * D + V; i += 256) {               // this head's q, k and v channels
-        const int c = i < D ? kvh * D + i : i < 2 * D ? KV * D + kvh * D + i - D : 2 * KV * D + h * V + i - 2 * D;
-        const float own = to_f32(row[c]);
+    const int channels = 2 * D + V;                            // this head's q, k and v channels
+    auto channel = [&](int i) { return i < D ? kvh * D + i : i < 2 * D ? KV * D + kvh * D + i - D : 2 * KV * D + h * V + i - 2 * D; };
+    auto past = [&](int c) {                                   // the filter's sum over the inputs before this token
         float acc = 0.f;
         auto tap = [&](int j) {
             const int back = taps - 1 - j;
@@ -221,11 +217,32 @@ __global__ void __launch_bounds__(256) delta_step_kernel(const T* __restrict__ p
         } else {
             for (int j = 0; j + 1 < taps; ++j) tap(j);
         }
-        const float y = silu(fmaf(conv[(size_t)c * taps + taps - 1], own, acc));
+        return acc;
+    };
+    float early[2], last_tap[2];
+#pragma unroll
+    for (int k = 0; k < 2; ++k) {
+        const int i = tid + 256 * k, c = i < channels ? channel(i) : 0;
+        early[k] = i < channels ? past(c) : 0.f;
+        last_tap[k] = conv[(size_t)c * taps + taps - 1];
+    }
+    pdl_wait();
+    if (tid == 255) {
+        gates[0] = 1.f / (1.f + expf(-to_f32(row[C + H * V + h])));
+        gates[1] = decay_of(log_decay(to_f32(row[C + H * V + H + h]), dt_bias[h], rate[h]));
+    }
+    float sq = 0.f, sk = 0.f;
+    auto finish = [&](int i, int c, float acc, float w) {
+        const float own = to_f32(row[c]);
+        const float y = silu(fmaf(w, own, acc));
         qs[i] = y;
         if (i < D) sq = fmaf(y, y, sq); else if (i < 2 * D) sk = fmaf(y, y, sk);
         if (taps > 1 && (i >= 2 * D || h % rep == 0)) ring[(size_t)(pos % taps) * C + c] = own;      // one writer a channel
-    }
+    };
+#pragma unroll
+    for (int k = 0; k < 2; ++k)
+        if (tid + 256 * k < channels) finish(tid + 256 * k, channel(tid + 256 * k), early[k], last_tap[k]);
+    for (int i = tid + 512; i < channels; i += 256) finish(i, channel(i), past(channel(i)), conv[(size_t)channel(i) * taps + taps - 1]);
     sq = warp_sum(sq);
     sk = warp_sum(sk);
     if (lane == 0) squares[warp] = make_float2(sq, sk);
@@ -360,10 +377,10 @@ MI_EXPORT int mi_gated_delta_step(const void* p, int ldp, const float* conv, int
             if (e != cudaSuccess) return (int)e; \
             configured = true; \
         } \
-        delta_step_kernel<T, TAPS><<<grid, 256, smem, stream>>>((const T*)p, ldp, conv, taps, rate, dt_bias, state, state_stride, ring_off, norm, (T*)rows, positions, \
-                                                                seg_q_start, seg_slot, H, KV, D, V, unit_eps, q_scale, eps, error); } while (0)
-    if (dtype == MI_BF16) { if (taps == 4) GO(__nv_bfloat16, 4); else GO(__nv_bfloat16, 0); }
-    else { if (taps == 4) GO(float, 4); else GO(float, 0); }
+        return (int)launch_pdl(delta_step_kernel<T, TAPS>, grid, dim3(256), smem, stream, (const T*)p, ldp, conv, taps, rate, dt_bias, state, state_stride, ring_off, norm, \
+                               (T*)rows, positions, seg_q_start, seg_slot, H, KV, D, V, unit_eps, q_scale, eps, error); } while (0)
+    if (dtype == MI_BF16) { if (taps == 4) GO(__nv_bfloat16, 4); GO(__nv_bfloat16, 0); }
+    if (taps == 4) GO(float, 4);
+    GO(float, 0);
 #undef GO
-    return (int)cudaGetLastError();
 }

@@ -43,9 +43,11 @@ template <> __device__ __forceinline__ __nv_bfloat16 cvt_out<__nv_bfloat16>(floa
 // NT: 8-token tiles (M <= 8 NT); MT: 16-row weight tiles per block; U: windows in flight per warp
 template <int NT, int MT, int U, typename OutT>
 __global__ void __launch_bounds__(GW * 32)
-gemm_skinny_kernel(const __nv_bfloat16* __restrict__ X, int ldx, const __nv_bfloat16* __restrict__ W,
+gemm_skinny_kernel(const __nv_bfloat16* X, int ldx, const __nv_bfloat16* __restrict__ W,
                    OutT* __restrict__ out, int ldo, int M, int N, int K) {
     extern __shared__ float red[];                    // [GW][MT*16][NT*8]
+    pdl_trigger();
+    bool waited = false;                              // the first window's weights are requested before waiting for the kernel that makes X
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int g = lane >> 2, c = lane & 3;
     const int n0 = blockIdx.x * MT * 16;
@@ -84,6 +86,7 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ X, int ldx, const __nv_bflo
                 }
             }
         }
+        if (!waited) { pdl_wait(); waited = true; }
 #pragma unroll
         for (int u = 0; u < U; ++u) {
             const int w = w0 + u * GW;
@@ -91,7 +94,7 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ X, int ldx, const __nv_bflo
 #pragma unroll
                 for (int nt = 0; nt < NT; ++nt) {
                     uint4 b = make_uint4(0, 0, 0, 0);
-                    if (xok[nt]) b = __ldg(reinterpret_cast<const uint4*>(xrow[nt] + (size_t)w * 32));
+                    if (xok[nt]) b = *reinterpret_cast<const uint4*>(xrow[nt] + (size_t)w * 32);
 #pragma unroll
                     for (int mt = 0; mt < MT; ++mt) {
                         mma16816(acc[mt][nt], a[u][mt][0].x, a[u][mt][1].x, a[u][mt][0].y, a[u][mt][1].y, b.x, b.y);
@@ -102,6 +105,7 @@ gemm_skinny_kernel(const __nv_bfloat16* __restrict__ X, int ldx, const __nv_bflo
         }
     }
 
+    if (!waited) pdl_wait();
     // partial sums -> shared memory [warp][row][token], then a fixed-order sum over the warps
     constexpr int ROWS = MT * 16, TOK = NT * 8;
     float* mine = red + (size_t)warp * ROWS * TOK;
@@ -140,8 +144,7 @@ int launch(const void* X, int ldx, const void* W, void* out, int ldo, int M, int
         }
     }
     const int blocks = (N + MT * 16 - 1) / (MT * 16);
-    kern<<<blocks, GW * 32, smem, stream>>>((const __nv_bfloat16*)X, ldx, (const __nv_bfloat16*)W, (OutT*)out, ldo, M, N, K);
-    return (int)cudaGetLastError();
+    return (int)launch_pdl(kern, dim3(blocks), dim3(GW * 32), smem, stream, (const __nv_bfloat16*)X, ldx, (const __nv_bfloat16*)W, (OutT*)out, ldo, M, N, K);
 }
 
 template <typename OutT>

@@ -255,7 +255,7 @@ gemm_tc2_kernel(const __grid_constant__ CUtensorMap amap, const __grid_constant_
         };
         auto activate = [](float gate, float up) {
             const float gt = round_to<__nv_bfloat16>(gate), u = round_to<__nv_bfloat16>(up);
-            return gate_act(gt, ACT) * u;
+            return gate_act_fast(gt, ACT) * u;
         };
         for (int t = 0; !abort_flag && t2_work(sh, pair, t, nk, wk); ++t) {
             const int b = t & 1;

@@ -82,7 +82,8 @@ __global__ void __launch_bounds__(NT) stream_layernorm_vec_kernel(float* __restr
     __shared__ float4 scratch[2][NT / 32];
     const size_t r = (rows ? (size_t)rows[blockIdx.x] : (size_t)blockIdx.x) * hidden;
     const int quads = hidden >> 2;
-    constexpr bool AHEAD = VPT <= 2;                          // the weights are fetched with the row, so that no wait for them follows a sum
+    constexpr bool AHEAD = VPT <= 2;                          // the weights are fetched before the row, so that no wait for them follows a sum
+    pdl_trigger();
     float4 v[VPT], wv[AHEAD ? VPT : 1], wyv[AHEAD ? VPT : 1];
     if constexpr (AHEAD) {
 #pragma unroll
@@ -92,6 +93,7 @@ __global__ void __launch_bounds__(NT) stream_layernorm_vec_kernel(float* __restr
             wyv[k] = y && q < quads ? *reinterpret_cast<const float4*>(wy + 4 * q) : make_float4(0.f, 0.f, 0.f, 0.f);
         }
     }
+    pdl_wait();
 #pragma unroll
     for (int k = 0; k < VPT; ++k) {
         const int q = threadIdx.x + k * NT;
@@ -151,6 +153,8 @@ __global__ void __launch_bounds__(LOOP_NT) stream_layernorm_kernel(float* __rest
                                                               const float* __restrict__ pre, const float* __restrict__ w, TY* __restrict__ out,
                                                               const int* __restrict__ rows, int hidden, float eps, int keep) {
     __shared__ float4 scratch[2][LOOP_NT / 32];
+    pdl_trigger();
+    pdl_wait();
     const size_t r = (rows ? (size_t)rows[blockIdx.x] : (size_t)blockIdx.x) * hidden;
     Moments my{0.f, 0.f};
     if (y) my = loop_moments([&](int i) { return to_f32(y[r + i]); }, hidden, eps_y, scratch[0]);
@@ -182,17 +186,16 @@ MI_EXPORT int mi_stream_layernorm(float* x, const void* y, const float* wy, floa
     const uintptr_t all = (uintptr_t)x | (uintptr_t)y | (uintptr_t)wy | (uintptr_t)pre | (uintptr_t)w | (uintptr_t)out;
     const bool vec = hidden % 4 == 0 && hidden <= 8192 && all % 16 == 0;
     const int quads = hidden / 4;
-#define VEC(TD, TY, NT, VPT) stream_layernorm_vec_kernel<TD, TY, NT, VPT><<<n, NT, 0, stream>>>(x, (const TD*)y, wy, eps_y, pre, w, (TY*)out, rows, hidden, eps, keep)
+#define VEC(TD, TY, NT, VPT) return (int)launch_pdl(stream_layernorm_vec_kernel<TD, TY, NT, VPT>, dim3(n), dim3(NT), 0, stream, x, (const TD*)y, wy, eps_y, pre, w, (TY*)out, rows, hidden, eps, keep)
 #define GO(TD, TY) do { \
-        if (!vec) stream_layernorm_kernel<TD, TY><<<n, LOOP_NT, 0, stream>>>(x, (const TD*)y, wy, eps_y, pre, w, (TY*)out, rows, hidden, eps, keep); \
-        else if (n >= 512) { if (quads <= 128) VEC(TD, TY, 128, 1); else if (quads <= 256) VEC(TD, TY, 128, 2); else if (quads <= 512) VEC(TD, TY, 128, 4); \
-                             else if (quads <= 1024) VEC(TD, TY, 256, 4); else VEC(TD, TY, 256, 8); } \
-        else { if (quads <= 256) VEC(TD, TY, 256, 1); else if (quads <= 512) VEC(TD, TY, 256, 2); else if (quads <= 1024) VEC(TD, TY, 512, 2); \
-               else VEC(TD, TY, 512, 4); } } while (0)
+        if (!vec) return (int)launch_pdl(stream_layernorm_kernel<TD, TY>, dim3(n), dim3(LOOP_NT), 0, stream, x, (const TD*)y, wy, eps_y, pre, w, (TY*)out, rows, hidden, eps, keep); \
+        if (n >= 512) { if (quads <= 128) VEC(TD, TY, 128, 1); else if (quads <= 256) VEC(TD, TY, 128, 2); else if (quads <= 512) VEC(TD, TY, 128, 4); \
+                        else if (quads <= 1024) VEC(TD, TY, 256, 4); else VEC(TD, TY, 256, 8); } \
+        if (quads <= 256) VEC(TD, TY, 256, 1); else if (quads <= 512) VEC(TD, TY, 256, 2); else if (quads <= 1024) VEC(TD, TY, 512, 2); \
+        else VEC(TD, TY, 512, 4); } while (0)
     if (y_dtype == MI_BF16 && out_dtype == MI_BF16) GO(__nv_bfloat16, __nv_bfloat16);
     else if (y_dtype == MI_F32 && out_dtype == MI_F32) GO(float, float);
-    else return -1;
+    return -1;
 #undef GO
 #undef VEC
-    return (int)cudaGetLastError();
 }

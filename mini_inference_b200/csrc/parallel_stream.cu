@@ -142,6 +142,8 @@ __global__ void __launch_bounds__(NT) stream_rmsnorm_pair_vec_kernel(float* __re
 template <typename T>
 __global__ void rows_rmsnorm_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ w, T* __restrict__ y, int cols, float eps) {
     __shared__ float scratch[32];
+    pdl_trigger();
+    pdl_wait();
     const T* xr = x + (size_t)blockIdx.x * ldx;
     float ss = 0.f;
     for (int i = threadIdx.x; i < cols; i += NT) { const float v = to_f32(xr[i]); ss += v * v; }
@@ -161,6 +163,8 @@ template <typename T> __device__ __forceinline__ void store16v(T* p, const float
 // grid (rows, pieces of the row)
 template <typename T>
 __global__ void bias_glu_kernel(const T* __restrict__ gu, const float* __restrict__ bias, T* __restrict__ out, int inter, int act) {
+    pdl_trigger();
+    pdl_wait();
     const T* g = gu + (size_t)blockIdx.x * 2 * inter;
     T* o = out + (size_t)blockIdx.x * inter;
     for (int i = blockIdx.y * NT + threadIdx.x; i < inter; i += gridDim.y * NT) {
@@ -174,6 +178,8 @@ __global__ void bias_glu_kernel(const T* __restrict__ gu, const float* __restric
 template <typename T>
 __global__ void bias_glu_vec_kernel(const T* __restrict__ gu, const float* __restrict__ bias, T* __restrict__ out, int inter, int act) {
     constexpr int VN = Vec16<T>::N;
+    pdl_trigger();
+    pdl_wait();
     const T* g = gu + (size_t)blockIdx.x * 2 * inter;
     T* o = out + (size_t)blockIdx.x * inter;
     for (int i = (blockIdx.y * NT + threadIdx.x) * VN; i < inter; i += gridDim.y * NT * VN) {
@@ -238,9 +244,8 @@ MI_EXPORT int mi_stream_rmsnorm_pair(float* x, const void* a, const void* b, con
 
 MI_EXPORT int mi_rows_rmsnorm(const void* x, long long ldx, const float* w, void* y, int n, int cols, float eps, int dtype, cudaStream_t stream) {
     if (n == 0) return 0;
-    if (dtype == MI_BF16) rows_rmsnorm_kernel<__nv_bfloat16><<<n, NT, 0, stream>>>((const __nv_bfloat16*)x, ldx, w, (__nv_bfloat16*)y, cols, eps);
-    else rows_rmsnorm_kernel<float><<<n, NT, 0, stream>>>((const float*)x, ldx, w, (float*)y, cols, eps);
-    return (int)cudaGetLastError();
+    if (dtype == MI_BF16) return (int)launch_pdl(rows_rmsnorm_kernel<__nv_bfloat16>, dim3(n), dim3(NT), 0, stream, (const __nv_bfloat16*)x, ldx, w, (__nv_bfloat16*)y, cols, eps);
+    return (int)launch_pdl(rows_rmsnorm_kernel<float>, dim3(n), dim3(NT), 0, stream, (const float*)x, ldx, w, (float*)y, cols, eps);
 }
 
 // act: 0 relu, 1 silu, 2 gelu_tanh
@@ -251,11 +256,11 @@ MI_EXPORT int mi_bias_glu(const void* gu, const float* bias, void* out, int rows
     const bool vec = inter % vn == 0 && ((uintptr_t)gu % 16) == 0 && ((uintptr_t)out % 16) == 0 && ((uintptr_t)bias % 16) == 0;
     const int per = vec ? NT * vn : NT;
     dim3 grid(rows, rows >= 512 ? 1 : min(16, (inter + per - 1) / per));
-#define GO(T) do { if (vec) bias_glu_vec_kernel<T><<<grid, NT, 0, stream>>>((const T*)gu, bias, (T*)out, inter, act); \
-                   else bias_glu_kernel<T><<<grid, NT, 0, stream>>>((const T*)gu, bias, (T*)out, inter, act); } while (0)
-    if (dtype == MI_BF16) GO(__nv_bfloat16); else GO(float);
+#define GO(T) do { if (vec) return (int)launch_pdl(bias_glu_vec_kernel<T>, grid, dim3(NT), 0, stream, (const T*)gu, bias, (T*)out, inter, act); \
+                   return (int)launch_pdl(bias_glu_kernel<T>, grid, dim3(NT), 0, stream, (const T*)gu, bias, (T*)out, inter, act); } while (0)
+    if (dtype == MI_BF16) GO(__nv_bfloat16);
+    GO(float);
 #undef GO
-    return (int)cudaGetLastError();
 }
 
 MI_EXPORT int mi_scale_f32(float* z, long long n, float s, cudaStream_t stream) {

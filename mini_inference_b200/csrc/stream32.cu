@@ -154,6 +154,8 @@ __global__ void head_gate_kernel(const T* __restrict__ o, const T* __restrict__ 
 // grid (tokens, pieces of the row); VN neighbouring entries per thread and step (1, or 16 bytes of T)
 template <typename T, int VN>
 __global__ void sigmoid_gate_kernel(T* __restrict__ rows, const T* __restrict__ gate, int gate_stride, int n) {
+    pdl_trigger();
+    pdl_wait();
     T* r = rows + (size_t)blockIdx.x * n;
     const T* g = gate + (size_t)blockIdx.x * gate_stride;
     for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * VN; i < n; i += gridDim.y * blockDim.x * VN) {
@@ -348,9 +350,9 @@ MI_EXPORT int mi_sigmoid_gate(void* rows, const void* gate, int gate_stride, int
     const int per = vec ? vn : 1, nt = n / per >= 256 ? 256 : 128;
     const int pieces = (n + nt * per - 1) / (nt * per);
     dim3 grid(T_, pieces < 65535 ? pieces : 65535);
-#define GO(T, VN) sigmoid_gate_kernel<T, VN><<<grid, nt, 0, stream>>>((T*)rows, (const T*)gate, gate_stride, n)
-    if (dtype == MI_BF16) { if (vec) GO(__nv_bfloat16, 8); else GO(__nv_bfloat16, 1); }
-    else { if (vec) GO(float, 4); else GO(float, 1); }
+#define GO(T, VN) return (int)launch_pdl(sigmoid_gate_kernel<T, VN>, grid, dim3(nt), 0, stream, (T*)rows, (const T*)gate, gate_stride, n)
+    if (dtype == MI_BF16) { if (vec) GO(__nv_bfloat16, 8); GO(__nv_bfloat16, 1); }
+    if (vec) GO(float, 4);
+    GO(float, 1);
 #undef GO
-    return (int)cudaGetLastError();
 }

@@ -350,7 +350,7 @@ class CudaOps:
                 return b
         return 0
 
-    def tune_linear(self, weights, out_dtypes=None, iters=16, min_bytes=256 << 20, deferrable=(), gated=()):
+    def tune_linear(self, weights, out_dtypes=None, iters=16, min_bytes=256 << 20, copy_bytes=2 << 20, deferrable=(), gated=()):
         """Per weight shape and row-count bucket, time this package's few-row kernels against the
         library GEMM on the model's own weights and remember the fastest.  The reference does the
         same kind of start-up timing to choose a weight layout per shape
@@ -366,9 +366,12 @@ class CudaOps:
             self._linear_choice = None
             for (N, K), ws in groups.items():
                 od = (out_dtypes or {}).get((N, K))
-                # one weight cannot defeat the L2 by rotation; leave such shapes to the default rule
+                # the rotation over the weights must defeat the L2: shapes with few weights rotate over copies of them as well (made and
+                # dropped here); small shapes, which live in the L2 in a step too, are left to the default rule
                 if len(ws) * N * K * 2 < min_bytes:
-                    continue
+                    if N * K * 2 < copy_bytes:
+                        continue
+                    ws = ws + [ws[i % len(ws)].clone() for i in range(min(-(-min_bytes // (N * K * 2)) - len(ws), 128))]
                 for M in self.ROW_BUCKETS:
                     x = torch.randn(M, K, device=ws[0].device, dtype=torch.bfloat16)
                     times = {}

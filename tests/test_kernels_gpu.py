@@ -232,10 +232,11 @@ def test_gemm_tc2_random_shapes(ops):
             assert err < 2e-2, (M, N, K, err)
 
 
+@pytest.mark.parametrize("act", ["silu", "gelu_tanh"])
 @pytest.mark.parametrize("M,inter,K", [(512, 128, 64), (700, 264, 192), (2048, 9728, 2560), (600, 1000, 640), (513, 40, 128), (129, 64, 128),
                                        (256, 1024, 2560), (1024, 648, 512)])
-def test_gemm_tc2_swiglu(ops, M, inter, K):
-    """The same with the gate rows loaded by the even block and the up rows by the odd one, silu(gate) * up in the epilogue."""
+def test_gemm_tc2_gated(ops, M, inter, K, act):
+    """The same with the gate rows loaded by the even block and the up rows by the odd one, act(gate) * up in the epilogue."""
     g = torch.Generator().manual_seed(M + inter)
     x = torch.randn(M, K, generator=g).to(torch.bfloat16).to(DEV)
     w = (torch.randn(2 * inter, K, generator=g) * K ** -0.5).to(torch.bfloat16).to(DEV)
@@ -243,13 +244,30 @@ def test_gemm_tc2_swiglu(ops, M, inter, K):
     ops.tc_gemm = True
     try:
         before = ops.launches
-        got = ops.gated_linear(x, w)
+        got = ops.gated_linear(x, w, act)
         assert ops.launches == before + 1
     finally:
         ops.tc_gemm = saved
     ops.check_errors()
     ref = TorchRefOps()
-    close(got, ref.swiglu(ref.linear(x, w)), torch.bfloat16)
+    close(got, ref.gated_linear(x, w, act), torch.bfloat16)
+
+
+@pytest.mark.parametrize("act", ["silu", "gelu_tanh"])
+@pytest.mark.parametrize("M,inter,K", [(1, 512, 256), (8, 1000, 640), (17, 2688, 1024), (32, 96, 2048)])
+def test_gated_product_of_a_few_rows(ops, M, inter, K, act):
+    """The few-row product left as partial sums, act(gate) * up applied by the kernel that adds them."""
+    g = torch.Generator().manual_seed(M + inter)
+    x = torch.randn(M, K, generator=g).to(torch.bfloat16).to(DEV)
+    w = (torch.randn(2 * inter, K, generator=g) * K ** -0.5).to(torch.bfloat16).to(DEV)
+    saved = ops._linear_choice
+    ops._linear_choice = {(ops._row_bucket(M), 2 * inter, K): "stream"}
+    try:
+        got = ops.gated_linear(x, w, act)
+    finally:
+        ops._linear_choice = saved
+    ops.check_errors()
+    close(got, TorchRefOps().gated_linear(x, w, act), torch.bfloat16)
 
 
 def make_meta(page_size, segs, num_pages, seed, tile=64, indirect=False, window=None):
