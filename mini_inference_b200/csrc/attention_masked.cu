@@ -224,7 +224,28 @@ __device__ __forceinline__ void put_head(const T* x, T* dst, int D, float r, con
     }
 }
 
+// The same two neighbouring coordinates at a time (D and half even, rows on the pair's boundary)
 template <typename T>
+__device__ __forceinline__ void put_head_pairs(const T* x, T* dst, int D, float r, const float* __restrict__ w, int half, const float* turn, int lane) {
+    for (int d = 2 * lane; d < D; d += 64) {
+        if (d >= half && d < 2 * half) continue;
+        float a0, a1;
+        load2(x + d, a0, a1);
+        a0 *= r; a1 *= r;
+        if (w) { a0 *= w[d]; a1 *= w[d + 1]; }
+        if (d >= half) { store2(dst + d, a0, a1); continue; }
+        float b0, b1;
+        load2(x + d + half, b0, b1);
+        b0 *= r; b1 *= r;
+        if (w) { b0 *= w[d + half]; b1 *= w[d + half + 1]; }
+        const float c0 = turn[d], c1 = turn[d + 1], s0 = turn[half + d], s1 = turn[half + d + 1];
+        store2(dst + d, a0 * c0 - b0 * s0, a1 * c1 - b1 * s1);
+        store2(dst + d + half, b0 * c0 + a0 * s0, b1 * c1 + a1 * s1);
+    }
+}
+
+// PAIRS: D, Dv, half and the row strides are even and everything lies on the boundary of two neighbouring entries
+template <typename T, bool PAIRS>
 __global__ void unit_qk_cache_kernel(T* __restrict__ p, int ldp, const T* __restrict__ v_src, int ld_src, const float* __restrict__ lam,
                                      const int* __restrict__ slots, T* __restrict__ k_cache, T* __restrict__ v_cache,
                                      int H, int KV, int D, int Dv, int ps, float eps, int unit, const float* __restrict__ q_w,
@@ -248,15 +269,22 @@ __global__ void unit_qk_cache_kernel(T* __restrict__ p, int ldp, const T* __rest
         float r = 1.f;
         if (unit) {
             float ss = 0.f;
-            for (int d = lane; d < D; d += 32) { const float v = to_f32(x[d]); ss += v * v; }
+            if constexpr (PAIRS) {
+                for (int d = 2 * lane; d < D; d += 64) { float a, b; load2(x + d, a, b); ss += a * a + b * b; }
+            } else {
+                for (int d = lane; d < D; d += 32) { const float v = to_f32(x[d]); ss += v * v; }
+            }
             r = rsqrtf(warp_sum(ss) / D + eps);
         }
+        auto put = [&](T* dst, float scale, const float* w) {
+            if constexpr (PAIRS) put_head_pairs<T>(x, dst, D, scale, w, half, turn, lane);
+            else put_head<T>(x, dst, D, scale, w, half, turn, lane);
+        };
         if (u < H) {
-            if (unit || q_w || temp_every > 0 || half > 0)
-                put_head<T>(x, x, D, r * temp, q_w, half, turn, lane);
+            if (unit || q_w || temp_every > 0 || half > 0) put(x, r * temp, q_w);
         } else if (k_cache) {
             T* dst = k_cache + ((page * KV + (u - H)) * ps + off) * D;
-            put_head<T>(x, dst, D, r, k_w, half, turn, lane);
+            put(dst, r, k_w);
             if (v_is_k && v_cache) {                           // the values are these keys as projected
                 T* vd = v_cache + ((page * KV + (u - H)) * ps + off) * D;
                 for (int d = lane; d < D; d += 32) vd[d] = x[d];
@@ -267,6 +295,14 @@ __global__ void unit_qk_cache_kernel(T* __restrict__ p, int ldp, const T* __rest
     const float l = lam ? lam[0] : 0.f;
     const T* v = row + (size_t)(H + KV) * D;
     const T* vs = v_src ? v_src + (size_t)t * ld_src : nullptr;
+    if (PAIRS && !vs) {
+        for (int i = 2 * threadIdx.x; i < KV * Dv; i += 2 * blockDim.x) {
+            float a, b;
+            load2(v + i, a, b);
+            store2(v_cache + ((page * KV + i / Dv) * ps + off) * Dv + i % Dv, a, b);
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < KV * Dv; i += blockDim.x) {
         float val = to_f32(v[i]);
         if (vs) val = (1.f - l) * val + l * to_f32(vs[i]);
@@ -287,11 +323,14 @@ MI_EXPORT int mi_normed_qk_cache(void* p, int ldp, const void* v_src, int ld_src
         (half > 0 && (!positions || !inv_freq || 2 * half > D || half > 4096))) return -2;
     const size_t turn = half > 0 ? 2 * (size_t)half * sizeof(float) : 0;
     // few tokens (decode steps): a warp per head, so that no warp walks several heads one after the other
-    const int nt = T_ >= 256 ? 128 : min(1024, max(128, 32 * (H + KV)));
-#define GO(T) return (int)launch_pdl(unit_qk_cache_kernel<T>, dim3(T_), dim3(nt), turn, stream, (T*)p, ldp, (const T*)v_src, ld_src, lam, slots, (T*)k_cache, (T*)v_cache, \
-                  H, KV, D, Dv, ps, eps, unit, q_w, k_w, positions, temp_coef, temp_every, v_is_k, inv_freq, half)
-    if (dtype == MI_BF16) GO(__nv_bfloat16);
-    GO(float);
+    const int nt = T_ >= 256 ? 256 : min(1024, max(128, 32 * (H + KV)));
+    const int el = dtype == MI_BF16 ? 2 : 4;
+    const bool pairs = D % 2 == 0 && Dv % 2 == 0 && half % 2 == 0 && ldp % 2 == 0 && ((uintptr_t)p | (uintptr_t)k_cache | (uintptr_t)v_cache) % (2 * el) == 0;
+#define GO(T, PAIRS) return (int)launch_pdl(unit_qk_cache_kernel<T, PAIRS>, dim3(T_), dim3(nt), turn, stream, (T*)p, ldp, (const T*)v_src, ld_src, lam, slots, (T*)k_cache, \
+                         (T*)v_cache, H, KV, D, Dv, ps, eps, unit, q_w, k_w, positions, temp_coef, temp_every, v_is_k, inv_freq, half)
+    if (dtype == MI_BF16) { if (pairs) GO(__nv_bfloat16, true); GO(__nv_bfloat16, false); }
+    if (pairs) GO(float, true);
+    GO(float, false);
 #undef GO
 }
 

@@ -152,6 +152,28 @@ __global__ void rows_rmsnorm_kernel(const T* __restrict__ x, long long ldx, cons
     for (int i = threadIdx.x; i < cols; i += NT) yr[i] = from_f32<T>(to_f32(xr[i]) * s * w[i]);
 }
 
+// rows of up to 8 NT entries of whole 16-byte pieces: a piece a thread, held between the statistic and the output
+template <typename T>
+__global__ void __launch_bounds__(NT) rows_rmsnorm_vec_kernel(const T* __restrict__ x, long long ldx, const float* __restrict__ w, T* __restrict__ y, int cols, float eps) {
+    constexpr int VN = Vec16<T>::N;
+    __shared__ float scratch[32];
+    pdl_trigger();
+    const int i = threadIdx.x * VN;
+    float wv[VN], v[VN], ss = 0.f;
+#pragma unroll
+    for (int e = 0; e < VN; ++e) { wv[e] = i < cols ? w[i + e] : 0.f; v[e] = 0.f; }
+    pdl_wait();
+    if (i < cols) load16(x + (size_t)blockIdx.x * ldx + i, v);
+#pragma unroll
+    for (int e = 0; e < VN; ++e) ss += v[e] * v[e];
+    const float s = rsqrtf(block_sum<NT>(ss, scratch) / cols + eps);
+    if (i < cols) {
+        T* o = y + (size_t)blockIdx.x * cols + i;
+#pragma unroll
+        for (int e = 0; e < VN; e += 2) store2(o + e, v[e] * s * wv[e], v[e + 1] * s * wv[e + 1]);
+    }
+}
+
 template <typename T> __device__ __forceinline__ void store16v(T* p, const float* v) {
     if constexpr (sizeof(T) == 4) {
         *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]);
@@ -244,6 +266,12 @@ MI_EXPORT int mi_stream_rmsnorm_pair(float* x, const void* a, const void* b, con
 
 MI_EXPORT int mi_rows_rmsnorm(const void* x, long long ldx, const float* w, void* y, int n, int cols, float eps, int dtype, cudaStream_t stream) {
     if (n == 0) return 0;
+    const int vn = dtype == MI_BF16 ? 8 : 4;
+    if (cols % vn == 0 && cols <= NT * vn && ldx % vn == 0 && ((uintptr_t)x | (uintptr_t)y) % 16 == 0) {
+        if (dtype == MI_BF16)
+            return (int)launch_pdl(rows_rmsnorm_vec_kernel<__nv_bfloat16>, dim3(n), dim3(NT), 0, stream, (const __nv_bfloat16*)x, ldx, w, (__nv_bfloat16*)y, cols, eps);
+        return (int)launch_pdl(rows_rmsnorm_vec_kernel<float>, dim3(n), dim3(NT), 0, stream, (const float*)x, ldx, w, (float*)y, cols, eps);
+    }
     if (dtype == MI_BF16) return (int)launch_pdl(rows_rmsnorm_kernel<__nv_bfloat16>, dim3(n), dim3(NT), 0, stream, (const __nv_bfloat16*)x, ldx, w, (__nv_bfloat16*)y, cols, eps);
     return (int)launch_pdl(rows_rmsnorm_kernel<float>, dim3(n), dim3(NT), 0, stream, (const float*)x, ldx, w, (float*)y, cols, eps);
 }
