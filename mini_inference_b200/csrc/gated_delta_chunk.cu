@@ -52,34 +52,6 @@ __device__ __forceinline__ void mma3(float (&c)[N][4], const uint32_t (&ah)[4], 
     for (int t = 0; t < N; ++t) mma16816(c[t], al, bh[t / 2][2 * (t % 2)], bh[t / 2][2 * (t % 2) + 1]);
 }
 
-// The same for few tiles, where a tile's products would wait for one another: the two smaller products add into sums of their own, which
-// join the first at the end of the chain (fold).
-template <int N> struct SideSums {
-    float hl[N][4], lh[N][4];
-    __device__ __forceinline__ SideSums() {
-#pragma unroll
-        for (int t = 0; t < N; ++t)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) hl[t][e] = lh[t][e] = 0.f;
-    }
-    __device__ __forceinline__ void fold(float (&c)[N][4]) const {
-#pragma unroll
-        for (int t = 0; t < N; ++t)
-#pragma unroll
-            for (int e = 0; e < 4; ++e) c[t][e] += hl[t][e] + lh[t][e];
-    }
-};
-template <int N>
-__device__ __forceinline__ void mma3(float (&c)[N][4], SideSums<N>& side, const uint32_t (&ah)[4], const uint32_t (&al)[4], const uint32_t (&bh)[(N + 1) / 2][4],
-                                     const uint32_t (&bl)[(N + 1) / 2][4]) {
-#pragma unroll
-    for (int t = 0; t < N; ++t) {
-        mma16816(c[t], ah, bh[t / 2][2 * (t % 2)], bh[t / 2][2 * (t % 2) + 1]);
-        mma16816(side.hl[t], ah, bl[t / 2][2 * (t % 2)], bl[t / 2][2 * (t % 2) + 1]);
-        mma16816(side.lh[t], al, bh[t / 2][2 * (t % 2)], bh[t / 2][2 * (t % 2) + 1]);
-    }
-}
-
 // byte offset of the 16-byte piece `ch` of row `row` in a tile of rows of N bfloat16 (N a multiple of 64; pieces XOR-ed with the row so that
 // ldmatrix meets no bank twice), and in a tile of rows of 32 or 16 of them
 template <int N> __device__ __forceinline__ uint32_t at(int row, int ch) {
@@ -473,8 +445,6 @@ __global__ void __launch_bounds__(NTH, 1) delta_pass_kernel(const unsigned char*
         if (k + 1 < chunks) fetch_u(k + 1);
         await(bar_wq, k);
         const uint32_t mine = base + L::WQ + (has_u ? 0 : 2 * W::KD);
-        SideSums<NT> u_side, o_side;
-        SideSums<SNT> s_side;
 #pragma unroll
         for (int ks = 0; ks < D / 16; ++ks) {                      // U = U_0 - W S;  O = Q' S
             uint32_t ah[4], al[4], bh[1][4], bl[1][4];
@@ -485,18 +455,17 @@ __global__ void __launch_bounds__(NTH, 1) delta_pass_kernel(const unsigned char*
             if constexpr (ROLES) {
                 ldsm4(ah, mine + ao);
                 ldsm4(al, mine + W::KD + ao);
-                mma3<NT>(u, u_side, ah, al, bh, bl);               // U, or O held in u
+                mma3<NT>(u, ah, al, bh, bl);                       // U, or O held in u
             } else {
                 uint32_t qh[4], ql[4];
                 ldsm4(ah, base + L::WQ + ao);
                 ldsm4(al, base + L::WQ + W::KD + ao);
                 ldsm4(qh, base + L::WQ + 2 * W::KD + ao);
                 ldsm4(ql, base + L::WQ + 3 * W::KD + ao);
-                mma3<NT>(u, u_side, ah, al, bh, bl);
-                mma3<NT>(o, o_side, qh, ql, bh, bl);
+                mma3<NT>(u, ah, al, bh, bl);
+                mma3<NT>(o, qh, ql, bh, bl);
             }
         }
-        u_side.fold(u);
         if constexpr (ROLES) {
 #pragma unroll
             for (int nt = 0; nt < NT; ++nt)
@@ -530,7 +499,7 @@ __global__ void __launch_bounds__(NTH, 1) delta_pass_kernel(const unsigned char*
                 const uint32_t bo = at<NC>(kb * 16 + (m & 1) * 8 + (lane & 7), nc0 / 8 + (m >> 1));
                 ldsm4t(uh[0], base + L::U + bo);
                 ldsm4t(ul[0], base + L::U + Q * NC * 2 + bo);
-                mma3<NT>(o, o_side, ph, pl, uh, ul);
+                mma3<NT>(o, ph, pl, uh, ul);
             }
             uint32_t ah[4], al[4], uh[(SNT + 1) / 2][4], ul[(SNT + 1) / 2][4];      // S += K'^T U
             const uint32_t ao = at<D>(kb * 16 + (m >> 1) * 8 + (lane & 7), sb * 2 + (m & 1));
@@ -543,10 +512,8 @@ __global__ void __launch_bounds__(NTH, 1) delta_pass_kernel(const unsigned char*
                 ldsm4t(uh[np], base + L::U + bo);
                 ldsm4t(ul[np], base + L::U + Q * NC * 2 + bo);
             }
-            mma3<SNT>(s, s_side, ah, al, uh, ul);
+            mma3<SNT>(s, ah, al, uh, ul);
         }
-        o_side.fold(o);
-        s_side.fold(s);
         spread_state();
         if (has_o)
 #pragma unroll
