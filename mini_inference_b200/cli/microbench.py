@@ -8,6 +8,7 @@ bench/micro/bench_attention.py (:61-167: paged decode attention over batch x con
     python -m mini_inference_b200.cli.microbench prefill   [--tokens 2048] [--ctx-before 0]
     python -m mini_inference_b200.cli.microbench design    [--design-size 2k|4k]   (the Naditar kernels beside Qwen3's)
     python -m mini_inference_b200.cli.microbench namesun   [--design-size 2k|4k]   (the Namesun kernels beside Qwen3's)
+    python -m mini_inference_b200.cli.microbench nununex|megovik|fetodra|kofutar   (those designs' kernels beside their closest predecessor's)
 
 Each line: kernel, shape, microseconds (CUDA events, after warm-up), GB/s of the bytes the
 kernel has to read, and that as a share of the measured copy bandwidth."""

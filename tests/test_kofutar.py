@@ -73,7 +73,7 @@ CONFIGS = {
                     loop=(0, 3, 2), eps=1e-6), 8),
     # pages of 16 and the sizes the tensor-core kernels take (heads of 64 and 128, latent rows of 64 and 128); more than 16 latent heads;
     # a span run "once" still passes the joining product; a layer behind the span
-    "pages": (config(64, 150, [attn(4, 2, 64, 64, rotation(32, 1e4, 8.0), scale=0.125, mlp=dense(72)), delta(4, 2, 32, 32, mlp=dense(24)),
+    "pages": (config(64, 150, [attn(4, 2, 64, 64, rotation(32, 1e4, 6.0), scale=0.125, mlp=dense(72)), delta(4, 2, 32, 32, mlp=dense(24)),
                                latent(18, 16, 16, 8, 48, 24, rotation(16, 5e3), scale=0.2), attn(3, 1, 128, 128, rotation(64, 3e5), scale=0.09),
                                latent(4, 24, 32, 16, 96, 40, rotation(32, 1e5), scale=0.13, mlp=dense(36)), delta(2, 1, 64, 128, conv=3)], loop=(1, 3, 1)), 16),
 }
@@ -242,7 +242,7 @@ SINGLE = {
     "attention_all_rotated": config(32, 61, [attn(2, 1, 16, 16, rotation(16, 10.0, 3.0))]),
     "attention_none_rotated": config(32, 61, [attn(2, 1, 16, 16, rotation(0, 10.0))]),
     "attention_odd": config(27, 53, [attn(3, 3, 7, 9, rotation(6, 40.0))]),
-    "attention_rows96": config(48, 61, [attn(4, 2, 96, 96, rotation(48, 1e4, 8.0), scale=0.1)]),
+    "attention_rows112": config(48, 61, [attn(6, 3, 112, 112, rotation(40, 1e4, 3.0), scale=0.1)]),
     "attention_rows64": config(48, 61, [attn(4, 2, 64, 64, rotation(20, 1e4), scale=0.1)]),
     "latent": config(32, 61, [latent(4, 8, 4, 8, 12, 10, rotation(4, 100.0))]),
     "latent_odd": config(27, 53, [latent(3, 7, 6, 5, 9, 11, rotation(6, 30.0, 2.0))]),
@@ -559,8 +559,8 @@ def test_each_mechanism_alone_on_gpu(tmp_path, name, dtype):
 @pytest.mark.parametrize("L,hot", HOT + [(1500, 3), (1500, 700), (1500, 1499), (1100, 1023)])
 def test_far_keys_and_the_sink_on_gpu(L, hot, dtype):
     ops = cuda_ops()
-    for kind, H, D, V in (("grouped", 4, 24, 24), ("grouped", 4, 64, 64), ("grouped", 6, 96, 96), ("grouped", 4, 40, 12), ("grouped", 4, 128, 128),
-                          ("latent", 4, 80, 64), ("latent", 5, 64, 48), ("latent", 20, 128, 96), ("latent", 3, 24, 17)):
+    for kind, H, D, V in (("grouped", 4, 24, 24), ("grouped", 4, 64, 64), ("grouped", 6, 112, 112), ("grouped", 4, 40, 12), ("grouped", 4, 128, 128),
+                          ("latent", 4, 88, 72), ("latent", 5, 64, 48), ("latent", 20, 128, 96), ("latent", 3, 24, 17)):
         for rows in (1, 3, 70):
             for splits in (None, 3):
                 ops.force_splits = splits
@@ -643,7 +643,7 @@ def test_kernels_against_the_stand_ins(dtype, lens, starts):
     cache_slots = (torch.randperm(2 * T, generator=g)[:T] + page).to(torch.int32)
     n_pages = 2 * T // page + 2
     ca, cg = SimpleNamespace(slots=cache_slots, positions=cpu.positions, page_size=page), SimpleNamespace(slots=cache_slots.to(dev), positions=gpu_b.positions, page_size=page)
-    for H, KV, D, V, half in ((6, 2, 8, 24, 3), (3, 1, 7, 5, 3), (4, 4, 16, 16, 8), (4, 2, 96, 96, 24), (2, 1, 33, 33, 0), (8, 2, 128, 128, 32), (1, 1, 256, 40, 128)):
+    for H, KV, D, V, half in ((6, 2, 8, 24, 3), (3, 1, 7, 5, 3), (4, 4, 16, 16, 8), (4, 2, 80, 80, 20), (2, 1, 33, 33, 0), (8, 2, 128, 128, 32), (1, 1, 256, 40, 128)):
         p, qw, kw, inv = rnd(T, (H + KV) * D + KV * V), f32(D), f32(D), torch.rand(half, generator=g)
         ka, va = torch.zeros(n_pages, KV, page, D, dtype=dtype), torch.zeros(n_pages, KV, page, V, dtype=dtype)
         kb, vb, pb = ka.to(dev), va.to(dev), p.to(dev)
